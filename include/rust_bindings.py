@@ -27,6 +27,7 @@ TYPES = {
     "float *": "*mut f32",
     "const float *": "*const f32",
     "int64_t *": "*mut i64",
+    "const int64_t *": "*const i64",
     "const int32_t *": "*const i32",
     "uint32_t *": "*mut u32",
     "const uint32_t *": "*const u32",

@@ -588,12 +588,92 @@ int singe_matmul_bf16_swiglu_bf16(singe_stream_t stream, void *out, const void *
 
 /* Linear::forward (singe/src/nn/layers/linear/mod.rs:49-70): out[rows, columns] = x[rows, reduction] . weight[columns,
  * reduction]^T, bf16 in, f32 accumulate, bf16 out -- singe_matmul_bf16_bf16 with the layer's layout fixed and a `hints`
- * word (SINGE_HINT_STABLE_WEIGHTS).  gated != 0: the SwiGLU epilogue of singe_matmul_bf16_swiglu_bf16 (out is
- * columns / 2 wide). */
+ * word (SINGE_HINT_STABLE_WEIGHTS).  activation 1: the SwiGLU epilogue of singe_matmul_bf16_swiglu_bf16 (out is
+ * columns / 2 wide); 2: max(x, 0)^2 before the store. */
 int singe_linear_bf16(singe_stream_t stream, void *out, const void *x, const void *weight, size_t rows, size_t columns,
                       size_t reduction, size_t x_row_stride, size_t weight_row_stride, size_t output_row_stride,
-                      int gated, unsigned hints);
+                      int activation, unsigned hints);
 
+/* =================================================================================================
+ * Layer-list decoders: f32 residual stream, attention over latents, gated linear attention
+ * No reference counterpart: these operators serve designs the reference has no layers for.  `_bf16` takes bf16
+ * activations and weights, `_f32` f32 ones (true 32-bit products); arithmetic between the matrix products is f32 in both.
+ * Row strides are in elements.
+ * ================================================================================================= */
+
+/* residual[t, :] = layer_norm(table[ids[t], :]) with layer_norm(x) = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight;
+ * negative ids wrap, ids outside the table take row 0 and set *status = 1.  width <= 16384 (4096 unless it divides by 4). */
+int singe_embedding_layer_norm_bf16(singe_stream_t stream, float *residual, const void *table, const int64_t *ids,
+                                    const void *weight, size_t tokens, size_t width, size_t vocab, float eps,
+                                    uint32_t *status);
+int singe_embedding_layer_norm_f32(singe_stream_t stream, float *residual, const void *table, const int64_t *ids,
+                                   const void *weight, size_t tokens, size_t width, size_t vocab, float eps,
+                                   uint32_t *status);
+
+/* residual += delta (delta != NULL), then normed = layer_norm(residual) (normed != NULL). */
+int singe_add_layer_norm_bf16(singe_stream_t stream, float *residual, const void *delta, size_t delta_stride,
+                              void *normed, size_t normed_stride, const void *weight, size_t rows, size_t width,
+                              float eps);
+int singe_add_layer_norm_f32(singe_stream_t stream, float *residual, const void *delta, size_t delta_stride,
+                             void *normed, size_t normed_stride, const void *weight, size_t rows, size_t width, float eps);
+
+/* A projected row is [query latent (q_rank) | key/value latent (kv_rank) | ...]: both are RMS-normed with their weights;
+ * the first goes to q_out, the second to row (write_pages[t], write_slots[t]) of the latent cache [pages, page_size,
+ * cache_width], zero-padded to cache_width.  Bad slots are dropped and set *status = 1. */
+int singe_latent_norm_cache_write_bf16(singe_stream_t stream, void *q_out, size_t q_stride, void *cache,
+                                       size_t cache_width, const void *projected, size_t projected_stride,
+                                       const void *q_weight, size_t q_rank, const void *kv_weight, size_t kv_rank,
+                                       const int64_t *write_pages, const int64_t *write_slots, size_t tokens, size_t pages,
+                                       size_t page_size, float eps, uint32_t *status);
+int singe_latent_norm_cache_write_f32(singe_stream_t stream, void *q_out, size_t q_stride, void *cache,
+                                      size_t cache_width, const void *projected, size_t projected_stride,
+                                      const void *q_weight, size_t q_rank, const void *kv_weight, size_t kv_rank,
+                                      const int64_t *write_pages, const int64_t *write_slots, size_t tokens, size_t pages,
+                                      size_t page_size, float eps, uint32_t *status);
+
+/* out[i, :] = source[rows[i], :]; rows of row_bytes bytes (a multiple of 16), row numbers below source_rows. */
+int singe_gather_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, size_t count,
+                      size_t row_bytes, size_t source_rows, uint32_t *status);
+
+/* singe_argmax_bf16 over f32 logits. */
+int singe_argmax_f32(singe_stream_t stream, float *best_value, int64_t *best_index, const float *logits,
+                     size_t row_stride, size_t rows, size_t width, int64_t index_offset);
+
+/* singe_linear_bf16 in true 32-bit; activation 0 (none) or 2 (squared relu). */
+int singe_linear_f32(singe_stream_t stream, float *out, const float *x, const float *weight, size_t rows, size_t columns,
+                     size_t reduction, size_t x_row_stride, size_t weight_row_stride, size_t output_row_stride,
+                     int activation);
+
+/* One product per attention head: out[t, h, :] = x[t, h, :] . weight[h]^T, times sigmoid(gate[t * gate_row_stride + h])
+ * when gate != NULL.  weight[h] is [columns, reduction] starting weight_head_rows rows after weight[h - 1].  bf16: row
+ * strides and x_head_stride are multiples of 8 elements; elements of x between heads, if any, must be finite. */
+int singe_head_linear_bf16(singe_stream_t stream, void *out, const void *x, const void *weight, size_t rows, size_t heads,
+                           size_t columns, size_t reduction, size_t x_row_stride, size_t x_head_stride,
+                           size_t weight_row_stride, size_t weight_head_rows, size_t out_row_stride,
+                           size_t out_head_stride, const void *gate, size_t gate_row_stride, unsigned hints);
+int singe_head_linear_f32(singe_stream_t stream, float *out, const float *x, const float *weight, size_t rows,
+                          size_t heads, size_t columns, size_t reduction, size_t x_row_stride, size_t x_head_stride,
+                          size_t weight_row_stride, size_t weight_head_rows, size_t out_row_stride,
+                          size_t out_head_stride, const float *gate, size_t gate_row_stride);
+
+/* Gated linear attention, one head's state S [dim, vdim] in f32 per sequence:
+ *   S_t = diag(sigmoid(z_t)^(1/tau)) S_(t-1) + k_t v_t^T,  o_t = query_scale * S_t^T q_t,  z_t = decay_weight a_t + decay_bias,
+ *   out = rms_norm(o_t) * norm_weight * silu(g_t)
+ * projected rows are [q (heads*dim) | k (heads*dim) | v (heads*vdim) | g (heads*vdim) | a (rank)]; decay_weight
+ * [heads*dim, rank], decay_bias [heads*dim], norm_weight [vdim]; out [rows, heads*vdim]; state [sequences, heads, dim, vdim].
+ * Sequence s owns rows [first[s], first[s] + count[s]); context[s] == 0 starts its state from zero.  count[s] == 0 leaves
+ * the state and zeroes row first[s] of out. */
+/* Token by token, for steps of few tokens; sequences of more than `longest` new tokens are left alone. */
+int singe_gated_linear_step_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *projected,
+                                 size_t projected_stride, const void *decay_weight, const void *decay_bias,
+                                 const void *norm_weight, float *state, const int32_t *first, const int32_t *count,
+                                 const int32_t *context, size_t rows, size_t sequences, size_t heads, size_t dim,
+                                 size_t vdim, size_t rank, float tau, float query_scale, float eps, size_t longest);
+int singe_gated_linear_step_f32(singe_stream_t stream, void *out, size_t out_stride, const void *projected,
+                                size_t projected_stride, const void *decay_weight, const void *decay_bias,
+                                const void *norm_weight, float *state, const int32_t *first, const int32_t *count,
+                                const int32_t *context, size_t rows, size_t sequences, size_t heads, size_t dim,
+                                size_t vdim, size_t rank, float tau, float query_scale, float eps, size_t longest);
 /* Explicit tile choice for the two GEMM entry points, process-wide: block_n in {32,64,128,256},
  * k_slices_per_stage in {1,2,4,8}; 0 = choose from the problem shape.
  * Replaces: TuningChoice::Explicit(MatmulTuning { tile, .. }) (singe-kernel/src/cuda/matmul.rs:58-77). */

@@ -23,6 +23,7 @@ import struct
 
 import numpy as np
 
+from .hybrid import GatedLinearConfig, HybridConfig, LatentAttentionConfig, LayerConfig
 from .llama import LlamaConfig, Shard
 
 CHECKPOINT_STEMS = ("model", "diffusion_pytorch_model")   # transformers' name first, then diffusers'
@@ -290,3 +291,125 @@ def load_llama(directory: str, shard: Shard | None = None, shard_lm_head: bool =
         "gate_up_interleaved": interleave_gate_up,
     }
     return config, weights
+
+
+# ------------------------------------------------------------------------------------------------
+# layer-list decoders (Kavalorn)
+# ------------------------------------------------------------------------------------------------
+
+def _section(fields: dict, where: str, *names):
+    """The named values of one object of the configuration; a missing or an unknown name is an error, so that nothing a
+    model asks for is passed over."""
+    if not isinstance(fields, dict):
+        raise UnsupportedConfig(f"{where} is not an object")
+    missing, unknown = sorted(set(names) - set(fields)), sorted(set(fields) - set(names))
+    if missing or unknown:
+        raise UnsupportedConfig(f"{where}: missing {missing}, unknown {unknown}")
+    return [fields[name] for name in names]
+
+
+def _positive(value, where: str) -> int:
+    if int(value) != value or value <= 0:
+        raise UnsupportedConfig(f"{where}: {value}")
+    return int(value)
+
+
+def _latent_attention(fields: dict, where: str, tensor_shape) -> LatentAttentionConfig:
+    heads, dim, vdim, q_rank, kv_rank, scale, mask = _section(fields, where, "heads", "dim", "vdim", "q_rank", "kv_rank",
+                                                              "scale", "mask")
+    (window,) = _section(mask, f"{where}.mask", "size")
+    sizes = [_positive(value, where) for value in (heads, dim, vdim, q_rank, kv_rank)]
+    return LatentAttentionConfig(*sizes, scale=float(scale), window=_positive(window, f"{where}.mask.size"))
+
+
+def _gated_linear(fields: dict, where: str, tensor_shape) -> GatedLinearConfig:
+    heads, dim, vdim, tau = _section(fields, where, "heads", "dim", "vdim", "tau")
+    if not float(tau) > 0.0:
+        raise UnsupportedConfig(f"{where}.tau: {tau}")
+    return GatedLinearConfig(*[_positive(value, where) for value in (heads, dim, vdim)],
+                             rank=int(tensor_shape("mix.a1")[0]), tau=float(tau))
+
+
+_MIXERS = {"latent_attention": _latent_attention, "gla": _gated_linear}
+
+
+def read_hybrid_config(directory: str, snapshot: "Snapshot") -> HybridConfig:
+    """``config.json`` of a layer-list model.  Sizes the configuration leaves out (the rank of the decay projection) come
+    from the tensors of the layer that owns the weights."""
+    with open(os.path.join(directory, "config.json")) as handle:
+        fields = json.load(handle)
+    _, entries, norm, vocab, width = _section(fields, "config.json", "architecture", "layers", "norm", "vocab", "width")
+    (eps,) = _section(norm, "norm", "eps")
+    config = HybridConfig(width=_positive(width, "width"), vocab=_positive(vocab, "vocab"), eps=float(eps))
+    borrowed = HybridConfig(layers=[LayerConfig(None, 0, entry.get("weights_of")) for entry in entries])
+    for index, entry in enumerate(entries):
+        where = f"layers[{index}]"
+        entry = {"mlp": None, "weights_of": None, **entry}
+        kind, mixer, mlp, _ = _section(entry, where, "type", "mixer", "mlp", "weights_of")
+        if kind not in _MIXERS:
+            raise UnsupportedConfig(f"{where}: mixer {kind}")
+        ffn = 0
+        if mlp is not None:
+            mlp_kind, ffn = _section(mlp, f"{where}.mlp", "kind", "ff")
+            if mlp_kind != "dense":
+                raise UnsupportedConfig(f"{where}.mlp: kind {mlp_kind}")
+            ffn = _positive(ffn, f"{where}.mlp.ff")
+        try:
+            owner = borrowed.owner(index)
+        except ValueError as error:
+            raise UnsupportedConfig(str(error)) from error
+
+        def tensor_shape(name, owner=owner):
+            full = f"l{owner}.{name}"
+            if full not in snapshot.where:
+                raise CheckpointError(f"checkpoint keys: missing {full}")
+            return snapshot.array(full).shape
+
+        config.layers.append(LayerConfig(_MIXERS[kind](mixer, f"{where}.mixer", tensor_shape), ffn,
+                                         entry["weights_of"]))
+    for index, layer in enumerate(config.layers):
+        source = config.layers[config.owner(index)]
+        if (layer.mixer, layer.ffn) != (source.mixer, source.ffn):
+            raise UnsupportedConfig(f"layers[{index}] differs from the layer whose weights it uses")
+    return config
+
+
+def hybrid_names(config: HybridConfig) -> dict:
+    """Parameter name -> expected shape, for the whole model."""
+    w = config.width
+    names = {"embed": (config.vocab, w), "embed.norm": (w,), "final.norm": (w,), "head": (config.vocab, w)}
+    for index, layer in enumerate(config.layers):
+        if layer.weights_of is not None:
+            continue
+        prefix, m = f"l{index}.", layer.mixer
+        names[prefix + "norm1"] = (w,)
+        if layer.ffn:
+            names.update({prefix + "norm2": (w,), prefix + "mlp.up": (layer.ffn, w), prefix + "mlp.down": (w, layer.ffn)})
+        if isinstance(m, LatentAttentionConfig):
+            mix = {"dq": (m.q_rank, w), "dq.norm": (m.q_rank,), "uq": (m.heads * m.dim, m.q_rank),
+                   "dkv": (m.kv_rank, w), "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank),
+                   "uv": (m.heads * m.vdim, m.kv_rank), "g": (m.heads, w), "o": (w, m.heads * m.vdim)}
+        else:
+            mix = {"q": (m.heads * m.dim, w), "k": (m.heads * m.dim, w), "v": (m.heads * m.vdim, w),
+                   "g": (m.heads * m.vdim, w), "o": (w, m.heads * m.vdim), "norm": (m.vdim,), "a1": (m.rank, w),
+                   "a2": (m.heads * m.dim, m.rank), "a2.b": (m.heads * m.dim,)}
+        names.update({f"{prefix}mix.{name}": shape for name, shape in mix.items()})
+    return names
+
+
+def load_hybrid(directory: str):
+    """Reads a snapshot and returns ``(config, weights)``, ``weights`` mapping names to device tensors of the stored
+    type."""
+    import torch
+
+    snapshot = Snapshot(directory)
+    config = read_hybrid_config(directory, snapshot)
+    check_keys(snapshot, hybrid_names(config))
+
+    def take(name):
+        host = np.array(snapshot.array(name), copy=True)
+        if snapshot.dtype(name) == "BF16":
+            return torch.from_numpy(host.view(np.int16)).cuda().view(torch.bfloat16)
+        return torch.from_numpy(host).cuda()
+
+    return config, {name: take(name) for name in snapshot.names()}

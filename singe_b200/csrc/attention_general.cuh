@@ -29,9 +29,10 @@ struct RowPlan {
                        // (sinks of Tensor::attend, singe/src/backend/cpu/normalization/attention.rs:253-263)
 };
 
-constexpr int kMaxPerLane = 8;  // head_dim <= 256
+constexpr int kMaxPerLane = 8;    // head_dim <= 256
+constexpr int kWidePerLane = 32;  // head_dim <= 1024: attention over latents, where a "head" is a whole cached row
 
-template <typename T, typename Policy>
+template <typename T, typename Policy, int MAX>
 __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, size_t rows, int head_dim, float scale,
                                                                 LseKind lse_kind, float empty_lse,
                                                                 uint32_t *status, float softcap) {
@@ -55,10 +56,10 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
         return;
     }
     const int per_lane = (head_dim + 31) >> 5;
-    float q[kMaxPerLane];
-    float acc[kMaxPerLane];
+    float q[MAX];
+    float acc[MAX];
 #pragma unroll
-    for (int i = 0; i < kMaxPerLane; ++i) {
+    for (int i = 0; i < MAX; ++i) {
         const int d = lane + 32 * i;
         q[i] = (i < per_lane && d < head_dim) ? to_float<T>(plan.query[d]) * scale : 0.0f;
         acc[i] = 0.0f;
@@ -81,7 +82,7 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
                 } else {
                     const T *key = policy.key_base() + offset[j];
 #pragma unroll
-                    for (int i = 0; i < kMaxPerLane; ++i) {
+                    for (int i = 0; i < MAX; ++i) {
                         const int d = lane + 32 * i;
                         if (i < per_lane && d < head_dim) {
                             score[j] = fmaf(q[i], to_float<T>(key[d]), score[j]);
@@ -114,7 +115,7 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
         running_sum = running_sum * correction + tile_sum;
         running_max = next_max;
 #pragma unroll
-        for (int i = 0; i < kMaxPerLane; ++i) {
+        for (int i = 0; i < MAX; ++i) {
             acc[i] *= correction;
         }
 #pragma unroll
@@ -122,7 +123,7 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
             if (pos + j < plan.end) {
                 const T *value = policy.value_base() + offset[j];
 #pragma unroll
-                for (int i = 0; i < kMaxPerLane; ++i) {
+                for (int i = 0; i < MAX; ++i) {
                     const int d = lane + 32 * i;
                     if (i < per_lane && d < head_dim) {
                         acc[i] = fmaf(weight[j], to_float<T>(value[d]), acc[i]);
@@ -138,7 +139,7 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
     const bool empty = plan.end <= plan.start && plan.sink == -INFINITY;
     const float inverse = empty ? 0.0f : 1.0f / running_sum;
 #pragma unroll
-    for (int i = 0; i < kMaxPerLane; ++i) {
+    for (int i = 0; i < MAX; ++i) {
         const int d = lane + 32 * i;
         if (i < per_lane && d < head_dim) {
             plan.out[d] = from_float<T>(acc[i] * inverse);
@@ -156,7 +157,7 @@ __global__ void __launch_bounds__(128) attention_general_kernel(Policy policy, s
 template <typename T, typename Policy>
 int launch_attention_general(cudaStream_t stream, const Policy &policy, size_t rows, size_t head_dim, float scale,
                              LseKind lse_kind, float empty_lse, uint32_t *status, float softcap = 0.0f) {
-    if (head_dim > 32 * kMaxPerLane) {
+    if (head_dim > 32 * kWidePerLane) {
         return SINGE_ERR_UNSUPPORTED_WIDTH;
     }
     if (rows == 0) {
@@ -166,9 +167,15 @@ int launch_attention_general(cudaStream_t stream, const Policy &policy, size_t r
     if (blocks > 0x7fffffffull) {
         return SINGE_ERR_LENGTH_EXCEEDS_I32;
     }
-    SINGE_CUDA_TRY(launch_dependent(attention_general_kernel<T, Policy>, dim3(static_cast<unsigned>(blocks)), dim3(128), 0,
-                                    stream, kLaunchGlue, 1, policy, rows, static_cast<int>(head_dim), scale, lse_kind,
-                                    empty_lse, status, softcap));
+    if (head_dim <= 32 * kMaxPerLane) {
+        SINGE_CUDA_TRY(launch_dependent(attention_general_kernel<T, Policy, kMaxPerLane>, dim3(static_cast<unsigned>(blocks)),
+                                        dim3(128), 0, stream, kLaunchGlue, 1, policy, rows, static_cast<int>(head_dim),
+                                        scale, lse_kind, empty_lse, status, softcap));
+    } else {
+        SINGE_CUDA_TRY(launch_dependent(attention_general_kernel<T, Policy, kWidePerLane>, dim3(static_cast<unsigned>(blocks)),
+                                        dim3(128), 0, stream, kLaunchGlue, 1, policy, rows, static_cast<int>(head_dim),
+                                        scale, lse_kind, empty_lse, status, softcap));
+    }
     return launch_status();
 }
 

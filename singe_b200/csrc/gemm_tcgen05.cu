@@ -52,6 +52,15 @@ struct GemmParams {
     int tiles_m, tiles_n, k_blocks;  // k_blocks counts stages: KPS 64-wide slices each
     int vector_store;  // 16-byte stores are legal (alignment and stride)
     int gated;         // 1: columns are (gate, up) pairs; the epilogue stores bf16(bf16(silu(gate)) * up), n / 2 wide
+    int squared_relu;  // 1: the epilogue stores max(x, 0)^2
+    // Batched form (one small product per attention head, see singe_head_linear_bf16): problem b reads lhs columns from
+    // b * lhs_batch_columns on, rhs rows from b * rhs_batch_rows on and writes out columns from b * out_batch_columns on.
+    int batch;         // 1: a single product
+    int lhs_batch_columns;
+    int rhs_batch_rows;
+    long long out_batch_columns;
+    const __nv_bfloat16 *row_gate;  // nullptr, or row i of problem b is multiplied by sigmoid(row_gate[i * row_gate_stride + b])
+    long long row_gate_stride;
     int stable_rhs;    // 1: the caller vouches that rhs (a weight matrix) is not written by work still in flight, so
                        //    its first tiles are fetched before the wait on the preceding kernels
     int prefetch_blocks;  // with stable_rhs: k-blocks beyond the ring whose rhs tiles are pulled into L2 before the wait
@@ -69,6 +78,13 @@ __device__ __forceinline__ float gated_value(float gate_acc, float up_acc) {
     const float up = __bfloat162float(__float2bfloat16_rn(up_acc));
     const float activated = __bfloat162float(__float2bfloat16_rn(silu_fast(gate)));
     return activated * up;
+}
+
+__device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + __expf(-x)); }
+
+__device__ __forceinline__ float squared_relu_f32(float x) {
+    const float positive = fmaxf(x, 0.0f);
+    return positive * positive;
 }
 
 // One 64-wide K slice of the B operand into shared memory (BN x 128 bytes either way).  [N, K] weights: one box of BN
@@ -147,7 +163,8 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
     const int a_bytes = p.a_rows * 128;
-    const int total_tiles = p.tiles_m * p.tiles_n;
+    const int batch_tiles = p.tiles_m * p.tiles_n;
+    const int total_tiles = batch_tiles * p.batch;
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < p.stages; ++s) {
@@ -184,7 +201,9 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
         int preloaded = 0;
         if (p.stable_rhs && blockIdx.x < total_tiles) {
             int tm, tn;
-            tile_coordinates(blockIdx.x, p.tiles_m, p.tiles_n, tm, tn);
+            const int batch = blockIdx.x / batch_tiles;
+            tile_coordinates(blockIdx.x - batch * batch_tiles, p.tiles_m, p.tiles_n, tm, tn);
+            const int b_row = batch * p.rhs_batch_rows + tn * BN;
             preloaded = min(p.stages, p.k_blocks);
             if (lane == 0) {
                 for (int kb = 0; kb < preloaded; ++kb) {
@@ -194,13 +213,13 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
 #pragma unroll
                     for (int sub = 0; sub < KPS; ++sub) {
                         load_b_slice<BN, KN>(stage + KPS * MT * a_bytes + sub * kBBytes, &b_map, full, (kb * KPS + sub) * kBlockK,
-                                         tn * BN);
+                                         b_row);
                     }
                 }
                 const int last = min(p.k_blocks, preloaded + p.prefetch_blocks);
                 for (int kb = preloaded; kb < last; ++kb) {
 #pragma unroll
-                    for (int sub = 0; sub < KPS; ++sub) prefetch_b_slice<BN, KN>(&b_map, (kb * KPS + sub) * kBlockK, tn * BN);
+                    for (int sub = 0; sub < KPS; ++sub) prefetch_b_slice<BN, KN>(&b_map, (kb * KPS + sub) * kBlockK, b_row);
                 }
             }
         }
@@ -208,7 +227,10 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
         int it = 0;
         for (int tile = blockIdx.x; tile < total_tiles && !failed; tile += gridDim.x) {
             int tm, tn;
-            tile_coordinates(tile, p.tiles_m, p.tiles_n, tm, tn);
+            const int batch = tile / batch_tiles;
+            tile_coordinates(tile - batch * batch_tiles, p.tiles_m, p.tiles_n, tm, tn);
+            const int a_column = batch * p.lhs_batch_columns;
+            const int b_row = batch * p.rhs_batch_rows + tn * BN;
             for (int kb = 0; kb < p.k_blocks; ++kb, ++it) {
                 const int s = it % p.stages;
                 const uint32_t phase = (it / p.stages) & 1;
@@ -235,7 +257,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
                                 tma_load_2d(a_at, &a_map, full, row0, (kb * KPS + sub) * kBlockK);
                                 tma_load_2d(a_at + 8192, &a_map, full, row0 + 64, (kb * KPS + sub) * kBlockK);
                             } else {
-                                tma_load_2d(a_at, &a_map, full, (kb * KPS + sub) * kBlockK, row0);
+                                tma_load_2d(a_at, &a_map, full, a_column + (kb * KPS + sub) * kBlockK, row0);
                             }
                         }
                     }
@@ -243,7 +265,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
 #pragma unroll
                         for (int sub = 0; sub < KPS; ++sub) {
                             load_b_slice<BN, KN>(stage + KPS * MT * a_bytes + sub * kBBytes, &b_map, full,
-                                             (kb * KPS + sub) * kBlockK, tn * BN);
+                                             (kb * KPS + sub) * kBlockK, b_row);
                         }
                     }
                 }
@@ -307,7 +329,9 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
         int local = 0;
         for (int tile = blockIdx.x; tile < total_tiles && !failed; tile += gridDim.x, ++local) {
             int tm, tn;
-            tile_coordinates(tile, p.tiles_m, p.tiles_n, tm, tn);
+            const int batch = tile / batch_tiles;
+            tile_coordinates(tile - batch * batch_tiles, p.tiles_m, p.tiles_n, tm, tn);
+            const long long out_column = batch * p.out_batch_columns;
             const int acc = MT == 2 ? 0 : (local & 1);
             const uint32_t acc_phase = MT == 2 ? (local & 1) : ((local >> 1) & 1);
             if (!__all_sync(0xffffffffu, mbar_wait(bar_acc_full + acc * 8, acc_phase) ? 1 : 0)) {
@@ -325,6 +349,15 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
                 tmem_ld_x32(taddr + c, r);
                 tmem_wait_ld();
                 const int col = tn * BN + c;
+                if (p.squared_relu) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(squared_relu_f32(__uint_as_float(r[j])));
+                }
+                if (p.row_gate != nullptr && row < p.m) {
+                    const float gate = sigmoid_f32(__bfloat162float(p.row_gate[row * p.row_gate_stride + batch]));
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * gate);
+                }
                 if (row < p.m && col < p.n && p.gated) {
                     __nv_bfloat16 *dst =
                         static_cast<__nv_bfloat16 *>(p.out) + static_cast<long long>(row) * p.ldo + col / 2;
@@ -352,7 +385,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
                     }
                 } else if (row < p.m && col < p.n) {
                     if (p.out_f32) {
-                        float *dst = static_cast<float *>(p.out) + static_cast<long long>(row) * p.ldo + col;
+                        float *dst = static_cast<float *>(p.out) + static_cast<long long>(row) * p.ldo + out_column + col;
                         if (p.vector_store && col + 32 <= p.n) {
 #pragma unroll
                             for (int j = 0; j < 32; j += 4) {
@@ -366,7 +399,7 @@ __global__ void __launch_bounds__(kGemmThreads, 1)
                         }
                     } else {
                         __nv_bfloat16 *dst =
-                            static_cast<__nv_bfloat16 *>(p.out) + static_cast<long long>(row) * p.ldo + col;
+                            static_cast<__nv_bfloat16 *>(p.out) + static_cast<long long>(row) * p.ldo + out_column + col;
                         if (p.vector_store && col + 32 <= p.n) {
 #pragma unroll
                             for (int j = 0; j < 32; j += 8) {
@@ -703,6 +736,12 @@ __global__ void __launch_bounds__(kSplitKThreads, 1)
                         sum.w += part[u][s].w;
                     }
                 }
+                if (p.squared_relu) {
+                    sum.x = squared_relu_f32(sum.x);
+                    sum.y = squared_relu_f32(sum.y);
+                    sum.z = squared_relu_f32(sum.z);
+                    sum.w = squared_relu_f32(sum.w);
+                }
                 const float values[4] = {sum.x, sum.y, sum.z, sum.w};
                 if (p.gated) {
                     __nv_bfloat16 *dst =
@@ -879,7 +918,10 @@ int launch_gemm(cudaStream_t stream, GemmParams params, const void *lhs, const v
         SINGE_TRY(encode_tensor_map(&a_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, lhs, dims, strides, box,
                                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     } else {
-        const uint64_t dims[2] = {static_cast<uint64_t>(params.k), static_cast<uint64_t>(params.m)};
+        // batched: the problems' columns lie side by side; a K tail that reads into the next problem's columns meets the
+        // zero fill of rhs
+        const uint64_t columns = static_cast<uint64_t>(params.batch - 1) * params.lhs_batch_columns + params.k;
+        const uint64_t dims[2] = {columns, static_cast<uint64_t>(params.m)};
         const uint64_t strides[1] = {static_cast<uint64_t>(lhs_row_stride) * 2};
         const uint32_t box[2] = {kBlockK, static_cast<uint32_t>(params.a_rows)};
         SINGE_TRY(encode_tensor_map(&a_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, lhs, dims, strides, box,
@@ -892,13 +934,14 @@ int launch_gemm(cudaStream_t stream, GemmParams params, const void *lhs, const v
         SINGE_TRY(encode_tensor_map(&b_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rhs, dims, strides, box,
                                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     } else {
-        const uint64_t dims[2] = {static_cast<uint64_t>(params.k), static_cast<uint64_t>(params.n)};
+        const uint64_t weight_rows = static_cast<uint64_t>(params.batch - 1) * params.rhs_batch_rows + params.n;
+        const uint64_t dims[2] = {static_cast<uint64_t>(params.k), weight_rows};
         const uint64_t strides[1] = {static_cast<uint64_t>(rhs_row_stride) * 2};
         const uint32_t box[2] = {kBlockK, static_cast<uint32_t>(BN)};
         SINGE_TRY(encode_tensor_map(&b_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rhs, dims, strides, box,
                                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     }
-    const int total = params.tiles_m * params.tiles_n;
+    const int total = params.tiles_m * params.tiles_n * params.batch;
     const int grid = total < device_sm_count() ? total : device_sm_count();
     if (params.rhs_kn) {
         SINGE_CUDA_TRY(launch_dependent(gemm_bf16_kernel<BN, KPS, kHasKN, AT, MT>, dim3(grid), dim3(kGemmThreads), smem,
@@ -912,10 +955,23 @@ int launch_gemm(cudaStream_t stream, GemmParams params, const void *lhs, const v
 
 }  // namespace
 
+// What a call asks of the epilogue beyond the plain store, and the batched form's strides (elements).
+struct GemmOptions {
+    bool gated = false;
+    bool squared_relu = false;
+    size_t batch = 1;
+    size_t lhs_batch_columns = 0;
+    size_t rhs_batch_rows = 0;
+    size_t out_batch_columns = 0;
+    const void *row_gate = nullptr;
+    size_t row_gate_stride = 0;
+};
+
 // validate_matmul (singe-kernel/src/cuda/matmul.rs:2977-3020), then the layout gate of the tensor-core path.
 int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, const void *rhs, size_t rows,
               size_t columns, size_t reduction, size_t lhs_row_stride, size_t rhs_row_stride,
-              size_t output_row_stride, int transpose_lhs, int transpose_rhs, bool gated, unsigned hints) {
+              size_t output_row_stride, int transpose_lhs, int transpose_rhs, const GemmOptions &options, unsigned hints) {
+    const bool gated = options.gated;
     const size_t lhs_min = transpose_lhs ? rows : reduction;
     const size_t rhs_min = transpose_rhs ? reduction : columns;
     if (rows == 0 || columns == 0 || reduction == 0 || lhs_row_stride < lhs_min || rhs_row_stride < rhs_min ||
@@ -942,6 +998,13 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
     params.out = out;
     params.out_f32 = out_f32 ? 1 : 0;
     params.gated = gated ? 1 : 0;
+    params.squared_relu = options.squared_relu ? 1 : 0;
+    params.batch = static_cast<int>(options.batch);
+    params.lhs_batch_columns = static_cast<int>(options.lhs_batch_columns);
+    params.rhs_batch_rows = static_cast<int>(options.rhs_batch_rows);
+    params.out_batch_columns = static_cast<long long>(options.out_batch_columns);
+    params.row_gate = static_cast<const __nv_bfloat16 *>(options.row_gate);
+    params.row_gate_stride = static_cast<long long>(options.row_gate_stride);
     params.stable_rhs = (hints & SINGE_HINT_STABLE_WEIGHTS) != 0 ? 1 : 0;
     params.warm = take_pending_warm();
     params.rhs_kn = transpose_rhs ? 0 : 1;
@@ -960,11 +1023,12 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
     params.a_rows = a_rows;
     const size_t element = out_f32 ? 4 : 2;
     params.vector_store =
-        ((reinterpret_cast<uintptr_t>(out) & 15u) == 0 && (output_row_stride * element) % 16 == 0) ? 1 : 0;
+        ((reinterpret_cast<uintptr_t>(out) & 15u) == 0 && (output_row_stride * element) % 16 == 0 &&
+         (options.out_batch_columns * element) % 16 == 0) ? 1 : 0;
     // Widest tile that still gives every SM a tile; narrow tiles for skinny (HBM-bound) problems, which also take
     // several K slices per stage so that each weight row is requested in long contiguous runs.
     const int sms = device_sm_count();
-    auto tiles = [&](int bn) { return params.tiles_m * ((params.n + bn - 1) / bn); };
+    auto tiles = [&](int bn) { return params.batch * params.tiles_m * ((params.n + bn - 1) / bn); };
     int bn = 32;
     int slices = 1;
     if (params.m > kBlockM) {
@@ -995,7 +1059,7 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
     const int forced_splits = g_tuning_splits.load(std::memory_order_relaxed);
     const int forced_block_n = g_tuning_block_n.load(std::memory_order_relaxed);
     const int forced_slices = g_tuning_slices.load(std::memory_order_relaxed);
-    if (params.m <= kBlockM && tiles(128) < (sms * 2) / 3 && forced_splits != 1) {
+    if (params.m <= kBlockM && tiles(128) < (sms * 2) / 3 && forced_splits != 1 && params.batch == 1) {
         int wide = 128;
         int wanted = 1;
         while (wanted < 4 && tiles(wide) * wanted * 2 <= sms) wanted <<= 1;
@@ -1013,7 +1077,7 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
             slices = 2;
         }
     }
-    if (forced_splits != 0) splits = forced_splits;
+    if (forced_splits != 0 && params.batch == 1) splits = forced_splits;
     if (forced_block_n != 0) bn = forced_block_n;
     if (params.rhs_kn && bn < 64) {
         // [K, N] tiles are staged in boxes of 64 columns
@@ -1048,7 +1112,7 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
         return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     }
     // Many 256 x 256 tiles: the form with two M sub-tiles per CTA, which halves the A-and-B bytes an SM pulls per flop.
-    if (bn == 256 && slices == 1 && params.m >= 2 * kBlockM &&
+    if (bn == 256 && slices == 1 && params.m >= 2 * kBlockM && params.batch == 1 &&
         ((params.m + 2 * kBlockM - 1) / (2 * kBlockM)) * ((params.n + 255) / 256) >= sms) {
         return launch_gemm<256, 1, false, 2>(stream, params, lhs, rhs, lhs_row_stride, rhs_row_stride);
     }
@@ -1070,6 +1134,17 @@ int gemm_bf16(cudaStream_t stream, void *out, bool out_f32, const void *lhs, con
     return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
 }
 
+namespace {
+
+// activation: 0 none, 1 SwiGLU over interleaved (gate, up) columns, 2 squared relu
+GemmOptions gemm_activation(int activation) {
+    GemmOptions options;
+    options.gated = activation == 1;
+    options.squared_relu = activation == 2;
+    return options;
+}
+
+}  // namespace
 }  // namespace singe
 
 extern "C" {
@@ -1078,7 +1153,7 @@ int singe_matmul_bf16_bf16(singe_stream_t stream, void *out, const void *lhs, co
                            size_t columns, size_t reduction, size_t lhs_row_stride, size_t rhs_row_stride,
                            size_t output_row_stride, int transpose_lhs, int transpose_rhs) {
     return singe::gemm_bf16(static_cast<cudaStream_t>(stream), out, false, lhs, rhs, rows, columns, reduction,
-                            lhs_row_stride, rhs_row_stride, output_row_stride, transpose_lhs, transpose_rhs, false, 0u);
+                            lhs_row_stride, rhs_row_stride, output_row_stride, transpose_lhs, transpose_rhs, {}, 0u);
 }
 
 // out[M, N/2] = bf16(bf16(silu(g)) * u) with g = bf16(lhs . rhs[2j]^T), u = bf16(lhs . rhs[2j+1]^T): the gate and up
@@ -1088,23 +1163,52 @@ int singe_matmul_bf16_swiglu_bf16(singe_stream_t stream, void *out, const void *
                                   size_t columns, size_t reduction, size_t lhs_row_stride, size_t rhs_row_stride,
                                   size_t output_row_stride) {
     return singe::gemm_bf16(static_cast<cudaStream_t>(stream), out, false, lhs, rhs, rows, columns, reduction,
-                            lhs_row_stride, rhs_row_stride, output_row_stride, 0, 1, true, 0u);
+                            lhs_row_stride, rhs_row_stride, output_row_stride, 0, 1, singe::gemm_activation(1), 0u);
 }
 
 int singe_matmul_bf16_f32(singe_stream_t stream, float *out, const void *lhs, const void *rhs, size_t rows,
                           size_t columns, size_t reduction, size_t lhs_row_stride, size_t rhs_row_stride,
                           size_t output_row_stride, int transpose_lhs, int transpose_rhs) {
     return singe::gemm_bf16(static_cast<cudaStream_t>(stream), out, true, lhs, rhs, rows, columns, reduction,
-                            lhs_row_stride, rhs_row_stride, output_row_stride, transpose_lhs, transpose_rhs, false, 0u);
+                            lhs_row_stride, rhs_row_stride, output_row_stride, transpose_lhs, transpose_rhs, {}, 0u);
 }
 
 // Linear::forward with the weight matrix as a parameter of the layer: out[M, N] = x[M, K] . weight[N, K]^T.  `hints`
-// may carry SINGE_HINT_STABLE_WEIGHTS; `gated` != 0 selects the SwiGLU epilogue of singe_matmul_bf16_swiglu_bf16.
+// may carry SINGE_HINT_STABLE_WEIGHTS; `activation` 1 selects the SwiGLU epilogue of singe_matmul_bf16_swiglu_bf16, 2 the
+// squared relu.
 int singe_linear_bf16(singe_stream_t stream, void *out, const void *x, const void *weight, size_t rows,
                       size_t columns, size_t reduction, size_t x_row_stride, size_t weight_row_stride,
-                      size_t output_row_stride, int gated, unsigned hints) {
+                      size_t output_row_stride, int activation, unsigned hints) {
+    if (activation < 0 || activation > 2) return SINGE_ERR_INVALID_ARGUMENT;
     return singe::gemm_bf16(static_cast<cudaStream_t>(stream), out, false, x, weight, rows, columns, reduction,
-                            x_row_stride, weight_row_stride, output_row_stride, 0, 1, gated != 0, hints);
+                            x_row_stride, weight_row_stride, output_row_stride, 0, 1,
+                            singe::gemm_activation(activation), hints);
+}
+
+// One product per head on the persistent kernel: every head's tiles are items of the same grid.
+int singe_head_linear_bf16(singe_stream_t stream, void *out, const void *x, const void *weight, size_t rows, size_t heads,
+                           size_t columns, size_t reduction, size_t x_row_stride, size_t x_head_stride,
+                           size_t weight_row_stride, size_t weight_head_rows, size_t out_row_stride,
+                           size_t out_head_stride, const void *gate, size_t gate_row_stride, unsigned hints) {
+    if (heads == 0 || columns == 0 || weight_head_rows < columns || x_head_stride < reduction ||
+        out_head_stride < columns || x_row_stride < (heads - 1) * x_head_stride + reduction ||
+        out_row_stride < (heads - 1) * out_head_stride + columns || (gate != nullptr && gate_row_stride < heads)) {
+        return SINGE_ERR_INVALID_LENGTH;
+    }
+    if (!singe::fits_i32(heads * weight_head_rows) || !singe::fits_i32(x_row_stride) || !singe::fits_i32(out_row_stride) ||
+        !singe::fits_i32(heads * ((rows + 127) / 128) * ((columns + 31) / 32))) {
+        return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    }
+    if (x_head_stride % 8 != 0) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;  // a head starts on a 16-byte boundary
+    singe::GemmOptions options;
+    options.batch = heads;
+    options.lhs_batch_columns = x_head_stride;
+    options.rhs_batch_rows = weight_head_rows;
+    options.out_batch_columns = out_head_stride;
+    options.row_gate = gate;
+    options.row_gate_stride = gate_row_stride;
+    return singe::gemm_bf16(static_cast<cudaStream_t>(stream), out, false, x, weight, rows, columns, reduction,
+                            x_row_stride, weight_row_stride, out_row_stride, 0, 1, options, hints);
 }
 
 // Overrides the tile choice of the GEMM entry points for this process: block_n in {32, 64, 128, 256} and

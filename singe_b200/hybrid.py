@@ -1,0 +1,558 @@
+"""Decoder whose configuration lists its layers one by one, each with its own mixer and an optional feed-forward.
+
+``HybridDecoder`` is a ``PagedDecoder``: the page table, the one-token step and its CUDA graph, the generation loop and
+the checkpoint reader are the ones every decoder here uses.  What is new stands beside them:
+
+  ``LatentAttention``   attention over a low-rank latent of the context.  The cache holds one normalised latent row per
+                        token, shared by all heads, behind the page table; a sliding window bounds what a token sees and
+                        lets the page table take unseen pages back.
+  ``GatedLinear``       gated linear attention: a recurrent state per sequence, [heads, dim, vdim] in f32, in the
+                        sequence's row; a sequence's first token starts it from zero, so a row that is used again needs
+                        no clearing.
+  feed-forward          down(relu(up(h))^2)
+
+A layer may borrow another layer's weights; its cache or state is always its own.  The residual stream and all norms
+are f32.  ``dtype`` "bfloat16" keeps weights and activations in bf16 (f32 accumulation, tensor-core kernels); "float32"
+computes everything in true 32-bit with the library's f32 kernels.
+
+Latent attention has two forms of the same product.  Per head, score = (W_uq c_q) . (W_uk c) and value = W_uv c:
+  absorbed   q' = W_uk^T q, then attention of q' over the latents themselves, then W_uv on the attended latent: reads only
+             the cache, for steps of few tokens per sequence;
+  expanded   k and v of every visible latent are computed by one GEMM and attended on the tensor core: for prompts.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+
+import numpy as np
+
+from . import kernel_sys as ks
+from .decoder import PagedDecoder, PageTable
+
+EXPANDED_HEAD_SIZES = (64, 128)  # head sizes of the tensor-core prompt attention; smaller heads are padded with zeros
+ABSORBED_LATENT_LIMIT = 512      # widest latent the tensor-core decode attention takes
+FEW_TOKENS = 8                   # a sequence with at most this many new tokens takes the decode kernels
+
+
+# ------------------------------------------------------------------------------------------------
+# configuration
+# ------------------------------------------------------------------------------------------------
+
+@dataclass(frozen=True)
+class LatentAttentionConfig:
+    heads: int
+    dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    window: int
+
+
+@dataclass(frozen=True)
+class GatedLinearConfig:
+    heads: int
+    dim: int
+    vdim: int
+    rank: int      # of the decay projection
+    tau: float
+
+
+@dataclass(frozen=True)
+class LayerConfig:
+    mixer: object
+    ffn: int = 0               # 0: the layer has no feed-forward
+    weights_of: int | None = None
+
+
+@dataclass
+class HybridConfig:
+    layers: list = field(default_factory=list)
+    width: int = 0
+    vocab: int = 0
+    eps: float = 1e-6
+    page_size: int = 16
+
+    def owner(self, index: int) -> int:
+        """The layer whose weights layer ``index`` uses."""
+        seen = {index}
+        while self.layers[index].weights_of is not None:
+            index = self.layers[index].weights_of
+            if not 0 <= index < len(self.layers) or index in seen:
+                raise ValueError(f"layer {index}: borrowed weights lead nowhere")
+            seen.add(index)
+        return index
+
+    def window(self) -> int:
+        """The most tokens any layer looks back over through the cache."""
+        return max((layer.mixer.window for layer in self.layers if isinstance(layer.mixer, LatentAttentionConfig)),
+                   default=1)
+
+
+def round_up(value: int, multiple: int) -> int:
+    return (value + multiple - 1) // multiple * multiple
+
+
+# ------------------------------------------------------------------------------------------------
+# kernels behind one activation type
+# ------------------------------------------------------------------------------------------------
+
+class Ops:
+    """The library's entry points for one activation type, and buffers laid out the way they want them (rows of whole
+    16-byte pieces)."""
+
+    def __init__(self, dtype: str):
+        import torch
+
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError(f"activation type {dtype}")
+        self.torch = torch
+        self.dtype = getattr(torch, dtype)
+        self.is_bf16 = dtype == "bfloat16"
+        self.suffix = "bf16" if self.is_bf16 else "f32"
+
+    def call(self, name: str, *arguments) -> None:
+        code = getattr(ks.lib(), name)(*[a.data_ptr() if hasattr(a, "data_ptr") else a for a in arguments])
+        if code != ks.OK:
+            raise RuntimeError(f"{name}: status {code} ({ks.status_string(code)})")
+
+    def rows(self, rows: int, columns: int):
+        """[rows, columns] of the activation type with padded row stride."""
+        return self.torch.empty((rows, round_up(columns, 8)), dtype=self.dtype, device="cuda")[:, :columns]
+
+    def weight(self, array):
+        """A matrix on the device with padded row stride, or a vector; the padding is zero."""
+        torch = self.torch
+        tensor = torch.as_tensor(array).to("cuda").to(self.dtype)
+        if tensor.dim() < 2:
+            return tensor.contiguous()
+        out = torch.zeros((tensor.shape[0], round_up(tensor.shape[1], 8)), dtype=self.dtype, device="cuda")
+        out[:, : tensor.shape[1]] = tensor
+        return out[:, : tensor.shape[1]]
+
+    def linear(self, stream, out, x, weight, activation: int = 0) -> None:
+        m, k = x.shape
+        n = weight.shape[0]
+        if self.is_bf16:
+            self.call("singe_linear_bf16", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0), out.stride(0),
+                      activation, ks.HINT_STABLE_WEIGHTS)
+        else:
+            self.call("singe_linear_f32", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0), out.stride(0),
+                      activation)
+
+    def linear_f32_out(self, stream, out, x, weight) -> None:
+        """f32 results whatever the activation type (logits)."""
+        m, k = x.shape
+        n = weight.shape[0]
+        if self.is_bf16:
+            self.call("singe_matmul_bf16_f32", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0),
+                      out.stride(0), 0, 1)
+        else:
+            self.linear(stream, out, x, weight)
+
+    def head_linear(self, stream, out, x, weight, heads: int, gate=None) -> None:
+        """out[t, h] = x[t, h] . weight[h]^T (* sigmoid(gate[t, h])); x and out hold the heads side by side, weight stacks
+        them [heads, columns, reduction]."""
+        columns, reduction = weight.shape[1], weight.shape[2]
+        arguments = [stream, out, x, weight, x.shape[0], heads, columns, reduction, x.stride(0), x.shape[1] // heads,
+                     weight.stride(1), weight.stride(0) // weight.stride(1), out.stride(0), out.shape[1] // heads,
+                     gate, 0 if gate is None else gate.stride(0)]
+        if self.is_bf16:
+            arguments.append(ks.HINT_STABLE_WEIGHTS)
+        self.call(f"singe_head_linear_{self.suffix}", *arguments)
+
+    def add_layer_norm(self, stream, residual, delta, normed, weight, eps: float) -> None:
+        self.call(f"singe_add_layer_norm_{self.suffix}", stream, residual, delta,
+                  0 if delta is None else delta.stride(0), normed, 0 if normed is None else normed.stride(0), weight,
+                  residual.shape[0], residual.shape[1], eps)
+
+
+# ------------------------------------------------------------------------------------------------
+# one step's rows, as the mixers read them
+# ------------------------------------------------------------------------------------------------
+
+@dataclass
+class StepRows:
+    """Device inputs of a step.  int64: tokens, positions, pages, slots per packed row and the paging lists of the
+    Tensor-surface attention; int32: each sequence's first row, new tokens and earlier tokens, the block table, and the
+    rows that take the decode attention with the sequence and the number of visible keys of each."""
+    count: int
+    tokens: object
+    pages: object
+    slots: object
+    query_offsets: object
+    page_offsets: object
+    page_list: object
+    last_page_lengths: object
+    first: object
+    fresh_tokens: object
+    context: object
+    table: object
+    short_rows: object        # int32 [n], or None: row i of the step is query i
+    short_sequences: object
+    short_lens: object
+    short_count: int
+    longest: int              # most new tokens of any sequence
+    expanded: dict = field(default_factory=dict)   # window -> ExpandedRows of the longer sequences
+
+
+@dataclass
+class ExpandedRows:
+    """What the prompt attention reads for one window: the cache rows whose keys and values it needs, packed sequence by
+    sequence, and each sequence's lengths and offsets."""
+    gather: object
+    keys: int
+    lens_q: object
+    lens_kv: object
+    offsets_q: object
+    offsets_kv: object
+    sequences: int
+
+
+# ------------------------------------------------------------------------------------------------
+# mixers
+# ------------------------------------------------------------------------------------------------
+
+class LatentAttention:
+    """Weights of one latent-attention layer and its step.  ``source`` maps tensor names to arrays."""
+
+    def __init__(self, config: LatentAttentionConfig, source, ops: Ops, eps: float):
+        torch = ops.torch
+        self.config, self.ops, self.eps = config, ops, eps
+        c = config
+        take = lambda name: torch.as_tensor(source(name)).to("cuda").to(ops.dtype)
+        widest = max(c.dim, c.vdim)
+        # the tensor-core kernels: heads of a size the prompt attention has, latents the decode attention takes
+        self.tiled = ops.is_bf16 and widest <= EXPANDED_HEAD_SIZES[-1] and c.kv_rank <= ABSORBED_LATENT_LIMIT
+        if self.tiled:
+            self.key_size = self.value_size = next(size for size in EXPANDED_HEAD_SIZES if widest <= size)
+            self.latent = round_up(c.kv_rank, 64)
+        else:
+            unit = 8 if ops.is_bf16 else 1   # 16-byte rows for the bf16 GEMM
+            self.key_size, self.value_size = round_up(c.dim, unit), round_up(c.vdim, unit)
+            self.latent = round_up(c.kv_rank, unit)
+        self.down = ops.weight(torch.cat([take("dq"), take("dkv"), take("g")]))
+        self.q_norm, self.kv_norm = ops.weight(take("dq.norm")), ops.weight(take("dkv.norm"))
+        # every head's rows (or columns) padded to the head size, the latent's columns to the cache row
+        padded = lambda array, size: torch.nn.functional.pad(
+            array.reshape(c.heads, -1, array.shape[1]), (0, 0, 0, size - array.shape[0] // c.heads))
+        self.uq = ops.weight(padded(take("uq"), self.key_size).reshape(c.heads * self.key_size, c.q_rank))
+        pad_latent = lambda array: torch.nn.functional.pad(array, (0, self.latent - c.kv_rank))
+        uk, uv = pad_latent(padded(take("uk"), self.key_size)), pad_latent(padded(take("uv"), self.value_size))
+        self.absorb = uk.transpose(1, 2).contiguous()          # [heads, latent, key_size]
+        if self.tiled:                                         # [2 * heads * size, latent]: keys, then values
+            self.expand = torch.cat([uk, uv]).reshape(2 * c.heads * self.key_size, self.latent).contiguous()
+            self.uv = self.expand[c.heads * self.key_size:].view(c.heads, self.value_size, self.latent)
+        else:
+            self.expand, self.uv = None, uv.contiguous()
+        out = take("o")
+        out = torch.nn.functional.pad(out.reshape(out.shape[0], c.heads, c.vdim), (0, self.value_size - c.vdim))
+        self.out = ops.weight(out.reshape(out.shape[0], c.heads * self.value_size))
+
+    def new_cache(self, table: PageTable, sequences: int):
+        torch = self.ops.torch
+        return torch.zeros((table.page_count(), table.page_size, 1, self.latent), dtype=self.ops.dtype, device="cuda")
+
+    def scratch(self, rows: int, key_bound: int):
+        """Partial results of the split decode attention for ``rows`` queries over at most ``key_bound`` keys."""
+        if not self.tiled:
+            return None
+        torch, c = self.ops.torch, self.config
+        splits = int(ks.lib().singe_latent_decode_splits(rows, c.heads, min(key_bound, c.window)))
+        attn = torch.empty((rows, splits, c.heads, self.latent), dtype=torch.float32, device="cuda")
+        lse = torch.empty((rows, splits, c.heads), dtype=torch.float32, device="cuda")
+        return splits, attn, lse
+
+    def run(self, stream, step: StepRows, normed, cache, delta, status, scratch=None) -> None:
+        """delta = W_o of the gated heads' outputs for the rows of ``normed``."""
+        ops, c = self.ops, self.config
+        t = normed.shape[0]
+        pages, page_size = cache.shape[0], cache.shape[1]
+        projected = ops.rows(t, c.q_rank + c.kv_rank + c.heads)
+        ops.linear(stream, projected, normed, self.down)
+        latent_query = ops.rows(t, c.q_rank)
+        ops.call(f"singe_latent_norm_cache_write_{ops.suffix}", stream, latent_query, latent_query.stride(0), cache,
+                 self.latent, projected, projected.stride(0), self.q_norm, c.q_rank, self.kv_norm, c.kv_rank, step.pages,
+                 step.slots, t, pages, page_size, self.eps, status)
+        query = ops.rows(t, c.heads * self.key_size)
+        ops.linear(stream, query, latent_query, self.uq)
+        gate = projected[:, c.q_rank + c.kv_rank:]
+        attended = ops.rows(t, c.heads * self.value_size)
+        if not self.tiled:
+            self._general(stream, step, query, cache, gate, attended, status)
+        else:
+            if c.window in step.expanded:
+                self._expanded(stream, step.expanded[c.window], query, cache, gate, attended, status)
+            if step.short_count > 0:
+                self._absorbed(stream, step, query, cache, gate, attended, status, scratch)
+        ops.linear(stream, delta, attended, self.out)
+
+    def _general(self, stream, step, query, cache, gate, attended, status) -> None:
+        """Absorbed attention of every row on the general kernel: any sizes, either activation type."""
+        ops, c = self.ops, self.config
+        t = query.shape[0]
+        latent_queries, latents = ops.rows(t, c.heads * self.latent), ops.rows(t, c.heads * self.latent)
+        ops.head_linear(stream, latent_queries, query, self.absorb, c.heads)
+        lse = ops.torch.empty((t, c.heads), dtype=ops.torch.float32, device="cuda")
+        ops.call(f"singe_paged_attention_{ops.suffix}", stream, latents, lse, latent_queries, cache, cache,
+                 step.query_offsets, step.page_offsets, step.page_list, step.last_page_lengths, 8, t, c.heads, 1,
+                 self.latent, cache.shape[1], cache.shape[0], step.last_page_lengths.numel(), step.page_list.numel(),
+                 c.scale, 1, c.window, status)
+        ops.head_linear(stream, attended, latents, self.uv, c.heads, gate)
+
+    def _absorbed(self, stream, step, query, cache, gate, attended, status, scratch) -> None:
+        """Absorbed attention of the rows whose sequences have few new tokens."""
+        ops, c = self.ops, self.config
+        rows, n = step.short_rows, step.short_count
+        values = attended
+        if rows is not None:
+            query, gate = query.index_select(0, rows), gate.index_select(0, rows)
+            values = ops.rows(n, c.heads * self.value_size)
+        latent_queries, latents = ops.rows(n, c.heads * self.latent), ops.rows(n, c.heads * self.latent)
+        ops.head_linear(stream, latent_queries, query, self.absorb, c.heads)
+        splits, attn, lse = scratch or self.scratch(n, step.table.shape[1] * cache.shape[1])
+        ops.call("singe_latent_decode_bf16", stream, latents, attn, lse, latent_queries, cache, step.short_sequences,
+                 step.short_lens, step.table, n, c.heads, self.latent, cache.shape[1], cache.shape[0],
+                 step.table.shape[0], step.table.shape[1], c.window, splits, c.scale, status)
+        ops.head_linear(stream, values, latents, self.uv, c.heads, gate)
+        if rows is not None:
+            attended.index_copy_(0, rows, values)
+
+    def _expanded(self, stream, rows: ExpandedRows, query, cache, gate, attended, status) -> None:
+        ops, c, size = self.ops, self.config, self.key_size
+        torch = ops.torch
+        latents = torch.empty((rows.keys, self.latent), dtype=ops.dtype, device="cuda")
+        ops.call("singe_gather_rows", stream, latents, cache, rows.gather, rows.keys, self.latent * 2,
+                 cache.shape[0] * cache.shape[1], status)
+        keys_values = torch.empty((rows.keys, 2 * c.heads * size), dtype=ops.dtype, device="cuda")
+        ops.linear(stream, keys_values, latents, self.expand)
+        ops.call("singe_windowed_prefill_attention_bf16", stream, attended, query, keys_values,
+                 keys_values.data_ptr() + c.heads * size * 2, keys_values.stride(0), rows.lens_q, rows.lens_kv,
+                 rows.offsets_q, rows.offsets_kv, gate, gate.stride(0), rows.sequences, query.shape[0], rows.keys,
+                 c.heads, size, c.window, c.scale)
+
+
+class GatedLinear:
+    """Weights of one gated-linear-attention layer and its step."""
+
+    def __init__(self, config: GatedLinearConfig, source, ops: Ops, eps: float):
+        torch = ops.torch
+        self.config, self.ops, self.eps = config, ops, eps
+        take = lambda name: torch.as_tensor(source(name)).to("cuda").to(ops.dtype)
+        self.project = ops.weight(torch.cat([take("q"), take("k"), take("v"), take("g"), take("a1")]))
+        self.decay, self.bias, self.norm = take("a2").contiguous(), take("a2.b").contiguous(), take("norm").contiguous()
+        self.out = ops.weight(take("o"))
+
+    def new_cache(self, table: PageTable, sequences: int):
+        c = self.config
+        return self.ops.torch.zeros((sequences, c.heads, c.dim, c.vdim), dtype=self.ops.torch.float32, device="cuda")
+
+    def scratch(self, rows: int, key_bound: int):
+        return None
+
+    def run(self, stream, step: StepRows, normed, state, delta, status, scratch=None) -> None:
+        ops, c = self.ops, self.config
+        t = normed.shape[0]
+        projected = ops.rows(t, self.project.shape[0])
+        ops.linear(stream, projected, normed, self.project)
+        attended = ops.rows(t, c.heads * c.vdim)
+        shape = [attended, attended.stride(0), projected, projected.stride(0), self.decay, self.bias, self.norm, state,
+                 step.first, step.fresh_tokens, step.context, t, state.shape[0], c.heads, c.dim, c.vdim, c.rank, c.tau,
+                 c.dim ** -0.5, self.eps]
+        ops.call(f"singe_gated_linear_step_{ops.suffix}", stream, *shape, 0x7fffffff)
+        ops.linear(stream, delta, attended, self.out)
+
+
+MIXERS = {LatentAttentionConfig: LatentAttention, GatedLinearConfig: GatedLinear}
+
+
+# ------------------------------------------------------------------------------------------------
+# decoder
+# ------------------------------------------------------------------------------------------------
+
+@dataclass
+class _Layer:
+    mixer: object
+    norm1: object
+    norm2: object = None
+    up: object = None
+    down: object = None
+
+
+class HybridDecoder(PagedDecoder):
+    """The decoder: weights, caches and states, and its steps.  ``weights`` maps tensor names to arrays (what
+    ``singe_b200.checkpoint.load_hybrid`` returns); ``cache_tokens`` sizes a cache pool shared by the sequences
+    (default: room for every sequence's whole capacity)."""
+
+    def __init__(self, config: HybridConfig, sequences: int, capacity: int, weights: dict, dtype: str = "bfloat16",
+                 cache_tokens: int | None = None):
+        import torch
+
+        self.config = config
+        self.dtype = dtype
+        self.ops = ops = Ops(dtype)
+        whole = sequences * round_up(capacity, config.page_size)
+        table = PageTable.create_shared(sequences, capacity, config.page_size, cache_tokens or whole, config.window())
+        self._init_step_inputs(table, sequences, capacity, config.page_size)
+        take = lambda name: torch.as_tensor(weights[name])
+        built = {}
+        for index, layer in enumerate(config.layers):
+            if layer.weights_of is not None:
+                continue
+            prefix = f"l{index}."
+            mixer = MIXERS[type(layer.mixer)](layer.mixer, lambda name, p=prefix: take(p + "mix." + name), ops, config.eps)
+            built[index] = _Layer(mixer, ops.weight(take(prefix + "norm1")))
+            if layer.ffn:
+                built[index].norm2 = ops.weight(take(prefix + "norm2"))
+                built[index].up = ops.weight(take(prefix + "mlp.up"))
+                built[index].down = ops.weight(take(prefix + "mlp.down"))
+        self.layers = [built[config.owner(index)] for index in range(len(config.layers))]
+        self.caches = [layer.mixer.new_cache(table, sequences) for layer in self.layers]
+        self.embed = torch.as_tensor(weights["embed"]).to("cuda").to(ops.dtype).contiguous()
+        self.embed_norm, self.final_norm = ops.weight(take("embed.norm")), ops.weight(take("final.norm"))
+        self.head = ops.weight(take("head"))
+        # persistent inputs of the one-token step beyond those every decoder has
+        i32, i64 = torch.int32, torch.int64
+        zeros = lambda shape, kind: torch.zeros(shape, dtype=kind, device="cuda")
+        self.d_first = torch.arange(sequences, dtype=i32, device="cuda")
+        self.d_fresh = zeros(sequences, i32)
+        self.d_context = zeros(sequences, i32)
+        self.d_query_offsets = torch.arange(sequences + 1, dtype=i64, device="cuda")
+        self.d_page_offsets = zeros(sequences + 1, i64)
+        self.d_page_list = zeros(table.table_length(), i64)
+        self.d_last_lengths = zeros(sequences, i64)
+        self.logits = torch.empty((sequences, config.vocab), dtype=torch.float32, device="cuda")
+        self.scratches = {id(layer): layer.mixer.scratch(sequences, self.stride * config.page_size)
+                          for layer in built.values()}
+        self.decode_rows = StepRows(sequences, self.d_tokens, self.d_pages, self.d_slots, self.d_query_offsets,
+                                    self.d_page_offsets, self.d_page_list, self.d_last_lengths, self.d_first,
+                                    self.d_fresh, self.d_context, self.d_table, None, self.d_first, self.d_lens,
+                                    sequences, 1)
+        self.trail = None   # set to a list to collect the residual stream after every layer (for inspection)
+
+    # ---- the layers, over a step of any shape ----
+
+    def _layers(self, rows: StepRows, scratches):
+        """Runs the layers; returns the final norm's output for the step's rows."""
+        torch, ops, c = self.torch, self.ops, self.config
+        stream = self._stream()
+        t = rows.count
+        residual = torch.empty((t, c.width), dtype=torch.float32, device="cuda")
+        normed, delta = ops.rows(t, c.width), ops.rows(t, c.width)
+        ops.call(f"singe_embedding_layer_norm_{ops.suffix}", stream, residual, self.embed, rows.tokens, self.embed_norm, t,
+                 c.width, c.vocab, c.eps, self.status)
+        pending = None   # the sublayer output not yet added to the residual
+        for layer, cache in zip(self.layers, self.caches):
+            ops.add_layer_norm(stream, residual, pending, normed, layer.norm1, c.eps)
+            layer.mixer.run(stream, rows, normed, cache, delta, self.status, scratches.get(id(layer)))
+            pending = delta
+            if layer.up is not None:
+                ops.add_layer_norm(stream, residual, pending, normed, layer.norm2, c.eps)
+                inner = ops.rows(t, layer.up.shape[0])
+                ops.linear(stream, inner, normed, layer.up, activation=2)
+                ops.linear(stream, delta, inner, layer.down)
+            if self.trail is not None:
+                self.trail.append(residual + delta.float())
+        ops.add_layer_norm(stream, residual, pending, normed, self.final_norm, c.eps)
+        return normed
+
+    def forward(self) -> None:
+        """One token per sequence, from the persistent step inputs; idle rows have nothing in ``d_fresh``."""
+        stream = self._stream()
+        normed = self._layers(self.decode_rows, self.scratches)
+        self.ops.linear_f32_out(stream, self.logits, normed, self.head)
+        self.ops.call("singe_argmax_f32", stream, self.best_value, self.next_tokens, self.logits, self.logits.stride(0),
+                      self.sequences, self.config.vocab, 0)
+
+    def _plan_lists(self, tokens):
+        step = super()._plan_lists(tokens)
+        torch = self.torch
+        to = lambda target, array: target.copy_(torch.from_numpy(np.ascontiguousarray(array)))
+        to(self.d_fresh, step.real_tokens.astype(np.int32))
+        to(self.d_context, (np.asarray(self.table.lengths) - step.real_tokens).astype(np.int32))
+        to(self.d_page_offsets, step.page_offsets)
+        to(self.d_page_list, step.pages)
+        to(self.d_last_lengths, step.last_page_lengths)
+        return step
+
+    def capture(self) -> None:
+        """The captured step must not leave anything behind: it is recorded with every row idle."""
+        self.d_pages.fill_(self.table.scratch_page)
+        for idle in (self.d_tokens, self.d_slots, self.d_lens, self.d_fresh):
+            idle.zero_()
+        super().capture()
+
+    def step_tokens(self, tokens, want=None):
+        """Extends each sequence with its ``tokens`` (an empty list leaves a row idle) and returns the logits of each
+        sequence's last token, f32 [sequences, vocab]; with ``want`` (one list of places among its new tokens per
+        sequence) the logits of those tokens, [wanted, vocab], in that order.  A step that cannot get its pages raises
+        before anything changed."""
+        torch = self.torch
+        tokens = [[int(v) for v in t] for t in tokens]
+        if all(len(t) <= 1 for t in tokens):
+            step = self._plan_lists(tokens)
+            self.run()
+            return self.logits if want is None else self.logits[torch.from_numpy(step.wanted_rows(want)).cuda()]
+        step = self.table.step(tokens)
+        rows = self._upload(step)
+        normed = self._layers(rows, {})
+        picked = step.last_rows if want is None else step.wanted_rows(want)
+        logits = torch.empty((len(picked), self.config.vocab), dtype=torch.float32, device="cuda")
+        if len(picked) > 0:
+            last = self.ops.rows(len(picked), self.config.width)
+            last.copy_(normed.index_select(0, torch.from_numpy(picked).cuda()))
+            self.ops.linear_f32_out(self._stream(), logits, last, self.head)
+        return logits
+
+    def _upload(self, step) -> StepRows:
+        """The device inputs of a step of any shape: two copies, one per integer width."""
+        torch, c = self.torch, self.config
+        table = self.table
+        lengths = np.asarray(table.lengths, dtype=np.int64)
+        fresh = step.real_tokens
+        context = lengths - fresh
+        first = step.query_offsets[:-1]
+        page_counts = np.asarray([max(len(held), 1) for held in table.pages])
+        block_table = np.full((self.sequences, int(page_counts.max())), table.scratch_page, dtype=np.int64)
+        for b, held in enumerate(table.pages):
+            block_table[b, : len(held)] = held
+        few = fresh <= FEW_TOKENS
+        short = np.nonzero(few[step.sequence_ids])[0]
+        sequences = step.sequence_ids[short]
+        lens = np.where(fresh[sequences] > 0, step.positions[short] + 1, 0)
+        narrow = {"first": first, "fresh": fresh, "context": context, "table": block_table.reshape(-1),
+                  "short_sequences": sequences, "short_lens": lens}
+        long = np.nonzero(~few)[0]
+        windows = sorted({layer.mixer.window for layer in c.layers if isinstance(layer.mixer, LatentAttentionConfig)})
+        for window in windows if len(long) else []:
+            start = np.maximum(context[long] - window + 1, 0)
+            lens_kv = lengths[long] - start
+            gather = [block_table[b, np.arange(s, lengths[b]) // c.page_size] * c.page_size
+                      + np.arange(s, lengths[b]) % c.page_size for b, s in zip(long, start)]
+            narrow.update({f"gather{window}": np.concatenate(gather), f"lens_q{window}": fresh[long],
+                           f"lens_kv{window}": lens_kv, f"offsets_q{window}": first[long],
+                           f"offsets_kv{window}": np.cumsum(lens_kv) - lens_kv})
+        wide = {"tokens": step.tokens, "pages": step.write_pages, "slots": step.write_slots,
+                "query_offsets": step.query_offsets, "page_offsets": step.page_offsets, "page_list": step.pages,
+                "last": step.last_page_lengths, "short_rows": short}
+        w, n = self._send(wide, np.int64), self._send(narrow, np.int32)
+        expanded = {}
+        for window in windows if len(long) else []:
+            part = lambda name: n[f"{name}{window}"]
+            expanded[window] = ExpandedRows(part("gather"), part("gather").numel(), part("lens_q"), part("lens_kv"),
+                                            part("offsets_q"), part("offsets_kv"), len(long))
+        everything = len(short) == len(step.tokens)
+        return StepRows(len(step.tokens), w["tokens"], w["pages"], w["slots"], w["query_offsets"], w["page_offsets"],
+                        w["page_list"], w["last"], n["first"], n["fresh"], n["context"],
+                        n["table"].view(block_table.shape), None if everything else w["short_rows"],
+                        n["short_sequences"], n["short_lens"], len(short), int(fresh.max()), expanded)
+
+    def _send(self, arrays: dict, kind) -> dict:
+        torch = self.torch
+        sizes = [len(array) for array in arrays.values()]
+        starts = np.cumsum([0] + [round_up(size, 4) for size in sizes])
+        packed = np.zeros(int(starts[-1]), dtype=kind)
+        for (start, size), array in zip(zip(starts, sizes), arrays.values()):
+            packed[start: start + size] = array
+        sent = torch.from_numpy(packed).cuda()
+        return {name: sent[start: start + size] for name, start, size in zip(arrays, starts, sizes)}

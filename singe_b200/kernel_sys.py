@@ -115,6 +115,21 @@ SIGNATURES = {
     "singe_peer_buffer_destroy": [_p],
     "singe_allreduce_add_rms_norm_bf16": [_p, _p, _p, _p, _p, _p, _p, _i, _i, _z, _z, _f, _p],
     "singe_allreduce_two_phase_add_rms_norm_bf16": [_p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _z, _z, _f, _i, _p],
+    "singe_embedding_layer_norm_bf16": [_p, _p, _p, _p, _p, _z, _z, _z, _f, _p],
+    "singe_embedding_layer_norm_f32": [_p, _p, _p, _p, _p, _z, _z, _z, _f, _p],
+    "singe_add_layer_norm_bf16": [_p, _p, _p, _z, _p, _z, _p, _z, _z, _f],
+    "singe_add_layer_norm_f32": [_p, _p, _p, _z, _p, _z, _p, _z, _z, _f],
+    "singe_latent_norm_cache_write_bf16": [_p, _p, _z, _p, _z, _p, _z, _p, _z, _p, _z, _p, _p, _z, _z, _z, _f, _p],
+    "singe_latent_norm_cache_write_f32": [_p, _p, _z, _p, _z, _p, _z, _p, _z, _p, _z, _p, _p, _z, _z, _z, _f, _p],
+    "singe_gather_rows": [_p, _p, _p, _p, _z, _z, _z, _p],
+    "singe_argmax_f32": [_p, _p, _p, _p, _z, _z, _z, ctypes.c_int64],
+    "singe_linear_f32": [_p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _i],
+    "singe_head_linear_bf16": [_p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _z, _z, _z, _z, _p, _z, ctypes.c_uint],
+    "singe_head_linear_f32": [_p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _z, _z, _z, _z, _p, _z],
+    "singe_gated_linear_step_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _f, _f, _f,
+                                     _z],
+    "singe_gated_linear_step_f32": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _f, _f, _f,
+                                    _z],
 }
 
 _RESTYPES = {

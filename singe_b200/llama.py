@@ -1,6 +1,6 @@
 """Llama-shaped decode step over the C-ABI kernels, tensor-parallel across the GPUs of one box.
 
-Host-side mirror of the reference's decode path: ``PageTable``/``DecodeStep`` (singe/src/nn/decode/step.rs),
+Host-side mirror of the reference's decode path (``PageTable`` and the step's inputs are in ``singe_b200.decoder``):
 ``RotaryTable`` (singe/src/nn/layers/positional/rotary.rs:166-219), the pre-norm block
 (singe/src/nn/layers/blocks/mod.rs:56-83: ``h += o(attn(norm h))``, ``h += down(silu(gate(norm h)) * up(norm h))``),
 ``GroupedQueryAttention::decode`` (singe/src/nn/layers/attention/grouped.rs:92-115) and
@@ -18,184 +18,12 @@ torch supplies device buffers, streams, CUDA graphs and ``torch.distributed``; e
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass, field
+from dataclasses import dataclass
 
 import numpy as np
 
 from . import kernel_sys as ks
-
-
-# ------------------------------------------------------------------------------------------------
-# PageTable: singe/src/nn/decode/step.rs:131-475 (pure host integer planning)
-# ------------------------------------------------------------------------------------------------
-
-class PageTableError(ValueError):
-    pass
-
-
-@dataclass
-class DecodeStep:
-    """The paging tensors of one step (singe/src/nn/decode/step.rs:13-30), as int64 numpy arrays."""
-    tokens: np.ndarray
-    positions: np.ndarray
-    write_pages: np.ndarray
-    write_slots: np.ndarray
-    query_offsets: np.ndarray
-    page_offsets: np.ndarray
-    pages: np.ndarray
-    last_page_lengths: np.ndarray
-    last_rows: np.ndarray
-    real_tokens: np.ndarray
-    sequence_ids: np.ndarray
-
-
-class PageTable:
-    """Hands out cache pages to sequences in increasing order from page zero and writes each step's paging
-    tensors.  After the pages sequences can hold comes one scratch page that held/idle rows and padding write."""
-
-    def __init__(self, sequences: int, capacity: int, page_size: int, pool: int):
-        self.page_size = page_size
-        self.capacity = capacity
-        self.pool = pool
-        self.padding = 0
-        self.free: list[int] = []
-        self.pages: list[list[int]] = [[] for _ in range(sequences)]
-        self.lengths: list[int] = [0] * sequences
-        self.reset()
-
-    @classmethod
-    def create(cls, sequences: int, capacity: int, page_size: int) -> "PageTable":
-        if sequences == 0 or capacity <= 0 or page_size <= 0:
-            raise PageTableError("page table size")
-        return cls(sequences, capacity, page_size, sequences * ((capacity - 1) // page_size + 1))
-
-    @classmethod
-    def create_shared(cls, sequences: int, capacity: int, page_size: int, cache_tokens: int) -> "PageTable":
-        if sequences == 0 or capacity <= 0 or page_size <= 0 or cache_tokens <= 0:
-            raise PageTableError("page table size")
-        return cls(sequences, capacity, page_size, (cache_tokens - 1) // page_size + 1)
-
-    def with_padding(self, padding: int) -> "PageTable":
-        self.padding = padding
-        return self
-
-    def reset(self) -> None:
-        self.free = list(range(self.pool - 1, -1, -1))
-        self.pages = [[] for _ in self.pages]
-        self.lengths = [0] * len(self.lengths)
-
-    def release(self, sequence: int) -> None:
-        if not 0 <= sequence < len(self.pages):
-            raise PageTableError("decoder sequence")
-        self.free.extend(reversed(self.pages[sequence]))
-        self.pages[sequence] = []
-        self.lengths[sequence] = 0
-
-    def free_pages(self) -> int:
-        return len(self.free)
-
-    def page_count(self) -> int:
-        return self.pool + 1
-
-    @property
-    def scratch_page(self) -> int:
-        return self.pool
-
-    def table_length(self) -> int:
-        return self.pool + len(self.pages) + (self.padding + self.page_size - 1) // self.page_size
-
-    @staticmethod
-    def step_tokens(tokens) -> int:
-        return sum(max(len(t), 1) for t in tokens)
-
-    def step(self, tokens) -> DecodeStep:
-        return self.step_padded(tokens, self.step_tokens(tokens))
-
-    def step_padded(self, tokens, total: int) -> DecodeStep:
-        sequences = len(self.pages)
-        if len(tokens) != sequences or all(len(t) == 0 for t in tokens):
-            raise PageTableError("decode step needs a slice for every sequence, and tokens in one")
-        padding = total - self.step_tokens(tokens)
-        if padding < 0:
-            raise PageTableError("a decode step is padded to fewer rows than it has")
-        if padding > self.padding:
-            raise PageTableError("a decode step is padded past what its page table allows")
-        padded = max(i for i, t in enumerate(tokens) if len(t) > 0)
-        for length, t in zip(self.lengths, tokens):
-            if length + len(t) > self.capacity:
-                raise PageTableError("decoder cache capacity")
-        fresh = 0
-        for length, held, t in zip(self.lengths, self.pages, tokens):
-            if len(t) > 0:
-                end = length + len(t)
-                fresh += max((end - 1) // self.page_size + 1 - len(held), 0)
-        if fresh > len(self.free):
-            raise PageTableError("decoder cache pages")
-
-        flat, positions, write_pages, write_slots = [], [], [], []
-        query_offsets, last_rows, real_tokens, sequence_ids, visible = [0], [], [], [], []
-        for row, t in enumerate(tokens):
-            held = self.pages[row]
-            for token in t:
-                position = self.lengths[row]
-                page = position // self.page_size
-                if page == len(held):
-                    held.append(self.free.pop())
-                flat.append(int(token))
-                positions.append(position)
-                write_pages.append(held[page])
-                write_slots.append(position % self.page_size)
-                self.lengths[row] += 1
-            if len(t) == 0:
-                flat.append(0)
-                positions.append(min(self.lengths[row], self.capacity - 1))
-                write_pages.append(self.pool)
-                write_slots.append(0)
-            last = len(flat) - 1
-            keys = self.lengths[row]
-            if row == padded:
-                for position in range(self.lengths[row], self.lengths[row] + padding):
-                    flat.append(0)
-                    positions.append(min(position, self.capacity - 1))
-                    write_pages.append(self.pool)
-                    write_slots.append(position % self.page_size)
-                keys += padding
-            visible.append(keys)
-            sequence_ids.extend([row] * (len(flat) - len(sequence_ids)))
-            query_offsets.append(len(flat))
-            last_rows.append(last)
-            real_tokens.append(len(t))
-
-        pages, page_offsets, last_page_lengths = [], [0], []
-        for held, seen in zip(self.pages, visible):
-            if seen == 0:
-                pages.append(self.pool)
-                last_page_lengths.append(1)
-            else:
-                used = (seen - 1) // self.page_size + 1
-                kept = min(used, len(held))
-                pages.extend(held[:kept])
-                pages.extend([self.pool] * (used - kept))
-                last_page_lengths.append((seen - 1) % self.page_size + 1)
-            page_offsets.append(len(pages))
-        pages.extend([0] * (self.table_length() - len(pages)))
-        as_array = lambda values: np.asarray(values, dtype=np.int64)
-        return DecodeStep(as_array(flat), as_array(positions), as_array(write_pages), as_array(write_slots),
-                          as_array(query_offsets), as_array(page_offsets), as_array(pages),
-                          as_array(last_page_lengths), as_array(last_rows), as_array(real_tokens),
-                          as_array(sequence_ids))
-
-    def place_prompts(self, lengths) -> None:
-        """Advances every sequence by ``lengths[b]`` tokens without building step tensors (bulk prompt placement)."""
-        for row, count in enumerate(lengths):
-            if self.lengths[row] + count > self.capacity:
-                raise PageTableError("decoder cache capacity")
-            need = (self.lengths[row] + count - 1) // self.page_size + 1 - len(self.pages[row]) if count > 0 else 0
-            if need > len(self.free):
-                raise PageTableError("decoder cache pages")
-            for _ in range(max(need, 0)):
-                self.pages[row].append(self.free.pop())
-            self.lengths[row] += count
+from .decoder import CachedDecoder, DecodeStep, PagedDecoder, PageTable, PageTableError  # noqa: F401 (one import for users)
 
 
 # ------------------------------------------------------------------------------------------------
@@ -295,7 +123,7 @@ def shard_layer_weights(full: dict, config: LlamaConfig, shard: Shard, interleav
 PEER_ONE_SHOT_UP_TO = 4
 
 
-class LlamaDecoder:
+class LlamaDecoder(PagedDecoder):
     """One rank of a tensor-parallel Llama decoder: weights, KV caches, page table and the decode step."""
 
     def __init__(self, config: LlamaConfig, sequences: int, capacity: int, shard: Shard | None = None, seed: int = 4,
@@ -304,12 +132,10 @@ class LlamaDecoder:
                  fold_in_kernel: bool = False, fuse_attention: bool = True):
         import torch
 
-        self.torch = torch
         self.config = config
         self.shard = shard or Shard()
-        self.sequences = sequences
-        self.capacity = capacity
-        self.table = PageTable.create(sequences, capacity, config.page_size)
+        self._init_step_inputs(PageTable.create(sequences, capacity, config.page_size), sequences, capacity,
+                               config.page_size)
         self.shard_lm_head = shard_lm_head and self.shard.world > 1
         tp = self.shard.world
         if config.heads % tp or config.kv_heads % tp or config.ffn % tp:
@@ -352,18 +178,9 @@ class LlamaDecoder:
         shape = (pages, config.page_size, self.kv_heads, config.head_dim)
         self.key_caches = [torch.zeros(shape, dtype=bf16, device=dev) for _ in range(config.layers)]
         self.value_caches = [torch.zeros(shape, dtype=bf16, device=dev) for _ in range(config.layers)]
-        # persistent step buffers (device) and their pinned host mirrors
+        # persistent step buffers (device)
         t = sequences
-        self.stride = (capacity + config.page_size - 1) // config.page_size
         i64, i32 = torch.int64, torch.int32
-        self.d_tokens = torch.zeros(t, dtype=i64, device=dev)
-        self.d_positions = torch.zeros(t, dtype=i64, device=dev)
-        self.d_pages = torch.zeros(t, dtype=i64, device=dev)
-        self.d_slots = torch.zeros(t, dtype=i64, device=dev)
-        self.d_lens = torch.zeros(t, dtype=i32, device=dev)
-        self.d_table = torch.zeros((t, self.stride), dtype=i32, device=dev)
-        self.h_table = np.zeros((t, self.stride), dtype=np.uint32)
-        self.status = torch.zeros(1, dtype=i32, device=dev)
         w = config.hidden
         self.hidden = torch.empty((t, w), dtype=bf16, device=dev)
         self.normed = torch.empty((t, w), dtype=bf16, device=dev)
@@ -395,9 +212,6 @@ class LlamaDecoder:
         self.gate_up = torch.empty((t, 2 * self.ffn), dtype=bf16, device=dev)
         self.activated = torch.empty((t, self.ffn), dtype=bf16, device=dev)
         self.logits = torch.empty((t, self.lm_head.shape[0]), dtype=bf16, device=dev)
-        self.best_value = torch.empty(t, dtype=torch.float32, device=dev)
-        self.best_index = torch.empty(t, dtype=i64, device=dev)
-        self.next_tokens = torch.empty(t, dtype=i64, device=dev)
         if self.shard_lm_head:
             self.all_values = torch.empty((tp, t), dtype=torch.float32, device=dev)
             self.all_indices = torch.empty((tp, t), dtype=i64, device=dev)
@@ -419,7 +233,6 @@ class LlamaDecoder:
         sms = torch.cuda.get_device_properties(0).multi_processor_count
         self.tickets = (torch.zeros(t * self.kv_heads, dtype=i32, device=dev)
                         if fold_in_kernel and t * self.kv_heads * max_splits <= 3 * sms else None)
-        self.graph = None
 
     def _device(self, array):
         torch = self.torch
@@ -439,34 +252,13 @@ class LlamaDecoder:
             cache.copy_(torch.randn(cache.shape, generator=generator, device="cuda").to(torch.bfloat16))
         self._refresh_block_table()
 
-    def _refresh_block_table(self) -> None:
-        for b, held in enumerate(self.table.pages):
-            self.h_table[b, : len(held)] = held
-        self.d_table.copy_(self.torch.from_numpy(self.h_table.view(np.int32)))
-
     # ---- the step ----
-
-    def plan(self, tokens) -> DecodeStep:
-        """One token per sequence -> the step's paging tensors, uploaded into the persistent device buffers."""
-        torch = self.torch
-        step = self.table.step([[int(t)] for t in tokens])
-        self._refresh_block_table()
-        self.d_tokens.copy_(torch.from_numpy(step.tokens))
-        self.d_positions.copy_(torch.from_numpy(step.positions))
-        self.d_pages.copy_(torch.from_numpy(step.write_pages))
-        self.d_slots.copy_(torch.from_numpy(step.write_slots))
-        self.d_lens.copy_(torch.from_numpy((step.positions + 1).astype(np.int32)))
-        return step
 
     def _warm(self, weight) -> None:
         """Attaches (the first part of) a weight matrix to the next launch as an L2 warm-ahead range."""
         if self.warm_bytes > 0:
             size = min(weight.numel() * weight.element_size(), self.warm_bytes)
             self._check(ks.lib().singe_warm_l2_with_next_launch(weight.data_ptr(), size), "warm")
-
-    def _check(self, code: int, where: str) -> None:
-        if code != ks.OK:
-            raise RuntimeError(f"{where}: status {code} ({ks.status_string(code)})")
 
     def _linear(self, out, x, weight, stream) -> None:
         m, k = x.shape
@@ -592,17 +384,19 @@ class LlamaDecoder:
 
     # ---- steps of any shape: prompts, prompt chunks behind a context, idle rows ----
 
-    def step_tokens(self, tokens):
+    def step_tokens(self, tokens, want=None):
         """Extends each sequence with its ``tokens`` (an empty list leaves a row idle) and returns the logits of each
         sequence's last token, [sequences, vocab] -- ``Decoder::step`` of the reference (singe/src/generation/mod.rs:25-36,
         ``CachedDecoder::step`` :715-744).  A step of one token per sequence takes the decode path (``step``); anything
         else is a prompt step: every new token's K/V go into the cache first, then the packed causal prefill kernel
         attends each sequence's new tokens over all of its cached keys (``causal = 2``: the queries are the sequence's
-        last tokens).  A step that cannot get its pages raises before anything changed."""
+        last tokens).  A step that cannot get its pages raises before anything changed.  ``want`` (one list of places among
+        its new tokens per sequence) asks for the logits of those tokens instead, [wanted, vocab] in that order."""
         torch, lib, c = self.torch, ks.lib(), self.config
         if all(len(t) == 1 for t in tokens):
             self.step([t[0] for t in tokens])
-            return self._full_logits(self.logits)
+            logits = self._full_logits(self.logits)
+            return logits if want is None else logits[[row for row, places in enumerate(want) for _ in places]]
         step = self.table.step([[int(v) for v in t] for t in tokens])
         stream = int(torch.cuda.current_stream().cuda_stream)
         dev, bf16 = "cuda", torch.bfloat16
@@ -620,7 +414,8 @@ class LlamaDecoder:
         d_lens_q, d_lens_kv = to_device(lens_q, torch.int32), to_device(lens_kv, torch.int32)
         d_offsets = to_device(step.query_offsets[:-1].astype(np.int32), torch.int32)
         d_table = to_device(table.view(np.int32), torch.int32)
-        d_last = to_device(step.last_rows, torch.int64)
+        rows = step.last_rows if want is None else step.wanted_rows(want)
+        d_last = to_device(rows, torch.int64)
         status = self.status.data_ptr()
         hidden = torch.empty((t, w), dtype=bf16, device=dev)
         normed = torch.empty((t, w), dtype=bf16, device=dev)
@@ -668,8 +463,10 @@ class LlamaDecoder:
             delta = projected
         self._check(lib.singe_add_rms_norm_bf16(stream, hidden.data_ptr(), delta.data_ptr(), normed.data_ptr(),
                                                 self.final_norm.data_ptr(), t, w, c.eps), "final norm")
+        if len(rows) == 0:
+            return torch.empty((0, c.vocab), dtype=bf16, device=dev)
         last = normed.index_select(0, d_last).contiguous()   # CausalLm::forward_embedded keeps the last rows only
-        logits = torch.empty((s, self.lm_head.shape[0]), dtype=bf16, device=dev)
+        logits = torch.empty((len(rows), self.lm_head.shape[0]), dtype=bf16, device=dev)
         self._linear(logits, last, self.lm_head, stream)
         return self._full_logits(logits)
 
@@ -681,57 +478,6 @@ class LlamaDecoder:
         pieces = [torch.empty_like(logits) for _ in range(self.shard.world)]
         self.shard.group.all_gather(pieces, logits.contiguous())
         return torch.cat(pieces, dim=1)
-
-    def capture(self) -> None:
-        """Captures ``forward`` into a CUDA graph that later steps replay (the reference replays a captured
-        step the same way, singe/src/generation/mod.rs:529-579)."""
-        torch = self.torch
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            self.forward()  # warm-up outside capture: loads modules, sizes nothing (all buffers are preallocated)
-        torch.cuda.current_stream().wait_stream(side)
-        torch.cuda.synchronize()
-        self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph):
-            self.forward()
-
-    def step(self, tokens) -> "object":
-        """Plans and runs one decode step; returns the device tensor of greedy next tokens [sequences]."""
-        self.plan(tokens)
-        if self.graph is not None:
-            self.graph.replay()
-        else:
-            self.forward()
-        return self.next_tokens
-
-
-class CachedDecoder:
-    """``LlamaDecoder`` behind the reference's ``Decoder`` trait (singe/src/generation/mod.rs:25-52), which is what
-    ``singe_b200.generation`` drives: ``sequences()``, ``step(tokens)``, ``reset()``, ``release(row)``,
-    ``largest_chunk()``.  Prompt steps read at most the largest prompt chunk of extra tokens (16, 64, 256, ... 1024,
-    ``PromptChunks``, :367-417)."""
-
-    def __init__(self, model: LlamaDecoder, prompt_chunks=None):
-        from .generation import PromptChunks
-
-        self.model = model
-        self.chunks = (prompt_chunks or PromptChunks.STANDARD).sizes(model.capacity)
-
-    def sequences(self) -> int:
-        return self.model.sequences
-
-    def step(self, tokens):
-        return self.model.step_tokens(tokens)
-
-    def reset(self) -> None:
-        self.model.table.reset()
-
-    def release(self, sequence: int) -> None:
-        self.model.table.release(sequence)
-
-    def largest_chunk(self):
-        return self.chunks[-1] if self.chunks else 0
 
 
 def random_weights(config: LlamaConfig, seed: int = 4) -> dict:
