@@ -656,6 +656,32 @@ int singe_head_linear_f32(singe_stream_t stream, float *out, const float *x, con
                           size_t weight_row_stride, size_t weight_head_rows, size_t out_row_stride,
                           size_t out_head_stride, const float *gate, size_t gate_row_stride);
 
+/* Attention of few query rows over a latent cache [pages, page_size, latent] shared by all heads: the cached rows are
+ * keys and values at once.  Query i belongs to sequence sequence_of[i] (a row of block_table [sequences, table_stride])
+ * and sees its keys max(0, lens[i] - window) .. lens[i] - 1 (window == 0: from 0; lens[i] == 0: zeros).
+ * query, out [queries, heads, latent] bf16; attn_scratch f32 [queries, splits, heads, latent] and lse_scratch
+ * [queries, splits, heads].  latent: a multiple of 64 up to 512.  Page ids outside the cache set *status = 1. */
+int singe_latent_decode_bf16(singe_stream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                             const void *cache, const int32_t *sequence_of, const int32_t *lens,
+                             const int32_t *block_table, size_t queries, size_t heads, size_t latent, size_t page_size,
+                             size_t pages, size_t sequences, size_t table_stride, size_t window, size_t splits,
+                             float scale, uint32_t *status);
+/* The split count that fills the machine for a call of this shape. */
+size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t key_bound);
+
+/* Causal prompt attention with a sliding window on the tensor core (the kernel of singe_ragged_kv_prefill_attention_bf16):
+ * query, out [total_query_tokens, heads, head_dim]; key and value rows of kv_row_stride elements, heads side by side.
+ * Sequence b owns query rows [offsets_q[b], offsets_q[b] + lens_q[b]) and key rows [offsets_kv[b], ...+ lens_kv[b]); the
+ * queries are the sequence's last tokens, and a query sees itself and the window - 1 tokens before it.  gate != NULL: row t
+ * of head h is multiplied by sigmoid(gate[t * gate_row_stride + h]).  lse [total_query_tokens, heads], natural log.
+ * head_dim 64 or 128. */
+int singe_windowed_prefill_attention_bf16(singe_stream_t stream, void *out, float *lse, const void *query,
+                                          const void *key, const void *value, size_t kv_row_stride, const int32_t *lens_q,
+                                          const int32_t *lens_kv, const int32_t *offsets_q, const int32_t *offsets_kv,
+                                          const void *gate, size_t gate_row_stride, size_t batch,
+                                          size_t total_query_tokens, size_t total_kv_tokens, size_t heads,
+                                          size_t head_dim, size_t window, float scale);
+
 /* Gated linear attention, one head's state S [dim, vdim] in f32 per sequence:
  *   S_t = diag(sigmoid(z_t)^(1/tau)) S_(t-1) + k_t v_t^T,  o_t = query_scale * S_t^T q_t,  z_t = decay_weight a_t + decay_bias,
  *   out = rms_norm(o_t) * norm_weight * silu(g_t)

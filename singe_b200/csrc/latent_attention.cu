@@ -1,0 +1,400 @@
+// Attention of few query rows (a decode step) over a paged latent cache: one cached row of `latent` bf16 per token serves
+// every head as key and as value,
+//     score[h, j] = scale * q[h] . c[j],   out[h] = sum_j softmax(score[h])_j c[j],
+// with q already multiplied into the latent space.  A sliding window bounds the keys of a query.
+//
+// The cache is the traffic: a tile of 64 cached rows is read from HBM once for up to 32 heads and used twice, as keys and
+// as values.  One CTA per (query, split of its keys, 32 heads), one warp per 64 columns of the latent:
+//   load      a warp copies its own 64-column slice of the tile (cp.async, two tiles in flight) and is the only reader of it
+//   scores    its share of q . c over its 64 columns (q stays in registers), f32 partials to shared memory
+//   softmax   partials of all warps summed, f32 online softmax, weights to shared memory as bf16
+//   values    weights x its slice into f32 accumulators [heads, 64]
+// mma.sync m16n8k16: at 32 heads the tile costs about 64 flops per byte read, well under what HBM leaves room for.
+// With more than one split the normalised partial and its log-sum-exp (base 2) go to scratch and a second kernel folds them.
+#include "common.cuh"
+
+namespace singe {
+namespace {
+
+constexpr int kTileKeys = 64;
+constexpr int kSlice = 64;                        // latent columns of one warp
+constexpr int kSliceBytes = kTileKeys * kSlice * 2;
+constexpr int kScoreStride = kTileKeys + 8;       // floats; spreads the fragment stores over the banks
+constexpr int kWeightStride = kTileKeys + 8;      // bf16
+constexpr int kLatentStages = 2;
+constexpr int kMaxLatent = 512;
+
+struct LatentDecode {
+    __nv_bfloat16 *out;
+    float *attn;  // [queries, splits, heads, latent]
+    float *lse;   // [queries, splits, heads]
+    const __nv_bfloat16 *query;
+    const __nv_bfloat16 *cache;
+    const int32_t *sequence_of, *lens, *table;
+    int heads, latent, page_size, pages, sequences, table_stride, window, splits;
+    float scale_log2;
+    uint32_t *status;
+};
+
+__device__ __forceinline__ void copy_async_16(uint32_t target, const void *source, bool valid) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(target), "l"(source), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void copy_async_wait() {
+    asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
+}
+
+// Byte offset of 16-byte piece `piece` of key row `key` in a slice: pieces are permuted within a row so that eight rows
+// read at one piece position touch all banks.
+__device__ __forceinline__ uint32_t slice_at(int key, int piece) {
+    return static_cast<uint32_t>(key * 128 + ((piece ^ (key & 7)) << 4));
+}
+
+int latent_shared_bytes(int warps, int head_tiles) {
+    return kLatentStages * warps * kSliceBytes + warps * head_tiles * 16 * kScoreStride * 4 +
+           head_tiles * 16 * kWeightStride * 2 + 3 * head_tiles * 16 * 4;
+}
+
+template <int MT>  // 16-head tiles of a CTA
+__global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentDecode p) {
+    constexpr int kHeads = MT * 16;
+    grid_launch_dependents();
+    grid_dependency_wait();
+    extern __shared__ __align__(128) uint8_t shared[];
+    const int warps = blockDim.x >> 5;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int g = lane >> 2, q2 = (lane & 3) * 2;  // fragment row and column pair
+    uint8_t *tiles = shared;
+    float *scores = reinterpret_cast<float *>(shared + kLatentStages * warps * kSliceBytes);  // [warps][kHeads][stride]
+    __nv_bfloat16 *weights = reinterpret_cast<__nv_bfloat16 *>(scores + warps * kHeads * kScoreStride);
+    float *row_max = reinterpret_cast<float *>(weights + kHeads * kWeightStride);
+    float *row_sum = row_max + kHeads;
+    float *row_factor = row_sum + kHeads;
+
+    const int query = blockIdx.x, split = blockIdx.y, head0 = blockIdx.z * kHeads;
+    const int sequence = p.sequence_of[query];
+    const bool known = sequence >= 0 && sequence < p.sequences;
+    if (!known && threadIdx.x == 0) report_status(p.status, kStatusIndexOutOfBounds);
+    const int end_all = known ? min(p.lens[query], p.table_stride * p.page_size) : 0;
+    const int start_all = p.window > 0 ? max(end_all - p.window, 0) : 0;
+    const int per_split = ((max(end_all - start_all, 0) + p.splits - 1) / p.splits + kTileKeys - 1) / kTileKeys * kTileKeys;
+    const int start = start_all + split * per_split;
+    const int end = min(start + per_split, end_all);
+    const int tile_count = end > start ? (end - start + kTileKeys - 1) / kTileKeys : 0;
+    const int column0 = warp * kSlice;
+
+    if (tile_count == 0) {
+        for (int r = threadIdx.x; r < kHeads; r += blockDim.x) {
+            if (p.splits > 1 && head0 + r < p.heads) {
+                p.lse[(static_cast<size_t>(query) * p.splits + split) * p.heads + head0 + r] = -INFINITY;
+            }
+        }
+        if (p.splits == 1) {
+            for (int i = threadIdx.x; i < kHeads * p.latent; i += blockDim.x) {
+                const int head = head0 + i / p.latent;
+                if (head < p.heads) {
+                    p.out[(static_cast<size_t>(query) * p.heads + head) * p.latent + i % p.latent] = __float2bfloat16_rn(0.0f);
+                }
+            }
+        }
+        return;
+    }
+
+    const int32_t *table = p.table + static_cast<size_t>(sequence) * p.table_stride;
+    const uint32_t slice = smem_u32(tiles) + warp * kSliceBytes;
+    const int stage_bytes = warps * kSliceBytes;
+    auto load_tile = [&](int tile) {
+        // lanes look up the cache rows of two keys each, then all copy four keys at a time, eight 16-byte pieces each
+        int row[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int key = start + tile * kTileKeys + lane + 32 * i;
+            row[i] = -1;
+            if (key < end) {
+                const int page = table[key / p.page_size];
+                if (page >= 0 && page < p.pages) {
+                    row[i] = page * p.page_size + key % p.page_size;
+                } else {
+                    report_status(p.status, kStatusIndexOutOfBounds);
+                }
+            }
+        }
+        const uint32_t target = slice + (tile % kLatentStages) * stage_bytes;
+        const int piece = lane & 7;
+#pragma unroll
+        for (int i = 0; i < kTileKeys / 4; ++i) {
+            const int key = (lane >> 3) + 4 * i;
+            const int at = __shfl_sync(0xffffffffu, row[i / 8], key & 31);
+            const __nv_bfloat16 *source = p.cache + static_cast<size_t>(max(at, 0)) * p.latent + column0 + piece * 8;
+            copy_async_16(target + slice_at(key, piece), source, at >= 0);
+        }
+    };
+    load_tile(0);
+    copy_async_commit();
+    if (tile_count > 1) load_tile(1);
+    copy_async_commit();
+
+    // q fragments of this warp's columns, for the whole kernel
+    uint32_t qf[MT][4][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int head = head0 + m * 16 + g + (i & 1) * 8;
+                const int column = column0 + ks * 16 + q2 + (i >> 1) * 8;
+                qf[m][ks][i] = head < p.heads ? *reinterpret_cast<const uint32_t *>(
+                                                    p.query + (static_cast<size_t>(query) * p.heads + head) * p.latent + column)
+                                              : 0u;
+            }
+        }
+    }
+    for (int r = threadIdx.x; r < kHeads; r += blockDim.x) {
+        row_max[r] = -INFINITY;
+        row_sum[r] = 0.0f;
+    }
+    float acc[MT][8][4] = {};
+    __syncthreads();
+
+    for (int tile = 0; tile < tile_count; ++tile) {
+        copy_async_wait<kLatentStages - 1>();
+        __syncwarp();
+        const uint32_t here = slice + (tile % kLatentStages) * stage_bytes;
+        {
+            float s[MT][8][4] = {};
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) {
+#pragma unroll
+                for (int pair = 0; pair < 4; ++pair) {  // two 8-key tiles at a time
+                    uint32_t b0, b1, b2, b3;
+                    const int key = pair * 16 + (lane & 7) + ((lane >> 4) << 3);
+                    ldmatrix_x4(here + slice_at(key, ks * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        mma_m16n8k16<__nv_bfloat16>(s[m][2 * pair], qf[m][ks][0], qf[m][ks][1], qf[m][ks][2], qf[m][ks][3], b0, b1);
+                        mma_m16n8k16<__nv_bfloat16>(s[m][2 * pair + 1], qf[m][ks][0], qf[m][ks][1], qf[m][ks][2], qf[m][ks][3], b2, b3);
+                    }
+                }
+            }
+            float *mine = scores + warp * kHeads * kScoreStride;
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+#pragma unroll
+                for (int n = 0; n < 8; ++n) {
+                    *reinterpret_cast<float2 *>(mine + (m * 16 + g) * kScoreStride + n * 8 + q2) = make_float2(s[m][n][0], s[m][n][1]);
+                    *reinterpret_cast<float2 *>(mine + (m * 16 + g + 8) * kScoreStride + n * 8 + q2) = make_float2(s[m][n][2], s[m][n][3]);
+                }
+            }
+        }
+        __syncthreads();
+        const int visible = end - start - tile * kTileKeys;  // keys of this tile
+        for (int r = warp; r < kHeads; r += warps) {
+            float a = 0.0f, b = 0.0f;
+            for (int w = 0; w < warps; ++w) {
+                a += scores[(w * kHeads + r) * kScoreStride + lane];
+                b += scores[(w * kHeads + r) * kScoreStride + lane + 32];
+            }
+            a = lane < visible ? a * p.scale_log2 : -INFINITY;
+            b = lane + 32 < visible ? b * p.scale_log2 : -INFINITY;
+            const float before = row_max[r];
+            const float now = fmaxf(before, warp_max(fmaxf(a, b)));  // finite: the tile has at least one key
+            a = exp2f(a - now);
+            b = exp2f(b - now);
+            const float sum = warp_sum(a + b);
+            weights[r * kWeightStride + lane] = __float2bfloat16_rn(a);
+            weights[r * kWeightStride + lane + 32] = __float2bfloat16_rn(b);
+            __syncwarp();
+            if (lane == 0) {
+                const float factor = exp2f(before - now);
+                row_factor[r] = factor;
+                row_max[r] = now;
+                row_sum[r] = row_sum[r] * factor + sum;
+            }
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const float f0 = row_factor[m * 16 + g], f1 = row_factor[m * 16 + g + 8];
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+                acc[m][n][0] *= f0;
+                acc[m][n][1] *= f0;
+                acc[m][n][2] *= f1;
+                acc[m][n][3] *= f1;
+            }
+        }
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            uint32_t a[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                const __nv_bfloat16 *at = weights + (m * 16 + (lane & 15)) * kWeightStride + ks * 16 + (lane >> 4) * 8;
+                ldmatrix_x4(smem_u32(at), a[m][0], a[m][1], a[m][2], a[m][3]);
+            }
+#pragma unroll
+            for (int pair = 0; pair < 4; ++pair) {  // two 8-column tiles at a time
+                uint32_t b0, b1, b2, b3;
+                const int key = ks * 16 + (lane & 15);
+                ldmatrix_x4_trans(here + slice_at(key, pair * 2 + (lane >> 4)), b0, b1, b2, b3);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    mma_m16n8k16<__nv_bfloat16>(acc[m][2 * pair], a[m][0], a[m][1], a[m][2], a[m][3], b0, b1);
+                    mma_m16n8k16<__nv_bfloat16>(acc[m][2 * pair + 1], a[m][0], a[m][1], a[m][2], a[m][3], b2, b3);
+                }
+            }
+        }
+        __syncwarp();
+        if (tile + kLatentStages < tile_count) load_tile(tile + kLatentStages);
+        copy_async_commit();
+    }
+    copy_async_wait<0>();
+
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int r = m * 16 + g + half * 8;
+            const int head = head0 + r;
+            if (head >= p.heads) continue;
+            const float inverse = 1.0f / row_sum[r];
+#pragma unroll
+            for (int n = 0; n < 8; ++n) {
+                const int column = column0 + n * 8 + q2;
+                const float x = acc[m][n][2 * half] * inverse, y = acc[m][n][2 * half + 1] * inverse;
+                if (p.splits == 1) {
+                    *reinterpret_cast<uint32_t *>(p.out + (static_cast<size_t>(query) * p.heads + head) * p.latent + column) =
+                        pack2<__nv_bfloat16>(x, y);
+                } else {
+                    *reinterpret_cast<float2 *>(
+                        p.attn + ((static_cast<size_t>(query) * p.splits + split) * p.heads + head) * p.latent + column) =
+                        make_float2(x, y);
+                }
+            }
+            if (p.splits > 1 && warp == 0 && q2 == 0) {
+                p.lse[(static_cast<size_t>(query) * p.splits + split) * p.heads + head] = row_max[r] + log2f(row_sum[r]);
+            }
+        }
+    }
+}
+
+// out[query, head] = sum over the splits of exp2(lse_s - max) * attn_s, normalised.
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentDecode p) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int query = blockIdx.x, head = blockIdx.y;
+    const float *lse = p.lse + static_cast<size_t>(query) * p.splits * p.heads + head;
+    float top = -INFINITY;
+    for (int s = 0; s < p.splits; ++s) top = fmaxf(top, lse[s * p.heads]);
+    float total = 0.0f;
+    for (int s = 0; s < p.splits; ++s) total += top == -INFINITY ? 0.0f : exp2f(lse[s * p.heads] - top);
+    const float inverse = total > 0.0f ? 1.0f / total : 0.0f;
+    for (int c = threadIdx.x * 4; c < p.latent; c += blockDim.x * 4) {
+        float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        for (int s = 0; s < p.splits; ++s) {
+            const float value = lse[s * p.heads];
+            if (value == -INFINITY) continue;  // a split without keys wrote nothing
+            const float weight = exp2f(value - top) * inverse;
+            const float4 x = *reinterpret_cast<const float4 *>(
+                p.attn + ((static_cast<size_t>(query) * p.splits + s) * p.heads + head) * p.latent + c);
+            sum.x = fmaf(weight, x.x, sum.x);
+            sum.y = fmaf(weight, x.y, sum.y);
+            sum.z = fmaf(weight, x.z, sum.z);
+            sum.w = fmaf(weight, x.w, sum.w);
+        }
+        *reinterpret_cast<uint2 *>(p.out + (static_cast<size_t>(query) * p.heads + head) * p.latent + c) =
+            make_uint2(pack2<__nv_bfloat16>(sum.x, sum.y), pack2<__nv_bfloat16>(sum.z, sum.w));
+    }
+}
+
+template <int MT>
+int launch_latent_decode(cudaStream_t stream, const LatentDecode &p, size_t queries) {
+    const int warps = p.latent / kSlice;
+    const int bytes = latent_shared_bytes(warps, MT);
+    static int configured[kMaxDevices] = {0};
+    SINGE_CUDA_TRY(ensure_dynamic_shared(latent_decode_kernel<MT>, bytes, configured));
+    const dim3 grid(static_cast<unsigned>(queries), static_cast<unsigned>(p.splits),
+                    static_cast<unsigned>((p.heads + MT * 16 - 1) / (MT * 16)));
+    SINGE_CUDA_TRY(launch_dependent(latent_decode_kernel<MT>, grid, dim3(warps * 32), bytes, stream, kLaunchDecode, 1, p));
+    if (p.splits > 1) {
+        const int threads = (p.latent / 4 + 31) / 32 * 32;
+        SINGE_CUDA_TRY(launch_dependent(latent_combine_kernel, dim3(static_cast<unsigned>(queries), static_cast<unsigned>(p.heads)),
+                                        dim3(threads), 0, stream, kLaunchCombine, 1, p));
+    }
+    return launch_status();
+}
+
+}  // namespace
+}  // namespace singe
+
+using namespace singe;
+
+extern "C" {
+
+size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t key_bound) {
+    // One CTA per SM at a time, in waves: a CTA costs a fixed ramp and a time per key; each split adds to the fold.
+    const double slots = device_sm_count();
+    const double groups = static_cast<double>((heads + 31) / 32);
+    const size_t finest = key_bound / (2 * kTileKeys) > 0 ? key_bound / (2 * kTileKeys) : 1;
+    size_t best = 1;
+    double best_time = 1e30;
+    for (size_t splits = 1; splits <= finest && splits <= 64; ++splits) {
+        const double ctas = static_cast<double>(queries) * groups * static_cast<double>(splits);
+        const double waves = static_cast<double>(static_cast<long long>((ctas + slots - 1) / slots));
+        const double keys = static_cast<double>((key_bound + splits - 1) / splits);
+        const double time = waves * (4.0 + 0.025 * keys) + (splits > 1 ? 2.0 + 0.3 * static_cast<double>(splits) : 0.0);
+        if (time < best_time) {
+            best_time = time;
+            best = splits;
+        }
+    }
+    return best;
+}
+
+int singe_latent_decode_bf16(singe_stream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                             const void *cache, const int32_t *sequence_of, const int32_t *lens,
+                             const int32_t *block_table, size_t queries, size_t heads, size_t latent, size_t page_size,
+                             size_t pages, size_t sequences, size_t table_stride, size_t window, size_t splits,
+                             float scale, uint32_t *status) {
+    if (queries == 0 || heads == 0 || latent == 0 || page_size == 0 || pages == 0 || sequences == 0 || table_stride == 0 ||
+        splits == 0 || !(scale == scale)) {
+        return SINGE_ERR_INVALID_LENGTH;
+    }
+    if (!fits_i32(queries) || !fits_i32(heads) || !fits_i32(pages * page_size) || !fits_i32(table_stride * page_size) ||
+        !fits_i32(window)) {
+        return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    }
+    if (out == nullptr || query == nullptr || cache == nullptr || sequence_of == nullptr || lens == nullptr ||
+        block_table == nullptr || (splits > 1 && (attn_scratch == nullptr || lse_scratch == nullptr))) {
+        return SINGE_ERR_NULL_POINTER;
+    }
+    if (latent % kSlice != 0 || latent > kMaxLatent || splits > 65535 || heads > 65535 ||
+        ((reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(query) | reinterpret_cast<uintptr_t>(out) |
+          reinterpret_cast<uintptr_t>(attn_scratch)) & 15u) != 0) {
+        return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    }
+    LatentDecode p;
+    p.out = static_cast<__nv_bfloat16 *>(out);
+    p.attn = attn_scratch;
+    p.lse = lse_scratch;
+    p.query = static_cast<const __nv_bfloat16 *>(query);
+    p.cache = static_cast<const __nv_bfloat16 *>(cache);
+    p.sequence_of = sequence_of;
+    p.lens = lens;
+    p.table = block_table;
+    p.heads = static_cast<int>(heads);
+    p.latent = static_cast<int>(latent);
+    p.page_size = static_cast<int>(page_size);
+    p.pages = static_cast<int>(pages);
+    p.sequences = static_cast<int>(sequences);
+    p.table_stride = static_cast<int>(table_stride);
+    p.window = static_cast<int>(window);
+    p.splits = static_cast<int>(splits);
+    p.scale_log2 = scale * 1.4426950408889634f;
+    p.status = status;
+    return heads <= 16 ? launch_latent_decode<1>(static_cast<cudaStream_t>(stream), p, queries)
+                       : launch_latent_decode<2>(static_cast<cudaStream_t>(stream), p, queries);
+}
+
+}  // extern "C"

@@ -34,6 +34,9 @@
 // Tensor memory (all 512 columns): S_A/P_A [0,128), S_B/P_B [128,256), O_A [256,384), O_B [384,512).
 // Shared memory: Q_A, Q_B, 2 x K, 2 x V tiles of 32 KB = 192 KB.
 // Under a causal mask tile A sees one key tile less than tile B; CTAs are dispatched heaviest-first.
+// WINDOW: a query sees itself and the window - 1 keys before it.  Both tiles of a pair start at the key tile where the
+// pair's first row begins to see; a row whose first visible key lies in a later tile takes its base from that tile.
+// Keys have offsets and a row stride of their own, and the epilogue may gate a head's rows by a sigmoid.
 // Every mbarrier wait is bounded; on a timeout the CTA records status 2, frees tensor memory and leaves.
 #include <type_traits>
 
@@ -86,6 +89,11 @@ struct PrefillParams {
                     // 2: the queries are the sequence's last tokens (query i sits at position len_kv - len_q + i)
     float scale_log2;
     uint32_t *error;
+    // windowed form
+    int window;
+    const int32_t *offsets_kv;
+    const __nv_bfloat16 *gate;  // nullptr, or row t of head h is multiplied by sigmoid(gate[t * gate_stride + h])
+    long long gate_stride;
 };
 
 // Lengths and first rows of sequence b.  DENSE is a template argument of the kernel: as run-time branches these four
@@ -96,8 +104,10 @@ template <bool DENSE>
 __device__ __forceinline__ int seq_len_kv(const PrefillParams &p, int b) { return DENSE ? p.uniform_kv : p.lens_kv[b]; }
 template <bool DENSE>
 __device__ __forceinline__ int seq_offset_q(const PrefillParams &p, int b) { return DENSE ? b * p.uniform_q : p.offsets[b]; }
-template <bool DENSE>
-__device__ __forceinline__ int seq_offset_kv(const PrefillParams &p, int b) { return DENSE ? b * p.uniform_kv : p.offsets[b]; }
+template <bool DENSE, bool WINDOW>
+__device__ __forceinline__ int seq_offset_kv(const PrefillParams &p, int b) {
+    return DENSE ? b * p.uniform_kv : (WINDOW ? p.offsets_kv[b] : p.offsets[b]);
+}
 
 __device__ __forceinline__ float exp2_approx(float x) {
     float y;
@@ -111,17 +121,25 @@ __device__ __forceinline__ float max3(float a, float b, float c) {
     return d;
 }
 
-// Folds the 32 raw scores of one chunk into four running maxima (independent chains).  MASKED handles tiles where
-// some keys are hidden (the diagonal tile and a sequence's last tile) and a negative scale; `limit` counts the
-// visible columns from the chunk's first.
-template <bool MASKED>
-__device__ __forceinline__ void chunk_max(const uint32_t (&sc)[kChunk], int limit, float sign, float (&m)[4]) {
-    if (MASKED) {
+// Which columns of a tile may be hidden: none, those from `limit` on (the diagonal tile and a sequence's last tile), or
+// also those before `low` (where a sliding window begins).
+constexpr int kMaskNone = 0, kMaskEnd = 1, kMaskBoth = 2;
+
+template <int MASK>
+__device__ __forceinline__ bool column_visible(int column, int low, int limit) {
+    return MASK == kMaskBoth ? (column >= low && column < limit) : column < limit;
+}
+
+// Folds the 32 raw scores of one chunk into four running maxima (independent chains).  A mask other than none also
+// handles a negative scale; `low` and `limit` count columns from the chunk's first.
+template <int MASK>
+__device__ __forceinline__ void chunk_max(const uint32_t (&sc)[kChunk], int low, int limit, float sign, float (&m)[4]) {
+    if (MASK != kMaskNone) {
 #pragma unroll
         for (int i = 0; i < kChunk; i += 4) {
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                if (i + u < limit) m[u] = fmaxf(m[u], __uint_as_float(sc[i + u]) * sign);
+                if (column_visible<MASK>(i + u, low, limit)) m[u] = fmaxf(m[u], __uint_as_float(sc[i + u]) * sign);
             }
         }
     } else {
@@ -139,9 +157,9 @@ __device__ __forceinline__ void chunk_max(const uint32_t (&sc)[kChunk], int limi
 // columns at `tmem_p`), the unrounded values are added to two running f32x2 sums.  Scores are handled as f32x2
 // pairs.  (Evaluating part of the exponentials as a polynomial on the FMA pipe was measured slower at every ratio:
 // with one softmax warp per scheduler the extra instructions cost more than the special-function unit saves.)
-template <typename T, bool MASKED>
+template <typename T, int MASK>
 __device__ __forceinline__ void chunk_exp_store(const uint32_t (&sc)[kChunk], uint32_t tmem_p, float2 scale2,
-                                                float2 bias2, int limit, float2 (&sum)[2]) {
+                                                float2 bias2, int low, int limit, float2 (&sum)[2]) {
     uint32_t packed[kChunk / 2];
 #pragma unroll
     for (int i = 0; i < kChunk; i += 2) {
@@ -149,9 +167,9 @@ __device__ __forceinline__ void chunk_exp_store(const uint32_t (&sc)[kChunk], ui
         float2 e;
         e.x = exp2_approx(x.x);
         e.y = exp2_approx(x.y);
-        if (MASKED) {
-            e.x = (i < limit) ? e.x : 0.0f;
-            e.y = (i + 1 < limit) ? e.y : 0.0f;
+        if (MASK != kMaskNone) {
+            e.x = column_visible<MASK>(i, low, limit) ? e.x : 0.0f;
+            e.y = column_visible<MASK>(i + 1, low, limit) ? e.y : 0.0f;
         }
         sum[(i >> 1) & 1] = __fadd2_rn(sum[(i >> 1) & 1], e);
         packed[i >> 1] = pack2<T>(e.x, e.y);
@@ -161,21 +179,22 @@ __device__ __forceinline__ void chunk_exp_store(const uint32_t (&sc)[kChunk], ui
 
 // One row of one key tile: S (128 f32 columns at `tmem_s`) -> P (64 packed columns over the same place), chunk by
 // chunk with the next chunk's load in flight.
-template <typename T, bool MASKED>
-__device__ __forceinline__ void tile_exp(uint32_t tmem_s, float2 scale2, float2 bias2, int limit, float2 (&sum)[2]) {
+template <typename T, int MASK>
+__device__ __forceinline__ void tile_exp(uint32_t tmem_s, float2 scale2, float2 bias2, int low, int limit, float2 (&sum)[2]) {
     uint32_t buf[2][kChunk];
     tmem_ld_x32(tmem_s, buf[0]);
 #pragma unroll
     for (int c = 0; c < kTile / kChunk; ++c) {
         tmem_wait_ld_into(buf[c & 1]);
         if (c + 1 < kTile / kChunk) tmem_ld_x32(tmem_s + (c + 1) * kChunk, buf[(c + 1) & 1]);
-        chunk_exp_store<T, MASKED>(buf[c & 1], tmem_s + c * (kChunk / 2), scale2, bias2, limit - c * kChunk, sum);
+        chunk_exp_store<T, MASK>(buf[c & 1], tmem_s + c * (kChunk / 2), scale2, bias2, low - c * kChunk, limit - c * kChunk,
+                                 sum);
     }
 }
 
 // Exact maximum of the visible raw scores (times `sign`) of one row of one key tile.
-template <bool MASKED>
-__device__ __forceinline__ float tile_max(uint32_t tmem_s, int limit, float sign) {
+template <int MASK>
+__device__ __forceinline__ float tile_max(uint32_t tmem_s, int low, int limit, float sign) {
     float m[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
     uint32_t buf[2][kChunk];
     tmem_ld_x32(tmem_s, buf[0]);
@@ -183,7 +202,7 @@ __device__ __forceinline__ float tile_max(uint32_t tmem_s, int limit, float sign
     for (int c = 0; c < kTile / kChunk; ++c) {
         tmem_wait_ld_into(buf[c & 1]);
         if (c + 1 < kTile / kChunk) tmem_ld_x32(tmem_s + (c + 1) * kChunk, buf[(c + 1) & 1]);
-        chunk_max<MASKED>(buf[c & 1], limit - c * kChunk, sign, m);
+        chunk_max<MASK>(buf[c & 1], low - c * kChunk, limit - c * kChunk, sign, m);
     }
     return fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3]));
 }
@@ -215,7 +234,8 @@ struct Item {
     int len_kv;
     int shift;      // causal mask: query row i sees keys 0 .. max(i + shift, 0); 0 for the sequence-local mask,
                     // len_kv - len_q when the queries are the sequence's last tokens
-    int tiles[2];   // key tiles tile A / tile B need (0: no real row, or no visible key)
+    int start;      // first key tile either tile needs (0 unless a window hides the ones before)
+    int tiles[2];   // one past the last key tile tile A / tile B needs (0: no real row, or no visible key)
     int key_tiles;  // max of the two
     bool valid;     // false: the sequence's offsets leave the packed tensors
 };
@@ -226,7 +246,7 @@ __device__ __forceinline__ int pairs_of(int len_q) { return (max(len_q, 0) + kPa
 // pair index down (under a causal mask a pair's work grows with its index), head = index % heads.  `counts[t]` is
 // the number of sequences that have a pair t, `tmax` the largest pair count.  Every lane of the calling warp
 // takes part and receives the same answer.
-template <bool DENSE>
+template <bool DENSE, bool WINDOW>
 __device__ __forceinline__ Item decode_item(const PrefillParams &p, const int *counts, int tmax, int index, int lane) {
     constexpr unsigned kFull = 0xffffffffu;
     Item item;
@@ -272,18 +292,20 @@ __device__ __forceinline__ Item decode_item(const PrefillParams &p, const int *c
     item.len_q = 0;
     item.len_kv = 0;
     item.shift = 0;
+    item.start = 0;
     item.tiles[0] = item.tiles[1] = 0;
     item.key_tiles = 0;
     if (seq < 0) return item;
     item.len_q = max(seq_len_q<DENSE>(p, seq), 0);
     item.len_kv = max(seq_len_kv<DENSE>(p, seq), 0);
     item.offset = seq_offset_q<DENSE>(p, seq);
-    item.offset_kv = seq_offset_kv<DENSE>(p, seq);
-    item.valid = item.offset >= 0 && item.offset + item.len_q <= p.total_q &&
+    item.offset_kv = seq_offset_kv<DENSE, WINDOW>(p, seq);
+    item.valid = item.offset >= 0 && item.offset_kv >= 0 && item.offset + item.len_q <= p.total_q &&
                  (p.block_table != nullptr ? item.len_kv <= p.table_stride * kPageTokens
                                            : item.offset_kv + item.len_kv <= p.total_kv);
     if (!item.valid) return item;
     item.shift = p.causal == 2 ? item.len_kv - item.len_q : 0;
+    if (WINDOW) item.start = max(item.q0 + item.shift - p.window + 1, 0) / kTile;
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
         const int first = item.q0 + x * kTile;
@@ -306,7 +328,7 @@ __device__ __forceinline__ Item decode_item(const PrefillParams &p, const int *c
 // 128-key tile and 64-wide half; the boxes land back to back, which is the layout one 128-row box would have).
 // HD = 128 or 64: with 64 a tile is a single 128-byte-wide box (the second half of every 32 KB buffer stays unused).
 // DENSE: uniform lengths, sequences back to back, LSE laid out [batch, heads, queries] (fmha_prefill_lse).
-template <typename T, int HD, bool SAFE, bool PAGED, bool DENSE>
+template <typename T, int HD, bool SAFE, bool PAGED, bool DENSE, bool WINDOW>
 __global__ void __launch_bounds__(kPrefillThreads, 1)
     prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                            const __grid_constant__ CUtensorMap v_map, const PrefillParams p) {
@@ -386,7 +408,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         for (int round = 0;; ++round) {
             const int index = share_index(round);
             if (index < 0) break;
-            const Item item = decode_item<DENSE>(p, counts, tmax, index, lane);
+            const Item item = decode_item<DENSE, WINDOW>(p, counts, tmax, index, lane);
             const int row = item.q0 + tid;
             const bool marked = item.valid && item.key_tiles > 0 && tid < kPair && row < item.len_q &&
                                 isnan(*lse_at(item, row));
@@ -444,7 +466,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         for (int round = 0; !failed; ++round) {
             const int index = item_index(round);
             if (index < 0) break;
-            const Item item = decode_item<DENSE>(p, counts, tmax, index, lane);
+            const Item item = decode_item<DENSE, WINDOW>(p, counts, tmax, index, lane);
             if (item.key_tiles == 0) continue;
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
@@ -465,7 +487,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     }
                 }
             }
-            for (int j = 0; j < item.key_tiles && !failed; ++j, ++g) {
+            for (int j = item.start; j < item.key_tiles && !failed; ++j, ++g) {
                 const int stage = g & 1;
                 const int row0 = item.offset_kv + j * kTile;
                 if (g >= 2 && !wait_lane0(bar_k_empty + stage * 8, ((g >> 1) - 1) & 1)) {
@@ -578,7 +600,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     return item;
                 }
                 ++round;
-                item = decode_item<DENSE>(p, counts, tmax, index, lane);
+                item = decode_item<DENSE, WINDOW>(p, counts, tmax, index, lane);
                 if (item.key_tiles > 0) return item;
             }
         };
@@ -588,7 +610,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             if (!wait_all(bar_q_full + x * 8, q_uses[x] & 1)) return false;
             ++q_uses[x];
             tcgen05_fence_after();
-            issue_qk(x, stage, item.tiles[x] == 1);
+            issue_qk(x, stage, item.tiles[x] == item.start + 1);
             return true;
         };
         Item item = next_item();
@@ -602,7 +624,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         }
         while (item.key_tiles > 0 && !failed) {
             const Item following = next_item();
-            for (int j = 0; j < item.key_tiles && !failed; ++j, ++g) {
+            for (int j = item.start; j < item.key_tiles && !failed; ++j, ++g) {
                 const int stage = g & 1;
                 const int next = (g + 1) & 1;
                 const bool more = j + 1 < item.key_tiles;          // this item has another key tile
@@ -616,7 +638,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     if (failed) continue;
                     if (j < item.tiles[x]) {
                         // the previous item's epilogue must have taken O out of tensor memory
-                        if (j == 0 && o_done[x] > 0 && !wait_all(bar_o_empty + x * 8, (o_done[x] - 1) & 1)) {
+                        if (j == item.start && o_done[x] > 0 && !wait_all(bar_o_empty + x * 8, (o_done[x] - 1) & 1)) {
                             failed = true;
                             continue;
                         }
@@ -627,7 +649,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                         ++p_uses[x];
                         tcgen05_fence_after();
                         const bool last = j == item.tiles[x] - 1;
-                        issue_pv(x, stage, j > 0, last);
+                        issue_pv(x, stage, j > item.start, last);
                         if (last) ++o_done[x];
                     }
                     if (x == 1) {
@@ -672,7 +694,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         for (int round = 0; !failed; ++round) {
             const int index = item_index(round);
             if (index < 0) break;
-            const Item item = decode_item<DENSE>(p, counts, tmax, index, lane);
+            const Item item = decode_item<DENSE, WINDOW>(p, counts, tmax, index, lane);
             if (!item.valid) {
                 if (warp == 0 && lane == 0) report_status(p.error, kStatusIndexOutOfBounds);
                 continue;
@@ -695,7 +717,8 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             float base_log2 = -INFINITY;  // what P, O and the row sum are relative to (log2 units); finite after tile 0
             float row_sum = 0.0f;
             bool in_range = true;
-            for (int j = 0; j < my_tiles && !failed; ++j, ++s_uses) {
+            bool unseen = WINDOW && real;  // no key seen yet: O and the sum are zero, so the base is free
+            for (int j = item.start; j < my_tiles && !failed; ++j, ++s_uses) {
                 if (!__all_sync(0xffffffffu, mbar_wait(bar_s_full + x * 8, s_uses & 1) ? 1 : 0)) {
                     failed = true;
                     break;
@@ -705,23 +728,34 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                 int limit = item.len_kv - j * kTile;
                 if (p.causal) limit = min(limit, max(row + item.shift, 0) + 1 - j * kTile);
                 limit = real ? limit : 0;
+                const int low = WINDOW ? row + item.shift - p.window + 1 - j * kTile : 0;  // first column the row sees
                 const bool partial = __any_sync(0xffffffffu, limit < kTile);
+                const bool lower = WINDOW && __any_sync(0xffffffffu, low > 0);
 
-                if (SAFE || j == 0) {
-                    float wanted = (partial || sign < 0.0f) ? tile_max<true>(tmem_s, limit, sign)
-                                                            : tile_max<false>(tmem_s, limit, sign);
+                if (SAFE || j == item.start || (WINDOW && __any_sync(0xffffffffu, unseen))) {
+                    float wanted;
+                    if (WINDOW && lower) {
+                        wanted = tile_max<kMaskBoth>(tmem_s, low, limit, sign);
+                    } else if (partial || sign < 0.0f) {
+                        wanted = tile_max<kMaskEnd>(tmem_s, low, limit, sign);
+                    } else {
+                        wanted = tile_max<kMaskNone>(tmem_s, low, limit, sign);
+                    }
                     wanted = fmaxf(base_log2, wanted * fabsf(p.scale_log2));
                     wanted = wanted == -INFINITY ? 0.0f : wanted;  // nothing visible yet: any base will do
+                    const bool free_base = WINDOW && unseen;
+                    if (WINDOW && unseen && max(low, 0) < min(limit, kTile)) unseen = false;
                     // Re-base O only when some row's max grew past the threshold; then every row of the warp does.
-                    const bool grow = wanted > base_log2 + kRescaleThreshold;
+                    const bool grow = !free_base && wanted > base_log2 + kRescaleThreshold;
                     if (__any_sync(0xffffffffu, grow)) {
-                        if (j > 0) {
-                            const float factor = exp2_approx(base_log2 - wanted);
+                        if (j > item.start) {
+                            const float factor = free_base ? 1.0f : exp2_approx(base_log2 - wanted);
                             row_sum *= factor;
                             scale_o_row<HD>(tmem_o, factor);
                         }
                         base_log2 = wanted;
                     }
+                    if (free_base) base_log2 = unseen ? -INFINITY : wanted;
                 } else if (__any_sync(0xffffffffu, row_sum > kRebaseLimit)) {
                     // Single-pass tiles: pull the row back by the exponent of its sum, an exact power of two.
                     const int exponent = row_sum > kRebaseLimit ? ((__float_as_int(row_sum) >> 23) & 0xff) - 127 : 0;
@@ -730,12 +764,15 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     base_log2 += static_cast<float>(exponent);
                     scale_o_row<HD>(tmem_o, factor);
                 }
-                const float2 bias2 = make_float2(-base_log2, -base_log2);
+                const float bias = WINDOW && unseen ? 0.0f : -base_log2;
+                const float2 bias2 = make_float2(bias, bias);
                 float2 sum[2] = {make_float2(row_sum, 0.0f), make_float2(0.0f, 0.0f)};
-                if (partial) {
-                    tile_exp<T, true>(tmem_s, scale2, bias2, limit, sum);
+                if (WINDOW && lower) {
+                    tile_exp<T, kMaskBoth>(tmem_s, scale2, bias2, low, limit, sum);
+                } else if (partial) {
+                    tile_exp<T, kMaskEnd>(tmem_s, scale2, bias2, low, limit, sum);
                 } else {
-                    tile_exp<T, false>(tmem_s, scale2, bias2, limit, sum);
+                    tile_exp<T, kMaskNone>(tmem_s, scale2, bias2, low, limit, sum);
                 }
                 row_sum = (sum[0].x + sum[0].y) + (sum[1].x + sum[1].y);
                 tmem_wait_st();
@@ -755,7 +792,10 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             ++o_uses;
             tcgen05_fence_after();
             const bool empty = row_sum == 0.0f;
-            const float inverse = empty ? 0.0f : 1.0f / row_sum;
+            float inverse = empty ? 0.0f : 1.0f / row_sum;
+            if (WINDOW && p.gate != nullptr) {
+                inverse /= 1.0f + __expf(-__bfloat162float(p.gate[token * p.gate_stride + item.head]));
+            }
 #pragma unroll 1
             for (int c = 0; c < HD; c += 32) {
                 uint32_t r[32];
@@ -817,21 +857,21 @@ bool prefill_fast_path(size_t heads, size_t kv_heads, size_t head_dim, size_t to
 
 namespace {
 
-template <typename T, int HD, bool PAGED, bool DENSE = false>
+template <typename T, int HD, bool PAGED, bool DENSE = false, bool WINDOW = false>
 int launch_prefill(cudaStream_t stream, const CUtensorMap &q_map, const CUtensorMap &k_map, const CUtensorMap &v_map,
                    const PrefillParams &params, unsigned persistent) {
-    SINGE_CUDA_TRY(cudaFuncSetAttribute(prefill_tcgen05_kernel<T, HD, true, PAGED, DENSE>,
+    SINGE_CUDA_TRY(cudaFuncSetAttribute(prefill_tcgen05_kernel<T, HD, true, PAGED, DENSE, WINDOW>,
                                         cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
     if (std::is_same<T, __nv_bfloat16>::value) {
-        SINGE_CUDA_TRY(cudaFuncSetAttribute(prefill_tcgen05_kernel<__nv_bfloat16, HD, false, PAGED, DENSE>,
+        SINGE_CUDA_TRY(cudaFuncSetAttribute(prefill_tcgen05_kernel<__nv_bfloat16, HD, false, PAGED, DENSE, WINDOW>,
                                             cudaFuncAttributeMaxDynamicSharedMemorySize, kPrefillSmem));
-        prefill_tcgen05_kernel<__nv_bfloat16, HD, false, PAGED, DENSE>
+        prefill_tcgen05_kernel<__nv_bfloat16, HD, false, PAGED, DENSE, WINDOW>
             <<<persistent, kPrefillThreads, kPrefillSmem, stream>>>(q_map, k_map, v_map, params);
         SINGE_TRY(launch_status());
     }
     // bf16: the redo pass over the same shares, a no-op while the device's out-of-range flag has never been raised.
     // f16 (params.exact): the only pass.  P must stay below 65504 there, so every tile takes its exact row maximum.
-    prefill_tcgen05_kernel<T, HD, true, PAGED, DENSE><<<persistent, kPrefillThreads, kPrefillSmem, stream>>>(q_map, k_map, v_map,
+    prefill_tcgen05_kernel<T, HD, true, PAGED, DENSE, WINDOW><<<persistent, kPrefillThreads, kPrefillSmem, stream>>>(q_map, k_map, v_map,
                                                                                                   params);
     return launch_status();
 }
@@ -878,7 +918,7 @@ int prefill_tcgen05(cudaStream_t stream, bool is_f16, void *out, float *lse, con
         SINGE_TRY(encode_tensor_map(&v_map, type, 3, value, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
                                     CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     }
-    PrefillParams params;
+    PrefillParams params = {};
     params.out = out;
     params.lse = lse;
     params.lens_q = lens_q;
@@ -930,6 +970,55 @@ int prefill_tcgen05(cudaStream_t stream, bool is_f16, void *out, float *lse, con
                  : launch_prefill<__nv_bfloat16, 128, false>(stream, q_map, k_map, v_map, params, persistent);
 }
 
+// The windowed form: keys and values are rows of kv_row_stride elements (heads side by side) with offsets of their own;
+// the queries are their sequences' last tokens.
+int prefill_tcgen05_windowed(cudaStream_t stream, void *out, float *lse, const void *query, const void *key,
+                             const void *value, size_t kv_row_stride, const int32_t *lens_q, const int32_t *lens_kv,
+                             const int32_t *offsets_q, const int32_t *offsets_kv, const void *gate, size_t gate_stride,
+                             size_t batch, size_t total_query_tokens, size_t total_kv_tokens, size_t heads,
+                             size_t head_dim, size_t window, float scale) {
+    const uint64_t kHeadDim = head_dim;
+    const CUtensorMapDataType type = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+    CUtensorMap q_map, k_map, v_map;
+    const uint32_t box[3] = {64, 1, kTile};
+    const uint64_t q_dims[3] = {kHeadDim, heads, total_query_tokens};
+    const uint64_t q_strides[2] = {kHeadDim * 2, kHeadDim * 2 * heads};
+    const uint64_t kv_dims[3] = {kHeadDim, heads, total_kv_tokens};
+    const uint64_t kv_strides[2] = {kHeadDim * 2, static_cast<uint64_t>(kv_row_stride) * 2};
+    SINGE_TRY(encode_tensor_map(&q_map, type, 3, query, q_dims, q_strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
+                                CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    SINGE_TRY(encode_tensor_map(&k_map, type, 3, key, kv_dims, kv_strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
+                                CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    SINGE_TRY(encode_tensor_map(&v_map, type, 3, value, kv_dims, kv_strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
+                                CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    PrefillParams params = {};
+    params.out = out;
+    params.lse = lse;
+    params.lens_q = lens_q;
+    params.lens_kv = lens_kv;
+    params.offsets = offsets_q;
+    params.offsets_kv = offsets_kv;
+    params.batch = static_cast<int>(batch);
+    params.heads = static_cast<int>(heads);
+    params.kv_heads = static_cast<int>(heads);
+    params.total_q = static_cast<int>(total_query_tokens);
+    params.total_kv = static_cast<int>(total_kv_tokens);
+    params.causal = 2;
+    params.scale_log2 = scale * 1.4426950408889634f;
+    params.error = device_error_word();
+    params.window = static_cast<int>(window);
+    params.gate = static_cast<const __nv_bfloat16 *>(gate);
+    params.gate_stride = static_cast<long long>(gate_stride);
+    const size_t items = (total_query_tokens / kPair + batch) * heads;
+    if (items > 0x7fffffffull) return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    const size_t sms = static_cast<size_t>(device_sm_count());
+    const unsigned persistent = static_cast<unsigned>(items < sms ? items : sms);
+    if (head_dim == 64) {
+        return launch_prefill<__nv_bfloat16, 64, false, false, true>(stream, q_map, k_map, v_map, params, persistent);
+    }
+    return launch_prefill<__nv_bfloat16, 128, false, false, true>(stream, q_map, k_map, v_map, params, persistent);
+}
+
 int prefill_tcgen05_bf16(cudaStream_t stream, void *out, float *lse, const void *query, const void *key,
                          const void *value, const int32_t *lens_q, const int32_t *lens_kv, const int32_t *offsets,
                          size_t batch, size_t total_query_tokens, size_t total_kv_tokens, size_t heads,
@@ -941,3 +1030,29 @@ int prefill_tcgen05_bf16(cudaStream_t stream, void *out, float *lse, const void 
 }
 
 }  // namespace singe
+
+extern "C" int singe_windowed_prefill_attention_bf16(
+    singe_stream_t stream, void *out, float *lse, const void *query, const void *key, const void *value,
+    size_t kv_row_stride, const int32_t *lens_q, const int32_t *lens_kv, const int32_t *offsets_q,
+    const int32_t *offsets_kv, const void *gate, size_t gate_row_stride, size_t batch, size_t total_query_tokens,
+    size_t total_kv_tokens, size_t heads, size_t head_dim, size_t window, float scale) {
+    using namespace singe;
+    if (batch == 0 || total_query_tokens == 0 || total_kv_tokens == 0 || heads == 0 || window == 0 ||
+        kv_row_stride < heads * head_dim || (gate != nullptr && gate_row_stride < heads) || !(scale == scale)) {
+        return SINGE_ERR_INVALID_LENGTH;
+    }
+    if (!fits_i32(batch) || !fits_i32(total_query_tokens) || !fits_i32(total_kv_tokens) || !fits_i32(heads) ||
+        !fits_i32(window)) {
+        return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    }
+    if (out == nullptr || lse == nullptr || query == nullptr || key == nullptr || value == nullptr || lens_q == nullptr ||
+        lens_kv == nullptr || offsets_q == nullptr || offsets_kv == nullptr) {
+        return SINGE_ERR_NULL_POINTER;
+    }
+    if (kv_row_stride % 8 != 0 || !prefill_fast_path(heads, heads, head_dim, total_query_tokens, query, key, value, out)) {
+        return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    }
+    return prefill_tcgen05_windowed(static_cast<cudaStream_t>(stream), out, lse, query, key, value, kv_row_stride, lens_q,
+                                    lens_kv, offsets_q, offsets_kv, gate, gate_row_stride, batch, total_query_tokens,
+                                    total_kv_tokens, heads, head_dim, window, scale);
+}

@@ -326,7 +326,8 @@ class LatentAttention:
                  cache.shape[0] * cache.shape[1], status)
         keys_values = torch.empty((rows.keys, 2 * c.heads * size), dtype=ops.dtype, device="cuda")
         ops.linear(stream, keys_values, latents, self.expand)
-        ops.call("singe_windowed_prefill_attention_bf16", stream, attended, query, keys_values,
+        lse = torch.empty((query.shape[0], c.heads), dtype=torch.float32, device="cuda")
+        ops.call("singe_windowed_prefill_attention_bf16", stream, attended, lse, query, keys_values,
                  keys_values.data_ptr() + c.heads * size * 2, keys_values.stride(0), rows.lens_q, rows.lens_kv,
                  rows.offsets_q, rows.offsets_kv, gate, gate.stride(0), rows.sequences, query.shape[0], rows.keys,
                  c.heads, size, c.window, c.scale)

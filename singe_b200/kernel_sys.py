@@ -130,9 +130,14 @@ SIGNATURES = {
                                      _z],
     "singe_gated_linear_step_f32": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _f, _f, _f,
                                     _z],
+    "singe_latent_decode_bf16": [_p, _p, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _z, _z, _z, _f, _p],
+    "singe_latent_decode_splits": [_z, _z, _z],
+    "singe_windowed_prefill_attention_bf16": [_p, _p, _p, _p, _p, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z,
+                                              _z, _f],
 }
 
 _RESTYPES = {
+    "singe_latent_decode_splits": ctypes.c_size_t,
     "singe_status_string": ctypes.c_char_p,
     "singe_paged_kv_decode_split_tokens": ctypes.c_size_t,
     "singe_paged_kv_decode_default_splits": ctypes.c_size_t,
