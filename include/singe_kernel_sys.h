@@ -700,6 +700,20 @@ int singe_gated_linear_step_f32(singe_stream_t stream, void *out, size_t out_str
                                 const void *norm_weight, float *state, const int32_t *first, const int32_t *count,
                                 const int32_t *context, size_t rows, size_t sequences, size_t heads, size_t dim,
                                 size_t vdim, size_t rank, float tau, float query_scale, float eps, size_t longest);
+/* The same over prompts, block by block on the tensor core (two-term bf16 operands for what is f32; the state stays f32).
+ * The blocks of 16 tokens of all sequences served, in order: block_row / block_tokens [blocks], a sequence's last block may
+ * be short.  segments [segment_count][4] = {sequence, first block, blocks, segments of the same sequence before it}, in
+ * order, segment_last[i] = 1 for a sequence's last one; cut != 0 when any sequence has more than one.  scratch:
+ * singe_gated_linear_prompt_scratch bytes, which is 0 for sizes this form does not take (dim <= 256 and vdim in eights; the
+ * state of a head has to fit one CTA's registers). */
+int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *projected,
+                                   size_t projected_stride, const void *decay_weight, const void *decay_bias,
+                                   const void *norm_weight, float *state, const int32_t *context, size_t heads, size_t dim,
+                                   size_t vdim, size_t rank, float tau, float query_scale, float eps,
+                                   const int32_t *block_row, const int32_t *block_tokens, size_t blocks,
+                                   const int32_t *segments, const int32_t *segment_last, size_t segment_count, int cut,
+                                   void *scratch);
+size_t singe_gated_linear_prompt_scratch(size_t heads, size_t dim, size_t vdim, size_t blocks, size_t segments);
 /* Explicit tile choice for the two GEMM entry points, process-wide: block_n in {32,64,128,256},
  * k_slices_per_stage in {1,2,4,8}; 0 = choose from the problem shape.
  * Replaces: TuningChoice::Explicit(MatmulTuning { tile, .. }) (singe-kernel/src/cuda/matmul.rs:58-77). */

@@ -32,6 +32,8 @@ from .decoder import PagedDecoder, PageTable
 EXPANDED_HEAD_SIZES = (64, 128)  # head sizes of the tensor-core prompt attention; smaller heads are padded with zeros
 ABSORBED_LATENT_LIMIT = 512      # widest latent the tensor-core decode attention takes
 FEW_TOKENS = 8                   # a sequence with at most this many new tokens takes the decode kernels
+BLOCK_TOKENS = 16                # tokens of a block of the recurrence's prompt kernel
+LEAST_SEGMENT = 8                # blocks a long sequence's segments have at least
 
 
 # ------------------------------------------------------------------------------------------------
@@ -192,8 +194,8 @@ class StepRows:
     short_sequences: object
     short_lens: object
     short_count: int
-    longest: int              # most new tokens of any sequence
     expanded: dict = field(default_factory=dict)   # window -> ExpandedRows of the longer sequences
+    blocks: dict = field(default_factory=dict)     # heads -> BlockRows of the longer sequences
 
 
 @dataclass
@@ -207,6 +209,39 @@ class ExpandedRows:
     offsets_q: object
     offsets_kv: object
     sequences: int
+
+
+@dataclass
+class BlockRows:
+    """What the recurrence's prompt kernel reads: the blocks of the longer sequences and the segments that run side by side."""
+    rows: object
+    tokens: object
+    blocks: int
+    segments: object
+    last: object
+    count: int
+    cut: bool
+
+
+def plan_segments(blocks_of, heads: int, sms: int):
+    """Cuts each sequence's blocks into segments.  A cut costs a second pass over all but a sequence's last segment, so
+    only steps whose (sequence, head) pairs leave SMs idle are cut, into about two segments per SM.  Returns rows of
+    (place in ``blocks_of``, first block, blocks, earlier segments of the sequence, last of the sequence)."""
+    total = sum(blocks_of)
+    size = total
+    if len(blocks_of) * heads < sms:
+        size = max(LEAST_SEGMENT, -(-total // max(2 * sms // heads, 1)))
+    rows, first = [], 0
+    for place, blocks in enumerate(blocks_of):
+        pieces = -(-blocks // size)
+        each = -(-blocks // pieces)
+        done = 0
+        while done < blocks:
+            taken = min(each, blocks - done)
+            rows.append((place, first + done, taken, done // each, int(done + taken == blocks)))
+            done += taken
+        first += blocks
+    return rows
 
 
 # ------------------------------------------------------------------------------------------------
@@ -291,7 +326,8 @@ class LatentAttention:
         """Absorbed attention of every row on the general kernel: any sizes, either activation type."""
         ops, c = self.ops, self.config
         t = query.shape[0]
-        latent_queries, latents = ops.rows(t, c.heads * self.latent), ops.rows(t, c.heads * self.latent)
+        # rows without padding, as the attention wants them
+        latent_queries, latents = ops.torch.empty((2, t, c.heads * self.latent), dtype=ops.dtype, device="cuda")
         ops.head_linear(stream, latent_queries, query, self.absorb, c.heads)
         lse = ops.torch.empty((t, c.heads), dtype=ops.torch.float32, device="cuda")
         ops.call(f"singe_paged_attention_{ops.suffix}", stream, latents, lse, latent_queries, cache, cache,
@@ -343,6 +379,8 @@ class GatedLinear:
         self.project = ops.weight(torch.cat([take("q"), take("k"), take("v"), take("g"), take("a1")]))
         self.decay, self.bias, self.norm = take("a2").contiguous(), take("a2.b").contiguous(), take("norm").contiguous()
         self.out = ops.weight(take("o"))
+        # the prompt kernel, for sizes it takes
+        self.blocked = ops.is_bf16 and ks.lib().singe_gated_linear_prompt_scratch(config.heads, config.dim, config.vdim, 1, 1) > 0
 
     def new_cache(self, table: PageTable, sequences: int):
         c = self.config
@@ -357,10 +395,18 @@ class GatedLinear:
         projected = ops.rows(t, self.project.shape[0])
         ops.linear(stream, projected, normed, self.project)
         attended = ops.rows(t, c.heads * c.vdim)
-        shape = [attended, attended.stride(0), projected, projected.stride(0), self.decay, self.bias, self.norm, state,
-                 step.first, step.fresh_tokens, step.context, t, state.shape[0], c.heads, c.dim, c.vdim, c.rank, c.tau,
-                 c.dim ** -0.5, self.eps]
-        ops.call(f"singe_gated_linear_step_{ops.suffix}", stream, *shape, 0x7fffffff)
+        operands = [attended, attended.stride(0), projected, projected.stride(0), self.decay, self.bias, self.norm, state]
+        sizes = [c.heads, c.dim, c.vdim, c.rank, c.tau, c.dim ** -0.5, self.eps]
+        rows = step.blocks.get(c.heads) if self.blocked else None
+        if rows is not None:
+            scratch = ops.torch.empty(int(ks.lib().singe_gated_linear_prompt_scratch(c.heads, c.dim, c.vdim, rows.blocks,
+                                                                                     rows.count)),
+                                      dtype=ops.torch.uint8, device="cuda")
+            ops.call("singe_gated_linear_prompt_bf16", stream, *operands, step.context, *sizes, rows.rows, rows.tokens,
+                     rows.blocks, rows.segments, rows.last, rows.count, int(rows.cut), scratch)
+        if rows is None or step.short_count > 0:
+            ops.call(f"singe_gated_linear_step_{ops.suffix}", stream, *operands, step.first, step.fresh_tokens,
+                     step.context, t, state.shape[0], *sizes, 0x7fffffff if rows is None else FEW_TOKENS)
         ops.linear(stream, delta, attended, self.out)
 
 
@@ -428,7 +474,8 @@ class HybridDecoder(PagedDecoder):
         self.decode_rows = StepRows(sequences, self.d_tokens, self.d_pages, self.d_slots, self.d_query_offsets,
                                     self.d_page_offsets, self.d_page_list, self.d_last_lengths, self.d_first,
                                     self.d_fresh, self.d_context, self.d_table, None, self.d_first, self.d_lens,
-                                    sequences, 1)
+                                    sequences)
+        self.sms = torch.cuda.get_device_properties(0).multi_processor_count
         self.trail = None   # set to a list to collect the residual stream after every layer (for inspection)
 
     # ---- the layers, over a step of any shape ----
@@ -533,6 +580,18 @@ class HybridDecoder(PagedDecoder):
             narrow.update({f"gather{window}": np.concatenate(gather), f"lens_q{window}": fresh[long],
                            f"lens_kv{window}": lens_kv, f"offsets_q{window}": first[long],
                            f"offsets_kv{window}": np.cumsum(lens_kv) - lens_kv})
+        block_heads = sorted({layer.mixer.heads for layer in c.layers if isinstance(layer.mixer, GatedLinearConfig)})
+        cut = {}
+        if len(long):
+            starts = [first[b] + np.arange(0, fresh[b], BLOCK_TOKENS) for b in long]
+            narrow["block_rows"] = np.concatenate(starts)
+            narrow["block_tokens"] = np.concatenate([np.minimum(first[b] + fresh[b] - start, BLOCK_TOKENS)
+                                                     for b, start in zip(long, starts)])
+            for heads in block_heads:
+                plan = np.asarray(plan_segments([len(start) for start in starts], heads, self.sms))
+                narrow[f"segments{heads}"] = np.stack([long[plan[:, 0]], plan[:, 1], plan[:, 2], plan[:, 3]], 1).reshape(-1)
+                narrow[f"segment_last{heads}"] = plan[:, 4]
+                cut[heads] = bool((plan[:, 4] == 0).any())
         wide = {"tokens": step.tokens, "pages": step.write_pages, "slots": step.write_slots,
                 "query_offsets": step.query_offsets, "page_offsets": step.page_offsets, "page_list": step.pages,
                 "last": step.last_page_lengths, "short_rows": short}
@@ -542,11 +601,14 @@ class HybridDecoder(PagedDecoder):
             part = lambda name: n[f"{name}{window}"]
             expanded[window] = ExpandedRows(part("gather"), part("gather").numel(), part("lens_q"), part("lens_kv"),
                                             part("offsets_q"), part("offsets_kv"), len(long))
+        blocks = {heads: BlockRows(n["block_rows"], n["block_tokens"], n["block_rows"].numel(), n[f"segments{heads}"],
+                                   n[f"segment_last{heads}"], n[f"segment_last{heads}"].numel(), cut[heads])
+                  for heads in cut}
         everything = len(short) == len(step.tokens)
         return StepRows(len(step.tokens), w["tokens"], w["pages"], w["slots"], w["query_offsets"], w["page_offsets"],
                         w["page_list"], w["last"], n["first"], n["fresh"], n["context"],
                         n["table"].view(block_table.shape), None if everything else w["short_rows"],
-                        n["short_sequences"], n["short_lens"], len(short), int(fresh.max()), expanded)
+                        n["short_sequences"], n["short_lens"], len(short), expanded, blocks)
 
     def _send(self, arrays: dict, kind) -> dict:
         torch = self.torch

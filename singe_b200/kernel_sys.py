@@ -134,9 +134,13 @@ SIGNATURES = {
     "singe_latent_decode_splits": [_z, _z, _z],
     "singe_windowed_prefill_attention_bf16": [_p, _p, _p, _p, _p, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z,
                                               _z, _f],
+    "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _f, _f, _f, _p, _p, _z,
+                                       _p, _p, _z, _i, _p],
+    "singe_gated_linear_prompt_scratch": [_z, _z, _z, _z, _z],
 }
 
 _RESTYPES = {
+    "singe_gated_linear_prompt_scratch": ctypes.c_size_t,
     "singe_latent_decode_splits": ctypes.c_size_t,
     "singe_status_string": ctypes.c_char_p,
     "singe_paged_kv_decode_split_tokens": ctypes.c_size_t,

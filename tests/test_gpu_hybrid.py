@@ -1,0 +1,273 @@
+"""The layer-list decoder end to end: loader, steps of every shape, cache and state reuse, generation, trace replay --
+against the plain float64 restatement in ``oracle.hybrid_ref``."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+from oracle import hybrid_ref
+from singe_b200 import hybrid, models
+from singe_b200.decoder import CachedDecoder, PageTableError
+from singe_b200.generation import GenerationOptions, PromptChunks, RunningBatch, generate_batch
+from tests import hybrid_util as util
+from tests.conftest import ROOT
+
+pytestmark = pytest.mark.gpu
+
+# root mean square of a position's logit error over that of its logits
+LIMIT = {"float32": 3e-5, "bfloat16": 6e-2}
+CONFIGS = {"mixed": util.MIXED, "odd": util.ODD, "ones": util.ONES, "wide": util.WIDE}
+
+
+@pytest.fixture(scope="module")
+def snapshots(tmp_path_factory):
+    made = {}
+    for name, config in CONFIGS.items():
+        weights = util.make_weights(config, seed=len(name))
+        made[name] = (config, weights, util.write_snapshot(tmp_path_factory.mktemp(name), config, weights))
+    return made
+
+
+class Expect:
+    """Oracle logits of whole sequences, computed once each."""
+
+    def __init__(self, config, weights):
+        self.config, self.weights, self.known = config, weights, {}
+
+    def __call__(self, tokens):
+        key = tuple(tokens)
+        if key not in self.known:
+            self.known[key] = hybrid_ref.forward(self.config, self.weights, tokens)[0]
+        return self.known[key]
+
+
+@pytest.fixture(scope="module")
+def expects(snapshots):
+    return {name: Expect(config, weights) for name, (config, weights, _) in snapshots.items()}
+
+
+def tokens_of(config, seed, count):
+    return [int(t) for t in np.random.default_rng(seed).integers(0, config["vocab"], size=count)]
+
+
+def check(got, expect, dtype, what):
+    got, expect = got.float().cpu().numpy().astype(np.float64), np.asarray(expect)
+    error = np.sqrt(((got - expect) ** 2).mean(1) / (expect ** 2).mean(1))
+    assert np.isfinite(got).all(), what
+    assert error.max() < LIMIT[dtype], f"{what}: position {error.argmax()} of {len(error)}: {error.max():.2e}"
+
+
+def run_portions(decoder, row, tokens, portions):
+    """Steps one row through ``tokens`` in portions, everything wanted; returns all logits."""
+    outs, at = [], 0
+    for n in portions:
+        part, want = [[] for _ in range(decoder.sequences)], [[] for _ in range(decoder.sequences)]
+        part[row], want[row] = tokens[at: at + n], list(range(len(tokens[at: at + n])))
+        outs.append(decoder.step_tokens(part, want=want).clone())
+        at += n
+    assert at >= len(tokens) and int(decoder.status.item()) == 0
+    return torch.cat(outs)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,length", [("mixed", 180), ("odd", 90), ("ones", 40), ("wide", 420)])
+def test_whole_prompts_and_every_layer(snapshots, expects, name, length, dtype):
+    config, weights, directory = snapshots[name]
+    decoder = models.load_decoder(directory, 1, 512, dtype)
+    decoder.trail = []
+    tokens = tokens_of(config, 1, length)
+    logits = run_portions(decoder, 0, tokens, [length])
+    expect, trail = hybrid_ref.forward(config, weights, tokens)
+    for index, residual in enumerate(decoder.trail):
+        check(residual, trail[index], dtype, f"layer {index}")
+    check(logits, expect, dtype, "logits")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,length", [("mixed", 170), ("odd", 70), ("ones", 30)])
+def test_token_by_token_equals_the_prompt(snapshots, expects, name, length, dtype):
+    config, _, directory = snapshots[name]
+    decoder = models.load_decoder(directory, 2, 256, dtype)
+    decoder.capture()
+    tokens = tokens_of(config, 2, length)
+    check(run_portions(decoder, 1, tokens, [1] * length), expects[name](tokens), dtype, "decoded from the first token")
+    decoder.release(1)
+    check(run_portions(decoder, 0, tokens, [length // 2] + [1] * (length - length // 2)), expects[name](tokens), dtype,
+          "prompt, then decoded")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("portion", [2, 3, 8, 9, 16, 17, 63, 64, 65])
+def test_portions_of_every_size(snapshots, expects, portion, dtype):
+    config, _, directory = snapshots["mixed"]
+    decoder = models.load_decoder(directory, 1, 256, dtype)
+    tokens = tokens_of(config, 3, 181)
+    portions = [portion] * (-(-len(tokens) // portion))
+    check(run_portions(decoder, 0, tokens, portions), expects["mixed"](tokens), dtype, f"portions of {portion}")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_portions_of_changing_size_on_the_wide_model(snapshots, expects, dtype):
+    config, _, directory = snapshots["wide"]
+    decoder = models.load_decoder(directory, 1, 512, dtype)
+    tokens = tokens_of(config, 4, 430)
+    portions = [2, 64, 1, 129, 3, 8, 9, 128, 1, 1, 60, 24]
+    check(run_portions(decoder, 0, tokens, portions), expects["wide"](tokens), dtype, "portions")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["mixed", "odd"])
+def test_batches_of_unequal_requests_equal_each_alone(snapshots, expects, name, dtype):
+    config, _, directory = snapshots[name]
+    decoder = models.load_decoder(directory, 5, 256, dtype)
+    requests = [tokens_of(config, 10 + i, n) for i, n in enumerate((120, 1, 33, 77, 64))]
+    plans = [[50, 1, 1, 30, 8, 29, 1], [0, 0, 1, 0, 0, 0, 0], [1, 1, 1, 9, 1, 19, 1], [9, 8, 60, 0, 0, 0, 0], [0, 64, 0, 0, 0, 0, 0]]
+    at, outs = [0] * 5, [[] for _ in range(5)]
+    for index in range(7):
+        parts = [request[a: a + plan[index]] for request, a, plan in zip(requests, at, plans)]
+        want = [list(range(len(part))) for part in parts]
+        logits = decoder.step_tokens(parts, want=want).clone()
+        counts = np.cumsum([0] + [len(part) for part in parts])
+        for row in range(5):
+            outs[row].append(logits[counts[row]: counts[row + 1]])
+            at[row] += len(parts[row])
+    assert int(decoder.status.item()) == 0
+    for row, request in enumerate(requests):
+        check(torch.cat(outs[row]), expects[name](request[: at[row]]), dtype, f"request {row}")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_freed_pages_and_rows_are_used_again(snapshots, expects, dtype):
+    """A pool just large enough for the windows: pages move between sequences all the time, and a row's recurrent state
+    starts over with its next request."""
+    config, _, directory = snapshots["mixed"]
+    decoder = models.load_decoder(directory, 2, 400, dtype, cache_tokens=2 * (70 + 64 + 32))
+    decoder.capture()
+    long = tokens_of(config, 20, 330)
+    outs, at = [], 0
+    other, other_at, other_outs, finished = tokens_of(config, 21, 50), 0, [], 0
+    while at < len(long):
+        n = (64, 1, 1, 20, 1, 3)[len(outs) % 6]
+        part, spare = long[at: at + n], other[other_at: other_at + (1 if n == 1 else 16)]
+        logits = decoder.step_tokens([part, spare], want=[range(len(part)), range(len(spare))]).clone()
+        outs.append(logits[: len(part)])
+        other_outs.append(logits[len(part):])
+        at += len(part)
+        other_at += len(spare)
+        if other_at == len(other):
+            check(torch.cat(other_outs), expects["mixed"](other), dtype, "short-lived request")
+            decoder.release(1)
+            finished += 1
+            other, other_at, other_outs = tokens_of(config, 22 + finished % 2, 40), 0, []
+    assert finished >= 3 and int(decoder.status.item()) == 0
+    check(torch.cat(outs), expects["mixed"](long), dtype, "long request")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_decoding(snapshots, expects, dtype):
+    config, _, directory = snapshots["mixed"]
+    decoder = models.load_decoder(directory, 1, 700, dtype, cache_tokens=112)
+    decoder.capture()
+    tokens = tokens_of(config, 5, 640)
+    check(run_portions(decoder, 0, tokens, [9] + [1] * 631), expects["mixed"](tokens), dtype, "long decoding")
+
+
+def test_a_step_without_room_changes_nothing(snapshots, expects):
+    config, _, directory = snapshots["mixed"]
+    decoder = models.load_decoder(directory, 2, 128, "float32", cache_tokens=96)
+    tokens = tokens_of(config, 6, 60)
+    first = run_portions(decoder, 0, tokens[:40], [40])
+    with pytest.raises(PageTableError):
+        decoder.step_tokens([tokens[40:], [1] * 60])
+    with pytest.raises(PageTableError):
+        decoder.step_tokens([[1] * 100, []])
+    rest = run_portions(decoder, 0, tokens[40:], [20])
+    check(torch.cat([first, rest]), expects["mixed"](tokens), "float32", "around a refused step")
+
+
+def greedy(expect, prompt, count):
+    tokens = list(prompt)
+    for _ in range(count):
+        tokens.append(int(expect(tokens)[-1].argmax()))
+    return tokens[len(prompt):]
+
+
+def test_greedy_generation_through_the_scheduler(snapshots, expects):
+    """Requests of unequal lengths join and leave a running batch of two rows, prompts in chunks."""
+    config, _, directory = snapshots["mixed"]
+    decoder = models.load_decoder(directory, 2, 256, "float32")
+    decoder.capture()
+    prompts = [tokens_of(config, 30 + i, n) for i, n in enumerate((70, 3, 41, 1))]
+    batch = RunningBatch.create(CachedDecoder(decoder, PromptChunks(16, 16)), GenerationOptions(6))
+    waiting, got = list(prompts), {}
+    while waiting or not batch.is_empty():
+        while waiting and (joined := batch.join(waiting[0])) is not None:
+            got[joined] = []
+            waiting.pop(0)
+        for token in batch.advance():
+            got[token.sequence].append(token.token)
+    assert [got[i] for i in range(4)] == [greedy(expects["mixed"], prompt, 6) for prompt in prompts]
+    assert generate_batch(CachedDecoder(decoder), prompts[:2], GenerationOptions(4)) == [got[0][:4], got[1][:4]]
+
+
+def test_device_argmax_follows_the_logits(snapshots):
+    config, _, directory = snapshots["wide"]
+    decoder = models.load_decoder(directory, 3, 64)
+    decoder.step_tokens([tokens_of(config, 40 + i, 5 + 9 * i) for i in range(3)])
+    chosen = decoder.step([1, 2, 3])
+    assert chosen.tolist() == decoder.logits.argmax(1).tolist()
+
+
+def test_command_line_generates(snapshots, expects):
+    config, _, directory = snapshots["mixed"]
+    prompts = [tokens_of(config, 50, 20), tokens_of(config, 51, 5)]
+    command = [sys.executable, "-m", "singe_b200", "generate", "--model", directory, "--dtype", "float32",
+               "--max-new-tokens", "5"] + [part for prompt in prompts for part in ("--prompt", ",".join(map(str, prompt)))]
+    result = subprocess.run(command, capture_output=True, text=True, cwd=ROOT, timeout=300)
+    assert result.returncode == 0, result.stderr[-2000:]
+    lines = [[int(t) for t in line.split(",")] for line in result.stdout.split()]
+    assert lines == [greedy(expects["mixed"], prompt, 5) for prompt in prompts]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_trace_runner(snapshots, expects, tmp_path, dtype):
+    config, _, directory = snapshots["mixed"]
+    first, second = tokens_of(config, 60, 90), tokens_of(config, 61, 30)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": first[:70], "want": [0, 69, 21]}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": first[70:72], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "x", "tokens": first[72:], "want": [17]}], "end": ["x"]},
+             {"step": 3, "entries": [{"id": "y", "tokens": second, "want": [29, 0]}], "end": ["y"]}]
+    result = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", directory, "--dtype", dtype, "--out",
+                             str(tmp_path), "--max-tokens", "100"], input="\n".join(map(json.dumps, steps)) + "\n",
+                            capture_output=True, text=True, timeout=300)
+    assert result.returncode == 0, result.stderr[-2000:]
+    assert result.stdout.split("\n")[:4] == [f"done {i}" for i in range(4)]
+    read = lambda i: torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4").reshape(-1, config["vocab"]))
+    check(read(0), expects["mixed"](first)[[0, 69, 21]], dtype, "step 0")
+    assert not (tmp_path / "1.f32").exists()
+    check(read(2), expects["mixed"](first)[[89]], dtype, "step 2")
+    check(read(3), expects["mixed"](second)[[29, 0]], dtype, "step 3")
+
+
+def test_prompts_and_short_portions_take_the_kernels_meant_for_them(snapshots, monkeypatch):
+    """bf16 steps: the tiled kernels for sizes they take, the general one otherwise."""
+    called = set()
+    original = hybrid.Ops.call
+
+    def record(self, name, *arguments):
+        called.add(name)
+        original(self, name, *arguments)
+
+    monkeypatch.setattr(hybrid.Ops, "call", record)
+    tiled = {"singe_windowed_prefill_attention_bf16", "singe_latent_decode_bf16", "singe_gated_linear_prompt_bf16",
+             "singe_gated_linear_step_bf16"}
+    for name, expected in (("mixed", True), ("odd", False)):
+        config, _, directory = snapshots[name]
+        decoder = models.load_decoder(directory, 2, 64)
+        called.clear()
+        decoder.step_tokens([tokens_of(config, 1, 40), [1, 2]])
+        assert (tiled <= called) == expected and ("singe_paged_attention_bf16" in called) != expected
