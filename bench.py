@@ -709,6 +709,21 @@ def run_only(args):
     print(json.dumps({"only": args.only, "launches": args.warmup + args.steps, "device_error": ops.take_device_error()}))
 
 
+def run_model(args):
+    """``--model kavalorn``: one JSON line of decode and prompt throughput and kernel rooflines (bench_hybrid.py)."""
+    import torch
+
+    if not torch.cuda.is_available():
+        raise SystemExit("bench.py needs a CUDA device: the operators have no CPU path")
+    import bench_hybrid
+
+    peaks = measured_peaks()
+    with ClockSampler(0) as clocks:
+        figures = bench_hybrid.run(peaks)
+    print(json.dumps({"model": args.model, "dtype": "bf16", "data": "synthetic", "peaks": peaks, "clocks": clocks.summary(),
+                      "sizes": figures}), flush=True)
+
+
 def main():
     parser = argparse.ArgumentParser()
     parser.add_argument("--gpus", type=int, default=1)
@@ -719,6 +734,9 @@ def main():
     parser.add_argument("--no-decode-step", action="store_true", help="skip the Llama-shaped decode step figure")
     parser.add_argument("--collective", default="peer", choices=["peer", "oneshot", "twophase", "pushall", "nccl"],
                         help="how the decode step's two collectives per layer run at --gpus > 1")
+    parser.add_argument("--model", default="", choices=["", "kavalorn"],
+                        help="instead of the headline workload: this model beside the Llama-shaped one at equal size "
+                        "(throughput and kernels; one GPU)")
     parser.add_argument("--only", default="", help="profiling aid: launch one kernel a few times and exit "
                         "(decode | paged_attention | gemm:M,N,K | prefill[:len,len,...] | kvwrite | step:LAYERS[:TP])")
     args = parser.parse_args()
@@ -728,6 +746,9 @@ def main():
         return
     if args.only:
         run_only(args)
+        return
+    if args.model:
+        run_model(args)
         return
 
     import torch

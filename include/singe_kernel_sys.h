@@ -660,14 +660,15 @@ int singe_head_linear_f32(singe_stream_t stream, float *out, const float *x, con
  * keys and values at once.  Query i belongs to sequence sequence_of[i] (a row of block_table [sequences, table_stride])
  * and sees its keys max(0, lens[i] - window) .. lens[i] - 1 (window == 0: from 0; lens[i] == 0: zeros).
  * query, out [queries, heads, latent] bf16; attn_scratch f32 [queries, splits, heads, latent] and lse_scratch
- * [queries, splits, heads].  latent: a multiple of 64 up to 512.  Page ids outside the cache set *status = 1. */
+ * [queries, splits, heads].  latent: a multiple of 64 up to 512; the cache holds finite values.  Page ids outside the cache
+ * set *status = 1. */
 int singe_latent_decode_bf16(singe_stream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
                              const void *cache, const int32_t *sequence_of, const int32_t *lens,
                              const int32_t *block_table, size_t queries, size_t heads, size_t latent, size_t page_size,
                              size_t pages, size_t sequences, size_t table_stride, size_t window, size_t splits,
                              float scale, uint32_t *status);
 /* The split count that fills the machine for a call of this shape. */
-size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t key_bound);
+size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t latent, size_t key_bound);
 
 /* Causal prompt attention with a sliding window on the tensor core (the kernel of singe_ragged_kv_prefill_attention_bf16):
  * query, out [total_query_tokens, heads, head_dim]; key and value rows of kv_row_stride elements, heads side by side.

@@ -54,11 +54,21 @@ __device__ __forceinline__ float &part(typename StatePack<VEC>::type &x, int i) 
 // One CTA per (head, sequence): token by token, the state streamed from global memory (a decode step reads and writes it
 // once).  A thread owns VEC adjacent columns and every `groups`-th key channel, so it only ever touches its own elements.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kStepThreads) gated_linear_step_kernel(const GatedLinear p) {
+__global__ void __launch_bounds__(kStepThreads, 4) gated_linear_step_kernel(const GatedLinear p) {
     using Pack = typename StatePack<VEC>::type;
     grid_launch_dependents();
-    grid_dependency_wait();
     const int head = blockIdx.x, sequence = blockIdx.y;
+    float *state = p.state + (static_cast<size_t>(sequence) * p.heads + head) * p.dim * p.vdim;
+    if (VEC == 4 && threadIdx.x < 32) {
+        // the state crosses HBM while the projection is still running (a hint: nothing is read before the wait)
+        const int bytes = p.dim * p.vdim * 4;
+        for (int at = threadIdx.x * 4096; at < bytes; at += 32 * 4096) {
+            asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<const char *>(state) + at),
+                         "r"(min(4096, bytes - at))
+                         : "memory");
+        }
+    }
+    grid_dependency_wait();
     const int tokens = p.count[sequence];
     const int row0 = p.first[sequence];
     const int tid = threadIdx.x;
@@ -81,23 +91,34 @@ __global__ void __launch_bounds__(kStepThreads) gated_linear_step_kernel(const G
     const int groups = kStepThreads / columns;
     const int column = tid % columns, group = tid / columns;
     const bool active = group < groups;
-    float *state = p.state + (static_cast<size_t>(sequence) * p.heads + head) * p.dim * p.vdim;
     const int key_at = p.heads * p.dim, value_at = 2 * p.heads * p.dim, gate_at = value_at + p.heads * p.vdim;
     const int low_at = gate_at + p.heads * p.vdim;
     bool fresh = p.context[sequence] == 0;
+    const bool in_batch = p.dim <= groups * kStepBatch && packs <= columns;  // a thread's whole share is one batch of packs
     for (int t = 0; t < tokens; ++t, fresh = false) {
+        // the share of the state is on its way while the decays are computed
+        Pack held[kStepBatch];
+        if (in_batch && active) {
+#pragma unroll
+            for (int u = 0; u < kStepBatch; ++u) {
+                const int c = group + u * groups;
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) part<VEC>(held[u], i) = 0.0f;
+                if (c < p.dim && !fresh) held[u] = (reinterpret_cast<Pack *>(state) + column)[static_cast<size_t>(c) * packs];
+            }
+        }
         const T *row = static_cast<const T *>(p.projected) + (row0 + t) * p.stride;
         for (int r = tid; r < p.rank; r += kStepThreads) low[r] = to_float<T>(row[low_at + r]);
         __syncthreads();
         for (int c = tid; c < p.dim; c += kStepThreads) {
             const int channel = head * p.dim + c;
             const T *weight = static_cast<const T *>(p.decay_weight) + static_cast<size_t>(channel) * p.rank;
-            float z = 0.0f;
-            for (int r = 0; r < p.rank; ++r) z = fmaf(to_float<T>(weight[r]), low[r], z);
-            z += to_float<T>(static_cast<const T *>(p.decay_bias)[channel]);
-            alpha[c] = expf(log_sigmoid(z) * p.inverse_tau);
             query[c] = to_float<T>(row[channel]) * p.query_scale;
             key[c] = to_float<T>(row[key_at + channel]);
+            float z = to_float<T>(static_cast<const T *>(p.decay_bias)[channel]);
+#pragma unroll 16
+            for (int r = 0; r < p.rank; ++r) z = fmaf(to_float<T>(weight[r]), low[r], z);
+            alpha[c] = expf(log_sigmoid(z) * p.inverse_tau);
         }
         __syncthreads();
         for (int base = 0; base < packs; base += columns) {
@@ -114,13 +135,14 @@ __global__ void __launch_bounds__(kStepThreads) gated_linear_step_kernel(const G
                 }
                 Pack *cell = reinterpret_cast<Pack *>(state) + pack;
                 for (int c0 = group; c0 < p.dim; c0 += groups * kStepBatch) {
-                    Pack held[kStepBatch];
+                    if (!in_batch) {
 #pragma unroll
-                    for (int u = 0; u < kStepBatch; ++u) {
-                        const int c = c0 + u * groups;
+                        for (int u = 0; u < kStepBatch; ++u) {
+                            const int c = c0 + u * groups;
 #pragma unroll
-                        for (int i = 0; i < VEC; ++i) part<VEC>(held[u], i) = 0.0f;
-                        if (c < p.dim && !fresh) held[u] = cell[static_cast<size_t>(c) * packs];
+                            for (int i = 0; i < VEC; ++i) part<VEC>(held[u], i) = 0.0f;
+                            if (c < p.dim && !fresh) held[u] = cell[static_cast<size_t>(c) * packs];
+                        }
                     }
 #pragma unroll
                     for (int u = 0; u < kStepBatch; ++u) {

@@ -12,7 +12,8 @@
 // as two terms hi + lo, x = hi + lo up to 2^-17 |x|; v is bf16 from its projection and enters as it is.  Products of two
 // split operands keep hi hi + hi lo + lo hi.  Accumulators, and the state between the blocks, are f32.
 //
-//   prepare   one CTA per (block, head): decays, the split operands and P, to scratch
+//   prepare   one warp per (block, head): decays, the split operands and P, to scratch, laid out as the next kernel's
+//             shared memory wants them (rows padded against bank conflicts), so that a block arrives in one bulk copy
 //   advance   one CTA per (segment, head): the blocks of a segment in order, the state in registers as S^T [vdim, dim], whose
 //             accumulator layout is the A-operand layout of the next product.  A warp owns 16 (or 32) value rows.
 //             A long sequence is cut into segments that run side by side: a first pass (STATE_ONLY) takes every segment
@@ -24,9 +25,27 @@ namespace singe {
 namespace {
 
 constexpr int kBlock = 16;             // tokens
-constexpr int kPrepareThreads = 128;
+constexpr int kPrepareWarps = 4;
 constexpr int kStages = 3;
 constexpr float kFactoredLimit = -60.0f;
+constexpr int kPitchP = kBlock * 2 + 16;  // bytes of a padded row of P
+
+// The operands of one (block, head), bytes: q hi, q lo, P hi, P lo, and from `state_part` on what the state needs: k hi,
+// k lo, decay.
+struct OperandLayout {
+    int pitch;  // bytes of a padded row of q or k
+    int p_hi, state_part, decay, bytes;
+};
+
+__host__ __device__ constexpr OperandLayout operand_layout(int dim_pad) {
+    OperandLayout l = {};
+    l.pitch = dim_pad * 2 + 16;
+    l.p_hi = 2 * kBlock * l.pitch;
+    l.state_part = l.p_hi + 2 * kBlock * kPitchP;
+    l.decay = l.state_part + 2 * kBlock * l.pitch;
+    l.bytes = l.decay + dim_pad * 4;
+    return l;
+}
 
 struct PromptShape {
     int heads, dim, vdim, rank;
@@ -51,11 +70,10 @@ struct PromptParams {
     float *segment_start;                     // the same shape: the state a sequence's first segment starts from
     float *segment_decay;                     // [segments, heads, dim_pad]
     float inverse_tau, query_scale, eps;
+    uint32_t *error;
 };
 
-__host__ __device__ constexpr int operand_bytes(int dim_pad) { return 4 * kBlock * dim_pad * 2 + 2 * kBlock * kBlock * 2 + dim_pad * 4; }
-
-__device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
+__host__ __device__ constexpr int operand_bytes(int dim_pad) { return operand_layout(dim_pad).bytes; }
 
 // x = hi + lo
 __device__ __forceinline__ void split_bf16(float x, __nv_bfloat16 &hi, __nv_bfloat16 &lo) {
@@ -69,169 +87,214 @@ __device__ __forceinline__ void split_pair(float x, float y, uint32_t &hi, uint3
     lo = pack2<__nv_bfloat16>(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
-__device__ __forceinline__ void load_async_16(uint32_t target, const void *source, bool valid) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(target), "l"(source), "r"(valid ? 16 : 0) : "memory");
+// Bulk copy global -> shared, completing `bytes` on the mbarrier (16-byte aligned addresses and size).
+__device__ __forceinline__ void bulk_load(uint32_t target, const void *source, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(target),
+                 "l"(source), "r"(bytes), "r"(bar)
+                 : "memory");
 }
 
-__global__ void __launch_bounds__(kPrepareThreads) gated_linear_prepare_kernel(const PromptParams p) {
+// ldmatrix_x4_trans's inverse: four 8x8 matrices out of MMA fragments, transposed.
+__device__ __forceinline__ void stmatrix_x4_trans(uint32_t address, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
+    asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};" ::"r"(address), "r"(r0), "r"(r1),
+                 "r"(r2), "r"(r3)
+                 : "memory");
+}
+
+// Shared memory of one warp of the prepare kernel, in bytes: the factored operands of P (q hi, lo, k hi, lo) and the
+// logarithms of the decays.
+__host__ __device__ constexpr int prepare_warp_bytes(int dim_pad) {
+    return 4 * kBlock * (dim_pad * 2 + 16) + kBlock * dim_pad * 4;
+}
+
+__global__ void __launch_bounds__(kPrepareWarps * 32) gated_linear_prepare_kernel(const PromptParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
     const PromptShape &s = p.shape;
-    const int block = blockIdx.x, head = blockIdx.y;
+    const int block = blockIdx.x;
     const int row0 = p.block_row[block], tokens = p.block_tokens[block];
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int pitch = s.dim_pad + 8;  // bf16 elements of a padded operand row in shared memory
-    extern __shared__ __align__(16) float prepare_shared[];
-    float *low = prepare_shared;                       // [16][rank]
-    float *query = low + kBlock * s.rank;              // [16][dim_pad]: q, scaled
-    float *key = query + kBlock * s.dim_pad;           // [16][dim_pad]
-    float *alpha = key + kBlock * s.dim_pad;           // [16][dim_pad]
-    // factored operands of P, split: q exp(a_t) and k exp(-a_j)
-    __nv_bfloat16 *fq = reinterpret_cast<__nv_bfloat16 *>(alpha + kBlock * s.dim_pad);  // hi, lo [16][pitch] each
-    __nv_bfloat16 *fk = fq + 2 * kBlock * pitch;
-    uint8_t *pack = p.operands + (static_cast<size_t>(block) * s.heads + head) * operand_bytes(s.dim_pad);
-    __nv_bfloat16 *q_hi = reinterpret_cast<__nv_bfloat16 *>(pack);
-    __nv_bfloat16 *q_lo = q_hi + kBlock * s.dim_pad, *k_hi = q_lo + kBlock * s.dim_pad, *k_lo = k_hi + kBlock * s.dim_pad;
-    __nv_bfloat16 *p_hi = k_lo + kBlock * s.dim_pad, *p_lo = p_hi + kBlock * kBlock;
-    float *decay = reinterpret_cast<float *>(p_lo + kBlock * kBlock);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const OperandLayout layout = operand_layout(s.dim_pad);
+    extern __shared__ __align__(16) uint8_t prepare_shared[];
+    float *low = reinterpret_cast<float *>(prepare_shared);  // [rank][16]
+    uint8_t *own = prepare_shared + kBlock * s.rank * 4 + warp * prepare_warp_bytes(s.dim_pad);
+    uint8_t *fq = own, *fk = own + 2 * kBlock * layout.pitch;
+    float *steps = reinterpret_cast<float *>(own + 4 * kBlock * layout.pitch);  // [16][dim_pad]
 
     const int low_at = 2 * s.heads * (s.dim + s.vdim);
-    for (int i = tid; i < kBlock * s.rank; i += kPrepareThreads) {
-        const int t = i / s.rank;
-        low[i] = t < tokens ? __bfloat162float(p.projected[(row0 + t) * p.stride + low_at + i - t * s.rank]) : 0.0f;
+    for (int i = threadIdx.x; i < kBlock * s.rank; i += blockDim.x) {
+        const int t = i / s.rank, r = i - t * s.rank;
+        low[r * kBlock + t] = t < tokens ? __bfloat162float(p.projected[(row0 + t) * p.stride + low_at + r]) : 0.0f;
     }
     __syncthreads();
+    const int head = blockIdx.y * kPrepareWarps + warp;
+    if (head >= s.heads) return;
+    uint8_t *pack = p.operands + (static_cast<size_t>(block) * s.heads + head) * layout.bytes;
+    uint8_t *q_out = pack, *k_out = pack + layout.state_part;
+    float *decay = reinterpret_cast<float *>(pack + layout.decay);
+
     bool strong = false;
-    for (int c = tid; c < s.dim_pad; c += kPrepareThreads) {
-        const bool real = c < s.dim;
+    for (int c = 2 * lane; c < s.dim_pad; c += 64) {  // a lane takes two adjacent channels
+        const bool real = c < s.dim;                   // dim is a multiple of eight
         const int channel = head * s.dim + (real ? c : 0);
-        float z[kBlock] = {};
-        if (real) {
-            const __nv_bfloat16 *weight = p.decay_weight + static_cast<size_t>(channel) * s.rank;
-            for (int r = 0; r < s.rank; ++r) {
-                const float w = __bfloat162float(weight[r]);
-#pragma unroll
-                for (int t = 0; t < kBlock; ++t) z[t] = fmaf(w, low[t * s.rank + r], z[t]);
-            }
-        }
-        const float bias = real ? __bfloat162float(p.decay_bias[channel]) : 0.0f;
-        float running = 0.0f;
-#pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            const float step = real && t < tokens ? log_sigmoid_f32(z[t] + bias) * p.inverse_tau : 0.0f;
-            alpha[t * s.dim_pad + c] = expf(step);
-            running += step;
-            z[t] = running;
-        }
-        strong = strong || running < kFactoredLimit;
-        decay[c] = expf(running);
+        uint32_t q_raw[kBlock], k_raw[kBlock];
         const __nv_bfloat16 *source = p.projected + row0 * p.stride + channel;
 #pragma unroll
         for (int t = 0; t < kBlock; ++t) {
             const bool live = real && t < tokens;
-            const float q = live ? __bfloat162float(source[t * p.stride]) * p.query_scale : 0.0f;
-            const float k = live ? __bfloat162float(source[t * p.stride + s.heads * s.dim]) : 0.0f;
-            query[t * s.dim_pad + c] = q;
-            key[t * s.dim_pad + c] = k;
-            const float decayed = q * expf(z[t]);
-            __nv_bfloat16 hi, lo;
-            split_bf16(decayed, hi, lo);
-            q_hi[t * s.dim_pad + c] = hi;
-            q_lo[t * s.dim_pad + c] = lo;
-            fq[t * pitch + c] = hi;
-            fq[(kBlock + t) * pitch + c] = lo;
-            split_bf16(k * expf(running - z[t]), hi, lo);
-            k_hi[t * s.dim_pad + c] = hi;
-            k_lo[t * s.dim_pad + c] = lo;
-            split_bf16(k * expf(fminf(-z[t], -kFactoredLimit)), hi, lo);
-            fk[t * pitch + c] = hi;
-            fk[(kBlock + t) * pitch + c] = lo;
+            q_raw[t] = live ? *reinterpret_cast<const uint32_t *>(source + t * p.stride) : 0u;
+            k_raw[t] = live ? *reinterpret_cast<const uint32_t *>(source + t * p.stride + s.heads * s.dim) : 0u;
+        }
+        float z[2][kBlock] = {};
+        if (real) {
+            const __nv_bfloat16 *weight = p.decay_weight + static_cast<size_t>(channel) * s.rank;
+#pragma unroll 4
+            for (int r = 0; r < s.rank; ++r) {
+                const float w0 = __bfloat162float(weight[r]), w1 = __bfloat162float(weight[s.rank + r]);
+#pragma unroll
+                for (int t = 0; t < kBlock; t += 4) {
+                    const float4 x = *reinterpret_cast<const float4 *>(low + r * kBlock + t);
+                    z[0][t] = fmaf(w0, x.x, z[0][t]);
+                    z[0][t + 1] = fmaf(w0, x.y, z[0][t + 1]);
+                    z[0][t + 2] = fmaf(w0, x.z, z[0][t + 2]);
+                    z[0][t + 3] = fmaf(w0, x.w, z[0][t + 3]);
+                    z[1][t] = fmaf(w1, x.x, z[1][t]);
+                    z[1][t + 1] = fmaf(w1, x.y, z[1][t + 1]);
+                    z[1][t + 2] = fmaf(w1, x.z, z[1][t + 2]);
+                    z[1][t + 3] = fmaf(w1, x.w, z[1][t + 3]);
+                }
+            }
+        }
+        float total[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const float bias = real ? __bfloat162float(p.decay_bias[channel + i]) : 0.0f;
+            float running = 0.0f;
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) {
+                const float x = z[i][t] + bias;
+                // log(sigmoid(x)) / tau, without cancellation for either sign
+                const float step = real && t < tokens ? (fminf(x, 0.0f) - log1pf(__expf(-fabsf(x)))) * p.inverse_tau : 0.0f;
+                steps[t * s.dim_pad + c + i] = step;
+                running += step;
+                z[i][t] = running;
+            }
+            total[i] = running;
+        }
+        const bool factors = fminf(total[0], total[1]) >= kFactoredLimit;
+        strong = strong || !factors;
+        const float whole[2] = {__expf(total[0]), __expf(total[1])};
+        *reinterpret_cast<float2 *>(decay + c) = make_float2(whole[0], whole[1]);
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            float before[2], after[2], back[2];  // exp(a_t), exp(A - a_t), exp(-a_t)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                before[i] = __expf(z[i][t]);
+                if (factors) {
+                    back[i] = __fdividef(1.0f, before[i]);
+                    after[i] = whole[i] * back[i];
+                } else {
+                    back[i] = __expf(fminf(-z[i][t], -kFactoredLimit));
+                    after[i] = __expf(total[i] - z[i][t]);
+                }
+            }
+            const float q0 = __uint_as_float(q_raw[t] << 16) * p.query_scale, q1 = __uint_as_float(q_raw[t] & 0xffff0000u) * p.query_scale;
+            const float k0 = __uint_as_float(k_raw[t] << 16), k1 = __uint_as_float(k_raw[t] & 0xffff0000u);
+            const int at = t * layout.pitch + c * 2, low_half = kBlock * layout.pitch;
+            uint32_t hi, lo;
+            split_pair(q0 * before[0], q1 * before[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(q_out + at) = hi;
+            *reinterpret_cast<uint32_t *>(q_out + low_half + at) = lo;
+            *reinterpret_cast<uint32_t *>(fq + at) = hi;
+            *reinterpret_cast<uint32_t *>(fq + low_half + at) = lo;
+            split_pair(k0 * after[0], k1 * after[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(k_out + at) = hi;
+            *reinterpret_cast<uint32_t *>(k_out + low_half + at) = lo;
+            split_pair(k0 * back[0], k1 * back[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(fk + at) = hi;
+            *reinterpret_cast<uint32_t *>(fk + low_half + at) = lo;
         }
     }
-    if (__syncthreads_or(strong ? 1 : 0) == 0) {
+    __syncwarp();
+    uint8_t *p_hi = pack + layout.p_hi, *p_lo = p_hi + kBlock * kPitchP;
+    if (!__any_sync(0xffffffffu, strong)) {
         // P = (q exp(a)) (k exp(-a))^T, one 16 x 16 product of split operands
-        if (warp == 0) {
-            float acc[2][4] = {};
-            for (int k0 = 0; k0 < s.dim_pad; k0 += 16) {
-                uint32_t a[2][4], b[2][4];
+        float acc[2][4] = {};
+        const uint32_t a_at = smem_u32(fq) + (lane & 15) * layout.pitch + (lane >> 4) * 16;
+        const uint32_t b_at = smem_u32(fk) + ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch + ((lane >> 3) & 1) * 16;
+        for (int k0 = 0; k0 < s.dim_pad; k0 += 16) {
+            uint32_t a[2][4], b[2][4];
 #pragma unroll
-                for (int part = 0; part < 2; ++part) {
-                    ldmatrix_x4(smem_u32(fq + (part * kBlock + (lane & 15)) * pitch + k0 + (lane >> 4) * 8), a[part][0], a[part][1],
-                                a[part][2], a[part][3]);
-                    ldmatrix_x4(smem_u32(fk + (part * kBlock + (lane & 7) + ((lane >> 4) << 3)) * pitch + k0 + ((lane >> 3) & 1) * 8),
-                                b[part][0], b[part][1], b[part][2], b[part][3]);
-                }
-#pragma unroll
-                for (int n = 0; n < 2; ++n) {
-                    mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[0][2 * n], b[0][2 * n + 1]);
-                    mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[1][2 * n], b[1][2 * n + 1]);
-                    mma_m16n8k16<__nv_bfloat16>(acc[n], a[1][0], a[1][1], a[1][2], a[1][3], b[0][2 * n], b[0][2 * n + 1]);
-                }
+            for (int half = 0; half < 2; ++half) {
+                const uint32_t offset = half * kBlock * layout.pitch + k0 * 2;
+                ldmatrix_x4(a_at + offset, a[half][0], a[half][1], a[half][2], a[half][3]);
+                ldmatrix_x4(b_at + offset, b[half][0], b[half][1], b[half][2], b[half][3]);
             }
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-#pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    const int t = (lane >> 2) + half * 8, j = n * 8 + (lane & 3) * 2;
-                    const float x = j <= t ? acc[n][2 * half] : 0.0f, y = j + 1 <= t ? acc[n][2 * half + 1] : 0.0f;
-                    uint32_t hi, lo;
-                    split_pair(x, y, hi, lo);
-                    *reinterpret_cast<uint32_t *>(p_hi + t * kBlock + j) = hi;
-                    *reinterpret_cast<uint32_t *>(p_lo + t * kBlock + j) = lo;
-                }
+                mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[0][2 * n], b[0][2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[1][2 * n], b[1][2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(acc[n], a[1][0], a[1][1], a[1][2], a[1][3], b[0][2 * n], b[0][2 * n + 1]);
             }
         }
-    } else {
-        // Decays too strong to factor: k_j is carried to the later tokens by the decays themselves, one multiplication a
-        // token.  A warp takes four columns j, its lanes the channels; lane pair l ends up with the sum of row t = l.
-        for (int j = warp; j < kBlock; j += kPrepareThreads / 32) {
-            float sum[kBlock] = {};
-            for (int c = lane; c < s.dim_pad; c += 32) {
-                float carried = key[j * s.dim_pad + c];
 #pragma unroll
-                for (int t = 0; t < kBlock; ++t) {
-                    if (t > j) carried *= alpha[t * s.dim_pad + c];
-                    if (t >= j) sum[t] = fmaf(query[t * s.dim_pad + c], carried, sum[t]);
-                }
-            }
+        for (int n = 0; n < 2; ++n) {
 #pragma unroll
-            for (int half = 8; half >= 1; half >>= 1) {
-                const bool upper = (lane & (2 * half)) != 0;
+            for (int half = 0; half < 2; ++half) {
+                const int t = (lane >> 2) + half * 8, j = n * 8 + (lane & 3) * 2;
+                const float x = j <= t ? acc[n][2 * half] : 0.0f, y = j + 1 <= t ? acc[n][2 * half + 1] : 0.0f;
+                uint32_t hi, lo;
+                split_pair(x, y, hi, lo);
+                *reinterpret_cast<uint32_t *>(p_hi + t * kPitchP + j * 2) = hi;
+                *reinterpret_cast<uint32_t *>(p_lo + t * kPitchP + j * 2) = lo;
+            }
+        }
+        return;
+    }
+    // Decays too strong to factor: k_j is carried to the later tokens by the decays themselves, one multiplication a token.
+    // The lanes are the channels; lane pair l ends up with the sum of row t = l.
+    const __nv_bfloat16 *queries = p.projected + row0 * p.stride + head * s.dim, *keys = queries + s.heads * s.dim;
+    for (int j = 0; j < kBlock; ++j) {
+        float sum[kBlock] = {};
+        for (int c = lane; c < s.dim && j < tokens; c += 32) {
+            float carried = __bfloat162float(keys[j * p.stride + c]) * p.query_scale;
 #pragma unroll
-                for (int i = 0; i < half; ++i) {
-                    const float sent = upper ? sum[i] : sum[i + half];
-                    const float kept = upper ? sum[i + half] : sum[i];
-                    sum[i] = kept + __shfl_xor_sync(0xffffffffu, sent, 2 * half);
-                }
+            for (int t = 0; t < kBlock; ++t) {
+                if (t > j) carried *= __expf(steps[t * s.dim_pad + c]);
+                if (t >= j && t < tokens) sum[t] = fmaf(__bfloat162float(queries[t * p.stride + c]), carried, sum[t]);
             }
-            const float value = sum[0] + __shfl_xor_sync(0xffffffffu, sum[0], 1);
-            if ((lane & 1) == 0) {
-                const int t = lane >> 1;
-                __nv_bfloat16 hi, lo;
-                split_bf16(t >= j ? value : 0.0f, hi, lo);
-                p_hi[t * kBlock + j] = hi;
-                p_lo[t * kBlock + j] = lo;
+        }
+#pragma unroll
+        for (int half = 8; half >= 1; half >>= 1) {
+            const bool upper = (lane & (2 * half)) != 0;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float sent = upper ? sum[i] : sum[i + half];
+                const float kept = upper ? sum[i + half] : sum[i];
+                sum[i] = kept + __shfl_xor_sync(0xffffffffu, sent, 2 * half);
             }
+        }
+        const float value = sum[0] + __shfl_xor_sync(0xffffffffu, sum[0], 1);
+        if ((lane & 1) == 0) {
+            const int t = lane >> 1;
+            __nv_bfloat16 hi, lo;
+            split_bf16(t >= j ? value : 0.0f, hi, lo);
+            *reinterpret_cast<__nv_bfloat16 *>(p_hi + t * kPitchP + j * 2) = hi;
+            *reinterpret_cast<__nv_bfloat16 *>(p_lo + t * kPitchP + j * 2) = lo;
         }
     }
 }
 
-// Shared-memory stage of the advance kernel (bytes): q hi, q lo, k hi, k lo, P hi, P lo, decay, v, g with padded rows.
+// Shared-memory stage of the advance kernel (bytes): the operands as prepared, then v and g with padded rows.
 struct StageLayout {
-    int pitch_k, pitch_v;  // bytes of a row
-    int k_hi, p_hi, decay, v, g, bytes;
+    int pitch_v, v, g, bytes;
 };
-
-constexpr int kPitchP = kBlock * 2 + 16;
 
 __host__ __device__ inline StageLayout stage_layout(int dim_pad, int vdim_pad) {
     StageLayout l;
-    l.pitch_k = dim_pad * 2 + 16;
     l.pitch_v = vdim_pad * 2 + 16;
-    l.k_hi = 2 * kBlock * l.pitch_k;
-    l.p_hi = 4 * kBlock * l.pitch_k;
-    l.decay = l.p_hi + 2 * kBlock * kPitchP;
-    l.v = l.decay + dim_pad * 4;
+    l.v = operand_bytes(dim_pad);
     l.g = l.v + kBlock * l.pitch_v;
     l.bytes = l.g + kBlock * l.pitch_v;
     return l;
@@ -251,9 +314,22 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
     if (STATE_ONLY && last) return;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
     const int g = lane >> 2, q2 = (lane & 3) * 2;
+    constexpr OperandLayout kOperands = operand_layout(kDim);
     const StageLayout layout = stage_layout(kDim, s.vdim_pad);
     extern __shared__ __align__(128) uint8_t advance_shared[];
-    float *squares = reinterpret_cast<float *>(advance_shared + kStages * layout.bytes);  // [warps][16]
+    float *squares = reinterpret_cast<float *>(advance_shared + kStages * layout.bytes);  // [8 or more][16]
+    const uint32_t bars = smem_u32(squares + max(warps, 8) * kBlock);
+    // Nothing of a stage may hold a NaN: rows past a short block and columns past vdim meet zeros in the products.
+    for (int i = tid; i < kStages * layout.bytes / 16; i += blockDim.x) {
+        reinterpret_cast<uint4 *>(advance_shared)[i] = make_uint4(0u, 0u, 0u, 0u);
+    }
+    for (int i = tid; i < max(warps, 8) * kBlock; i += blockDim.x) squares[i] = 0.0f;
+    if (tid == 0) {
+        for (int i = 0; i < kStages; ++i) mbar_init(bars + 8 * i, 1);
+        mbar_init_fence();
+    }
+    fence_proxy_async_shared();
+    __syncthreads();
     const size_t state_size = static_cast<size_t>(s.vdim_pad) * kDim;
     const size_t slot = static_cast<size_t>(segment) * s.heads + head;
     const int value0 = warp * MT * 16;
@@ -313,52 +389,55 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
         }
     }
 
+    // One warp brings a block in: the operands in one bulk copy, v and g row by row.
     auto load_block = [&](int index) {
+        if (warp != 0) return;
         const int block = first_block + index;
+        const uint32_t bar = bars + 8 * (index % kStages);
         const uint32_t stage = smem_u32(advance_shared) + (index % kStages) * layout.bytes;
-        const uint8_t *pack = p.operands + (static_cast<size_t>(block) * s.heads + head) * operand_bytes(kDim);
-        constexpr int kPieces = kDim / 8;
-        // the state-only pass needs no queries
-        for (int i = tid + (STATE_ONLY ? 2 * kBlock * kPieces : 0); i < 4 * kBlock * kPieces; i += blockDim.x) {
-            load_async_16(stage + (i / kPieces) * layout.pitch_k + (i % kPieces) * 16, pack + i * 16, true);
-        }
-        const uint8_t *tail = pack + 4 * kBlock * kDim * 2;
-        if (!STATE_ONLY) {
-            for (int i = tid; i < 2 * kBlock * 2; i += blockDim.x) {
-                load_async_16(stage + layout.p_hi + (i >> 1) * kPitchP + (i & 1) * 16, tail + i * 16, true);
-            }
-        }
-        for (int i = tid; i < kDim / 4; i += blockDim.x) {
-            load_async_16(stage + layout.decay + i * 16, tail + 2 * kBlock * kBlock * 2 + i * 16, true);
-        }
         const int row0 = p.block_row[block], tokens = p.block_tokens[block];
-        const int value_pieces = s.vdim_pad / 8;
-        const __nv_bfloat16 *values = p.projected + 2 * s.heads * s.dim + head * s.vdim;
-        for (int i = tid; i < kBlock * value_pieces; i += blockDim.x) {
-            const int t = i / value_pieces, piece = i - t * value_pieces;
-            const bool valid = t < tokens && piece * 8 < s.vdim;
-            const __nv_bfloat16 *source = values + (row0 + (valid ? t : 0)) * p.stride + (valid ? piece * 8 : 0);
-            load_async_16(stage + layout.v + t * layout.pitch_v + piece * 16, source, valid);
-            if (!STATE_ONLY) {
-                load_async_16(stage + layout.g + t * layout.pitch_v + piece * 16, source + s.heads * s.vdim, valid);
-            }
+        constexpr uint32_t kFrom = STATE_ONLY ? kOperands.state_part : 0, kBytes = kOperands.bytes - kFrom;
+        const uint32_t row_bytes = s.vdim * 2;
+        if (lane == 0) {
+            mbar_expect_tx(bar, kBytes + tokens * row_bytes * (STATE_ONLY ? 1 : 2));
+            bulk_load(stage + kFrom, p.operands + (static_cast<size_t>(block) * s.heads + head) * kOperands.bytes + kFrom, kBytes, bar);
+        }
+        __syncwarp();
+        const int t = lane & 15;
+        if (t < tokens && (lane < 16 || !STATE_ONLY)) {
+            const __nv_bfloat16 *source = p.projected + (row0 + t) * p.stride + 2 * s.heads * s.dim +
+                                          (lane < 16 ? 0 : s.heads * s.vdim) + head * s.vdim;
+            bulk_load(stage + (lane < 16 ? layout.v : layout.g) + t * layout.pitch_v, source, row_bytes, bar);
         }
     };
-    for (int i = 0; i < kStages - 1; ++i) {
-        if (i < blocks) load_block(i);
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    }
+    for (int i = 0; i < kStages - 1 && i < blocks; ++i) load_block(i);
+    bool failed = false;
     float kept[2 * KT][2];  // product of the segment's decays (STATE_ONLY)
     if (STATE_ONLY) {
 #pragma unroll
         for (int n = 0; n < 2 * KT; ++n) kept[n][0] = kept[n][1] = 1.0f;
     }
 
+    const float inverse_vdim = 1.0f / static_cast<float>(s.vdim);
+    float weight[MT][2];
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int v = value0 + m * 16 + g + half * 8;
+            weight[m][half] = v < s.vdim ? __bfloat162float(p.norm_weight[v]) : 0.0f;
+        }
+    }
+
     for (int index = 0; index < blocks; ++index) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
-        __syncthreads();  // the block has arrived for every thread, and everyone is done with the stage loaded next
+        const bool arrived = mbar_wait(bars + 8 * (index % kStages), (index / kStages) & 1);
+        fence_proxy_async_shared();
+        // the block has arrived for every thread, and everyone is done with the stage loaded next
+        if (__syncthreads_or(arrived ? 0 : 1) != 0) {
+            failed = true;
+            break;
+        }
         if (index + kStages - 1 < blocks) load_block(index + kStages - 1);
-        asm volatile("cp.async.commit_group;" ::: "memory");
         uint8_t *here = advance_shared + (index % kStages) * layout.bytes;
         const uint32_t stage = smem_u32(here);
 
@@ -371,14 +450,15 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
         }
         float o[MT][2][4] = {};
         if (!STATE_ONLY) {
+            float cross[MT][2][4] = {};  // the small terms, a dependency chain of their own
             // ---- o^T = S^T (q exp(a))^T ----
             const int t = (lane & 7) + ((lane >> 4) << 3);
 #pragma unroll
             for (int kt = 0; kt < KT; ++kt) {
-                const uint32_t at = stage + t * layout.pitch_k + (kt * 16 + ((lane >> 3) & 1) * 8) * 2;
+                const uint32_t at = stage + t * kOperands.pitch + (kt * 16 + ((lane >> 3) & 1) * 8) * 2;
                 uint32_t hi[4], lo[4];
                 ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
-                ldmatrix_x4(at + kBlock * layout.pitch_k, lo[0], lo[1], lo[2], lo[3]);
+                ldmatrix_x4(at + kBlock * kOperands.pitch, lo[0], lo[1], lo[2], lo[3]);
 #pragma unroll
                 for (int m = 0; m < MT; ++m) {
                     uint32_t sh[4], sl[4];
@@ -389,14 +469,14 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
 #pragma unroll
                     for (int n = 0; n < 2; ++n) {
                         mma_m16n8k16<__nv_bfloat16>(o[m][n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
-                        mma_m16n8k16<__nv_bfloat16>(o[m][n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
-                        mma_m16n8k16<__nv_bfloat16>(o[m][n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+                        mma_m16n8k16<__nv_bfloat16>(cross[m][n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+                        mma_m16n8k16<__nv_bfloat16>(cross[m][n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
                     }
                 }
             }
             // ---- o^T += v^T P^T ----
             {
-                const uint32_t at = stage + layout.p_hi + t * kPitchP + ((lane >> 3) & 1) * 16;
+                const uint32_t at = stage + kOperands.p_hi + t * kPitchP + ((lane >> 3) & 1) * 16;
                 uint32_t hi[4], lo[4];
                 ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
                 ldmatrix_x4(at + kBlock * kPitchP, lo[0], lo[1], lo[2], lo[3]);
@@ -405,21 +485,29 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
 #pragma unroll
                     for (int n = 0; n < 2; ++n) {
                         mma_m16n8k16<__nv_bfloat16>(o[m][n], value[m][0], value[m][1], value[m][2], value[m][3], hi[2 * n], hi[2 * n + 1]);
-                        mma_m16n8k16<__nv_bfloat16>(o[m][n], value[m][0], value[m][1], value[m][2], value[m][3], lo[2 * n], lo[2 * n + 1]);
+                        mma_m16n8k16<__nv_bfloat16>(cross[m][n], value[m][0], value[m][1], value[m][2], value[m][3], lo[2 * n], lo[2 * n + 1]);
                     }
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) o[m][n][i] += cross[m][n][i];
                 }
             }
         }
         // ---- S^T = S^T exp(A) + v^T (k exp(A - a)) ----
 #pragma unroll
         for (int kt = 0; kt < KT; ++kt) {
-            const uint32_t at = stage + layout.k_hi + (lane & 15) * layout.pitch_k + (kt * 16 + (lane >> 4) * 8) * 2;
+            const uint32_t at = stage + kOperands.state_part + (lane & 15) * kOperands.pitch + (kt * 16 + (lane >> 4) * 8) * 2;
             uint32_t hi[4], lo[4];
             ldmatrix_x4_trans(at, hi[0], hi[1], hi[2], hi[3]);
-            ldmatrix_x4_trans(at + kBlock * layout.pitch_k, lo[0], lo[1], lo[2], lo[3]);
+            ldmatrix_x4_trans(at + kBlock * kOperands.pitch, lo[0], lo[1], lo[2], lo[3]);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                const float2 d = *reinterpret_cast<const float2 *>(here + layout.decay + (kt * 16 + n * 8 + q2) * 4);
+                const float2 d = *reinterpret_cast<const float2 *>(here + kOperands.decay + (kt * 16 + n * 8 + q2) * 4);
                 if (STATE_ONLY) {
                     kept[2 * kt + n][0] *= d.x;
                     kept[2 * kt + n][1] *= d.y;
@@ -452,34 +540,42 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
                 }
             }
             __syncthreads();
+            // every lane adds up one warp's (or two warps') squares of its four tokens, then the eight lanes of a column meet
             float scale[2][2];
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-#pragma unroll
-                for (int i = 0; i < 2; ++i) {
-                    float total = 0.0f;
-                    for (int w = 0; w < warps; ++w) total += squares[w * kBlock + n * 8 + q2 + i];
-                    scale[n][i] = 1.0f / sqrtf(total / static_cast<float>(s.vdim) + p.eps);
+                float2 total = *reinterpret_cast<const float2 *>(squares + g * kBlock + n * 8 + q2);
+                if (warps > 8 && g + 8 < warps) {
+                    const float2 more = *reinterpret_cast<const float2 *>(squares + (g + 8) * kBlock + n * 8 + q2);
+                    total.x += more.x;
+                    total.y += more.y;
                 }
+#pragma unroll
+                for (int d = 4; d <= 16; d <<= 1) {
+                    total.x += __shfl_xor_sync(0xffffffffu, total.x, d);
+                    total.y += __shfl_xor_sync(0xffffffffu, total.y, d);
+                }
+                scale[n][0] = rsqrtf(total.x * inverse_vdim + p.eps);
+                scale[n][1] = rsqrtf(total.y * inverse_vdim + p.eps);
             }
-            __nv_bfloat16 *gates = reinterpret_cast<__nv_bfloat16 *>(here + layout.g);  // overwritten by the result
-            const int pitch = layout.pitch_v / 2;
+            // the gates come out of shared memory in the layout of o^T, and the result goes back to where they were
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
+                const uint32_t at = stage + layout.g + ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch_v +
+                                    (value0 + m * 16 + ((lane >> 3) & 1) * 8) * 2;
+                uint32_t gate[4];
+                ldmatrix_x4_trans(at, gate[0], gate[1], gate[2], gate[3]);
 #pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    const int v = value0 + m * 16 + g + half * 8;
-                    const float weight = v < s.vdim ? __bfloat162float(p.norm_weight[v]) : 0.0f;
+                for (int n = 0; n < 2; ++n) {
 #pragma unroll
-                    for (int n = 0; n < 2; ++n) {
-#pragma unroll
-                        for (int i = 0; i < 2; ++i) {
-                            __nv_bfloat16 *cell = gates + (n * 8 + q2 + i) * pitch + v;
-                            const float gate = __bfloat162float(*cell);
-                            *cell = __float2bfloat16_rn(o[m][n][2 * half + i] * scale[n][i] * weight * silu_fast(gate));
-                        }
+                    for (int half = 0; half < 2; ++half) {
+                        const uint32_t pair = gate[2 * n + half];
+                        const float x = o[m][n][2 * half] * scale[n][0] * weight[m][half] * silu_fast(__uint_as_float(pair << 16));
+                        const float y = o[m][n][2 * half + 1] * scale[n][1] * weight[m][half] * silu_fast(__uint_as_float(pair & 0xffff0000u));
+                        gate[2 * n + half] = pack2<__nv_bfloat16>(x, y);
                     }
                 }
+                stmatrix_x4_trans(at, gate[0], gate[1], gate[2], gate[3]);
             }
             __syncthreads();
             const int block = first_block + index;
@@ -488,12 +584,15 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
             for (int i = tid; i < tokens * pieces; i += blockDim.x) {
                 const int t = i / pieces, piece = i - t * pieces;
                 *reinterpret_cast<uint4 *>(p.out + (row0 + t) * p.out_stride + head * s.vdim + piece * 8) =
-                    *reinterpret_cast<const uint4 *>(gates + t * pitch + piece * 8);
+                    *reinterpret_cast<const uint4 *>(here + layout.g + t * layout.pitch_v + piece * 16);
             }
         }
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-
+    if (failed) {
+        if (tid == 0) report_status(p.error, kStatusWaitTimeout);
+        linger_after_timeout();
+        return;
+    }
     if (STATE_ONLY) {
         float *end = p.segment_state + slot * state_size;
 #pragma unroll
@@ -530,7 +629,7 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
 template <int KT, int MT>
 int launch_advance(cudaStream_t stream, const PromptParams &p, size_t segments, bool cut, int warps) {
     const StageLayout layout = stage_layout(KT * 16, p.shape.vdim_pad);
-    const int bytes = kStages * layout.bytes + warps * kBlock * 4;
+    const int bytes = kStages * layout.bytes + (warps > 8 ? warps : 8) * kBlock * 4 + kStages * 8;
     if (bytes > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     static int configured[kMaxDevices] = {0};
     static int configured_state[kMaxDevices] = {0};
@@ -631,13 +730,14 @@ int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_
     p.query_scale = query_scale;
     p.eps = eps;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const size_t shared = (kBlock * rank + 3 * kBlock * dim_pad) * sizeof(float) + 4 * kBlock * (dim_pad + 8) * 2;
+    p.error = device_error_word();
+    const size_t shared = kBlock * rank * sizeof(float) + kPrepareWarps * prepare_warp_bytes(dim_pad);
     if (shared > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     static int configured[kMaxDevices] = {0};
     SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_prepare_kernel, static_cast<int>(shared), configured));
     SINGE_CUDA_TRY(launch_dependent(gated_linear_prepare_kernel,
-                                    dim3(static_cast<unsigned>(blocks), static_cast<unsigned>(heads)), dim3(kPrepareThreads),
-                                    shared, s, kLaunchGlue, 1, p));
+                                    dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((heads + kPrepareWarps - 1) / kPrepareWarps)),
+                                    dim3(kPrepareWarps * 32), shared, s, kLaunchGlue, 1, p));
     const bool segmented = cut != 0;
 #define SINGE_ADVANCE(KT_, MT_) \
     if (dim_pad == KT_ * 16 && value_tiles == MT_) return launch_advance<KT_, MT_>(s, p, segment_count, segmented, warps);

@@ -4,14 +4,13 @@
 // with q already multiplied into the latent space.  A sliding window bounds the keys of a query.
 //
 // The cache is the traffic: a tile of 64 cached rows is read from HBM once for up to 32 heads and used twice, as keys and
-// as values.  One CTA per (query, split of its keys, 32 heads), one warp per 64 columns of the latent:
-//   load      a warp copies its own 64-column slice of the tile (cp.async, two tiles in flight) and is the only reader of it
-//   scores    its share of q . c over its 64 columns (q stays in registers), f32 partials to shared memory
-//   softmax   partials of all warps summed, f32 online softmax, weights to shared memory as bf16
-//   values    weights x its slice into f32 accumulators [heads, 64]
-// mma.sync m16n8k16: at 32 heads the tile costs about 64 flops per byte read, well under what HBM leaves room for.
-// With more than one split the normalised partial and its log-sum-exp (base 2) go to scratch and a second kernel folds them.
+// as values.  Two kernels:
+//   latent_decode_tcgen05_kernel  pages of 8, 16, 32 or a multiple of 64 tokens: tiles by TMA, both products on the fifth-
+//                                 generation tensor core with the heads as the N side, scores and outputs in tensor memory
+//   latent_decode_kernel          any page size: cp.async and mma.sync
+// With more than one split the normalised partial and its log-sum-exp (base 2) go to scratch and a third kernel folds them.
 #include "common.cuh"
+#include "tcgen05.cuh"
 
 namespace singe {
 namespace {
@@ -34,6 +33,7 @@ struct LatentDecode {
     int heads, latent, page_size, pages, sequences, table_stride, window, splits;
     float scale_log2;
     uint32_t *status;
+    uint32_t *error;
 };
 
 __device__ __forceinline__ void copy_async_16(uint32_t target, const void *source, bool valid) {
@@ -56,6 +56,12 @@ int latent_shared_bytes(int warps, int head_tiles) {
            head_tiles * 16 * kWeightStride * 2 + 3 * head_tiles * 16 * 4;
 }
 
+// ---- any page size ----
+// One CTA per (query, split of its keys, 32 heads), one warp per 64 columns of the latent:
+//   load      a warp copies its own 64-column slice of the tile (cp.async, two tiles in flight) and is the only reader of it
+//   scores    its share of q . c over its 64 columns (q stays in registers), f32 partials to shared memory
+//   softmax   partials of all warps summed, f32 online softmax, weights to shared memory as bf16
+//   values    weights x its slice into f32 accumulators [heads, 64]
 template <int MT>  // 16-head tiles of a CTA
 __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentDecode p) {
     constexpr int kHeads = MT * 16;
@@ -279,6 +285,344 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentDecod
     }
 }
 
+// ---- tcgen05 ----
+// One CTA per (query, split of its keys, 32 heads); heads past the last one are zero rows of q.
+//   warp 0     TMA producer: q once, then tiles of 64 keys: one box per (page, 64 latent columns), SWIZZLE_128B, stored as
+//              [64-column chunk][64 keys][128 bytes]
+//   warp 1     MMA issuer and owner of tensor memory:
+//                S^T [keys, heads] = C q^T: A = the tile, K-major.  M is 128: rows 64.. read the chunk behind (or what lies
+//                behind the last one) and give scores nobody reads.
+//                O^T [latent, heads] += C^T P^T: A = the same tile, MN-major, 128 latent columns a product; B = P from
+//                shared memory.
+//              QK(t + 1) is issued before PV(t), so the tensor core works while the softmax of tile t runs.
+//   warps 2-5  softmax and epilogue.  A thread is a key: its tensor-memory lane holds the key's scores of all heads.  The
+//              tile's maximum per head comes from a butterfly across the lanes; O and the sums are re-based only when it
+//              grew by more than 2^8 over the base in use (the result does not depend on the base).
+// Tensor memory: S of even and odd tiles [0, 32) [32, 64), O^T from 64 on, 32 columns per 128 latent columns.
+// Every wait is bounded.
+constexpr int kTcHeads = 32;
+constexpr int kTcThreads = 192;
+constexpr int kTcMaxStages = 4;
+constexpr int kChunkBytes = kTileKeys * 128;       // 64 keys x 64 columns
+constexpr int kQueryChunkBytes = kTcHeads * 128;
+constexpr int kWeightBytes = kTcHeads * 128;       // P: 32 heads x 64 keys
+constexpr float kRebase = 8.0f;                    // log2 units
+
+struct LatentTcShape {
+    int chunks, stages, page_rows;  // page_rows: rows of a TMA box
+};
+
+__host__ __device__ inline int latent_tc_bytes(int chunks, int stages) {
+    // tiles, then q (also what over-reading products of the last tile touch), P twice, exchange area, barriers, alignment
+    const int query = chunks * kQueryChunkBytes > 2 * kChunkBytes ? chunks * kQueryChunkBytes : 2 * kChunkBytes;
+    return stages * chunks * kChunkBytes + query + 2 * kWeightBytes + 4 * kTcHeads * 4 + 8 * (2 * kTcMaxStages + 8) + 1024;
+}
+
+// Lane h ends up with op over all lanes of x[h].
+template <typename Op>
+__device__ __forceinline__ float transpose_reduce(float (&x)[32], int lane, Op op) {
+#pragma unroll
+    for (int half = 16; half >= 1; half >>= 1) {
+        const bool upper = (lane & half) != 0;
+#pragma unroll
+        for (int i = 0; i < half; ++i) {
+            const float sent = upper ? x[i] : x[i + half];
+            const float kept = upper ? x[i + half] : x[i];
+            x[i] = op(kept, __shfl_xor_sync(0xffffffffu, sent, half));
+        }
+    }
+    return x[0];
+}
+
+__device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+
+__global__ void __launch_bounds__(kTcThreads, 1)
+    latent_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap cache_map, const __grid_constant__ CUtensorMap query_map,
+                                 const LatentDecode p, const LatentTcShape shape) {
+    grid_dependency_wait();
+    extern __shared__ uint8_t smem_raw[];
+    const uint32_t raw = smem_u32(smem_raw);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    const int chunks = shape.chunks, stages = shape.stages;
+    const uint32_t stage_bytes = chunks * kChunkBytes;
+    const uint32_t query_at = base + stages * stage_bytes;
+    const uint32_t weights_at = query_at + max(chunks * kQueryChunkBytes, 2 * kChunkBytes);
+    const uint32_t exchange_at = weights_at + 2 * kWeightBytes;
+    float *exchange = reinterpret_cast<float *>(smem_raw + (exchange_at - raw));  // [4][32]
+    const uint32_t bars = exchange_at + 4 * kTcHeads * 4;
+    const uint32_t bar_full = bars, bar_empty = bars + 8 * kTcMaxStages;
+    const uint32_t bar_query = bars + 16 * kTcMaxStages;
+    const uint32_t bar_scores = bar_query + 8;    // [2]
+    const uint32_t bar_weights = bar_query + 24;  // [2], one arrival per softmax warp
+    const uint32_t bar_values = bar_query + 40;   // PV of a tile has retired
+    const uint32_t holder = bar_query + 48;
+    volatile uint32_t *holder_ptr = reinterpret_cast<volatile uint32_t *>(smem_raw + (holder - raw));
+
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int query = blockIdx.x, split = blockIdx.y, head0 = blockIdx.z * kTcHeads;
+    const int sequence = p.sequence_of[query];
+    const bool known = sequence >= 0 && sequence < p.sequences;
+    if (!known && threadIdx.x == 0) report_status(p.status, kStatusIndexOutOfBounds);
+    const int end_all = known ? min(p.lens[query], p.table_stride * p.page_size) : 0;
+    const int visible_from = p.window > 0 ? max(end_all - p.window, 0) : 0;
+    // tiles start on box boundaries; keys before the window are masked
+    const int start_all = visible_from / shape.page_rows * shape.page_rows;
+    const int per_split = ((max(end_all - start_all, 0) + p.splits - 1) / p.splits + kTileKeys - 1) / kTileKeys * kTileKeys;
+    const int start = start_all + split * per_split;
+    const int end = min(start + per_split, end_all);
+    const int tile_count = end > start ? (end - start + kTileKeys - 1) / kTileKeys : 0;
+
+    if (tile_count == 0) {
+        if (p.splits > 1) {
+            for (int r = threadIdx.x; r < kTcHeads; r += blockDim.x) {
+                if (head0 + r < p.heads) p.lse[(static_cast<size_t>(query) * p.splits + split) * p.heads + head0 + r] = -INFINITY;
+            }
+        } else {
+            for (int i = threadIdx.x; i < kTcHeads * p.latent; i += blockDim.x) {
+                const int head = head0 + i / p.latent;
+                if (head < p.heads) {
+                    p.out[(static_cast<size_t>(query) * p.heads + head) * p.latent + i % p.latent] = __float2bfloat16_rn(0.0f);
+                }
+            }
+        }
+        return;
+    }
+
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < stages; ++i) {
+            mbar_init(bar_full + 8 * i, 1);
+            mbar_init(bar_empty + 8 * i, 1);
+        }
+        mbar_init(bar_query, 1);
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(bar_scores + 8 * i, 1);
+            mbar_init(bar_weights + 8 * i, 4);
+        }
+        mbar_init(bar_values, 1);
+        mbar_init_fence();
+    }
+    if (warp == 1) {
+        tmem_alloc(holder, 256);
+        tmem_relinquish();
+    }
+    tcgen05_fence_before();
+    __syncthreads();
+    tcgen05_fence_after();
+    const uint32_t tmem = *holder_ptr;
+    bool failed = false;
+
+    if (warp == 0) {
+        // ---------------- TMA producer ----------------
+        if (lane == 0) {
+            prefetch_tensor_map(&cache_map);
+            prefetch_tensor_map(&query_map);
+            mbar_expect_tx(bar_query, chunks * kQueryChunkBytes);
+            for (int c = 0; c < chunks; ++c) tma_load_3d(query_at + c * kQueryChunkBytes, &query_map, bar_query, c * 64, head0, query);
+        }
+        const int32_t *table = p.table + static_cast<size_t>(sequence) * p.table_stride;
+        const int boxes = kTileKeys / shape.page_rows;  // boxes of one chunk
+        for (int tile = 0; tile < tile_count; ++tile) {
+            const int stage = tile % stages;
+            int ok = 1;
+            if (lane == 0 && tile >= stages) ok = mbar_wait(bar_empty + 8 * stage, (tile / stages - 1) & 1) ? 1 : 0;
+            if (__shfl_sync(0xffffffffu, ok, 0) == 0) {
+                failed = true;
+                break;
+            }
+            // lane b looks up box b's first cache row; boxes past the end repeat the tile's first box (masked)
+            int row = 0;
+            if (lane < boxes) {
+                int key = start + tile * kTileKeys + lane * shape.page_rows;
+                if (key >= end) key = start + tile * kTileKeys;
+                int page = table[key / p.page_size];
+                if (page < 0 || page >= p.pages) {
+                    report_status(p.status, kStatusIndexOutOfBounds);
+                    page = 0;
+                }
+                row = page * p.page_size + key % p.page_size;
+            }
+            if (lane == 0) mbar_expect_tx(bar_full + 8 * stage, stage_bytes);
+            __syncwarp();
+            for (int i = lane; i - lane < boxes * chunks; i += 32) {
+                const int box = i % boxes, chunk = i / boxes;
+                const int from = __shfl_sync(0xffffffffu, row, box);
+                if (i < boxes * chunks) {
+                    tma_load_2d(base + stage * stage_bytes + chunk * kChunkBytes + box * shape.page_rows * 128, &cache_map,
+                                bar_full + 8 * stage, chunk * 64, from);
+                }
+            }
+        }
+    } else if (warp == 1) {
+        // ---------------- MMA issuer ----------------
+        constexpr uint32_t kIdescScores = make_instr_desc(128, kTcHeads, true, 0, 0);
+        constexpr uint32_t kIdescValues = make_instr_desc(128, kTcHeads, true, 1, 0);  // A = C^T, MN-major
+        auto wait_all = [&](uint32_t bar, uint32_t parity) -> bool {
+            return __all_sync(0xffffffffu, mbar_wait(bar, parity) ? 1 : 0) != 0;
+        };
+        auto issue_values = [&](int tile) -> bool {
+            if (!wait_all(bar_weights + 8 * (tile & 1), (tile >> 1) & 1)) return false;
+            tcgen05_fence_after();
+            if (lane == 0) {
+                const int stage = tile % stages;
+                const uint32_t at = base + stage * stage_bytes;
+                const uint32_t weights = weights_at + (tile & 1) * kWeightBytes;
+                for (int m = 0; m < (chunks + 1) / 2; ++m) {
+#pragma unroll
+                    for (int ks = 0; ks < kTileKeys / 16; ++ks) {
+                        umma_ss(tmem + 64 + m * kTcHeads, make_smem_desc(at + 2 * m * kChunkBytes + ks * 2048, kChunkBytes, 1024),
+                                make_smem_desc(weights + ks * 32, 16, 1024), kIdescValues, (tile > 0 || ks > 0) ? 1u : 0u);
+                    }
+                }
+                tcgen05_commit(bar_empty + 8 * stage);
+                tcgen05_commit(bar_values);
+            }
+            __syncwarp();
+            return true;
+        };
+        if (!wait_all(bar_query, 0)) failed = true;
+        for (int tile = 0; tile < tile_count && !failed; ++tile) {
+            const int stage = tile % stages;
+            if (!wait_all(bar_full + 8 * stage, (tile / stages) & 1)) {
+                failed = true;
+                break;
+            }
+            tcgen05_fence_after();
+            if (lane == 0) {
+                const uint32_t at = base + stage * stage_bytes;
+                for (int c = 0; c < chunks; ++c) {
+#pragma unroll
+                    for (int ks = 0; ks < 4; ++ks) {
+                        umma_ss(tmem + (tile & 1) * kTcHeads, make_smem_desc(at + c * kChunkBytes + ks * 32, 16, 1024),
+                                make_smem_desc(query_at + c * kQueryChunkBytes + ks * 32, 16, 1024), kIdescScores,
+                                (c > 0 || ks > 0) ? 1u : 0u);
+                    }
+                }
+                tcgen05_commit(bar_scores + 8 * (tile & 1));
+            }
+            __syncwarp();
+            if (tile > 0 && !issue_values(tile - 1)) failed = true;
+        }
+        if (!failed && !issue_values(tile_count - 1)) failed = true;
+    } else {
+        // ---------------- softmax, epilogue ----------------
+        const int quarter = warp & 3;  // tensor-memory lanes 32 * quarter ..
+        const uint32_t lanes = static_cast<uint32_t>(quarter * 32) << 16;
+        const bool scoring = quarter < 2;  // 64 keys
+        const int my_key = quarter * 32 + lane;
+        float base_log2 = -INFINITY;       // of head `lane`; the same in all four warps
+        float bias[kTcHeads], sum[kTcHeads];
+#pragma unroll
+        for (int h = 0; h < kTcHeads; ++h) bias[h] = sum[h] = 0.0f;
+        auto maximum = [](float a, float b) { return fmaxf(a, b); };
+        auto addition = [](float a, float b) { return a + b; };
+        for (int tile = 0; tile < tile_count; ++tile) {
+            uint32_t scores[32];
+            const int key = start + tile * kTileKeys + my_key;
+            const bool visible = key >= visible_from && key < end;
+            if (!failed && !__all_sync(0xffffffffu, mbar_wait(bar_scores + 8 * (tile & 1), (tile >> 1) & 1) ? 1 : 0)) failed = true;
+            tcgen05_fence_after();
+            if (scoring && !failed) {
+                tmem_ld_x32(tmem + lanes + (tile & 1) * kTcHeads, scores);
+                tmem_wait_ld_into(scores);
+                float top[32];
+#pragma unroll
+                for (int h = 0; h < 32; ++h) {
+                    const float x = __uint_as_float(scores[h]) * p.scale_log2;
+                    scores[h] = __float_as_uint(x);
+                    top[h] = visible ? x : -INFINITY;
+                }
+                exchange[quarter * kTcHeads + lane] = transpose_reduce(top, lane, maximum);
+            }
+            softmax_barrier();
+            const float tile_top = fmaxf(exchange[lane], exchange[kTcHeads + lane]);
+            const bool grow = tile_top > base_log2 + kRebase || (base_log2 == -INFINITY && tile_top > -INFINITY);
+            if (__any_sync(0xffffffffu, grow)) {  // the same answer in all four warps
+                const float next = fmaxf(base_log2, tile_top);
+                const float factor = base_log2 == -INFINITY ? 0.0f : exp2f(base_log2 - next);
+                if (tile > 0) {
+                    // O holds P V up to the tile before
+                    if (!failed && !__all_sync(0xffffffffu, mbar_wait(bar_values, (tile - 1) & 1) ? 1 : 0)) failed = true;
+                    tcgen05_fence_after();
+                    for (int m = 0; m < (chunks + 1) / 2 && !failed; ++m) {
+                        uint32_t o[32];
+                        tmem_ld_x32(tmem + lanes + 64 + m * kTcHeads, o);
+                        tmem_wait_ld_into(o);
+#pragma unroll
+                        for (int h = 0; h < 32; ++h) {
+                            o[h] = __float_as_uint(__uint_as_float(o[h]) * __shfl_sync(0xffffffffu, factor, h));
+                        }
+                        tmem_st_x32(tmem + lanes + 64 + m * kTcHeads, o);
+                    }
+                    tmem_wait_st();
+                }
+                base_log2 = next;
+#pragma unroll
+                for (int h = 0; h < 32; ++h) {
+                    sum[h] *= __shfl_sync(0xffffffffu, factor, h);
+                    const float b = __shfl_sync(0xffffffffu, next, h);
+                    bias[h] = b == -INFINITY ? 0.0f : b;
+                }
+            }
+            if (scoring && !failed) {
+                // P[head, key], 128-byte rows with the 16-byte pieces permuted as SWIZZLE_128B has them
+                uint8_t *weights = smem_raw + (weights_at - raw) + (tile & 1) * kWeightBytes;
+                const int piece = my_key >> 3, within = (my_key & 7) * 2;
+#pragma unroll
+                for (int h = 0; h < 32; ++h) {
+                    const float x = visible ? exp2f(__uint_as_float(scores[h]) - bias[h]) : 0.0f;
+                    sum[h] += x;
+                    *reinterpret_cast<__nv_bfloat16 *>(weights + h * 128 + ((piece ^ (h & 7)) << 4) + within) = __float2bfloat16_rn(x);
+                }
+                fence_proxy_async_shared();
+            }
+            tcgen05_fence_before();
+            softmax_barrier();  // also: everyone has read the exchange area
+            if (lane == 0) mbar_arrive(bar_weights + 8 * (tile & 1));
+        }
+        grid_launch_dependents();  // late: the fold's many small CTAs would take the slots of CTAs still to come
+        // ---- O^T / sum ----
+        if (!failed && !__all_sync(0xffffffffu, mbar_wait(bar_values, (tile_count - 1) & 1) ? 1 : 0)) failed = true;
+        tcgen05_fence_after();
+        if (scoring) exchange[quarter * kTcHeads + lane] = transpose_reduce(sum, lane, addition);
+        softmax_barrier();
+        const float total = exchange[lane] + exchange[kTcHeads + lane];
+        const float inverse = total > 0.0f ? 1.0f / total : 0.0f;
+        if (p.splits > 1 && quarter == 0 && head0 + lane < p.heads) {
+            p.lse[(static_cast<size_t>(query) * p.splits + split) * p.heads + head0 + lane] =
+                total > 0.0f ? base_log2 + log2f(total) : -INFINITY;
+        }
+        for (int m = 0; m < (chunks + 1) / 2 && !failed; ++m) {
+            uint32_t o[32];
+            tmem_ld_x32(tmem + lanes + 64 + m * kTcHeads, o);
+            tmem_wait_ld_into(o);
+            const int column = m * 128 + my_key;
+            if (p.splits == 1) {
+                __nv_bfloat16 *out = p.out + (static_cast<size_t>(query) * p.heads + head0) * p.latent + column;
+#pragma unroll
+                for (int h = 0; h < 32; ++h) {
+                    const float x = __uint_as_float(o[h]) * __shfl_sync(0xffffffffu, inverse, h);
+                    if (head0 + h < p.heads && column < p.latent) out[h * p.latent] = __float2bfloat16_rn(x);
+                }
+            } else {
+                float *out = p.attn + ((static_cast<size_t>(query) * p.splits + split) * p.heads + head0) * p.latent + column;
+#pragma unroll
+                for (int h = 0; h < 32; ++h) {
+                    const float x = __uint_as_float(o[h]) * __shfl_sync(0xffffffffu, inverse, h);
+                    if (head0 + h < p.heads && column < p.latent) out[h * p.latent] = x;
+                }
+            }
+        }
+    }
+    if (failed && lane == 0) report_status(p.error, kStatusWaitTimeout);
+    if (failed) linger_after_timeout();
+    tcgen05_fence_before();
+    __syncthreads();
+    if (warp == 1) {
+        tcgen05_fence_after();
+        tmem_dealloc(tmem, 256);
+    }
+}
+
 // out[query, head] = sum over the splits of exp2(lse_s - max) * attn_s, normalised.
 __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentDecode p) {
     grid_launch_dependents();
@@ -308,6 +652,59 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentDecode 
     }
 }
 
+// Rows of a TMA box for a page size, or 0 for sizes the tcgen05 kernel does not take.
+int latent_box_rows(size_t page_size) {
+    if (page_size == 8 || page_size == 16 || page_size == 32) return static_cast<int>(page_size);
+    return page_size % 64 == 0 ? 64 : 0;
+}
+
+// Two CTAs share an SM where their tiles fit it twice.
+int latent_tc_stages(int chunks) {
+    int stages = kTcMaxStages;
+    const int limit = latent_tc_bytes(chunks, 2) <= 113 * 1024 ? 113 * 1024 : 227 * 1024;
+    while (stages > 2 && latent_tc_bytes(chunks, stages) > limit) --stages;
+    return stages;
+}
+
+int launch_fold(cudaStream_t stream, const LatentDecode &p, size_t queries) {
+    if (p.splits > 1) {
+        const int threads = (p.latent / 4 + 31) / 32 * 32;
+        SINGE_CUDA_TRY(launch_dependent(latent_combine_kernel, dim3(static_cast<unsigned>(queries), static_cast<unsigned>(p.heads)),
+                                        dim3(threads), 0, stream, kLaunchCombine, 1, p));
+    }
+    return launch_status();
+}
+
+int launch_latent_tcgen05(cudaStream_t stream, const LatentDecode &p, size_t queries, int box_rows) {
+    LatentTcShape shape;
+    shape.chunks = p.latent / 64;
+    shape.page_rows = box_rows;
+    shape.stages = latent_tc_stages(shape.chunks);
+    const int bytes = latent_tc_bytes(shape.chunks, shape.stages);
+    static int configured[kMaxDevices] = {0};
+    SINGE_CUDA_TRY(ensure_dynamic_shared(latent_decode_tcgen05_kernel, bytes, configured));
+    CUtensorMap cache_map, query_map;
+    {
+        const uint64_t dims[2] = {static_cast<uint64_t>(p.latent), static_cast<uint64_t>(p.pages) * p.page_size};
+        const uint64_t strides[1] = {static_cast<uint64_t>(p.latent) * 2};
+        const uint32_t box[2] = {64, static_cast<uint32_t>(box_rows)};
+        SINGE_TRY(encode_tensor_map(&cache_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.cache, dims, strides, box,
+                                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    }
+    {
+        const uint64_t dims[3] = {static_cast<uint64_t>(p.latent), static_cast<uint64_t>(p.heads), queries};
+        const uint64_t strides[2] = {static_cast<uint64_t>(p.latent) * 2, static_cast<uint64_t>(p.latent) * p.heads * 2};
+        const uint32_t box[3] = {64, kTcHeads, 1};
+        SINGE_TRY(encode_tensor_map(&query_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, p.query, dims, strides, box,
+                                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    }
+    const dim3 grid(static_cast<unsigned>(queries), static_cast<unsigned>(p.splits),
+                    static_cast<unsigned>((p.heads + kTcHeads - 1) / kTcHeads));
+    SINGE_CUDA_TRY(launch_dependent(latent_decode_tcgen05_kernel, grid, dim3(kTcThreads), bytes, stream, kLaunchDecode, 1,
+                                    cache_map, query_map, p, shape));
+    return launch_fold(stream, p, queries);
+}
+
 template <int MT>
 int launch_latent_decode(cudaStream_t stream, const LatentDecode &p, size_t queries) {
     const int warps = p.latent / kSlice;
@@ -317,12 +714,7 @@ int launch_latent_decode(cudaStream_t stream, const LatentDecode &p, size_t quer
     const dim3 grid(static_cast<unsigned>(queries), static_cast<unsigned>(p.splits),
                     static_cast<unsigned>((p.heads + MT * 16 - 1) / (MT * 16)));
     SINGE_CUDA_TRY(launch_dependent(latent_decode_kernel<MT>, grid, dim3(warps * 32), bytes, stream, kLaunchDecode, 1, p));
-    if (p.splits > 1) {
-        const int threads = (p.latent / 4 + 31) / 32 * 32;
-        SINGE_CUDA_TRY(launch_dependent(latent_combine_kernel, dim3(static_cast<unsigned>(queries), static_cast<unsigned>(p.heads)),
-                                        dim3(threads), 0, stream, kLaunchCombine, 1, p));
-    }
-    return launch_status();
+    return launch_fold(stream, p, queries);
 }
 
 }  // namespace
@@ -332,10 +724,14 @@ using namespace singe;
 
 extern "C" {
 
-size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t key_bound) {
-    // One CTA per SM at a time, in waves: a CTA costs a fixed ramp and a time per key; each split adds to the fold.
-    const double slots = device_sm_count();
-    const double groups = static_cast<double>((heads + 31) / 32);
+size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t latent, size_t key_bound) {
+    // CTAs run in waves; one costs a fixed ramp and a time per key (its share of what HBM gives an SM); each split adds to
+    // the fold.
+    const int chunks = static_cast<int>((latent + 63) / 64);
+    const double per_sm = latent_tc_bytes(chunks, 2) <= 113 * 1024 ? 2.0 : 1.0;
+    const double slots = device_sm_count() * per_sm;
+    const double groups = static_cast<double>((heads + kTcHeads - 1) / kTcHeads);
+    const double key_us = static_cast<double>(latent) * 2.0 * per_sm / 36e3;
     const size_t finest = key_bound / (2 * kTileKeys) > 0 ? key_bound / (2 * kTileKeys) : 1;
     size_t best = 1;
     double best_time = 1e30;
@@ -343,7 +739,7 @@ size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t key_bound
         const double ctas = static_cast<double>(queries) * groups * static_cast<double>(splits);
         const double waves = static_cast<double>(static_cast<long long>((ctas + slots - 1) / slots));
         const double keys = static_cast<double>((key_bound + splits - 1) / splits);
-        const double time = waves * (4.0 + 0.025 * keys) + (splits > 1 ? 2.0 + 0.3 * static_cast<double>(splits) : 0.0);
+        const double time = waves * (4.0 + key_us * keys) + (splits > 1 ? 2.0 + 0.3 * static_cast<double>(splits) : 0.0);
         if (time < best_time) {
             best_time = time;
             best = splits;
@@ -393,6 +789,9 @@ int singe_latent_decode_bf16(singe_stream_t stream, void *out, float *attn_scrat
     p.splits = static_cast<int>(splits);
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
+    p.error = device_error_word();
+    const int box_rows = latent_box_rows(page_size);
+    if (box_rows > 0) return launch_latent_tcgen05(static_cast<cudaStream_t>(stream), p, queries, box_rows);
     return heads <= 16 ? launch_latent_decode<1>(static_cast<cudaStream_t>(stream), p, queries)
                        : launch_latent_decode<2>(static_cast<cudaStream_t>(stream), p, queries);
 }

@@ -34,8 +34,8 @@
 // Tensor memory (all 512 columns): S_A/P_A [0,128), S_B/P_B [128,256), O_A [256,384), O_B [384,512).
 // Shared memory: Q_A, Q_B, 2 x K, 2 x V tiles of 32 KB = 192 KB.
 // Under a causal mask tile A sees one key tile less than tile B; CTAs are dispatched heaviest-first.
-// WINDOW: a query sees itself and the window - 1 keys before it.  Both tiles of a pair start at the key tile where the
-// pair's first row begins to see; a row whose first visible key lies in a later tile takes its base from that tile.
+// WINDOW: a query sees itself and the window - 1 keys before it.  A tile starts at the key tile where its first row begins
+// to see; a row whose first visible key lies in a later tile takes its base from that tile.
 // Keys have offsets and a row stride of their own, and the epilogue may gate a head's rows by a sigmoid.
 // Every mbarrier wait is bounded; on a timeout the CTA records status 2, frees tensor memory and leaves.
 #include <type_traits>
@@ -234,7 +234,7 @@ struct Item {
     int len_kv;
     int shift;      // causal mask: query row i sees keys 0 .. max(i + shift, 0); 0 for the sequence-local mask,
                     // len_kv - len_q when the queries are the sequence's last tokens
-    int start;      // first key tile either tile needs (0 unless a window hides the ones before)
+    int first[2];   // first key tile tile A / tile B needs (0 unless a window hides the ones before); A's is the lower
     int tiles[2];   // one past the last key tile tile A / tile B needs (0: no real row, or no visible key)
     int key_tiles;  // max of the two
     bool valid;     // false: the sequence's offsets leave the packed tensors
@@ -292,7 +292,7 @@ __device__ __forceinline__ Item decode_item(const PrefillParams &p, const int *c
     item.len_q = 0;
     item.len_kv = 0;
     item.shift = 0;
-    item.start = 0;
+    item.first[0] = item.first[1] = 0;
     item.tiles[0] = item.tiles[1] = 0;
     item.key_tiles = 0;
     if (seq < 0) return item;
@@ -305,7 +305,10 @@ __device__ __forceinline__ Item decode_item(const PrefillParams &p, const int *c
                                            : item.offset_kv + item.len_kv <= p.total_kv);
     if (!item.valid) return item;
     item.shift = p.causal == 2 ? item.len_kv - item.len_q : 0;
-    if (WINDOW) item.start = max(item.q0 + item.shift - p.window + 1, 0) / kTile;
+    if (WINDOW) {
+#pragma unroll
+        for (int x = 0; x < 2; ++x) item.first[x] = max(item.q0 + x * kTile + item.shift - p.window + 1, 0) / kTile;
+    }
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
         const int first = item.q0 + x * kTile;
@@ -487,7 +490,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     }
                 }
             }
-            for (int j = item.start; j < item.key_tiles && !failed; ++j, ++g) {
+            for (int j = item.first[0]; j < item.key_tiles && !failed; ++j, ++g) {
                 const int stage = g & 1;
                 const int row0 = item.offset_kv + j * kTile;
                 if (g >= 2 && !wait_lane0(bar_k_empty + stage * 8, ((g >> 1) - 1) & 1)) {
@@ -606,11 +609,11 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         };
         // first Q K^T of both tiles of `item` on key stage `stage` (already waited for)
         auto first_qk = [&](const Item &item, int x, int stage) -> bool {
-            if (item.tiles[x] == 0) return true;
+            if (item.tiles[x] == 0 || (WINDOW && item.first[x] != item.first[0])) return true;  // (tile B's may come later)
             if (!wait_all(bar_q_full + x * 8, q_uses[x] & 1)) return false;
             ++q_uses[x];
             tcgen05_fence_after();
-            issue_qk(x, stage, item.tiles[x] == item.start + 1);
+            issue_qk(x, stage, item.tiles[x] == item.first[x] + 1);
             return true;
         };
         Item item = next_item();
@@ -624,7 +627,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         }
         while (item.key_tiles > 0 && !failed) {
             const Item following = next_item();
-            for (int j = item.start; j < item.key_tiles && !failed; ++j, ++g) {
+            for (int j = item.first[0]; j < item.key_tiles && !failed; ++j, ++g) {
                 const int stage = g & 1;
                 const int next = (g + 1) & 1;
                 const bool more = j + 1 < item.key_tiles;          // this item has another key tile
@@ -636,9 +639,9 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
                     if (failed) continue;
-                    if (j < item.tiles[x]) {
+                    if (j < item.tiles[x] && (!WINDOW || j >= item.first[x])) {
                         // the previous item's epilogue must have taken O out of tensor memory
-                        if (j == item.start && o_done[x] > 0 && !wait_all(bar_o_empty + x * 8, (o_done[x] - 1) & 1)) {
+                        if (j == item.first[x] && o_done[x] > 0 && !wait_all(bar_o_empty + x * 8, (o_done[x] - 1) & 1)) {
                             failed = true;
                             continue;
                         }
@@ -649,7 +652,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                         ++p_uses[x];
                         tcgen05_fence_after();
                         const bool last = j == item.tiles[x] - 1;
-                        issue_pv(x, stage, j > item.start, last);
+                        issue_pv(x, stage, j > item.first[x], last);
                         if (last) ++o_done[x];
                     }
                     if (x == 1) {
@@ -665,7 +668,17 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                             tcgen05_fence_after();
                         }
                         if (more) {
-                            if (j + 1 < item.tiles[x]) issue_qk(x, next, j + 2 == item.tiles[x]);
+                            if (WINDOW && item.tiles[x] > 0 && item.first[x] != item.first[0] && j + 1 == item.first[x]) {
+                                if (!wait_all(bar_q_full + x * 8, q_uses[x] & 1)) {
+                                    failed = true;
+                                    continue;
+                                }
+                                ++q_uses[x];
+                                tcgen05_fence_after();
+                            }
+                            if (j + 1 < item.tiles[x] && (!WINDOW || j + 1 >= item.first[x])) {
+                                issue_qk(x, next, j + 2 == item.tiles[x]);
+                            }
                         } else if (!first_qk(following, x, next)) {
                             failed = true;
                             continue;
@@ -705,6 +718,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             T *dst = static_cast<T *>(p.out) + (token * p.heads + item.head) * HD;
             float *lse_row = lse_at(item, real ? row : 0);
             const int my_tiles = x == 0 ? item.tiles[0] : item.tiles[1];
+            const int my_first = x == 0 ? item.first[0] : item.first[1];
             if (my_tiles == 0) {
                 // No key is visible to this tile's rows: zeros and LSE -1e20.
                 if (real) {
@@ -718,7 +732,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             float row_sum = 0.0f;
             bool in_range = true;
             bool unseen = WINDOW && real;  // no key seen yet: O and the sum are zero, so the base is free
-            for (int j = item.start; j < my_tiles && !failed; ++j, ++s_uses) {
+            for (int j = my_first; j < my_tiles && !failed; ++j, ++s_uses) {
                 if (!__all_sync(0xffffffffu, mbar_wait(bar_s_full + x * 8, s_uses & 1) ? 1 : 0)) {
                     failed = true;
                     break;
@@ -732,7 +746,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                 const bool partial = __any_sync(0xffffffffu, limit < kTile);
                 const bool lower = WINDOW && __any_sync(0xffffffffu, low > 0);
 
-                if (SAFE || j == item.start || (WINDOW && __any_sync(0xffffffffu, unseen))) {
+                if (SAFE || j == my_first || (WINDOW && __any_sync(0xffffffffu, unseen))) {
                     float wanted;
                     if (WINDOW && lower) {
                         wanted = tile_max<kMaskBoth>(tmem_s, low, limit, sign);
@@ -748,7 +762,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                     // Re-base O only when some row's max grew past the threshold; then every row of the warp does.
                     const bool grow = !free_base && wanted > base_log2 + kRescaleThreshold;
                     if (__any_sync(0xffffffffu, grow)) {
-                        if (j > item.start) {
+                        if (j > my_first) {
                             const float factor = free_base ? 1.0f : exp2_approx(base_log2 - wanted);
                             row_sum *= factor;
                             scale_o_row<HD>(tmem_o, factor);

@@ -268,13 +268,30 @@ __global__ void __launch_bounds__(1024)
     const float *row = logits + blockIdx.x * stride;
     float best = -INFINITY;
     int where = 0x7fffffff;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float value = row[c];
+    auto look = [&](float value, int c) {  // in ascending order: a later equal value never replaces an earlier one
         if (value > best) {
             best = value;
             where = c;
         }
+    };
+    int c = 0;
+    if ((reinterpret_cast<uintptr_t>(row) & 15u) == 0) {
+        constexpr int kAhead = 4;  // independent loads of a thread
+        for (; c + 4096 * kAhead <= width; c += 4096 * kAhead) {
+            float4 x[kAhead];
+#pragma unroll
+            for (int u = 0; u < kAhead; ++u) x[u] = *reinterpret_cast<const float4 *>(row + c + u * 4096 + threadIdx.x * 4);
+#pragma unroll
+            for (int u = 0; u < kAhead; ++u) {
+                const int at = c + u * 4096 + threadIdx.x * 4;
+                look(x[u].x, at);
+                look(x[u].y, at + 1);
+                look(x[u].z, at + 2);
+                look(x[u].w, at + 3);
+            }
+        }
     }
+    for (c += threadIdx.x; c < width; c += 1024) look(row[c], c);
 #pragma unroll
     for (int offset = 16; offset > 0; offset >>= 1) {
         const float other = __shfl_xor_sync(0xffffffffu, best, offset);
@@ -302,8 +319,9 @@ __global__ void __launch_bounds__(1024)
 }
 
 unsigned norm_threads(size_t width, int vec) {
+    // four packs a thread: fewer warps to bring together than with one, and loads enough in flight
     const size_t packs = (width + vec - 1) / vec;
-    size_t threads = (packs + 31) / 32 * 32;
+    size_t threads = ((packs + 3) / 4 + 31) / 32 * 32;
     if (threads > kNormThreads) threads = kNormThreads;
     return static_cast<unsigned>(threads);
 }

@@ -293,7 +293,7 @@ class LatentAttention:
         if not self.tiled:
             return None
         torch, c = self.ops.torch, self.config
-        splits = int(ks.lib().singe_latent_decode_splits(rows, c.heads, min(key_bound, c.window)))
+        splits = int(ks.lib().singe_latent_decode_splits(rows, c.heads, self.latent, min(key_bound, c.window)))
         attn = torch.empty((rows, splits, c.heads, self.latent), dtype=torch.float32, device="cuda")
         lse = torch.empty((rows, splits, c.heads), dtype=torch.float32, device="cuda")
         return splits, attn, lse
@@ -478,6 +478,16 @@ class HybridDecoder(PagedDecoder):
         self.sms = torch.cuda.get_device_properties(0).multi_processor_count
         self.trail = None   # set to a list to collect the residual stream after every layer (for inspection)
 
+    def fill_context(self, tokens_per_sequence: int, seed: int = 4) -> None:
+        """Marks ``tokens_per_sequence`` tokens of every sequence as cached and fills caches and states with N(0,1) values
+        (a benchmark's stand-in for a processed prompt)."""
+        torch = self.torch
+        self.table.place_prompts([tokens_per_sequence] * self.sequences)
+        generator = torch.Generator(device="cuda").manual_seed(seed)
+        for cache in self.caches:
+            cache.normal_(generator=generator)
+        self._refresh_block_table()
+
     # ---- the layers, over a step of any shape ----
 
     def _layers(self, rows: StepRows, scratches):
@@ -619,3 +629,35 @@ class HybridDecoder(PagedDecoder):
             packed[start: start + size] = array
         sent = torch.from_numpy(packed).cuda()
         return {name: sent[start: start + size] for name, start, size in zip(arrays, starts, sizes)}
+
+
+def random_weights(config: HybridConfig, names: dict, seed: int = 4) -> dict:
+    """Random bf16 weights on the GPU for ``names`` (name -> shape): matrices ~ N(0, 1 / columns), norms 1, decay biases 2."""
+    import torch
+
+    generator = torch.Generator(device="cuda").manual_seed(seed)
+    weights = {}
+    for name, shape in names.items():
+        if len(shape) == 1:
+            weights[name] = torch.full(shape, 2.0 if name.endswith("a2.b") else 1.0, dtype=torch.bfloat16, device="cuda")
+        else:
+            values = torch.randn(shape, generator=generator, device="cuda", dtype=torch.float32)
+            weights[name] = (values * (1.0 if name == "embed" else shape[1] ** -0.5)).to(torch.bfloat16)
+    return weights
+
+
+def decode_step_bytes(config: HybridConfig, sequences: int, context: int) -> dict:
+    """Algorithmic HBM bytes of one bf16 decode step: every weight once (borrowed layers read their owner's again), the
+    visible latents of every sequence, the recurrent states read and written."""
+    weights, cache, state = config.vocab * config.width, 0, 0
+    for layer in config.layers:
+        m, w = layer.mixer, config.width
+        weights += 2 * layer.ffn * w
+        if isinstance(m, LatentAttentionConfig):
+            weights += (m.q_rank + m.kv_rank + m.heads) * w + m.heads * m.dim * (m.q_rank + m.kv_rank)
+            weights += m.heads * m.vdim * (m.kv_rank + w)
+            cache += sequences * min(context, m.window) * m.kv_rank
+        else:
+            weights += (2 * m.heads * (m.dim + m.vdim) + m.rank) * w + m.heads * m.dim * m.rank + m.heads * m.vdim * w
+            state += sequences * m.heads * m.dim * m.vdim
+    return {"weights": 2 * weights, "latents": 2 * cache, "states": 8 * state, "total": 2 * weights + 2 * cache + 8 * state}
