@@ -284,6 +284,21 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
     return done != 0;
 }
 
+// Whether the phase with `parity` has completed, without waiting (try_wait may suspend the thread for a while).
+__device__ __forceinline__ bool mbar_test_wait(uint32_t bar, uint32_t parity) {
+    uint32_t done;
+    asm volatile(
+        "{\n"
+        ".reg .pred p;\n"
+        "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n"
+        "selp.u32 %0, 1, 0, p;\n"
+        "}\n"
+        : "=r"(done)
+        : "r"(bar), "r"(parity)
+        : "memory");
+    return done != 0;
+}
+
 // Waits for the phase with `parity` to complete, for at most `kWaitLimitCycles` SM clock cycles
 // (about half a second at full clock).  Returns false when the limit ran out, so callers can flag the
 // failure and leave instead of spinning for ever.  The SM cycle counter is used because it is

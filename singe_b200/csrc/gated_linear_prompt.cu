@@ -26,7 +26,7 @@ namespace {
 
 constexpr int kBlock = 16;             // tokens
 constexpr int kPrepareWarps = 4;
-constexpr int kStages = 3;
+constexpr int kMaxStages = 6;
 constexpr float kFactoredLimit = -60.0f;
 constexpr int kPitchP = kBlock * 2 + 16;  // bytes of a padded row of P
 
@@ -71,6 +71,7 @@ struct PromptParams {
     float *segment_decay;                     // [segments, heads, dim_pad]
     float inverse_tau, query_scale, eps;
     uint32_t *error;
+    int stages;  // blocks on their way to a CTA, plus the one in use
 };
 
 __host__ __device__ constexpr int operand_bytes(int dim_pad) { return operand_layout(dim_pad).bytes; }
@@ -301,8 +302,9 @@ __host__ __device__ inline StageLayout stage_layout(int dim_pad, int vdim_pad) {
 }
 
 // KT = dim_pad / 16; MT = 16-row value tiles of a warp.
-template <int KT, int MT, bool STATE_ONLY>
-__global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kernel(const PromptParams p) {
+// THREADS bounds the CTA; small states leave registers for three CTAs of an SM, whose latencies then hide one another.
+template <int KT, int MT, int THREADS, bool STATE_ONLY>
+__global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 ? 3 : 1) gated_linear_advance_kernel(const PromptParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
     constexpr int kDim = KT * 16;
@@ -316,16 +318,17 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
     const int g = lane >> 2, q2 = (lane & 3) * 2;
     constexpr OperandLayout kOperands = operand_layout(kDim);
     const StageLayout layout = stage_layout(kDim, s.vdim_pad);
+    const int stages = p.stages;
     extern __shared__ __align__(128) uint8_t advance_shared[];
-    float *squares = reinterpret_cast<float *>(advance_shared + kStages * layout.bytes);  // [8 or more][16]
+    float *squares = reinterpret_cast<float *>(advance_shared + stages * layout.bytes);  // [8 or more][16]
     const uint32_t bars = smem_u32(squares + max(warps, 8) * kBlock);
     // Nothing of a stage may hold a NaN: rows past a short block and columns past vdim meet zeros in the products.
-    for (int i = tid; i < kStages * layout.bytes / 16; i += blockDim.x) {
+    for (int i = tid; i < stages * layout.bytes / 16; i += blockDim.x) {
         reinterpret_cast<uint4 *>(advance_shared)[i] = make_uint4(0u, 0u, 0u, 0u);
     }
     for (int i = tid; i < max(warps, 8) * kBlock; i += blockDim.x) squares[i] = 0.0f;
     if (tid == 0) {
-        for (int i = 0; i < kStages; ++i) mbar_init(bars + 8 * i, 1);
+        for (int i = 0; i < stages; ++i) mbar_init(bars + 8 * i, 1);
         mbar_init_fence();
     }
     fence_proxy_async_shared();
@@ -393,8 +396,8 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
     auto load_block = [&](int index) {
         if (warp != 0) return;
         const int block = first_block + index;
-        const uint32_t bar = bars + 8 * (index % kStages);
-        const uint32_t stage = smem_u32(advance_shared) + (index % kStages) * layout.bytes;
+        const uint32_t bar = bars + 8 * (index % stages);
+        const uint32_t stage = smem_u32(advance_shared) + (index % stages) * layout.bytes;
         const int row0 = p.block_row[block], tokens = p.block_tokens[block];
         constexpr uint32_t kFrom = STATE_ONLY ? kOperands.state_part : 0, kBytes = kOperands.bytes - kFrom;
         const uint32_t row_bytes = s.vdim * 2;
@@ -410,7 +413,7 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
             bulk_load(stage + (lane < 16 ? layout.v : layout.g) + t * layout.pitch_v, source, row_bytes, bar);
         }
     };
-    for (int i = 0; i < kStages - 1 && i < blocks; ++i) load_block(i);
+    for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
     bool failed = false;
     float kept[2 * KT][2];  // product of the segment's decays (STATE_ONLY)
     if (STATE_ONLY) {
@@ -429,16 +432,21 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
         }
     }
 
+    // the rows and the 16-byte piece of the output this thread stores (threads past whole rows store none)
+    const int pieces = s.vdim / 8, store_rows = max(static_cast<int>(blockDim.x) / pieces, 1);
+    const int store_piece = tid % pieces, store_row = tid / pieces < store_rows ? tid / pieces : kBlock;
+
     for (int index = 0; index < blocks; ++index) {
-        const bool arrived = mbar_wait(bars + 8 * (index % kStages), (index / kStages) & 1);
+        const int row0 = p.block_row[first_block + index], tokens = p.block_tokens[first_block + index];
+        const bool arrived = mbar_wait(bars + 8 * (index % stages), (index / stages) & 1);
         fence_proxy_async_shared();
         // the block has arrived for every thread, and everyone is done with the stage loaded next
         if (__syncthreads_or(arrived ? 0 : 1) != 0) {
             failed = true;
             break;
         }
-        if (index + kStages - 1 < blocks) load_block(index + kStages - 1);
-        uint8_t *here = advance_shared + (index % kStages) * layout.bytes;
+        if (index + stages - 1 < blocks) load_block(index + stages - 1);
+        uint8_t *here = advance_shared + (index % stages) * layout.bytes;
         const uint32_t stage = smem_u32(here);
 
         uint32_t value[MT][4];  // v^T of this warp: rows v, columns tokens
@@ -578,13 +586,9 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
                 stmatrix_x4_trans(at, gate[0], gate[1], gate[2], gate[3]);
             }
             __syncthreads();
-            const int block = first_block + index;
-            const int row0 = p.block_row[block], tokens = p.block_tokens[block];
-            const int pieces = s.vdim / 8;
-            for (int i = tid; i < tokens * pieces; i += blockDim.x) {
-                const int t = i / pieces, piece = i - t * pieces;
-                *reinterpret_cast<uint4 *>(p.out + (row0 + t) * p.out_stride + head * s.vdim + piece * 8) =
-                    *reinterpret_cast<const uint4 *>(here + layout.g + t * layout.pitch_v + piece * 16);
+            for (int t = store_row; t < tokens; t += store_rows) {
+                *reinterpret_cast<uint4 *>(p.out + (row0 + t) * p.out_stride + head * s.vdim + store_piece * 8) =
+                    *reinterpret_cast<const uint4 *>(here + layout.g + t * layout.pitch_v + store_piece * 16);
             }
         }
     }
@@ -626,21 +630,24 @@ __global__ void __launch_bounds__(KT <= 4 ? 512 : 256) gated_linear_advance_kern
     }
 }
 
-template <int KT, int MT>
-int launch_advance(cudaStream_t stream, const PromptParams &p, size_t segments, bool cut, int warps) {
+template <int KT, int MT, int THREADS>
+int launch_advance(cudaStream_t stream, PromptParams p, size_t segments, bool cut, int warps) {
     const StageLayout layout = stage_layout(KT * 16, p.shape.vdim_pad);
-    const int bytes = kStages * layout.bytes + (warps > 8 ? warps : 8) * kBlock * 4 + kStages * 8;
+    const auto shared_bytes = [&](int stages) { return stages * layout.bytes + (warps > 8 ? warps : 8) * kBlock * 4 + kMaxStages * 8; };
+    p.stages = kMaxStages;  // as many as leave room for two more CTAs, three at least
+    while (p.stages > 3 && shared_bytes(p.stages) > 75 * 1024) --p.stages;
+    const int bytes = shared_bytes(p.stages);
     if (bytes > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     static int configured[kMaxDevices] = {0};
     static int configured_state[kMaxDevices] = {0};
     const dim3 grid(static_cast<unsigned>(segments), static_cast<unsigned>(p.shape.heads));
     if (cut) {
-        SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, true>, bytes, configured_state));
-        SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, true>, grid, dim3(warps * 32), bytes, stream,
+        SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, THREADS, true>, bytes, configured_state));
+        SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, THREADS, true>, grid, dim3(warps * 32), bytes, stream,
                                         kLaunchGlue, 1, p));
     }
-    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, false>, bytes, configured));
-    SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, false>, grid, dim3(warps * 32), bytes, stream,
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, THREADS, false>, bytes, configured));
+    SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, THREADS, false>, grid, dim3(warps * 32), bytes, stream,
                                     kLaunchGlue, 1, p));
     return launch_status();
 }
@@ -739,17 +746,22 @@ int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_
                                     dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((heads + kPrepareWarps - 1) / kPrepareWarps)),
                                     dim3(kPrepareWarps * 32), shared, s, kLaunchGlue, 1, p));
     const bool segmented = cut != 0;
-#define SINGE_ADVANCE(KT_, MT_) \
-    if (dim_pad == KT_ * 16 && value_tiles == MT_) return launch_advance<KT_, MT_>(s, p, segment_count, segmented, warps);
-    SINGE_ADVANCE(1, 1)
-    SINGE_ADVANCE(1, 2)
-    SINGE_ADVANCE(2, 1)
-    SINGE_ADVANCE(2, 2)
-    SINGE_ADVANCE(4, 1)
-    SINGE_ADVANCE(4, 2)
-    SINGE_ADVANCE(8, 1)
-    SINGE_ADVANCE(8, 2)
-    SINGE_ADVANCE(16, 1)
+#define SINGE_ADVANCE(KT_, MT_, THREADS_)                                          \
+    if (dim_pad == KT_ * 16 && value_tiles == MT_ && warps * 32 <= THREADS_) {      \
+        return launch_advance<KT_, MT_, THREADS_>(s, p, segment_count, segmented, warps); \
+    }
+    SINGE_ADVANCE(1, 1, 256)
+    SINGE_ADVANCE(1, 1, 512)
+    SINGE_ADVANCE(1, 2, 512)
+    SINGE_ADVANCE(2, 1, 256)
+    SINGE_ADVANCE(2, 1, 512)
+    SINGE_ADVANCE(2, 2, 512)
+    SINGE_ADVANCE(4, 1, 256)
+    SINGE_ADVANCE(4, 1, 512)
+    SINGE_ADVANCE(4, 2, 512)
+    SINGE_ADVANCE(8, 1, 256)
+    SINGE_ADVANCE(8, 2, 256)
+    SINGE_ADVANCE(16, 1, 256)
 #undef SINGE_ADVANCE
     return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
 }

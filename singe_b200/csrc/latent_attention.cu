@@ -294,7 +294,8 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentDecod
 //                behind the last one) and give scores nobody reads.
 //                O^T [latent, heads] += C^T P^T: A = the same tile, MN-major, 128 latent columns a product; B = P from
 //                shared memory.
-//              QK(t + 1) is issued before PV(t), so the tensor core works while the softmax of tile t runs.
+//              QK(t + 1) is issued before PV(t) when its tile is there, so that the tensor core works while the softmax of
+//              tile t runs; a tile that is still on its way does not hold PV(t), whose end frees the stage after it.
 //   warps 2-5  softmax and epilogue.  A thread is a key: its tensor-memory lane holds the key's scores of all heads.  The
 //              tile's maximum per head comes from a butterfly across the lanes; O and the sums are re-based only when it
 //              grew by more than 2^8 over the base in use (the result does not depend on the base).
@@ -334,9 +335,15 @@ __device__ __forceinline__ float transpose_reduce(float (&x)[32], int lane, Op o
     return x[0];
 }
 
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 __device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(kTcThreads, 2)
     latent_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap cache_map, const __grid_constant__ CUtensorMap query_map,
                                  const LatentDecode p, const LatentTcShape shape) {
     grid_dependency_wait();
@@ -420,15 +427,10 @@ __global__ void __launch_bounds__(kTcThreads, 1)
             for (int c = 0; c < chunks; ++c) tma_load_3d(query_at + c * kQueryChunkBytes, &query_map, bar_query, c * 64, head0, query);
         }
         const int32_t *table = p.table + static_cast<size_t>(sequence) * p.table_stride;
-        const int boxes = kTileKeys / shape.page_rows;  // boxes of one chunk
+        const int boxes = kTileKeys / shape.page_rows;  // boxes of one chunk: 1, 2, 4 or 8
+        const int box_bits = 31 - __clz(boxes);
         for (int tile = 0; tile < tile_count; ++tile) {
             const int stage = tile % stages;
-            int ok = 1;
-            if (lane == 0 && tile >= stages) ok = mbar_wait(bar_empty + 8 * stage, (tile / stages - 1) & 1) ? 1 : 0;
-            if (__shfl_sync(0xffffffffu, ok, 0) == 0) {
-                failed = true;
-                break;
-            }
             // lane b looks up box b's first cache row; boxes past the end repeat the tile's first box (masked)
             int row = 0;
             if (lane < boxes) {
@@ -441,10 +443,16 @@ __global__ void __launch_bounds__(kTcThreads, 1)
                 }
                 row = page * p.page_size + key % p.page_size;
             }
+            int ok = 1;
+            if (lane == 0 && tile >= stages) ok = mbar_wait(bar_empty + 8 * stage, (tile / stages - 1) & 1) ? 1 : 0;
+            if (__shfl_sync(0xffffffffu, ok, 0) == 0) {
+                failed = true;
+                break;
+            }
             if (lane == 0) mbar_expect_tx(bar_full + 8 * stage, stage_bytes);
             __syncwarp();
             for (int i = lane; i - lane < boxes * chunks; i += 32) {
-                const int box = i % boxes, chunk = i / boxes;
+                const int box = i & (boxes - 1), chunk = i >> box_bits;
                 const int from = __shfl_sync(0xffffffffu, row, box);
                 if (i < boxes * chunks) {
                     tma_load_2d(base + stage * stage_bytes + chunk * kChunkBytes + box * shape.page_rows * 128, &cache_map,
@@ -459,50 +467,69 @@ __global__ void __launch_bounds__(kTcThreads, 1)
         auto wait_all = [&](uint32_t bar, uint32_t parity) -> bool {
             return __all_sync(0xffffffffu, mbar_wait(bar, parity) ? 1 : 0) != 0;
         };
+        // Descriptors advance by adding to their address field (16-byte units).
+        auto issue_scores = [&](int tile) {
+            if (lane == 0) {
+                uint64_t a = make_smem_desc(base + (tile % stages) * stage_bytes, 16, 1024);
+                uint64_t b = make_smem_desc(query_at, 16, 1024);
+                const uint32_t target = tmem + (tile & 1) * kTcHeads;
+                uint32_t accumulate = 0;
+#pragma unroll 2
+                for (int c = 0; c < chunks; ++c) {
+#pragma unroll
+                    for (int ks = 0; ks < 4; ++ks) {
+                        umma_ss(target, a + 2 * ks, b + 2 * ks, kIdescScores, accumulate);
+                        accumulate = 1;
+                    }
+                    a += kChunkBytes >> 4;
+                    b += kQueryChunkBytes >> 4;
+                }
+                tcgen05_commit(bar_scores + 8 * (tile & 1));
+            }
+            __syncwarp();
+        };
         auto issue_values = [&](int tile) -> bool {
             if (!wait_all(bar_weights + 8 * (tile & 1), (tile >> 1) & 1)) return false;
             tcgen05_fence_after();
             if (lane == 0) {
-                const int stage = tile % stages;
-                const uint32_t at = base + stage * stage_bytes;
-                const uint32_t weights = weights_at + (tile & 1) * kWeightBytes;
+                uint64_t a = make_smem_desc(base + (tile % stages) * stage_bytes, kChunkBytes, 1024);
+                const uint64_t b = make_smem_desc(weights_at + (tile & 1) * kWeightBytes, 16, 1024);
+                uint32_t target = tmem + 64;
+                const uint32_t accumulate = tile > 0 ? 1u : 0u;
+#pragma unroll 2
                 for (int m = 0; m < (chunks + 1) / 2; ++m) {
+                    umma_ss(target, a, b, kIdescValues, accumulate);
 #pragma unroll
-                    for (int ks = 0; ks < kTileKeys / 16; ++ks) {
-                        umma_ss(tmem + 64 + m * kTcHeads, make_smem_desc(at + 2 * m * kChunkBytes + ks * 2048, kChunkBytes, 1024),
-                                make_smem_desc(weights + ks * 32, 16, 1024), kIdescValues, (tile > 0 || ks > 0) ? 1u : 0u);
-                    }
+                    for (int ks = 1; ks < kTileKeys / 16; ++ks) umma_ss(target, a + 128 * ks, b + 2 * ks, kIdescValues, 1u);
+                    a += (2 * kChunkBytes) >> 4;
+                    target += kTcHeads;
                 }
-                tcgen05_commit(bar_empty + 8 * stage);
+                tcgen05_commit(bar_empty + 8 * (tile % stages));
                 tcgen05_commit(bar_values);
             }
             __syncwarp();
             return true;
         };
         if (!wait_all(bar_query, 0)) failed = true;
+        int scored = 0;  // tiles whose scores have been issued
         for (int tile = 0; tile < tile_count && !failed; ++tile) {
-            const int stage = tile % stages;
-            if (!wait_all(bar_full + 8 * stage, (tile / stages) & 1)) {
-                failed = true;
-                break;
-            }
-            tcgen05_fence_after();
-            if (lane == 0) {
-                const uint32_t at = base + stage * stage_bytes;
-                for (int c = 0; c < chunks; ++c) {
-#pragma unroll
-                    for (int ks = 0; ks < 4; ++ks) {
-                        umma_ss(tmem + (tile & 1) * kTcHeads, make_smem_desc(at + c * kChunkBytes + ks * 32, 16, 1024),
-                                make_smem_desc(query_at + c * kQueryChunkBytes + ks * 32, 16, 1024), kIdescScores,
-                                (c > 0 || ks > 0) ? 1u : 0u);
-                    }
+            // scores of this tile if they are still to come, and of the next one if its keys have arrived
+            for (int ahead = tile; ahead < tile + 2 && ahead < tile_count && !failed; ++ahead) {
+                if (ahead < scored) continue;
+                const uint32_t bar = bar_full + 8 * (ahead % stages), parity = (ahead / stages) & 1;
+                if (ahead > tile) {
+                    if (__shfl_sync(0xffffffffu, mbar_test_wait(bar, parity) ? 1 : 0, 0) == 0) break;
                 }
-                tcgen05_commit(bar_scores + 8 * (tile & 1));
+                if (!wait_all(bar, parity)) {
+                    failed = true;
+                    break;
+                }
+                tcgen05_fence_after();
+                issue_scores(ahead);
+                scored = ahead + 1;
             }
-            __syncwarp();
-            if (tile > 0 && !issue_values(tile - 1)) failed = true;
+            if (!failed && !issue_values(tile)) failed = true;
         }
-        if (!failed && !issue_values(tile_count - 1)) failed = true;
     } else {
         // ---------------- softmax, epilogue ----------------
         const int quarter = warp & 3;  // tensor-memory lanes 32 * quarter ..
@@ -510,9 +537,10 @@ __global__ void __launch_bounds__(kTcThreads, 1)
         const bool scoring = quarter < 2;  // 64 keys
         const int my_key = quarter * 32 + lane;
         float base_log2 = -INFINITY;       // of head `lane`; the same in all four warps
-        float bias[kTcHeads], sum[kTcHeads];
+        float sum[kTcHeads];               // of this thread's key
 #pragma unroll
-        for (int h = 0; h < kTcHeads; ++h) bias[h] = sum[h] = 0.0f;
+        for (int h = 0; h < kTcHeads; ++h) sum[h] = 0.0f;
+        float *bases = exchange + 2 * kTcHeads;  // the base in use per head
         auto maximum = [](float a, float b) { return fmaxf(a, b); };
         auto addition = [](float a, float b) { return a + b; };
         for (int tile = 0; tile < tile_count; ++tile) {
@@ -557,21 +585,30 @@ __global__ void __launch_bounds__(kTcThreads, 1)
                 }
                 base_log2 = next;
 #pragma unroll
-                for (int h = 0; h < 32; ++h) {
-                    sum[h] *= __shfl_sync(0xffffffffu, factor, h);
-                    const float b = __shfl_sync(0xffffffffu, next, h);
-                    bias[h] = b == -INFINITY ? 0.0f : b;
-                }
+                for (int h = 0; h < 32; ++h) sum[h] *= __shfl_sync(0xffffffffu, factor, h);
+                if (quarter == 0) bases[lane] = next == -INFINITY ? 0.0f : next;
+                softmax_barrier();
             }
             if (scoring && !failed) {
                 // P[head, key], 128-byte rows with the 16-byte pieces permuted as SWIZZLE_128B has them
                 uint8_t *weights = smem_raw + (weights_at - raw) + (tile & 1) * kWeightBytes;
                 const int piece = my_key >> 3, within = (my_key & 7) * 2;
 #pragma unroll
-                for (int h = 0; h < 32; ++h) {
-                    const float x = visible ? exp2f(__uint_as_float(scores[h]) - bias[h]) : 0.0f;
-                    sum[h] += x;
-                    *reinterpret_cast<__nv_bfloat16 *>(weights + h * 128 + ((piece ^ (h & 7)) << 4) + within) = __float2bfloat16_rn(x);
+                for (int h0 = 0; h0 < 32; h0 += 8) {  // eight heads at a time, so that their latencies overlap
+                    const float4 low = *reinterpret_cast<const float4 *>(bases + h0);
+                    const float4 high = *reinterpret_cast<const float4 *>(bases + h0 + 4);
+                    const float subtracted[8] = {low.x, low.y, low.z, low.w, high.x, high.y, high.z, high.w};
+                    float x[8];
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        x[i] = visible ? exp2_fast(__uint_as_float(scores[h0 + i]) - subtracted[i]) : 0.0f;
+                        sum[h0 + i] += x[i];
+                    }
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        *reinterpret_cast<__nv_bfloat16 *>(weights + (h0 + i) * 128 + ((piece ^ i) << 4) + within) =
+                            __float2bfloat16_rn(x[i]);
+                    }
                 }
                 fence_proxy_async_shared();
             }

@@ -225,12 +225,12 @@ class BlockRows:
 
 def plan_segments(blocks_of, heads: int, sms: int):
     """Cuts each sequence's blocks into segments.  A cut costs a second pass over all but a sequence's last segment, so
-    only steps whose (sequence, head) pairs leave SMs idle are cut, into about two segments per SM.  Returns rows of
+    only steps whose (sequence, head) pairs leave SMs idle are cut, into about three (segment, head) pairs per SM.  Returns rows of
     (place in ``blocks_of``, first block, blocks, earlier segments of the sequence, last of the sequence)."""
     total = sum(blocks_of)
     size = total
     if len(blocks_of) * heads < sms:
-        size = max(LEAST_SEGMENT, -(-total // max(2 * sms // heads, 1)))
+        size = max(LEAST_SEGMENT, -(-total // max(3 * sms // heads, 1)))
     rows, first = [], 0
     for place, blocks in enumerate(blocks_of):
         pieces = -(-blocks // size)
