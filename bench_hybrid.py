@@ -17,6 +17,7 @@ SIZES = {
     "2048": (2048, 16, 128, 768, 256, 1024, 8192, 16, 64, 128, 32000),
     "4096": (4096, 32, 128, 1536, 512, 4096, 14336, 32, 64, 128, 128256),
 }
+PAGE = hybrid.HybridConfig().page_size
 PATTERN = "aagaag"   # a: latent attention and feed-forward; g: gated linear attention and feed-forward
 
 
@@ -130,7 +131,7 @@ def normal(*shape, scale=1.0, kind=torch.bfloat16):
 def latent_decode_kernel(size: str, sequences: int, context: int, peaks) -> dict:
     _, heads, _, _, latent, window, *_ = SIZES[size]
     o = hybrid.Ops("bfloat16")
-    stride = -(-context // 16)
+    stride = -(-context // PAGE)
     from singe_b200 import kernel_sys as ks
 
     seen = min(context, window)
@@ -142,11 +143,11 @@ def latent_decode_kernel(size: str, sequences: int, context: int, peaks) -> dict
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
 
     def make(i):
-        cache = normal(sequences * stride, 16, latent)
+        cache = normal(sequences * stride, PAGE, latent)
         table = torch.randperm(sequences * stride, device="cuda").to(torch.int32).view(sequences, stride)
         query, out = normal(sequences, heads, latent), torch.empty((sequences, heads, latent), dtype=torch.bfloat16, device="cuda")
         return lambda: o.call("singe_latent_decode_bf16", _stream(), out, attn, lse, query, cache, order, lens, table, sequences,
-                              heads, latent, 16, sequences * stride, sequences, stride, window, splits, latent ** -0.5, status)
+                              heads, latent, PAGE, sequences * stride, sequences, stride, window, splits, latent ** -0.5, status)
 
     moved = sequences * (seen + 2 * heads) * latent * 2
     call, _ = rotating(make, moved)

@@ -287,19 +287,23 @@ __global__ void __launch_bounds__(256, 1) latent_decode_kernel(const LatentDecod
 
 // ---- tcgen05 ----
 // One CTA per (query, split of its keys, 32 heads); heads past the last one are zero rows of q.
-//   warp 0     TMA producer: q once, then tiles of 64 keys: one box per (page, 64 latent columns), SWIZZLE_128B, stored as
-//              [64-column chunk][64 keys][128 bytes]
+//   warp 0     TMA producer: q once, then tiles of 64 keys, SWIZZLE_128B, stored as [64-column chunk][64 keys][128 bytes].
+//              Pages of 64 tokens arrive in one box a tile; smaller pages take one box per page and chunk, which the TMA
+//              unit works off at about 12 bytes a clock, a quarter of the large boxes' rate.
 //   warp 1     MMA issuer and owner of tensor memory:
-//                S^T [keys, heads] = C q^T: A = the tile, K-major.  M is 128: rows 64.. read the chunk behind (or what lies
-//                behind the last one) and give scores nobody reads.
+//                S^T [keys, heads] = C q^T: A = the tile, K-major, M = 64: key k lands in tensor-memory lane
+//                32 * (k / 16) + k % 16.
 //                O^T [latent, heads] += C^T P^T: A = the same tile, MN-major, 128 latent columns a product; B = P from
 //                shared memory.
+//              Neighbouring products go to different accumulators: with 32 columns a product is all latency.
 //              QK(t + 1) is issued before PV(t) when its tile is there, so that the tensor core works while the softmax of
 //              tile t runs; a tile that is still on its way does not hold PV(t), whose end frees the stage after it.
-//   warps 2-5  softmax and epilogue.  A thread is a key: its tensor-memory lane holds the key's scores of all heads.  The
-//              tile's maximum per head comes from a butterfly across the lanes; O and the sums are re-based only when it
-//              grew by more than 2^8 over the base in use (the result does not depend on the base).
-// Tensor memory: S of even and odd tiles [0, 32) [32, 64), O^T from 64 on, 32 columns per 128 latent columns.
+//   warps 2-5  softmax and epilogue.  A thread of a warp's first half is a key: its lane holds the key's scores of all
+//              heads.  Weights are taken relative to a base per head, on which the result does not depend; when a score
+//              exceeds its head's base by more than 2^8, the tile's maxima (a butterfly across the lanes) give new bases,
+//              and O and the sums are scaled.
+// Tensor memory: S of even tiles [0, 64), of odd tiles [64, 128), two accumulators each, whose sum is the score; O^T from
+// 128 on, 32 columns per 128 latent columns.
 // Every wait is bounded.
 constexpr int kTcHeads = 32;
 constexpr int kTcThreads = 192;
@@ -310,13 +314,14 @@ constexpr int kWeightBytes = kTcHeads * 128;       // P: 32 heads x 64 keys
 constexpr float kRebase = 8.0f;                    // log2 units
 
 struct LatentTcShape {
-    int chunks, stages, page_rows;  // page_rows: rows of a TMA box
+    int chunks, stages;
+    int page_rows, box_chunks;  // rows and 64-column chunks of a TMA box
 };
 
 __host__ __device__ inline int latent_tc_bytes(int chunks, int stages) {
-    // tiles, then q (also what over-reading products of the last tile touch), P twice, exchange area, barriers, alignment
+    // tiles, then q (also what the over-reading product of an odd last chunk touches), P twice, exchange area, barriers
     const int query = chunks * kQueryChunkBytes > 2 * kChunkBytes ? chunks * kQueryChunkBytes : 2 * kChunkBytes;
-    return stages * chunks * kChunkBytes + query + 2 * kWeightBytes + 4 * kTcHeads * 4 + 8 * (2 * kTcMaxStages + 8) + 1024;
+    return stages * chunks * kChunkBytes + query + 2 * kWeightBytes + 5 * kTcHeads * 4 + 16 + 8 * (2 * kTcMaxStages + 8) + 1024;
 }
 
 // Lane h ends up with op over all lanes of x[h].
@@ -355,8 +360,8 @@ __global__ void __launch_bounds__(kTcThreads, 2)
     const uint32_t query_at = base + stages * stage_bytes;
     const uint32_t weights_at = query_at + max(chunks * kQueryChunkBytes, 2 * kChunkBytes);
     const uint32_t exchange_at = weights_at + 2 * kWeightBytes;
-    float *exchange = reinterpret_cast<float *>(smem_raw + (exchange_at - raw));  // [4][32]
-    const uint32_t bars = exchange_at + 4 * kTcHeads * 4;
+    float *exchange = reinterpret_cast<float *>(smem_raw + (exchange_at - raw));  // [5][32]: one row per softmax warp, then the bases
+    const uint32_t bars = exchange_at + 5 * kTcHeads * 4 + 16;
     const uint32_t bar_full = bars, bar_empty = bars + 8 * kTcMaxStages;
     const uint32_t bar_query = bars + 16 * kTcMaxStages;
     const uint32_t bar_scores = bar_query + 8;    // [2]
@@ -429,6 +434,7 @@ __global__ void __launch_bounds__(kTcThreads, 2)
         const int32_t *table = p.table + static_cast<size_t>(sequence) * p.table_stride;
         const int boxes = kTileKeys / shape.page_rows;  // boxes of one chunk: 1, 2, 4 or 8
         const int box_bits = 31 - __clz(boxes);
+        const int columns = chunks / shape.box_chunks;  // boxes side by side
         for (int tile = 0; tile < tile_count; ++tile) {
             const int stage = tile % stages;
             // lane b looks up box b's first cache row; boxes past the end repeat the tile's first box (masked)
@@ -451,36 +457,36 @@ __global__ void __launch_bounds__(kTcThreads, 2)
             }
             if (lane == 0) mbar_expect_tx(bar_full + 8 * stage, stage_bytes);
             __syncwarp();
-            for (int i = lane; i - lane < boxes * chunks; i += 32) {
-                const int box = i & (boxes - 1), chunk = i >> box_bits;
+            for (int i = lane; i - lane < boxes * columns; i += 32) {
+                const int box = i & (boxes - 1), chunk = (i >> box_bits) * shape.box_chunks;
                 const int from = __shfl_sync(0xffffffffu, row, box);
-                if (i < boxes * chunks) {
-                    tma_load_2d(base + stage * stage_bytes + chunk * kChunkBytes + box * shape.page_rows * 128, &cache_map,
-                                bar_full + 8 * stage, chunk * 64, from);
+                if (i < boxes * columns) {
+                    tma_load_3d(base + stage * stage_bytes + chunk * kChunkBytes + box * shape.page_rows * 128, &cache_map,
+                                bar_full + 8 * stage, 0, from, chunk);
                 }
             }
         }
     } else if (warp == 1) {
         // ---------------- MMA issuer ----------------
-        constexpr uint32_t kIdescScores = make_instr_desc(128, kTcHeads, true, 0, 0);
+        constexpr uint32_t kIdescScores = make_instr_desc(kTileKeys, kTcHeads, true, 0, 0);
         constexpr uint32_t kIdescValues = make_instr_desc(128, kTcHeads, true, 1, 0);  // A = C^T, MN-major
         auto wait_all = [&](uint32_t bar, uint32_t parity) -> bool {
             return __all_sync(0xffffffffu, mbar_wait(bar, parity) ? 1 : 0) != 0;
         };
         // Descriptors advance by adding to their address field (16-byte units).
         auto issue_scores = [&](int tile) {
-            if (lane == 0) {
+            if (elect_one()) {
                 uint64_t a = make_smem_desc(base + (tile % stages) * stage_bytes, 16, 1024);
                 uint64_t b = make_smem_desc(query_at, 16, 1024);
-                const uint32_t target = tmem + (tile & 1) * kTcHeads;
+                const uint32_t target = tmem + (tile & 1) * 2 * kTcHeads;
                 uint32_t accumulate = 0;
 #pragma unroll 2
                 for (int c = 0; c < chunks; ++c) {
-#pragma unroll
-                    for (int ks = 0; ks < 4; ++ks) {
-                        umma_ss(target, a + 2 * ks, b + 2 * ks, kIdescScores, accumulate);
-                        accumulate = 1;
-                    }
+                    umma_ss(target, a, b, kIdescScores, accumulate);
+                    umma_ss(target + kTcHeads, a + 2, b + 2, kIdescScores, accumulate);
+                    umma_ss(target, a + 4, b + 4, kIdescScores, 1u);
+                    umma_ss(target + kTcHeads, a + 6, b + 6, kIdescScores, 1u);
+                    accumulate = 1;
                     a += kChunkBytes >> 4;
                     b += kQueryChunkBytes >> 4;
                 }
@@ -491,18 +497,18 @@ __global__ void __launch_bounds__(kTcThreads, 2)
         auto issue_values = [&](int tile) -> bool {
             if (!wait_all(bar_weights + 8 * (tile & 1), (tile >> 1) & 1)) return false;
             tcgen05_fence_after();
-            if (lane == 0) {
-                uint64_t a = make_smem_desc(base + (tile % stages) * stage_bytes, kChunkBytes, 1024);
+            if (elect_one()) {
+                const uint64_t a = make_smem_desc(base + (tile % stages) * stage_bytes, kChunkBytes, 1024);
                 const uint64_t b = make_smem_desc(weights_at + (tile & 1) * kWeightBytes, 16, 1024);
-                uint32_t target = tmem + 64;
-                const uint32_t accumulate = tile > 0 ? 1u : 0u;
-#pragma unroll 2
-                for (int m = 0; m < (chunks + 1) / 2; ++m) {
-                    umma_ss(target, a, b, kIdescValues, accumulate);
+                uint32_t accumulate = tile > 0 ? 1u : 0u;
 #pragma unroll
-                    for (int ks = 1; ks < kTileKeys / 16; ++ks) umma_ss(target, a + 128 * ks, b + 2 * ks, kIdescValues, 1u);
-                    a += (2 * kChunkBytes) >> 4;
-                    target += kTcHeads;
+                for (int ks = 0; ks < kTileKeys / 16; ++ks) {
+#pragma unroll 4
+                    for (int m = 0; m < (chunks + 1) / 2; ++m) {
+                        umma_ss(tmem + 4 * kTcHeads + m * kTcHeads, a + m * ((2 * kChunkBytes) >> 4) + 128 * ks, b + 2 * ks,
+                                kIdescValues, accumulate);
+                    }
+                    accumulate = 1;
                 }
                 tcgen05_commit(bar_empty + 8 * (tile % stages));
                 tcgen05_commit(bar_values);
@@ -534,37 +540,53 @@ __global__ void __launch_bounds__(kTcThreads, 2)
         // ---------------- softmax, epilogue ----------------
         const int quarter = warp & 3;  // tensor-memory lanes 32 * quarter ..
         const uint32_t lanes = static_cast<uint32_t>(quarter * 32) << 16;
-        const bool scoring = quarter < 2;  // 64 keys
-        const int my_key = quarter * 32 + lane;
+        const bool has_key = lane < 16;
+        const int my_key = quarter * 16 + (lane & 15);
         float base_log2 = -INFINITY;       // of head `lane`; the same in all four warps
         float sum[kTcHeads];               // of this thread's key
 #pragma unroll
         for (int h = 0; h < kTcHeads; ++h) sum[h] = 0.0f;
-        float *bases = exchange + 2 * kTcHeads;  // the base in use per head
+        float *bases = exchange + 4 * kTcHeads;                                  // the base in use per head
+        volatile int *grown = reinterpret_cast<volatile int *>(bases + kTcHeads);  // [4]: a warp saw a score beyond its base
         auto maximum = [](float a, float b) { return fmaxf(a, b); };
         auto addition = [](float a, float b) { return a + b; };
         for (int tile = 0; tile < tile_count; ++tile) {
             uint32_t scores[32];
             const int key = start + tile * kTileKeys + my_key;
-            const bool visible = key >= visible_from && key < end;
+            const bool visible = has_key && key >= visible_from && key < end;
             if (!failed && !__all_sync(0xffffffffu, mbar_wait(bar_scores + 8 * (tile & 1), (tile >> 1) & 1) ? 1 : 0)) failed = true;
             tcgen05_fence_after();
-            if (scoring && !failed) {
-                tmem_ld_x32(tmem + lanes + (tile & 1) * kTcHeads, scores);
+            if (!failed) {
+                uint32_t other[32];
+                tmem_ld_x32(tmem + lanes + (tile & 1) * 2 * kTcHeads, scores);
+                tmem_ld_x32(tmem + lanes + (tile & 1) * 2 * kTcHeads + kTcHeads, other);
                 tmem_wait_ld_into(scores);
-                float top[32];
+                tmem_wait_ld_into(other);
+                float excess = tile == 0 ? INFINITY : -INFINITY;
 #pragma unroll
-                for (int h = 0; h < 32; ++h) {
-                    const float x = __uint_as_float(scores[h]) * p.scale_log2;
-                    scores[h] = __float_as_uint(x);
-                    top[h] = visible ? x : -INFINITY;
+                for (int h = 0; h < 32; h += 4) {
+                    const float4 b = *reinterpret_cast<const float4 *>(bases + h);
+                    const float subtracted[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const float both = __uint_as_float(scores[h + i]) + __uint_as_float(other[h + i]);
+                        const float x = visible ? both * p.scale_log2 : -INFINITY;
+                        scores[h + i] = __float_as_uint(x);
+                        if (tile > 0) excess = fmaxf(excess, x - subtracted[i]);
+                    }
                 }
-                exchange[quarter * kTcHeads + lane] = transpose_reduce(top, lane, maximum);
+                const bool beyond = __any_sync(0xffffffffu, excess > kRebase);
+                if (lane == 0) grown[quarter] = beyond ? 1 : 0;
             }
             softmax_barrier();
-            const float tile_top = fmaxf(exchange[lane], exchange[kTcHeads + lane]);
-            const bool grow = tile_top > base_log2 + kRebase || (base_log2 == -INFINITY && tile_top > -INFINITY);
-            if (__any_sync(0xffffffffu, grow)) {  // the same answer in all four warps
+            if ((grown[0] | grown[1] | grown[2] | grown[3]) != 0) {  // the same answer in all four warps
+                float top[32];
+#pragma unroll
+                for (int h = 0; h < 32; ++h) top[h] = __uint_as_float(scores[h]);
+                exchange[quarter * kTcHeads + lane] = transpose_reduce(top, lane, maximum);
+                softmax_barrier();
+                const float tile_top = fmaxf(fmaxf(exchange[lane], exchange[kTcHeads + lane]),
+                                             fmaxf(exchange[2 * kTcHeads + lane], exchange[3 * kTcHeads + lane]));
                 const float next = fmaxf(base_log2, tile_top);
                 const float factor = base_log2 == -INFINITY ? 0.0f : exp2f(base_log2 - next);
                 if (tile > 0) {
@@ -573,13 +595,13 @@ __global__ void __launch_bounds__(kTcThreads, 2)
                     tcgen05_fence_after();
                     for (int m = 0; m < (chunks + 1) / 2 && !failed; ++m) {
                         uint32_t o[32];
-                        tmem_ld_x32(tmem + lanes + 64 + m * kTcHeads, o);
+                        tmem_ld_x32(tmem + lanes + 4 * kTcHeads + m * kTcHeads, o);
                         tmem_wait_ld_into(o);
 #pragma unroll
                         for (int h = 0; h < 32; ++h) {
                             o[h] = __float_as_uint(__uint_as_float(o[h]) * __shfl_sync(0xffffffffu, factor, h));
                         }
-                        tmem_st_x32(tmem + lanes + 64 + m * kTcHeads, o);
+                        tmem_st_x32(tmem + lanes + 4 * kTcHeads + m * kTcHeads, o);
                     }
                     tmem_wait_st();
                 }
@@ -589,7 +611,7 @@ __global__ void __launch_bounds__(kTcThreads, 2)
                 if (quarter == 0) bases[lane] = next == -INFINITY ? 0.0f : next;
                 softmax_barrier();
             }
-            if (scoring && !failed) {
+            if (has_key && !failed) {
                 // P[head, key], 128-byte rows with the 16-byte pieces permuted as SWIZZLE_128B has them
                 uint8_t *weights = smem_raw + (weights_at - raw) + (tile & 1) * kWeightBytes;
                 const int piece = my_key >> 3, within = (my_key & 7) * 2;
@@ -601,7 +623,7 @@ __global__ void __launch_bounds__(kTcThreads, 2)
                     float x[8];
 #pragma unroll
                     for (int i = 0; i < 8; ++i) {
-                        x[i] = visible ? exp2_fast(__uint_as_float(scores[h0 + i]) - subtracted[i]) : 0.0f;
+                        x[i] = exp2_fast(__uint_as_float(scores[h0 + i]) - subtracted[i]);  // a hidden key's score is -inf
                         sum[h0 + i] += x[i];
                     }
 #pragma unroll
@@ -618,11 +640,15 @@ __global__ void __launch_bounds__(kTcThreads, 2)
         }
         grid_launch_dependents();  // late: the fold's many small CTAs would take the slots of CTAs still to come
         // ---- O^T / sum ----
-        if (!failed && !__all_sync(0xffffffffu, mbar_wait(bar_values, (tile_count - 1) & 1) ? 1 : 0)) failed = true;
+        // A parity wait tells neighbouring phases apart, not more: the last scores imply the values up to the third-last
+        // tile, so the second-last tile is waited for before the last.
+        for (int tile = max(tile_count - 2, 0); tile < tile_count && !failed; ++tile) {
+            if (!__all_sync(0xffffffffu, mbar_wait(bar_values, tile & 1) ? 1 : 0)) failed = true;
+        }
         tcgen05_fence_after();
-        if (scoring) exchange[quarter * kTcHeads + lane] = transpose_reduce(sum, lane, addition);
+        exchange[quarter * kTcHeads + lane] = transpose_reduce(sum, lane, addition);
         softmax_barrier();
-        const float total = exchange[lane] + exchange[kTcHeads + lane];
+        const float total = (exchange[lane] + exchange[kTcHeads + lane]) + (exchange[2 * kTcHeads + lane] + exchange[3 * kTcHeads + lane]);
         const float inverse = total > 0.0f ? 1.0f / total : 0.0f;
         if (p.splits > 1 && quarter == 0 && head0 + lane < p.heads) {
             p.lse[(static_cast<size_t>(query) * p.splits + split) * p.heads + head0 + lane] =
@@ -630,9 +656,9 @@ __global__ void __launch_bounds__(kTcThreads, 2)
         }
         for (int m = 0; m < (chunks + 1) / 2 && !failed; ++m) {
             uint32_t o[32];
-            tmem_ld_x32(tmem + lanes + 64 + m * kTcHeads, o);
+            tmem_ld_x32(tmem + lanes + 4 * kTcHeads + m * kTcHeads, o);
             tmem_wait_ld_into(o);
-            const int column = m * 128 + my_key;
+            const int column = m * 128 + quarter * 32 + lane;
             if (p.splits == 1) {
                 __nv_bfloat16 *out = p.out + (static_cast<size_t>(query) * p.heads + head0) * p.latent + column;
 #pragma unroll
@@ -716,16 +742,18 @@ int launch_latent_tcgen05(cudaStream_t stream, const LatentDecode &p, size_t que
     LatentTcShape shape;
     shape.chunks = p.latent / 64;
     shape.page_rows = box_rows;
+    shape.box_chunks = box_rows == kTileKeys ? shape.chunks : 1;
     shape.stages = latent_tc_stages(shape.chunks);
     const int bytes = latent_tc_bytes(shape.chunks, shape.stages);
     static int configured[kMaxDevices] = {0};
     SINGE_CUDA_TRY(ensure_dynamic_shared(latent_decode_tcgen05_kernel, bytes, configured));
     CUtensorMap cache_map, query_map;
     {
-        const uint64_t dims[2] = {static_cast<uint64_t>(p.latent), static_cast<uint64_t>(p.pages) * p.page_size};
-        const uint64_t strides[1] = {static_cast<uint64_t>(p.latent) * 2};
-        const uint32_t box[2] = {64, static_cast<uint32_t>(box_rows)};
-        SINGE_TRY(encode_tensor_map(&cache_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, p.cache, dims, strides, box,
+        // the latent's 64-column chunks as the outer dimension, so that a box lands chunk by chunk
+        const uint64_t dims[3] = {64, static_cast<uint64_t>(p.pages) * p.page_size, static_cast<uint64_t>(shape.chunks)};
+        const uint64_t strides[2] = {static_cast<uint64_t>(p.latent) * 2, 128};
+        const uint32_t box[3] = {64, static_cast<uint32_t>(box_rows), static_cast<uint32_t>(shape.box_chunks)};
+        SINGE_TRY(encode_tensor_map(&cache_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, p.cache, dims, strides, box,
                                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     }
     {

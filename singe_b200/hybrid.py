@@ -73,7 +73,7 @@ class HybridConfig:
     width: int = 0
     vocab: int = 0
     eps: float = 1e-6
-    page_size: int = 16
+    page_size: int = 64        # a page of this size is one tile of the decode attention
 
     def owner(self, index: int) -> int:
         """The layer whose weights layer ``index`` uses."""

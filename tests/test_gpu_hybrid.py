@@ -11,6 +11,7 @@ import torch
 
 from oracle import hybrid_ref
 from singe_b200 import hybrid, models
+from singe_b200.checkpoint import load_hybrid
 from singe_b200.decoder import CachedDecoder, PageTableError
 from singe_b200.generation import GenerationOptions, PromptChunks, RunningBatch, generate_batch
 from tests import hybrid_util as util
@@ -48,6 +49,13 @@ class Expect:
 @pytest.fixture(scope="module")
 def expects(snapshots):
     return {name: Expect(config, weights) for name, (config, weights, _) in snapshots.items()}
+
+
+def small_pages(directory, sequences, capacity, dtype, cache_tokens):
+    """A decoder whose cache pages hold 16 tokens, so that a small pool still has pages to move around."""
+    config, weights = load_hybrid(directory)
+    config.page_size = 16
+    return hybrid.HybridDecoder(config, sequences, capacity, weights, dtype, cache_tokens)
 
 
 def tokens_of(config, seed, count):
@@ -145,7 +153,7 @@ def test_freed_pages_and_rows_are_used_again(snapshots, expects, dtype):
     """A pool just large enough for the windows: pages move between sequences all the time, and a row's recurrent state
     starts over with its next request."""
     config, _, directory = snapshots["mixed"]
-    decoder = models.load_decoder(directory, 2, 400, dtype, cache_tokens=2 * (70 + 64 + 32))
+    decoder = small_pages(directory, 2, 400, dtype, 2 * (70 + 64 + 32))
     decoder.capture()
     long = tokens_of(config, 20, 330)
     outs, at = [], 0
@@ -170,7 +178,7 @@ def test_freed_pages_and_rows_are_used_again(snapshots, expects, dtype):
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_long_decoding(snapshots, expects, dtype):
     config, _, directory = snapshots["mixed"]
-    decoder = models.load_decoder(directory, 1, 700, dtype, cache_tokens=112)
+    decoder = small_pages(directory, 1, 700, dtype, 112)
     decoder.capture()
     tokens = tokens_of(config, 5, 640)
     check(run_portions(decoder, 0, tokens, [9] + [1] * 631), expects["mixed"](tokens), dtype, "long decoding")
@@ -178,7 +186,7 @@ def test_long_decoding(snapshots, expects, dtype):
 
 def test_a_step_without_room_changes_nothing(snapshots, expects):
     config, _, directory = snapshots["mixed"]
-    decoder = models.load_decoder(directory, 2, 128, "float32", cache_tokens=96)
+    decoder = small_pages(directory, 2, 128, "float32", 96)
     tokens = tokens_of(config, 6, 60)
     first = run_portions(decoder, 0, tokens[:40], [40])
     with pytest.raises(PageTableError):

@@ -173,7 +173,8 @@ def edge_queries(rng, keys, positions, window, heads, sharp=30.0):
 
 @pytest.mark.parametrize("heads,latent,page_size,window,splits", [
     (1, 64, 16, 1, 1), (5, 64, 16, 2, 1), (8, 128, 16, 136, 3), (16, 192, 4, 65, 2), (20, 256, 7, 64, 1),
-    (34, 512, 16, 300, 4), (32, 320, 16, 100000, 7), (3, 448, 1, 33, 5), (40, 64, 16, 0, 2)])
+    (34, 512, 16, 300, 4), (32, 320, 16, 100000, 7), (3, 448, 1, 33, 5), (40, 64, 16, 0, 2),
+    (32, 512, 64, 200, 2), (8, 256, 128, 129, 1), (33, 320, 64, 64, 3), (4, 64, 8, 77, 2), (16, 448, 32, 1, 1)])
 def test_decode_attention_at_window_and_page_edges(heads, latent, page_size, window, splits):
     rng = np.random.default_rng(heads * latent + window)
     capacity = 500
@@ -210,7 +211,8 @@ def test_decode_attention_at_window_and_page_edges(heads, latent, page_size, win
                          stride, window, splits, scale, status)
     got = host(out)
     assert np.isfinite(got).all() and int(status.item()) == 0
-    assert np.abs(got - np.stack(expect)).max() < 3e-2
+    error = np.abs(got - np.stack(expect)) / (1.0 + np.abs(np.stack(expect)))
+    assert error.max() < 1e-2, f"query, head, column {np.unravel_index(error.argmax(), error.shape)}: {error.max()}"
 
 
 def test_decode_attention_reports_bad_pages():
