@@ -193,7 +193,7 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) gated_linear_prepare_kerne
             for (int i = 0; i < 2; ++i) {
                 before[i] = __expf(z[i][t]);
                 if (factors) {
-                    back[i] = __fdividef(1.0f, before[i]);
+                    back[i] = __expf(-z[i][t]);
                     after[i] = whole[i] * back[i];
                 } else {
                     back[i] = __expf(fminf(-z[i][t], -kFactoredLimit));

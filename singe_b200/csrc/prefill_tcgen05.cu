@@ -558,7 +558,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         };
         // S_x = Q_x K(stage)^T; `last` releases the Q tile
         auto issue_qk = [&](int x, int stage, bool last) {
-            if (lane == 0) {
+            if (elect_one()) {
                 const uint32_t q_tile = q_smem + x * kTileBytes;
                 const uint32_t k_tile = k_smem + stage * kTileBytes;
 #pragma unroll
@@ -575,7 +575,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
         // O_x (+)= P_x V(stage): 16 keys per step, P advances 8 packed columns, V two 8-row groups (2 x 1024 bytes);
         // the second 64 dims of V are the next box, 16 KB further (leading byte offset).
         auto issue_pv = [&](int x, int stage, bool accumulate, bool last) {
-            if (lane == 0) {
+            if (elect_one()) {
                 const uint32_t v_tile = v_smem + stage * kTileBytes;
 #pragma unroll
                 for (int ks = 0; ks < kTile / 16; ++ks) {
@@ -621,7 +621,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
             if (!wait_all(bar_k_full, 0)) failed = true;
             if (!failed && (!first_qk(item, 0, 0) || !first_qk(item, 1, 0))) failed = true;
             if (!failed) {
-                if (lane == 0) tcgen05_commit(bar_k_empty);
+                if (elect_one()) tcgen05_commit(bar_k_empty);
                 __syncwarp();
             }
         }
@@ -656,7 +656,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                         if (last) ++o_done[x];
                     }
                     if (x == 1) {
-                        if (lane == 0) tcgen05_commit(bar_v_empty + stage * 8);
+                        if (elect_one()) tcgen05_commit(bar_v_empty + stage * 8);
                         __syncwarp();
                     }
                     if (onward) {
@@ -684,7 +684,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1)
                             continue;
                         }
                         if (x == 1) {
-                            if (lane == 0) tcgen05_commit(bar_k_empty + next * 8);
+                            if (elect_one()) tcgen05_commit(bar_k_empty + next * 8);
                             __syncwarp();
                         }
                     }
