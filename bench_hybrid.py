@@ -233,7 +233,7 @@ def recurrence_prompt_kernel(size: str, lengths, peaks) -> dict:
     rows, tokens, segments, last = i32(np.concatenate(starts)), i32(tokens), i32(plan[:, :4]), i32(plan[:, 4])
     scratch = torch.empty(int(ks.lib().singe_gated_linear_prompt_scratch(heads, key, value, rows.numel(), len(plan))), dtype=torch.uint8, device="cuda")
     call = lambda: o.call("singe_gated_linear_prompt_bf16", _stream(), out, out.stride(0), projected, projected.stride(0), decay, bias, norm,
-                          state, context, heads, key, value, rank, 16.0, key ** -0.5, 1e-6, rows, tokens, rows.numel(), segments, last,
+                          state, context, total, heads, key, value, rank, 16.0, key ** -0.5, 1e-6, rows, tokens, rows.numel(), segments, last,
                           len(plan), int((plan[:, 4] == 0).any()), scratch)
     moved = 2 * total * (width + heads * value)
     return {"shape": f"{len(lengths)} x {lengths[0]} tokens, {heads} heads, state {key} x {value}, {len(plan)} segments",

@@ -709,8 +709,8 @@ int singe_gated_linear_step_f32(singe_stream_t stream, void *out, size_t out_str
  * state of a head has to fit one CTA's registers). */
 int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *projected,
                                    size_t projected_stride, const void *decay_weight, const void *decay_bias,
-                                   const void *norm_weight, float *state, const int32_t *context, size_t heads, size_t dim,
-                                   size_t vdim, size_t rank, float tau, float query_scale, float eps,
+                                   const void *norm_weight, float *state, const int32_t *context, size_t rows, size_t heads,
+                                   size_t dim, size_t vdim, size_t rank, float tau, float query_scale, float eps,
                                    const int32_t *block_row, const int32_t *block_tokens, size_t blocks,
                                    const int32_t *segments, const int32_t *segment_last, size_t segment_count, int cut,
                                    void *scratch);

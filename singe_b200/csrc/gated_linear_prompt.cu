@@ -287,24 +287,33 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) gated_linear_prepare_kerne
     }
 }
 
-// Shared-memory stage of the advance kernel (bytes): the operands as prepared, then v and g with padded rows.
+// Shared-memory stage of the advance kernel (bytes): the operands as prepared, then v and g as TMA boxes of 16 tokens x 64
+// columns, SWIZZLE_128B.
 struct StageLayout {
-    int pitch_v, v, g, bytes;
+    int v, g, bytes;
 };
 
+constexpr int kValueBox = kBlock * 128;
+
 __host__ __device__ inline StageLayout stage_layout(int dim_pad, int vdim_pad) {
+    const int boxes = (vdim_pad + 63) / 64;
     StageLayout l;
-    l.pitch_v = vdim_pad * 2 + 16;
-    l.v = operand_bytes(dim_pad);
-    l.g = l.v + kBlock * l.pitch_v;
-    l.bytes = l.g + kBlock * l.pitch_v;
+    l.v = (operand_bytes(dim_pad) + 1023) / 1024 * 1024;
+    l.g = l.v + boxes * kValueBox;
+    l.bytes = l.g + boxes * kValueBox;
     return l;
+}
+
+// Byte offset of columns v .. v + 7 (v a multiple of eight) of token t in the boxes of v or g.
+__device__ __forceinline__ uint32_t value_at(int t, int v) {
+    return static_cast<uint32_t>((v >> 6) * kValueBox + t * 128 + ((((v >> 3) & 7) ^ (t & 7)) << 4));
 }
 
 // KT = dim_pad / 16; MT = 16-row value tiles of a warp.
 // THREADS bounds the CTA; small states leave registers for three CTAs of an SM, whose latencies then hide one another.
 template <int KT, int MT, int THREADS, bool STATE_ONLY>
-__global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 ? 3 : 1) gated_linear_advance_kernel(const PromptParams p) {
+__global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 ? 3 : 1) gated_linear_advance_kernel(
+    const __grid_constant__ CUtensorMap value_map, const PromptParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
     constexpr int kDim = KT * 16;
@@ -319,19 +328,15 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
     constexpr OperandLayout kOperands = operand_layout(kDim);
     const StageLayout layout = stage_layout(kDim, s.vdim_pad);
     const int stages = p.stages;
-    extern __shared__ __align__(128) uint8_t advance_shared[];
+    extern __shared__ uint8_t advance_raw[];
+    uint8_t *advance_shared = advance_raw + ((1024u - (smem_u32(advance_raw) & 1023u)) & 1023u);
     float *squares = reinterpret_cast<float *>(advance_shared + stages * layout.bytes);  // [8 or more][16]
     const uint32_t bars = smem_u32(squares + max(warps, 8) * kBlock);
-    // Nothing of a stage may hold a NaN: rows past a short block and columns past vdim meet zeros in the products.
-    for (int i = tid; i < stages * layout.bytes / 16; i += blockDim.x) {
-        reinterpret_cast<uint4 *>(advance_shared)[i] = make_uint4(0u, 0u, 0u, 0u);
-    }
     for (int i = tid; i < max(warps, 8) * kBlock; i += blockDim.x) squares[i] = 0.0f;
     if (tid == 0) {
         for (int i = 0; i < stages; ++i) mbar_init(bars + 8 * i, 1);
         mbar_init_fence();
     }
-    fence_proxy_async_shared();
     __syncthreads();
     const size_t state_size = static_cast<size_t>(s.vdim_pad) * kDim;
     const size_t slot = static_cast<size_t>(segment) * s.heads + head;
@@ -392,25 +397,25 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
         }
     }
 
-    // One warp brings a block in: the operands in one bulk copy, v and g row by row.
+    // One warp brings a block in: the operands in one bulk copy, v and g in boxes.  What a box holds past a short block or
+    // past the head's columns belongs to other rows or columns; it meets zeros in k and P, or is never stored.
+    const int value_boxes = (s.vdim_pad + 63) / 64;
     auto load_block = [&](int index) {
         if (warp != 0) return;
         const int block = first_block + index;
         const uint32_t bar = bars + 8 * (index % stages);
         const uint32_t stage = smem_u32(advance_shared) + (index % stages) * layout.bytes;
-        const int row0 = p.block_row[block], tokens = p.block_tokens[block];
         constexpr uint32_t kFrom = STATE_ONLY ? kOperands.state_part : 0, kBytes = kOperands.bytes - kFrom;
-        const uint32_t row_bytes = s.vdim * 2;
+        const int boxes = value_boxes * (STATE_ONLY ? 1 : 2);
         if (lane == 0) {
-            mbar_expect_tx(bar, kBytes + tokens * row_bytes * (STATE_ONLY ? 1 : 2));
+            mbar_expect_tx(bar, kBytes + boxes * kValueBox);
             bulk_load(stage + kFrom, p.operands + (static_cast<size_t>(block) * s.heads + head) * kOperands.bytes + kFrom, kBytes, bar);
         }
         __syncwarp();
-        const int t = lane & 15;
-        if (t < tokens && (lane < 16 || !STATE_ONLY)) {
-            const __nv_bfloat16 *source = p.projected + (row0 + t) * p.stride + 2 * s.heads * s.dim +
-                                          (lane < 16 ? 0 : s.heads * s.vdim) + head * s.vdim;
-            bulk_load(stage + (lane < 16 ? layout.v : layout.g) + t * layout.pitch_v, source, row_bytes, bar);
+        if (lane < boxes) {
+            const int gate = lane < value_boxes ? 0 : 1, box = lane - gate * value_boxes;
+            tma_load_2d(stage + (gate ? layout.g : layout.v) + box * kValueBox, &value_map, bar,
+                        2 * s.heads * s.dim + gate * s.heads * s.vdim + head * s.vdim + box * 64, p.block_row[block]);
         }
     };
     for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
@@ -453,7 +458,7 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
             const int t = (lane & 7) + ((lane >> 4) << 3);
-            ldmatrix_x4_trans(stage + layout.v + t * layout.pitch_v + (value0 + m * 16 + ((lane >> 3) & 1) * 8) * 2, value[m][0],
+            ldmatrix_x4_trans(stage + layout.v + value_at(t, value0 + m * 16 + ((lane >> 3) & 1) * 8), value[m][0],
                               value[m][1], value[m][2], value[m][3]);
         }
         float o[MT][2][4] = {};
@@ -540,7 +545,11 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
                 for (int i = 0; i < 2; ++i) {
                     float square = 0.0f;
 #pragma unroll
-                    for (int m = 0; m < MT; ++m) square += o[m][n][i] * o[m][n][i] + o[m][n][2 + i] * o[m][n][2 + i];
+                    for (int m = 0; m < MT; ++m) {
+                        const int v = value0 + m * 16 + g;  // rows past vdim hold what is not this head's
+                        square += v < s.vdim ? o[m][n][i] * o[m][n][i] : 0.0f;
+                        square += v + 8 < s.vdim ? o[m][n][2 + i] * o[m][n][2 + i] : 0.0f;
+                    }
                     square += __shfl_xor_sync(0xffffffffu, square, 4);
                     square += __shfl_xor_sync(0xffffffffu, square, 8);
                     square += __shfl_xor_sync(0xffffffffu, square, 16);
@@ -569,8 +578,7 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
             // the gates come out of shared memory in the layout of o^T, and the result goes back to where they were
 #pragma unroll
             for (int m = 0; m < MT; ++m) {
-                const uint32_t at = stage + layout.g + ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch_v +
-                                    (value0 + m * 16 + ((lane >> 3) & 1) * 8) * 2;
+                const uint32_t at = stage + layout.g + value_at((lane & 7) + ((lane >> 4) << 3), value0 + m * 16 + ((lane >> 3) & 1) * 8);
                 uint32_t gate[4];
                 ldmatrix_x4_trans(at, gate[0], gate[1], gate[2], gate[3]);
 #pragma unroll
@@ -588,7 +596,7 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
             __syncthreads();
             for (int t = store_row; t < tokens; t += store_rows) {
                 *reinterpret_cast<uint4 *>(p.out + (row0 + t) * p.out_stride + head * s.vdim + store_piece * 8) =
-                    *reinterpret_cast<const uint4 *>(here + layout.g + t * layout.pitch_v + store_piece * 16);
+                    *reinterpret_cast<const uint4 *>(here + layout.g + value_at(t, store_piece * 8));
             }
         }
     }
@@ -631,9 +639,9 @@ __global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 
 }
 
 template <int KT, int MT, int THREADS>
-int launch_advance(cudaStream_t stream, PromptParams p, size_t segments, bool cut, int warps) {
+int launch_advance(cudaStream_t stream, const CUtensorMap &value_map, PromptParams p, size_t segments, bool cut, int warps) {
     const StageLayout layout = stage_layout(KT * 16, p.shape.vdim_pad);
-    const auto shared_bytes = [&](int stages) { return stages * layout.bytes + (warps > 8 ? warps : 8) * kBlock * 4 + kMaxStages * 8; };
+    const auto shared_bytes = [&](int stages) { return stages * layout.bytes + (warps > 8 ? warps : 8) * kBlock * 4 + kMaxStages * 8 + 1024; };
     p.stages = kMaxStages;  // as many as leave room for two more CTAs, three at least
     while (p.stages > 3 && shared_bytes(p.stages) > 75 * 1024) --p.stages;
     const int bytes = shared_bytes(p.stages);
@@ -644,11 +652,11 @@ int launch_advance(cudaStream_t stream, PromptParams p, size_t segments, bool cu
     if (cut) {
         SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, THREADS, true>, bytes, configured_state));
         SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, THREADS, true>, grid, dim3(warps * 32), bytes, stream,
-                                        kLaunchGlue, 1, p));
+                                        kLaunchGlue, 1, value_map, p));
     }
     SINGE_CUDA_TRY(ensure_dynamic_shared(gated_linear_advance_kernel<KT, MT, THREADS, false>, bytes, configured));
     SINGE_CUDA_TRY(launch_dependent(gated_linear_advance_kernel<KT, MT, THREADS, false>, grid, dim3(warps * 32), bytes, stream,
-                                    kLaunchGlue, 1, p));
+                                    kLaunchGlue, 1, value_map, p));
     return launch_status();
 }
 
@@ -683,12 +691,12 @@ size_t singe_gated_linear_prompt_scratch(size_t heads, size_t dim, size_t vdim, 
 
 int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *projected,
                                    size_t projected_stride, const void *decay_weight, const void *decay_bias,
-                                   const void *norm_weight, float *state, const int32_t *context, size_t heads, size_t dim,
+                                   const void *norm_weight, float *state, const int32_t *context, size_t rows, size_t heads, size_t dim,
                                    size_t vdim, size_t rank, float tau, float query_scale, float eps,
                                    const int32_t *block_row, const int32_t *block_tokens, size_t blocks,
                                    const int32_t *segments, const int32_t *segment_last, size_t segment_count, int cut,
                                    void *scratch) {
-    if (heads == 0 || rank == 0 || blocks == 0 || segment_count == 0 || out_stride < heads * vdim ||
+    if (rows == 0 || heads == 0 || rank == 0 || blocks == 0 || segment_count == 0 || out_stride < heads * vdim ||
         projected_stride < 2 * heads * (dim + vdim) + rank) {
         return SINGE_ERR_INVALID_LENGTH;
     }
@@ -745,10 +753,18 @@ int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_
     SINGE_CUDA_TRY(launch_dependent(gated_linear_prepare_kernel,
                                     dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((heads + kPrepareWarps - 1) / kPrepareWarps)),
                                     dim3(kPrepareWarps * 32), shared, s, kLaunchGlue, 1, p));
+    CUtensorMap value_map;
+    {
+        const uint64_t dims[2] = {2 * heads * (dim + vdim) + rank, rows};
+        const uint64_t strides[1] = {projected_stride * 2};
+        const uint32_t box[2] = {64, kBlock};
+        SINGE_TRY(encode_tensor_map(&value_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, projected, dims, strides, box,
+                                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    }
     const bool segmented = cut != 0;
 #define SINGE_ADVANCE(KT_, MT_, THREADS_)                                          \
     if (dim_pad == KT_ * 16 && value_tiles == MT_ && warps * 32 <= THREADS_) {      \
-        return launch_advance<KT_, MT_, THREADS_>(s, p, segment_count, segmented, warps); \
+        return launch_advance<KT_, MT_, THREADS_>(s, value_map, p, segment_count, segmented, warps); \
     }
     SINGE_ADVANCE(1, 1, 256)
     SINGE_ADVANCE(1, 1, 512)

@@ -402,7 +402,7 @@ class GatedLinear:
             scratch = ops.torch.empty(int(ks.lib().singe_gated_linear_prompt_scratch(c.heads, c.dim, c.vdim, rows.blocks,
                                                                                      rows.count)),
                                       dtype=ops.torch.uint8, device="cuda")
-            ops.call("singe_gated_linear_prompt_bf16", stream, *operands, step.context, *sizes, rows.rows, rows.tokens,
+            ops.call("singe_gated_linear_prompt_bf16", stream, *operands, step.context, t, *sizes, rows.rows, rows.tokens,
                      rows.blocks, rows.segments, rows.last, rows.count, int(rows.cut), scratch)
         if rows is None or step.short_count > 0:
             ops.call(f"singe_gated_linear_step_{ops.suffix}", stream, *operands, step.first, step.fresh_tokens,

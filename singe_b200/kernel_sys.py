@@ -133,8 +133,8 @@ SIGNATURES = {
     "singe_latent_decode_bf16": [_p, _p, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _z, _z, _z, _f, _p],
     "singe_windowed_prefill_attention_bf16": [_p, _p, _p, _p, _p, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z,
                                               _z, _f],
-    "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _f, _f, _f, _p, _p, _z,
-                                       _p, _p, _z, _i, _p],
+    "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _z, _p, _z, _z, _z, _z, _f, _f, _f, _p, _p,
+                                       _z, _p, _p, _z, _i, _p],
     "singe_gated_linear_prompt_scratch": [_z, _z, _z, _z, _z],
     "singe_latent_decode_splits": [_z, _z, _z, _z],
 }

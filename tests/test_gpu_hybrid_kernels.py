@@ -367,7 +367,7 @@ def test_recurrence_block_by_block(heads, dim, vdim, rank, tau, bias, spread):
     size = int(ks.lib().singe_gated_linear_prompt_scratch(heads, dim, vdim, len(tokens), len(plan)))
     assert size > 0
     ops.call("singe_gated_linear_prompt_bf16", stream(), out, out.stride(0), projected, projected.stride(0),
-             dev(a2).to(ops.dtype), dev(b).to(ops.dtype), dev(norm).to(ops.dtype), state, i32(contexts), heads, dim, vdim, rank,
+             dev(a2).to(ops.dtype), dev(b).to(ops.dtype), dev(norm).to(ops.dtype), state, i32(contexts), len(x), heads, dim, vdim, rank,
              tau, dim ** -0.5, 1e-5, i32(np.concatenate(starts)), i32(tokens), len(tokens), i32(segments), i32(plan[:, 4]),
              len(plan), 1, torch.empty(size, dtype=torch.uint8, device="cuda"))
     got, after = host(out).reshape(-1, heads, vdim), host(state)
