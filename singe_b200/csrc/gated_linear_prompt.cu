@@ -312,7 +312,7 @@ __device__ __forceinline__ uint32_t value_at(int t, int v) {
 // KT = dim_pad / 16; MT = 16-row value tiles of a warp.
 // THREADS bounds the CTA; small states leave registers for three CTAs of an SM, whose latencies then hide one another.
 template <int KT, int MT, int THREADS, bool STATE_ONLY>
-__global__ void __launch_bounds__(THREADS, KT <= 4 && MT == 1 && THREADS <= 256 ? 3 : 1) gated_linear_advance_kernel(
+__global__ void __launch_bounds__(THREADS, KT <= 4 && THREADS <= 256 / MT ? 3 : 1) gated_linear_advance_kernel(
     const __grid_constant__ CUtensorMap value_map, const PromptParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
@@ -667,7 +667,8 @@ bool prompt_tiling(size_t dim, size_t vdim, int &dim_pad, int &value_tiles, int 
     while (static_cast<size_t>(dim_pad) < dim) dim_pad *= 2;
     const int tiles = static_cast<int>((vdim + 15) / 16);
     const int most = dim_pad <= 64 ? 16 : 8;  // warps: 32 (64) state registers a thread at one (two) tiles leave room for 512 threads
-    value_tiles = tiles <= most ? 1 : 2;
+    // two value tiles a warp share the operands it reads, where they leave the registers for it
+    value_tiles = tiles <= most && (tiles % 2 != 0 || dim_pad > 64) ? 1 : 2;
     warps = (tiles + value_tiles - 1) / value_tiles;
     return warps <= most && !(dim_pad == 256 && value_tiles == 2);
 }
@@ -768,12 +769,15 @@ int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_
     }
     SINGE_ADVANCE(1, 1, 256)
     SINGE_ADVANCE(1, 1, 512)
+    SINGE_ADVANCE(1, 2, 128)
     SINGE_ADVANCE(1, 2, 512)
     SINGE_ADVANCE(2, 1, 256)
     SINGE_ADVANCE(2, 1, 512)
+    SINGE_ADVANCE(2, 2, 128)
     SINGE_ADVANCE(2, 2, 512)
     SINGE_ADVANCE(4, 1, 256)
     SINGE_ADVANCE(4, 1, 512)
+    SINGE_ADVANCE(4, 2, 128)
     SINGE_ADVANCE(4, 2, 512)
     SINGE_ADVANCE(8, 1, 256)
     SINGE_ADVANCE(8, 2, 256)
