@@ -351,7 +351,6 @@ __device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, 12
 __global__ void __launch_bounds__(kTcThreads, 2)
     latent_decode_tcgen05_kernel(const __grid_constant__ CUtensorMap cache_map, const __grid_constant__ CUtensorMap query_map,
                                  const LatentDecode p, const LatentTcShape shape) {
-    grid_dependency_wait();
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -371,6 +370,29 @@ __global__ void __launch_bounds__(kTcThreads, 2)
     volatile uint32_t *holder_ptr = reinterpret_cast<volatile uint32_t *>(smem_raw + (holder - raw));
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < stages; ++i) {
+            mbar_init(bar_full + 8 * i, 1);
+            mbar_init(bar_empty + 8 * i, 1);
+        }
+        mbar_init(bar_query, 1);
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(bar_scores + 8 * i, 1);
+            mbar_init(bar_weights + 8 * i, 4);
+        }
+        mbar_init(bar_values, 1);
+        mbar_init_fence();
+    }
+    if (warp == 1) {
+        tmem_alloc(holder, 256);
+        tmem_relinquish();
+    }
+    tcgen05_fence_before();
+    __syncthreads();
+    tcgen05_fence_after();
+    const uint32_t tmem = *holder_ptr;
+    grid_dependency_wait();  // the set-up above ran beside the kernels before
+
     const int query = blockIdx.x, split = blockIdx.y, head0 = blockIdx.z * kTcHeads;
     const int sequence = p.sequence_of[query];
     const bool known = sequence >= 0 && sequence < p.sequences;
@@ -397,33 +419,13 @@ __global__ void __launch_bounds__(kTcThreads, 2)
                 }
             }
         }
-        return;
     }
 
-    if (threadIdx.x == 0) {
-        for (int i = 0; i < stages; ++i) {
-            mbar_init(bar_full + 8 * i, 1);
-            mbar_init(bar_empty + 8 * i, 1);
-        }
-        mbar_init(bar_query, 1);
-        for (int i = 0; i < 2; ++i) {
-            mbar_init(bar_scores + 8 * i, 1);
-            mbar_init(bar_weights + 8 * i, 4);
-        }
-        mbar_init(bar_values, 1);
-        mbar_init_fence();
-    }
-    if (warp == 1) {
-        tmem_alloc(holder, 256);
-        tmem_relinquish();
-    }
-    tcgen05_fence_before();
-    __syncthreads();
-    tcgen05_fence_after();
-    const uint32_t tmem = *holder_ptr;
     bool failed = false;
 
-    if (warp == 0) {
+    if (tile_count == 0) {
+        // nothing to attend to
+    } else if (warp == 0) {
         // ---------------- TMA producer ----------------
         if (lane == 0) {
             prefetch_tensor_map(&cache_map);
