@@ -49,9 +49,9 @@ ONES = model(64, 64, 1e-6,
 # more heads than one CTA of the decode kernel takes, the widest latent, a wide recurrence
 WIDE = model(256, 300, 1e-6,
              latent(34, 128, 96, 128, 512, 300, 0.088, ff=512),
-             gla(2, 128, 256, 16.0),
+             gla(2, 128, 256, 10.0),
              latent(18, 64, 64, 96, 320, 150, 0.125),
-             gla(4, 48, 64, 8.0, ff=128))
+             gla(4, 40, 72, 8.0, ff=128))
 
 
 def bf16(values):

@@ -92,7 +92,7 @@ def test_embedding_with_its_norm(dtype, width):
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
-@pytest.mark.parametrize("q_rank,kv_rank,cache_width", [(24, 40, 64), (7, 5, 8), (80, 96, 128), (1536, 512, 512)])
+@pytest.mark.parametrize("q_rank,kv_rank,cache_width", [(24, 40, 64), (7, 5, 8), (72, 104, 128), (1536, 512, 512)])
 def test_latent_norms_and_cache_write(dtype, q_rank, kv_rank, cache_width):
     rng = np.random.default_rng(q_rank)
     ops = Ops(dtype)
@@ -172,7 +172,7 @@ def edge_queries(rng, keys, positions, window, heads, sharp=30.0):
 
 
 @pytest.mark.parametrize("heads,latent,page_size,window,splits", [
-    (1, 64, 16, 1, 1), (5, 64, 16, 2, 1), (8, 128, 16, 136, 3), (16, 192, 4, 65, 2), (20, 256, 7, 64, 1),
+    (1, 64, 16, 1, 1), (5, 64, 16, 2, 1), (9, 128, 16, 150, 3), (16, 192, 4, 65, 2), (20, 256, 7, 64, 1),
     (34, 512, 16, 300, 4), (32, 320, 16, 100000, 7), (3, 448, 1, 33, 5), (40, 64, 16, 0, 2),
     (32, 512, 64, 200, 2), (8, 256, 128, 129, 1), (33, 320, 64, 64, 3), (4, 64, 8, 77, 2), (16, 448, 32, 1, 1)])
 def test_decode_attention_at_window_and_page_edges(heads, latent, page_size, window, splits):
@@ -309,10 +309,10 @@ def recurrence_expect(x, a2, b, norm, first, n, state, heads, dim, vdim, rank, t
 
 
 CASES = [  # heads, dim, vdim, rank, tau, bias, spread
-    (2, 48, 64, 16, 16.0, 2.0, 1.0),
+    (3, 56, 80, 20, 12.0, 2.0, 1.0),
     (3, 24, 40, 5, 4.0, 2.0, 1.0),
     (1, 8, 8, 1, 1.0, 0.0, 2.0),
-    (2, 128, 256, 16, 16.0, 2.0, 0.5),
+    (2, 128, 256, 24, 10.0, 2.0, 0.5),
     (1, 256, 128, 8, 8.0, 1.0, 0.5),
     (4, 64, 128, 16, 1.0, -6.0, 3.0),     # decays too strong to factor
     (2, 16, 272, 3, 2.0, -3.0, 6.0),      # some blocks are, some are not
