@@ -28,7 +28,9 @@ CONFIGS = {"mixed": util.MIXED, "odd": util.ODD, "ones": util.ONES, "wide": util
 def snapshots(tmp_path_factory):
     made = {}
     for name, config in CONFIGS.items():
-        weights = util.make_weights(config, seed=len(name))
+        # Seeds under which no sequence starts ill-conditioned: a recurrent layer's first output is (q . k) v, RMS-normed,
+        # and where q and k are all but orthogonal the norm blows their rounding up.
+        weights = util.make_weights(config, seed=len(name) + 1)
         made[name] = (config, weights, util.write_snapshot(tmp_path_factory.mktemp(name), config, weights))
     return made
 
