@@ -182,7 +182,7 @@ def prompt_attention_kernels(size: str, lengths, peaks) -> dict:
     lens = torch.tensor(lengths, dtype=torch.int32, device="cuda")
     offsets = torch.tensor(np.cumsum([0] + lengths)[:-1], dtype=torch.int32, device="cuda")
     windowed = lambda: o.call("singe_windowed_prefill_attention_bf16", _stream(), out, lse, query, rows, rows.data_ptr() + heads * dim * 2,
-                              2 * heads * dim, lens, lens, offsets, offsets, gate, heads, len(lengths), total, total, heads, dim,
+                              2 * heads * dim, lens, lens, offsets, offsets, gate, heads, len(lengths), total, total, heads, heads, dim,
                               window, dim ** -0.5)
     kv = heads // 4
     keys, values = normal(total, kv, dim), normal(total, kv, dim)

@@ -31,6 +31,8 @@ TYPES = {
     "const int32_t *": "*const i32",
     "uint32_t *": "*mut u32",
     "const uint32_t *": "*const u32",
+    "const uint8_t *": "*const u8",
+    "const double *": "*const f64",
     "uint32_t *const *": "*const *mut u32",
 }
 RETURNS = {"int": " -> c_int", "size_t": " -> usize", "const char *": " -> *const c_char", "void": ""}

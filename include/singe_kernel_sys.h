@@ -635,6 +635,10 @@ int singe_latent_norm_cache_write_f32(singe_stream_t stream, void *q_out, size_t
 int singe_gather_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, size_t count,
                       size_t row_bytes, size_t source_rows, uint32_t *status);
 
+/* out[targets[i], :] = source[rows[i], :], target rows below out_rows. */
+int singe_move_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, const int32_t *targets,
+                    size_t count, size_t row_bytes, size_t source_rows, size_t out_rows, uint32_t *status);
+
 /* singe_argmax_bf16 over f32 logits. */
 int singe_argmax_f32(singe_stream_t stream, float *best_value, int64_t *best_index, const float *logits,
                      size_t row_stride, size_t rows, size_t width, int64_t index_offset);
@@ -671,7 +675,7 @@ int singe_latent_decode_bf16(singe_stream_t stream, void *out, float *attn_scrat
 size_t singe_latent_decode_splits(size_t queries, size_t heads, size_t latent, size_t key_bound);
 
 /* Causal prompt attention with a sliding window on the tensor core (the kernel of singe_ragged_kv_prefill_attention_bf16):
- * query, out [total_query_tokens, heads, head_dim]; key and value rows of kv_row_stride elements, heads side by side.
+ * query, out [total_query_tokens, heads, head_dim]; key and value rows of kv_row_stride elements, kv_heads side by side.
  * Sequence b owns query rows [offsets_q[b], offsets_q[b] + lens_q[b]) and key rows [offsets_kv[b], ...+ lens_kv[b]); the
  * queries are the sequence's last tokens, and a query sees itself and the window - 1 tokens before it.  gate != NULL: row t
  * of head h is multiplied by sigmoid(gate[t * gate_row_stride + h]).  lse [total_query_tokens, heads], natural log.
@@ -681,7 +685,7 @@ int singe_windowed_prefill_attention_bf16(singe_stream_t stream, void *out, floa
                                           const int32_t *lens_kv, const int32_t *offsets_q, const int32_t *offsets_kv,
                                           const void *gate, size_t gate_row_stride, size_t batch,
                                           size_t total_query_tokens, size_t total_kv_tokens, size_t heads,
-                                          size_t head_dim, size_t window, float scale);
+                                          size_t kv_heads, size_t head_dim, size_t window, float scale);
 
 /* Gated linear attention, one head's state S [dim, vdim] in f32 per sequence:
  *   S_t = diag(sigmoid(z_t)^(1/tau)) S_(t-1) + k_t v_t^T,  o_t = query_scale * S_t^T q_t,  z_t = decay_weight a_t + decay_bias,
@@ -715,6 +719,120 @@ int singe_gated_linear_prompt_bf16(singe_stream_t stream, void *out, size_t out_
                                    const int32_t *segments, const int32_t *segment_last, size_t segment_count, int cut,
                                    void *scratch);
 size_t singe_gated_linear_prompt_scratch(size_t heads, size_t dim, size_t vdim, size_t blocks, size_t segments);
+
+/* ---- several residual streams, attention within chunks, short convolutions, the gated delta rule ---- */
+
+/* streams [rows, count, width] f32.  All streams of row t start as table[ids[t], :] (negative ids wrap, ids outside the table
+ * take row 0 and set *status = 1), then normed (may be NULL) = rms_norm(sum_s in[s] streams[s]) * weight, with rms_norm(x) =
+ * x / sqrt(mean(x^2) + eps).  in NULL: the plain sum.  count <= 16; width <= 51200. */
+int singe_stream_embedding_norm_bf16(singe_stream_t stream, float *streams, const void *table, const int64_t *ids,
+                                     const float *in, void *normed, size_t normed_stride, const void *weight, size_t rows,
+                                     size_t count, size_t width, size_t vocab, float eps, uint32_t *status);
+int singe_stream_embedding_norm_f32(singe_stream_t stream, float *streams, const void *table, const int64_t *ids,
+                                    const float *in, void *normed, size_t normed_stride, const void *weight, size_t rows,
+                                    size_t count, size_t width, size_t vocab, float eps, uint32_t *status);
+/* All streams at once from the old ones: streams[t] = sum_s mix[s, t] streams[s] + out[t] y (written back when store != 0), then
+ * normed (may be NULL) = rms_norm(sum_t in[t] streams[t]) * weight * normed_scale.  parts 1: delta is y.  parts 2: a delta row
+ * holds two outputs of `width`, the second from column second_at on, y = part_scale * (rms_norm(left) * left_weight + rms_norm(right) * right_weight). */
+int singe_stream_step_norm_bf16(singe_stream_t stream, float *streams, const void *delta, size_t delta_stride, int parts,
+                                size_t second_at, const void *left_weight, const void *right_weight, float part_scale, const float *mix,
+                                const float *out, const float *in, int store, void *normed, size_t normed_stride,
+                                const void *weight, float normed_scale, size_t rows, size_t count, size_t width, float eps);
+int singe_stream_step_norm_f32(singe_stream_t stream, float *streams, const void *delta, size_t delta_stride, int parts,
+                               size_t second_at, const void *left_weight, const void *right_weight, float part_scale, const float *mix,
+                               const float *out, const float *in, int store, void *normed, size_t normed_stride,
+                               const void *weight, float normed_scale, size_t rows, size_t count, size_t width, float eps);
+
+/* Attention of query rows over a paged cache in which a query sees only the chunk of `chunk` positions it stands in, counted
+ * from position 0 of its sequence: query i belongs to sequence_of[i] (a row of block_table [sequences, table_stride]) and sees
+ * positions floor((lens[i] - 1) / chunk) * chunk .. lens[i] - 1 (lens[i] == 0: zeros).  query, out [queries, heads, head_dim];
+ * caches [pages, page_size, kv_heads, head_dim].  bf16 with page_size 16, head_dim 64 or 128 and at most eight heads per
+ * kv head runs the tiled split-K decode kernel, given attn_scratch f32 [queries, heads, splits, head_dim] and lse_scratch
+ * [queries, heads, splits] (unused when splits is 1, but not NULL); everything else the general kernel. */
+int singe_chunked_attention_bf16(singe_stream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                                 const void *key_cache, const void *value_cache, const int32_t *sequence_of,
+                                 const int32_t *lens, const int32_t *block_table, size_t queries, size_t heads,
+                                 size_t kv_heads, size_t head_dim, size_t page_size, size_t pages, size_t sequences,
+                                 size_t table_stride, size_t chunk, size_t splits, float scale, uint32_t *status);
+int singe_chunked_attention_f32(singe_stream_t stream, float *out, const float *query, const float *key_cache,
+                                const float *value_cache, const int32_t *sequence_of, const int32_t *lens,
+                                const int32_t *block_table, size_t queries, size_t heads, size_t kv_heads, size_t head_dim,
+                                size_t page_size, size_t pages, size_t sequences, size_t table_stride, size_t chunk,
+                                float scale, uint32_t *status);
+
+/* Short causal convolution over time on every projected channel, y_t = sum_j taps[j] * u_(t - tap_count + 1 + j), zero before a
+ * sequence's start, and what follows it.  The convolved columns are the first `span` of a projected row; taps [tap_count, span];
+ * state [sequences, tap_count - 1, span] holds each sequence's last projected rows.  Token t belongs to sequence_of[t], which
+ * owns rows [first, first + fresh) and had `context` tokens before; fresh == 0 marks an idle row.  Sequences with one new token
+ * have their state moved on by these calls; for the others singe_conv_state must follow.  tap_count <= 16.
+ *
+ * Attention: u = projection + bias (bias [span] or NULL).  Columns [q (heads*dim) | k (kv_heads*dim) at key_at | v
+ * (kv_heads*vdim) at value_at]; q and k are RMS-normed over all their columns together with query_norm and key_norm, dimensions
+ * 2i and 2i + 1 of every head turn by position * frequencies[i] for i < pairs, cosines and sines times rotation_scale.  Heads are
+ * padded with zeros to key_size / value_size; queries go to rows of `query` (an idle row becomes zeros), keys and values to
+ * (write_pages[t], write_slots[t]) of the caches where cached is NULL or cached[t] != 0, and to row packed_rows[t] of the packed
+ * arrays where that is not negative. */
+int singe_conv_attention_inputs_bf16(
+    singe_stream_t stream, void *query, size_t query_stride, void *key_cache, void *value_cache, void *packed_keys,
+    void *packed_values, const void *projected, size_t projected_stride, const void *bias, const void *taps, void *state,
+    const void *query_norm, const void *key_norm, const double *frequencies, size_t pairs, float rotation_scale,
+    const int64_t *positions, const int32_t *sequence_of, const int32_t *first, const int32_t *fresh, const int32_t *context,
+    const int64_t *write_pages, const int64_t *write_slots, const uint8_t *cached, const int32_t *packed_rows,
+    size_t packed_count, size_t rows, size_t sequences, size_t tap_count, size_t heads, size_t kv_heads, size_t dim,
+    size_t vdim, size_t key_size, size_t value_size, size_t key_at, size_t value_at, size_t span, size_t pages,
+    size_t page_size, float eps, uint32_t *status);
+int singe_conv_attention_inputs_f32(
+    singe_stream_t stream, void *query, size_t query_stride, void *key_cache, void *value_cache, void *packed_keys,
+    void *packed_values, const void *projected, size_t projected_stride, const void *bias, const void *taps, void *state,
+    const void *query_norm, const void *key_norm, const double *frequencies, size_t pairs, float rotation_scale,
+    const int64_t *positions, const int32_t *sequence_of, const int32_t *first, const int32_t *fresh, const int32_t *context,
+    const int64_t *write_pages, const int64_t *write_slots, const uint8_t *cached, const int32_t *packed_rows,
+    size_t packed_count, size_t rows, size_t sequences, size_t tap_count, size_t heads, size_t kv_heads, size_t dim,
+    size_t vdim, size_t key_size, size_t value_size, size_t key_at, size_t value_at, size_t span, size_t pages,
+    size_t page_size, float eps, uint32_t *status);
+/* Recurrence: mixed = silu(convolution) for all columns (idle rows are left alone); inverse [rows, 2 * unit_heads] holds
+ * 1 / sqrt(sum(x^2) + eps) of the first unit_heads pieces of `dim` columns and of as many from second_at on. */
+int singe_conv_recurrence_inputs_bf16(singe_stream_t stream, void *mixed, size_t mixed_stride, float *inverse,
+                                      const void *projected, size_t projected_stride, const void *taps, void *state,
+                                      const int32_t *sequence_of, const int32_t *first, const int32_t *fresh,
+                                      const int32_t *context, size_t rows, size_t sequences, size_t tap_count,
+                                      size_t unit_heads, size_t dim, size_t second_at, size_t span, float eps);
+int singe_conv_recurrence_inputs_f32(singe_stream_t stream, void *mixed, size_t mixed_stride, float *inverse,
+                                     const void *projected, size_t projected_stride, const void *taps, void *state,
+                                     const int32_t *sequence_of, const int32_t *first, const int32_t *fresh,
+                                     const int32_t *context, size_t rows, size_t sequences, size_t tap_count,
+                                     size_t unit_heads, size_t dim, size_t second_at, size_t span, float eps);
+int singe_conv_state_bf16(singe_stream_t stream, const void *projected, size_t projected_stride, void *state,
+                          const int32_t *first, const int32_t *fresh, size_t rows, size_t sequences, size_t tap_count,
+                          size_t span);
+int singe_conv_state_f32(singe_stream_t stream, const void *projected, size_t projected_stride, void *state,
+                         const int32_t *first, const int32_t *fresh, size_t rows, size_t sequences, size_t tap_count,
+                         size_t span);
+
+/* Gated delta rule, one head's state S [dim, vdim] in f32 per sequence, token by token:
+ *   S <- diag(g) S;  u = sigmoid(b) (v - S^T k);  S <- S + k u^T;  o = S^T q,   g = exp(-exp(rate) softplus(z + bias)),
+ *   out = rms_norm(o) * norm_weight * sigmoid(gate)
+ * with q and k unit vectors, q also times dim^(-1/2).  mixed rows hold [q (kv_heads*dim) | k at key_at | v (heads*vdim) at
+ * value_at] and `inverse` their inverse lengths (singe_conv_recurrence_inputs); strength rows hold b (heads); decay rows hold z
+ * (heads*dim) and from gate_at on the gates (heads*vdim).  Rows, context, idle rows and `longest` as in
+ * singe_gated_linear_step. */
+int singe_gated_delta_step_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *mixed, size_t mixed_stride,
+                                const float *inverse, const void *strength, size_t strength_stride, const void *decay,
+                                size_t decay_stride, const float *rate, const float *bias, const void *norm_weight,
+                                float *state, const int32_t *first, const int32_t *count, const int32_t *context, size_t rows,
+                                size_t sequences, size_t heads, size_t kv_heads, size_t dim, size_t vdim, size_t key_at,
+                                size_t value_at, size_t gate_at, float eps, size_t longest);
+int singe_gated_delta_step_f32(singe_stream_t stream, void *out, size_t out_stride, const void *mixed, size_t mixed_stride,
+                               const float *inverse, const void *strength, size_t strength_stride, const void *decay,
+                               size_t decay_stride, const float *rate, const float *bias, const void *norm_weight,
+                               float *state, const int32_t *first, const int32_t *count, const int32_t *context, size_t rows,
+                               size_t sequences, size_t heads, size_t kv_heads, size_t dim, size_t vdim, size_t key_at,
+                               size_t value_at, size_t gate_at, float eps, size_t longest);
+
+/* out = silu(gate) * up, elementwise in f32. */
+int singe_silu_mul_f32(singe_stream_t stream, float *out, size_t output_row_stride, const float *gate, const float *up,
+                       size_t input_row_stride, size_t rows, size_t width);
+
 /* Explicit tile choice for the two GEMM entry points, process-wide: block_n in {32,64,128,256},
  * k_slices_per_stage in {1,2,4,8}; 0 = choose from the problem shape.
  * Replaces: TuningChoice::Explicit(MatmulTuning { tile, .. }) (singe-kernel/src/cuda/matmul.rs:58-77). */

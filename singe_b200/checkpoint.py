@@ -25,6 +25,7 @@ import numpy as np
 
 from .hybrid import GatedLinearConfig, HybridConfig, LatentAttentionConfig, LayerConfig
 from .llama import LlamaConfig, Shard
+from .parallel_mixer import (TILED_PAGE, ChunkedAttentionConfig, GatedDeltaConfig, ParallelConfig, Rotation, YarnScaling)
 
 CHECKPOINT_STEMS = ("model", "diffusion_pytorch_model")   # transformers' name first, then diffusers'
 
@@ -294,7 +295,7 @@ def load_llama(directory: str, shard: Shard | None = None, shard_lm_head: bool =
 
 
 # ------------------------------------------------------------------------------------------------
-# layer-list decoders (Kavalorn)
+# layer-list decoders (Kavalorn, Vatolorn)
 # ------------------------------------------------------------------------------------------------
 
 def _section(fields: dict, where: str, *names):
@@ -330,23 +331,73 @@ def _gated_linear(fields: dict, where: str, tensor_shape) -> GatedLinearConfig:
                              rank=int(tensor_shape("mix.a1")[0]), tau=float(tau))
 
 
-_MIXERS = {"latent_attention": _latent_attention, "gla": _gated_linear}
+def _rotation(fields: dict, where: str, dim: int) -> Rotation:
+    dims, base, scaling = _section({"scaling": None, **fields}, where, "dims", "base", "scaling")
+    dims, base = _positive(dims, f"{where}.dims"), float(base)
+    if dims % 2 or dims > dim or base <= 1.0:
+        raise UnsupportedConfig(f"{where}: dims {dims}, base {base}")
+    if scaling is None:
+        return Rotation(dims, base)
+    values = [float(value) for value in _section(scaling, f"{where}.scaling", "factor", "original", "fast", "slow")]
+    if min(values) <= 0.0:
+        raise UnsupportedConfig(f"{where}.scaling: {values}")
+    return Rotation(dims, base, YarnScaling(*values))
+
+
+def _grouped(heads, kv_heads, where: str):
+    heads, kv_heads = _positive(heads, f"{where}.heads"), _positive(kv_heads, f"{where}.kv_heads")
+    if heads % kv_heads:
+        raise UnsupportedConfig(f"{where}: {heads} heads on {kv_heads}")
+    return heads, kv_heads
+
+
+def _chunked_attention(fields: dict, where: str) -> ChunkedAttentionConfig:
+    heads, kv_heads, dim, vdim, scale, mask, conv, rot = _section(fields, where, "heads", "kv_heads", "dim", "vdim", "scale", "mask",
+                                                                  "conv", "rot")
+    (chunk,) = _section(mask, f"{where}.mask", "size")
+    dim, vdim, conv = [_positive(value, where) for value in (dim, vdim, conv)]
+    return ChunkedAttentionConfig(*_grouped(heads, kv_heads, where), dim, vdim, float(scale),
+                                  _positive(chunk, f"{where}.mask.size"), conv, _rotation(rot, f"{where}.rot", dim))
+
+
+def _gated_delta(fields: dict, where: str, tensor_shape) -> GatedDeltaConfig:
+    heads, kv_heads, dim, vdim, conv = _section(fields, where, "heads", "kv_heads", "dim", "vdim", "conv")
+    dim, vdim, conv = [_positive(value, where) for value in (dim, vdim, conv)]
+    return GatedDeltaConfig(*_grouped(heads, kv_heads, where), dim, vdim, conv, rank=int(tensor_shape("mix.right.a1")[0]),
+                            gate_rank=int(tensor_shape("mix.right.g1")[0]))
+
+
+def _parallel(fields: dict, where: str, tensor_shape) -> ParallelConfig:
+    left, right = _section(fields, where, "left", "right")
+    return ParallelConfig(_chunked_attention(left, f"{where}.left"), _gated_delta(right, f"{where}.right", tensor_shape))
+
+
+# design -> its mixers, whether its feed-forwards are gated, and the keys of config.json beyond those every design has
+_DESIGNS = {
+    "Kavalorn": ({"latent_attention": _latent_attention, "gla": _gated_linear}, False, ()),
+    "Vatolorn": ({"parallel": _parallel}, True, ("streams", "logit_scale")),
+}
 
 
 def read_hybrid_config(directory: str, snapshot: "Snapshot") -> HybridConfig:
-    """``config.json`` of a layer-list model.  Sizes the configuration leaves out (the rank of the decay projection) come
+    """``config.json`` of a layer-list model.  Sizes the configuration leaves out (the ranks of low-rank projections) come
     from the tensors of the layer that owns the weights."""
     with open(os.path.join(directory, "config.json")) as handle:
         fields = json.load(handle)
-    _, entries, norm, vocab, width = _section(fields, "config.json", "architecture", "layers", "norm", "vocab", "width")
+    if not isinstance(fields, dict) or fields.get("architecture") not in _DESIGNS:
+        raise UnsupportedConfig("config.json names no layer-list design")
+    mixers, gated, own = _DESIGNS[fields["architecture"]]
+    _, entries, norm, vocab, width, *rest = _section(fields, "config.json", "architecture", "layers", "norm", "vocab", "width", *own)
     (eps,) = _section(norm, "norm", "eps")
     config = HybridConfig(width=_positive(width, "width"), vocab=_positive(vocab, "vocab"), eps=float(eps))
+    if own:
+        config.streams, config.logit_scale, config.page_size = _positive(rest[0], "streams"), float(rest[1]), TILED_PAGE
     borrowed = HybridConfig(layers=[LayerConfig(None, 0, entry.get("weights_of")) for entry in entries])
     for index, entry in enumerate(entries):
         where = f"layers[{index}]"
         entry = {"mlp": None, "weights_of": None, **entry}
         kind, mixer, mlp, _ = _section(entry, where, "type", "mixer", "mlp", "weights_of")
-        if kind not in _MIXERS:
+        if kind not in mixers:
             raise UnsupportedConfig(f"{where}: mixer {kind}")
         ffn = 0
         if mlp is not None:
@@ -365,8 +416,7 @@ def read_hybrid_config(directory: str, snapshot: "Snapshot") -> HybridConfig:
                 raise CheckpointError(f"checkpoint keys: missing {full}")
             return snapshot.array(full).shape
 
-        config.layers.append(LayerConfig(_MIXERS[kind](mixer, f"{where}.mixer", tensor_shape), ffn,
-                                         entry["weights_of"]))
+        config.layers.append(LayerConfig(mixers[kind](mixer, f"{where}.mixer", tensor_shape), ffn, entry["weights_of"], gated))
     for index, layer in enumerate(config.layers):
         source = config.layers[config.owner(index)]
         if (layer.mixer, layer.ffn) != (source.mixer, source.ffn):
@@ -377,7 +427,9 @@ def read_hybrid_config(directory: str, snapshot: "Snapshot") -> HybridConfig:
 def hybrid_names(config: HybridConfig) -> dict:
     """Parameter name -> expected shape, for the whole model."""
     w = config.width
-    names = {"embed": (config.vocab, w), "embed.norm": (w,), "final.norm": (w,), "head": (config.vocab, w)}
+    names = {"embed": (config.vocab, w), "final.norm": (w,), "head": (config.vocab, w)}
+    if not config.streams:
+        names["embed.norm"] = (w,)
     for index, layer in enumerate(config.layers):
         if layer.weights_of is not None:
             continue
@@ -385,16 +437,37 @@ def hybrid_names(config: HybridConfig) -> dict:
         names[prefix + "norm1"] = (w,)
         if layer.ffn:
             names.update({prefix + "norm2": (w,), prefix + "mlp.up": (layer.ffn, w), prefix + "mlp.down": (w, layer.ffn)})
+            if layer.gated:
+                names[prefix + "mlp.gate"] = (layer.ffn, w)
+        for sublayer in range(1, 3 if layer.ffn else 2) if config.streams else ():
+            names.update({f"{prefix}hc{sublayer}.{name}": shape for name, shape in
+                          (("in", (config.streams,)), ("out", (config.streams,)), ("mix", (config.streams, config.streams)))})
         if isinstance(m, LatentAttentionConfig):
             mix = {"dq": (m.q_rank, w), "dq.norm": (m.q_rank,), "uq": (m.heads * m.dim, m.q_rank),
                    "dkv": (m.kv_rank, w), "dkv.norm": (m.kv_rank,), "uk": (m.heads * m.dim, m.kv_rank),
                    "uv": (m.heads * m.vdim, m.kv_rank), "g": (m.heads, w), "o": (w, m.heads * m.vdim)}
+        elif isinstance(m, ParallelConfig):
+            mix = _parallel_names(m, w)
         else:
             mix = {"q": (m.heads * m.dim, w), "k": (m.heads * m.dim, w), "v": (m.heads * m.vdim, w),
                    "g": (m.heads * m.vdim, w), "o": (w, m.heads * m.vdim), "norm": (m.vdim,), "a1": (m.rank, w),
                    "a2": (m.heads * m.dim, m.rank), "a2.b": (m.heads * m.dim,)}
         names.update({f"{prefix}mix.{name}": shape for name, shape in mix.items()})
     return names
+
+
+def _parallel_names(m: ParallelConfig, w: int) -> dict:
+    left, right = m.left, m.right
+    mix = {"left.out": (w,), "right.out": (w,), "left.o": (w, left.heads * left.vdim), "right.o": (w, right.heads * right.vdim),
+           "left.q.norm": (left.heads * left.dim,), "left.k.norm": (left.kv_heads * left.dim,), "right.norm": (right.vdim,),
+           "right.b": (right.heads, w), "right.A_log": (right.heads,), "right.dt_bias": (right.heads * right.dim,),
+           "right.a1": (right.rank, w), "right.a2": (right.heads * right.dim, right.rank),
+           "right.g1": (right.gate_rank, w), "right.g2": (right.heads * right.vdim, right.gate_rank)}
+    for name, rows in (("q", left.heads * left.dim), ("k", left.kv_heads * left.dim), ("v", left.kv_heads * left.vdim)):
+        mix.update({f"left.{name}": (rows, w), f"left.{name}.b": (rows,), f"left.{name}.conv": (rows, left.taps)})
+    for name, rows in (("q", right.kv_heads * right.dim), ("k", right.kv_heads * right.dim), ("v", right.heads * right.vdim)):
+        mix.update({f"right.{name}": (rows, w), f"right.{name}.conv": (rows, right.taps)})
+    return mix
 
 
 def load_hybrid(directory: str):

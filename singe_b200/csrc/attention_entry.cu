@@ -22,6 +22,10 @@ int paged_decode_splitk(cudaStream_t stream, int element, void *out, float *attn
                         size_t max_splits, float scale, bool partials_only, uint32_t *status,
                         const RaggedDecode *ragged, unsigned hints, const QueryRotation *rotation, uint32_t *tickets,
                         const FusedStep *fused);
+int paged_decode_chunked(cudaStream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                         const void *key_cache, const void *value_cache, const int32_t *lens, const uint32_t *block_table,
+                         const ChunkedDecode &chunked, size_t queries, size_t heads, size_t kv_heads, size_t head_dim,
+                         size_t pages, size_t table_stride, size_t splits, float scale, uint32_t *status);
 extern int g_decode_prefetch_pages;
 // prefill_tcgen05.cu
 bool prefill_fast_path(size_t heads, size_t kv_heads, size_t head_dim, size_t total_query_tokens, const void *query,
@@ -110,6 +114,43 @@ struct DecodePagedPolicy {
         plan.end = static_cast<int>(len);
         plan.kv_head = head / (heads / kv_heads);
         plan.handle = static_cast<long long>(b) * stride;
+        return 1;
+    }
+    __device__ long long key_offset(const RowPlan<T> &plan, int pos) const {
+        const long long block = table[plan.handle + pos / block_size];
+        if (block >= physical_blocks) return -1;
+        return ((block * block_size + pos % block_size) * kv_heads + plan.kv_head) * head_dim;
+    }
+    __device__ const T *key_base() const { return key_cache; }
+    __device__ const T *value_base() const { return value_cache; }
+};
+
+// Queries that see the chunk of positions they stand in, over the paged cache of the sequence each belongs to.
+template <typename T>
+struct ChunkedPolicy {
+    const T *query;
+    T *out;
+    const T *key_cache;
+    const T *value_cache;
+    const int32_t *lens;
+    const uint32_t *table;
+    ChunkedDecode chunked;
+    int heads, kv_heads, head_dim, block_size;
+    long long physical_blocks, stride;
+
+    __device__ int locate(size_t row, RowPlan<T> &plan) const {
+        const size_t i = row / heads;
+        const int head = static_cast<int>(row - i * heads);
+        const long long len = lens[i] < 0 ? 0 : lens[i];
+        const int sequence = chunked.sequence_of[i];
+        if (sequence < 0 || sequence >= chunked.sequences || len > stride * block_size) return -1;
+        plan.query = query + row * head_dim;
+        plan.out = out + row * head_dim;
+        plan.lse = nullptr;
+        plan.start = len > 0 ? static_cast<int>((len - 1) / chunked.size * chunked.size) : 0;
+        plan.end = static_cast<int>(len);
+        plan.kv_head = head / (heads / kv_heads);
+        plan.handle = static_cast<long long>(sequence) * stride;
         return 1;
     }
     __device__ long long key_offset(const RowPlan<T> &plan, int pos) const {
@@ -673,6 +714,43 @@ int packed_prefill_general(cudaStream_t stream, void *out, float *lse, const voi
                                        nullptr);
 }
 
+template <typename T>
+int chunked_attention(cudaStream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                      const void *key_cache, const void *value_cache, const int32_t *sequence_of, const int32_t *lens,
+                      const int32_t *block_table, size_t queries, size_t heads, size_t kv_heads, size_t head_dim,
+                      size_t page_size, size_t pages, size_t sequences, size_t table_stride, size_t chunk, size_t splits,
+                      float scale, uint32_t *status) {
+    if (queries == 0 || sequences == 0 || chunk == 0 || splits == 0) return SINGE_ERR_INVALID_LENGTH;
+    SINGE_TRY(validate_paged_decode(queries, heads, kv_heads, head_dim, page_size, pages, table_stride, scale));
+    if (!fits_i32(sequences) || !fits_i32(chunk) || !fits_i32(table_stride * page_size)) return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    if (out == nullptr || query == nullptr || key_cache == nullptr || value_cache == nullptr || sequence_of == nullptr ||
+        lens == nullptr || block_table == nullptr) {
+        return SINGE_ERR_NULL_POINTER;
+    }
+    const ChunkedDecode chunked = {sequence_of, static_cast<int>(sequences), static_cast<int>(chunk)};
+    const uint32_t *table = reinterpret_cast<const uint32_t *>(block_table);
+    if (sizeof(T) == 2 && attn_scratch != nullptr && lse_scratch != nullptr &&
+        paged_decode_fast_path(heads, kv_heads, head_dim, page_size, key_cache, value_cache, query)) {
+        return paged_decode_chunked(stream, out, attn_scratch, lse_scratch, query, key_cache, value_cache, lens, table, chunked,
+                                    queries, heads, kv_heads, head_dim, pages, table_stride, splits, scale, status);
+    }
+    ChunkedPolicy<T> policy;
+    policy.query = static_cast<const T *>(query);
+    policy.out = static_cast<T *>(out);
+    policy.key_cache = static_cast<const T *>(key_cache);
+    policy.value_cache = static_cast<const T *>(value_cache);
+    policy.lens = lens;
+    policy.table = table;
+    policy.chunked = chunked;
+    policy.heads = static_cast<int>(heads);
+    policy.kv_heads = static_cast<int>(kv_heads);
+    policy.head_dim = static_cast<int>(head_dim);
+    policy.block_size = static_cast<int>(page_size);
+    policy.physical_blocks = static_cast<long long>(pages);
+    policy.stride = static_cast<long long>(table_stride);
+    return launch_attention_general<T>(stream, policy, queries * heads, head_dim, scale, LseKind::None, 0.0f, status);
+}
+
 template <typename T, typename Index>
 int tensor_paged(cudaStream_t stream, void *out, float *lse, const void *query, const void *key_cache,
                  const void *value_cache, const void *query_offsets, const void *page_offsets, const void *pages,
@@ -1170,6 +1248,26 @@ int singe_fmha_decode_splitk_reduce_f32(singe_stream_t stream, float *out, float
     return singe_splitk_reduce_f32(stream, out, attn_scratch, lse_scratch, batch, heads, splits, head_dim,
                                    heads * splits * head_dim, splits * head_dim, head_dim, heads * splits, splits,
                                    heads * head_dim, head_dim);
+}
+
+int singe_chunked_attention_bf16(singe_stream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                                 const void *key_cache, const void *value_cache, const int32_t *sequence_of,
+                                 const int32_t *lens, const int32_t *block_table, size_t queries, size_t heads,
+                                 size_t kv_heads, size_t head_dim, size_t page_size, size_t pages, size_t sequences,
+                                 size_t table_stride, size_t chunk, size_t splits, float scale, uint32_t *status) {
+    return chunked_attention<__nv_bfloat16>(static_cast<cudaStream_t>(stream), out, attn_scratch, lse_scratch, query, key_cache,
+                                            value_cache, sequence_of, lens, block_table, queries, heads, kv_heads, head_dim,
+                                            page_size, pages, sequences, table_stride, chunk, splits, scale, status);
+}
+
+int singe_chunked_attention_f32(singe_stream_t stream, float *out, const float *query, const float *key_cache,
+                                const float *value_cache, const int32_t *sequence_of, const int32_t *lens,
+                                const int32_t *block_table, size_t queries, size_t heads, size_t kv_heads, size_t head_dim,
+                                size_t page_size, size_t pages, size_t sequences, size_t table_stride, size_t chunk,
+                                float scale, uint32_t *status) {
+    return chunked_attention<float>(static_cast<cudaStream_t>(stream), out, nullptr, nullptr, query, key_cache, value_cache,
+                                    sequence_of, lens, block_table, queries, heads, kv_heads, head_dim, page_size, pages,
+                                    sequences, table_stride, chunk, 1, scale, status);
 }
 
 int singe_paged_attention_bf16(singe_stream_t stream, void *out, float *lse, const void *query, const void *key_cache,

@@ -56,6 +56,14 @@ struct RaggedDecode {
                                // window hides (the planning kernel has already dropped the whole pages before it)
 };
 
+// Decode attention of queries that see only the chunk of `size` positions they stand in (chunks counted from position 0 of
+// the sequence): lens[i] counts the keys up to query i from position 0, and the visible ones begin at the chunk's first.
+struct ChunkedDecode {
+    const int32_t *sequence_of;  // [queries] row of the block table
+    int sequences;
+    int size;
+};
+
 // What the tiled decode kernel needs to rotate its queries itself (singe_rotary_paged_kv_decode_attention_bf16).
 struct QueryRotation {
     const void *cos;        // [capacity, head_dim / 2] in the cache dtype

@@ -19,12 +19,11 @@
 //             A long sequence is cut into segments that run side by side: a first pass (STATE_ONLY) takes every segment
 //             but the last from a zero state (the first one from the sequence's state) to its end, and in the second
 //             pass a segment starts from the fold of its predecessors' end states.
-#include "common.cuh"
+#include "split_bf16.cuh"
 
 namespace singe {
 namespace {
 
-constexpr int kBlock = 16;             // tokens
 constexpr int kPrepareWarps = 4;
 constexpr int kMaxStages = 6;
 constexpr float kFactoredLimit = -60.0f;
@@ -75,32 +74,6 @@ struct PromptParams {
 };
 
 __host__ __device__ constexpr int operand_bytes(int dim_pad) { return operand_layout(dim_pad).bytes; }
-
-// x = hi + lo
-__device__ __forceinline__ void split_bf16(float x, __nv_bfloat16 &hi, __nv_bfloat16 &lo) {
-    hi = __float2bfloat16_rn(x);
-    lo = __float2bfloat16_rn(x - __bfloat162float(hi));
-}
-
-// The same for a pair, packed as an MMA register.
-__device__ __forceinline__ void split_pair(float x, float y, uint32_t &hi, uint32_t &lo) {
-    hi = pack2<__nv_bfloat16>(x, y);
-    lo = pack2<__nv_bfloat16>(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
-}
-
-// Bulk copy global -> shared, completing `bytes` on the mbarrier (16-byte aligned addresses and size).
-__device__ __forceinline__ void bulk_load(uint32_t target, const void *source, uint32_t bytes, uint32_t bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(target),
-                 "l"(source), "r"(bytes), "r"(bar)
-                 : "memory");
-}
-
-// ldmatrix_x4_trans's inverse: four 8x8 matrices out of MMA fragments, transposed.
-__device__ __forceinline__ void stmatrix_x4_trans(uint32_t address, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
-    asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};" ::"r"(address), "r"(r0), "r"(r1),
-                 "r"(r2), "r"(r3)
-                 : "memory");
-}
 
 // Shared memory of one warp of the prepare kernel, in bytes: the factored operands of P (q hi, lo, k hi, lo) and the
 // logarithms of the decays.
@@ -293,8 +266,6 @@ struct StageLayout {
     int v, g, bytes;
 };
 
-constexpr int kValueBox = kBlock * 128;
-
 __host__ __device__ inline StageLayout stage_layout(int dim_pad, int vdim_pad) {
     const int boxes = (vdim_pad + 63) / 64;
     StageLayout l;
@@ -302,11 +273,6 @@ __host__ __device__ inline StageLayout stage_layout(int dim_pad, int vdim_pad) {
     l.g = l.v + boxes * kValueBox;
     l.bytes = l.g + boxes * kValueBox;
     return l;
-}
-
-// Byte offset of columns v .. v + 7 (v a multiple of eight) of token t in the boxes of v or g.
-__device__ __forceinline__ uint32_t value_at(int t, int v) {
-    return static_cast<uint32_t>((v >> 6) * kValueBox + t * 128 + ((((v >> 3) & 7) ^ (t & 7)) << 4));
 }
 
 // KT = dim_pad / 16; MT = 16-row value tiles of a warp.
@@ -672,8 +638,6 @@ bool prompt_tiling(size_t dim, size_t vdim, int &dim_pad, int &value_tiles, int 
     warps = (tiles + value_tiles - 1) / value_tiles;
     return warps <= most && !(dim_pad == 256 && value_tiles == 2);
 }
-
-size_t align256(size_t bytes) { return (bytes + 255) / 256 * 256; }
 
 }  // namespace
 }  // namespace singe

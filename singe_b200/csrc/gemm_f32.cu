@@ -89,6 +89,19 @@ int launch_linear_f32(singe_stream_t stream, const LinearF32 &p, size_t batch) {
     return launch_status();
 }
 
+__device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+
+// out = silu(gate) * up, elementwise.
+__global__ void __launch_bounds__(256) silu_mul_f32_kernel(float *out, long long out_stride, const float *gate, const float *up,
+                                                           long long in_stride, int width) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const long long row = blockIdx.x;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        out[row * out_stride + c] = silu_exact(gate[row * in_stride + c]) * up[row * in_stride + c];
+    }
+}
+
 }  // namespace
 }  // namespace singe
 
@@ -118,6 +131,18 @@ int singe_linear_f32(singe_stream_t stream, float *out, const float *x, const fl
     p.ldo = static_cast<long long>(output_row_stride);
     p.squared_relu = activation == 2 ? 1 : 0;
     return launch_linear_f32(stream, p, 1);
+}
+
+int singe_silu_mul_f32(singe_stream_t stream, float *out, size_t output_row_stride, const float *gate, const float *up,
+                       size_t input_row_stride, size_t rows, size_t width) {
+    if (rows == 0 || width == 0 || input_row_stride < width || output_row_stride < width) return SINGE_ERR_INVALID_LENGTH;
+    if (!fits_i32(rows) || !fits_i32(width)) return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    if (out == nullptr || gate == nullptr || up == nullptr) return SINGE_ERR_NULL_POINTER;
+    SINGE_CUDA_TRY(launch_dependent(silu_mul_f32_kernel, dim3(static_cast<unsigned>(rows)), dim3(256), 0,
+                                    static_cast<cudaStream_t>(stream), kLaunchGlue, 1, out,
+                                    static_cast<long long>(output_row_stride), gate, up, static_cast<long long>(input_row_stride),
+                                    static_cast<int>(width)));
+    return launch_status();
 }
 
 int singe_head_linear_f32(singe_stream_t stream, float *out, const float *x, const float *weight, size_t rows,

@@ -185,6 +185,27 @@ constexpr int decode_smem_bytes() {
     return kDecodeStages * decode_stage_bytes<HD>() + 2 * kDecodeWarps * 8 * 4 + 2 * kDecodeStages * 8 + 1024;
 }
 
+// What a query of the chunked form reads: the sequence's pages from first_page on, `keys` of them counted from that page's
+// first slot, of which the first `hidden` belong to the chunk before.
+struct ChunkView {
+    int sequence, first_page, keys, hidden;
+};
+
+__device__ __forceinline__ ChunkView chunk_view(const ChunkedDecode &chunked, int query, int len, int table_stride, uint32_t *status) {
+    ChunkView view = {chunked.sequence_of[query], 0, 0, 0};
+    if (view.sequence < 0 || view.sequence >= chunked.sequences || len > table_stride * kPageTokens) {
+        if (threadIdx.x == 0) report_status(status, kStatusIndexOutOfBounds);
+        view.sequence = 0;
+        return view;
+    }
+    if (len <= 0) return view;
+    const int start = (len - 1) / chunked.size * chunked.size;
+    view.first_page = start / kPageTokens;
+    view.hidden = start - view.first_page * kPageTokens;
+    view.keys = len - view.first_page * kPageTokens;
+    return view;
+}
+
 // RAGGED selects the Tensor-surface form: the pages of sequence b start at ragged.first[b] in ragged.pages (32- or 64-bit
 // entries), p.lens and ragged.control were written by the planning kernel of the same call (control[0] != 0: "not a plain
 // decode batch, the general kernel runs instead"; control[1] = tokens per split), and finished rows also get their
@@ -199,11 +220,14 @@ constexpr int decode_smem_bytes() {
 // one-wave grid, L2 warming, the rotation of the queries, the in-kernel fold); without it the classic form is the plain
 // drop-in kernel and carries none of their registers or branches (they cost it 2 us of 58 on the bench workload).
 // OPTIONS (ragged form): tanh-capped scores and / or a sliding window's partly hidden first page.
-template <typename T, int HD, bool RAGGED, bool FUSED = false, bool EXTRAS = false, bool OPTIONS = false>
+// CHUNKED (classic form): every query sees the chunk of positions it stands in; a query's pages are those of the sequence
+// it belongs to, from the page on that holds the chunk's first position.
+template <typename T, int HD, bool RAGGED, bool FUSED = false, bool EXTRAS = false, bool OPTIONS = false, bool CHUNKED = false>
 __device__ __forceinline__ void paged_decode_body(const CUtensorMap &k_map, const CUtensorMap &v_map,
                                                   const DecodeParams &p, const StepExtras &x,
-                                                  const RaggedDecode &ragged) {
+                                                  const RaggedDecode &ragged, const ChunkedDecode &chunked = {}) {
     static_assert(!(RAGGED && FUSED), "the fused step form is a classic-form kernel");
+    static_assert(!CHUNKED || !(RAGGED || FUSED || EXTRAS || OPTIONS), "the chunked form is a classic-form kernel");
     static_assert(!FUSED || EXTRAS, "the fused step form is a decode-step kernel");
     static_assert(!(RAGGED && EXTRAS) && !(OPTIONS && !RAGGED), "extras: classic form; options: ragged form");
     constexpr int NHALF = HD / 64;
@@ -245,18 +269,26 @@ __device__ __forceinline__ void paged_decode_body(const CUtensorMap &k_map, cons
     // The ragged form's page list hangs off two more device values and is read below.
     int len = p.lens[b];
     uint32_t early_page = 0u;
+    const uint32_t *pages = p.table + static_cast<size_t>(b) * p.table_stride;
+    int page_room = p.table_stride;
+    int chunk_hidden = 0;
+    if (CHUNKED) {
+        const ChunkView view = chunk_view(chunked, b, len, p.table_stride, p.status);
+        len = view.keys;
+        chunk_hidden = view.hidden;
+        pages = p.table + static_cast<size_t>(view.sequence) * p.table_stride + view.first_page;
+        page_room = p.table_stride - view.first_page;
+    }
     if (!RAGGED && warp == kDecodeWarps) {
         const int at = split * (p.split_tokens / kPageTokens) + lane;
-        if (lane < p.split_tokens / kPageTokens && at < p.table_stride) {
-            early_page = p.table[static_cast<size_t>(b) * p.table_stride + at];
-        }
+        if (lane < p.split_tokens / kPageTokens && at < page_room) early_page = pages[at];
     }
     // A grid covers the longest possible sequence, so under mixed lengths many CTAs of split >= 1 have nothing to
     // do (40 % on config 2): those leave as soon as the length is here.
     const int bound = RAGGED ? 0x7ffffff0 : p.table_stride * kPageTokens;
     len = len < 0 ? 0 : (len > bound ? bound : len);
     const int piece = RAGGED ? ragged.control[1] : p.split_tokens;
-    const int hidden_keys = (OPTIONS && ragged.hidden != nullptr) ? ragged.hidden[b] : 0;
+    const int hidden_keys = CHUNKED ? chunk_hidden : (OPTIONS && ragged.hidden != nullptr) ? ragged.hidden[b] : 0;
     if (split > 0 && static_cast<long long>(split) * piece >= len && !p.partials_only) return;
     uint32_t qa[KSTEPS][2];
     if (warp < kDecodeWarps && !stable) {
@@ -324,7 +356,7 @@ __device__ __forceinline__ void paged_decode_body(const CUtensorMap &k_map, cons
             prefetch_tensor_map(&k_map);
             prefetch_tensor_map(&v_map);
         }
-        const uint32_t *table = p.table + static_cast<size_t>(b) * p.table_stride + first_page;
+        const uint32_t *table = pages + first_page;
         const long long ragged_at = RAGGED ? ragged.first[b] + first_page : 0;
         // Stable paging: the ring's first pages are requested ahead of the wait, up to (not including) the page that
         // holds the sequence's last key position, which the preceding kernel may still be writing.  `ahead` pages
@@ -489,11 +521,11 @@ __device__ __forceinline__ void paged_decode_body(const CUtensorMap &k_map, cons
                 s1[1] = outward * fast_tanh(s1[1] * inward) / p.scale_log2;
             }
             // visible keys: below the sequence's end and (sliding window) not among the hidden ones of its first page
-            // (the lower bound exists only in the OPTIONS form: the other kernels keep their single compare per key)
-            float x00 = (t0 < tok_end && (!OPTIONS || t0 >= hidden_keys)) ? s0[0] * p.scale_log2 : -INFINITY;
-            float x01 = (t0 + 1 < tok_end && (!OPTIONS || t0 + 1 >= hidden_keys)) ? s0[1] * p.scale_log2 : -INFINITY;
-            float x10 = (t0 + 8 < tok_end && (!OPTIONS || t0 + 8 >= hidden_keys)) ? s1[0] * p.scale_log2 : -INFINITY;
-            float x11 = (t0 + 9 < tok_end && (!OPTIONS || t0 + 9 >= hidden_keys)) ? s1[1] * p.scale_log2 : -INFINITY;
+            // (the lower bound exists only in the OPTIONS and CHUNKED forms: the other kernels keep their single compare per key)
+            float x00 = (t0 < tok_end && (!(OPTIONS || CHUNKED) || t0 >= hidden_keys)) ? s0[0] * p.scale_log2 : -INFINITY;
+            float x01 = (t0 + 1 < tok_end && (!(OPTIONS || CHUNKED) || t0 + 1 >= hidden_keys)) ? s0[1] * p.scale_log2 : -INFINITY;
+            float x10 = (t0 + 8 < tok_end && (!(OPTIONS || CHUNKED) || t0 + 8 >= hidden_keys)) ? s1[0] * p.scale_log2 : -INFINITY;
+            float x11 = (t0 + 9 < tok_end && (!(OPTIONS || CHUNKED) || t0 + 9 >= hidden_keys)) ? s1[1] * p.scale_log2 : -INFINITY;
             float tile_max = fmaxf(fmaxf(x00, x01), fmaxf(x10, x11));
             tile_max = fmaxf(tile_max, __shfl_xor_sync(0xffffffffu, tile_max, 1));
             tile_max = fmaxf(tile_max, __shfl_xor_sync(0xffffffffu, tile_max, 2));
@@ -740,14 +772,23 @@ __global__ void __launch_bounds__(kDecodeThreads, 3)
     paged_decode_body<T, HD, true, false, false, OPTIONS>(k_map, v_map, p, unused, ragged);
 }
 
+template <typename T, int HD>
+__global__ void __launch_bounds__(kDecodeThreads, 3)
+    paged_decode_chunked_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
+                                const DecodeParams p, const ChunkedDecode chunked) {
+    RaggedDecode none = {};  // never read by this form
+    StepExtras unused = {};
+    paged_decode_body<T, HD, false, false, false, false, true>(k_map, v_map, p, unused, none, chunked);
+}
+
 // Folds the split partials of every (sequence, head) row that needed more than one split.
 // Follows splitk_reduce_f32 (singe-kernel/src/cpu/attention.rs:2157-2193): out = sum_s exp(lse_s - M) attn_s / sum_s exp(lse_s - M).
 // RAGGED: the Tensor-surface form (split size and verdict from the planning kernel, base-2 LSE written too); the
 // classic form is a separate instantiation so that it carries none of that code (it measured 2 % slower with it).
-template <typename T, bool RAGGED>
+template <typename T, bool RAGGED, bool CHUNKED = false>
 __global__ void decode_combine_kernel(T *out, const float *attn_partial, const float *lse_partial, const int32_t *lens,
                                       int heads, int head_dim, int split_tokens, int max_splits, int bound,
-                                      const int *ragged_control, float *lse_out) {
+                                      const int *ragged_control, float *lse_out, const ChunkedDecode chunked) {
     grid_launch_dependents();
     grid_dependency_wait();
     if (RAGGED) {
@@ -758,6 +799,7 @@ __global__ void decode_combine_kernel(T *out, const float *attn_partial, const f
     const int b = blockIdx.y;
     const int head = blockIdx.x;
     int len = lens[b];
+    if (CHUNKED) len = chunk_view(chunked, b, len, bound / kPageTokens, nullptr).keys;
     len = len < 0 ? 0 : (len > bound ? bound : len);
     const int n = (len + split_tokens - 1) / split_tokens;
     if (n <= 1) {
@@ -779,6 +821,39 @@ __global__ void decode_combine_kernel(T *out, const float *attn_partial, const f
     if (RAGGED && threadIdx.x == 0) {
         lse_out[row] = (top + logf(denom)) * 1.4426950408889634f;  // natural log -> base 2
     }
+}
+
+struct DecodeMaps {
+    CUtensorMap k, v;
+};
+
+template <typename T, int HD>
+int encode_cache_maps(DecodeMaps &maps, const DecodeParams &params, const void *key_cache, const void *value_cache) {
+    const uint64_t dims[4] = {static_cast<uint64_t>(HD), static_cast<uint64_t>(params.kv_heads), kPageTokens,
+                              static_cast<uint64_t>(params.physical_blocks)};
+    const uint64_t strides[3] = {static_cast<uint64_t>(HD) * sizeof(T),
+                                 static_cast<uint64_t>(HD) * sizeof(T) * params.kv_heads,
+                                 static_cast<uint64_t>(HD) * sizeof(T) * params.kv_heads * kPageTokens};
+    const uint32_t box[4] = {64, 1, kPageTokens, 1};
+    SINGE_TRY(encode_tensor_map(&maps.k, TensorMapType<T>::value, 4, key_cache, dims, strides, box,
+                                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B));
+    return encode_tensor_map(&maps.v, TensorMapType<T>::value, 4, value_cache, dims, strides, box,
+                             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B);
+}
+
+template <int HD>
+int launch_chunked(cudaStream_t stream, const DecodeParams &params, const ChunkedDecode &chunked, const void *key_cache,
+                   const void *value_cache, size_t queries) {
+    using T = __nv_bfloat16;
+    static int configured[kMaxDevices] = {0};
+    constexpr int smem = decode_smem_bytes<HD>();
+    SINGE_CUDA_TRY(ensure_dynamic_shared(paged_decode_chunked_kernel<T, HD>, smem, configured));
+    DecodeMaps maps;
+    SINGE_TRY((encode_cache_maps<T, HD>(maps, params, key_cache, value_cache)));
+    const dim3 grid(static_cast<unsigned>(params.kv_heads), static_cast<unsigned>(params.max_splits), static_cast<unsigned>(queries));
+    SINGE_CUDA_TRY(launch_dependent(paged_decode_chunked_kernel<T, HD>, grid, dim3(kDecodeThreads), smem, stream,
+                                    kLaunchDecode, 1, maps.k, maps.v, params, chunked));
+    return launch_status();
 }
 
 template <typename T, int HD, bool RAGGED>
@@ -809,17 +884,9 @@ int launch_decode(cudaStream_t stream, const DecodeParams &params, const StepExt
     } else {
         SINGE_CUDA_TRY(ensure_dynamic_shared(paged_decode_kernel<T, HD>, smem, configured));
     }
-    CUtensorMap k_map, v_map;
-    const uint64_t dims[4] = {static_cast<uint64_t>(HD), static_cast<uint64_t>(params.kv_heads), kPageTokens,
-                              static_cast<uint64_t>(params.physical_blocks)};
-    const uint64_t strides[3] = {static_cast<uint64_t>(HD) * sizeof(T),
-                                 static_cast<uint64_t>(HD) * sizeof(T) * params.kv_heads,
-                                 static_cast<uint64_t>(HD) * sizeof(T) * params.kv_heads * kPageTokens};
-    const uint32_t box[4] = {64, 1, kPageTokens, 1};
-    SINGE_TRY(encode_tensor_map(&k_map, TensorMapType<T>::value, 4, key_cache, dims, strides, box,
-                                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B));
-    SINGE_TRY(encode_tensor_map(&v_map, TensorMapType<T>::value, 4, value_cache, dims, strides, box,
-                                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B));
+    DecodeMaps maps;
+    SINGE_TRY((encode_cache_maps<T, HD>(maps, params, key_cache, value_cache)));
+    const CUtensorMap &k_map = maps.k, &v_map = maps.v;
     // KV heads vary fastest: the CTAs that read the interleaved rows of the same cache pages start together.
     dim3 grid(static_cast<unsigned>(params.kv_heads), static_cast<unsigned>(params.max_splits),
               static_cast<unsigned>(batch));
@@ -966,7 +1033,8 @@ int paged_decode_splitk(cudaStream_t stream, int element, void *out, float *attn
     SINGE_CUDA_TRY(launch_dependent(decode_combine_kernel<T, RAGGED_>, grid, dim3(threads), 0, stream, kLaunchCombine, \
                                     1, static_cast<T *>(out), attn_scratch, lse_scratch, actual_seq_lens,            \
                                     params.heads, static_cast<int>(head_dim), params.split_tokens,                   \
-                                    params.max_splits, static_cast<int>(bound), shape.control, shape.lse_out))
+                                    params.max_splits, static_cast<int>(bound), shape.control, shape.lse_out,                 \
+                                    ChunkedDecode{}))
         if (element == 0) {
             if (ragged != nullptr) {
                 SINGE_COMBINE(__nv_bfloat16, true);
@@ -984,6 +1052,42 @@ int paged_decode_splitk(cudaStream_t stream, int element, void *out, float *attn
         return launch_status();
     }
     return SINGE_OK;
+}
+
+// Decode attention within chunks, for shapes paged_decode_fast_path takes: query i belongs to sequence_of[i] and sees the
+// keys of its chunk up to lens[i] - 1.  `splits` pieces of split_tokens keys cover any chunk.
+int paged_decode_chunked(cudaStream_t stream, void *out, float *attn_scratch, float *lse_scratch, const void *query,
+                         const void *key_cache, const void *value_cache, const int32_t *lens, const uint32_t *block_table,
+                         const ChunkedDecode &chunked, size_t queries, size_t heads, size_t kv_heads, size_t head_dim,
+                         size_t pages, size_t table_stride, size_t splits, float scale, uint32_t *status) {
+    if (queries > 65535 || splits > 65535) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    DecodeParams params = {};
+    params.out = out;
+    params.attn_partial = attn_scratch;
+    params.lse_partial = lse_scratch;
+    params.query = query;
+    params.lens = lens;
+    params.table = block_table;
+    params.batch = static_cast<int>(queries);
+    params.heads = static_cast<int>(heads);
+    params.kv_heads = static_cast<int>(kv_heads);
+    params.group = static_cast<int>(heads / kv_heads);
+    params.physical_blocks = static_cast<int>(pages);
+    params.table_stride = static_cast<int>(table_stride);
+    const size_t widest = static_cast<size_t>(chunked.size) + kPageTokens - 1, held = table_stride * kPageTokens;
+    params.split_tokens = static_cast<int>(paged_decode_split_tokens(widest < held ? widest : held, splits, kPageTokens));
+    params.max_splits = static_cast<int>(splits);
+    params.scale_log2 = scale * 1.4426950408889634f;
+    params.status = status;
+    SINGE_TRY(head_dim == 128 ? launch_chunked<128>(stream, params, chunked, key_cache, value_cache, queries)
+                              : launch_chunked<64>(stream, params, chunked, key_cache, value_cache, queries));
+    if (splits == 1) return SINGE_OK;
+    const dim3 grid(static_cast<unsigned>(heads), static_cast<unsigned>(queries));
+    SINGE_CUDA_TRY(launch_dependent(decode_combine_kernel<__nv_bfloat16, false, true>, grid, dim3(head_dim >= 128 ? 128 : 64), 0,
+                                    stream, kLaunchCombine, 1, static_cast<__nv_bfloat16 *>(out), attn_scratch, lse_scratch, lens,
+                                    params.heads, static_cast<int>(head_dim), params.split_tokens, params.max_splits,
+                                    static_cast<int>(held), nullptr, nullptr, chunked));
+    return launch_status();
 }
 
 }  // namespace singe

@@ -990,14 +990,14 @@ int prefill_tcgen05_windowed(cudaStream_t stream, void *out, float *lse, const v
                              const void *value, size_t kv_row_stride, const int32_t *lens_q, const int32_t *lens_kv,
                              const int32_t *offsets_q, const int32_t *offsets_kv, const void *gate, size_t gate_stride,
                              size_t batch, size_t total_query_tokens, size_t total_kv_tokens, size_t heads,
-                             size_t head_dim, size_t window, float scale) {
+                             size_t kv_heads, size_t head_dim, size_t window, float scale) {
     const uint64_t kHeadDim = head_dim;
     const CUtensorMapDataType type = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
     CUtensorMap q_map, k_map, v_map;
     const uint32_t box[3] = {64, 1, kTile};
     const uint64_t q_dims[3] = {kHeadDim, heads, total_query_tokens};
     const uint64_t q_strides[2] = {kHeadDim * 2, kHeadDim * 2 * heads};
-    const uint64_t kv_dims[3] = {kHeadDim, heads, total_kv_tokens};
+    const uint64_t kv_dims[3] = {kHeadDim, kv_heads, total_kv_tokens};
     const uint64_t kv_strides[2] = {kHeadDim * 2, static_cast<uint64_t>(kv_row_stride) * 2};
     SINGE_TRY(encode_tensor_map(&q_map, type, 3, query, q_dims, q_strides, box, CU_TENSOR_MAP_SWIZZLE_128B,
                                 CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
@@ -1014,7 +1014,7 @@ int prefill_tcgen05_windowed(cudaStream_t stream, void *out, float *lse, const v
     params.offsets_kv = offsets_kv;
     params.batch = static_cast<int>(batch);
     params.heads = static_cast<int>(heads);
-    params.kv_heads = static_cast<int>(heads);
+    params.kv_heads = static_cast<int>(kv_heads);
     params.total_q = static_cast<int>(total_query_tokens);
     params.total_kv = static_cast<int>(total_kv_tokens);
     params.causal = 2;
@@ -1049,10 +1049,10 @@ extern "C" int singe_windowed_prefill_attention_bf16(
     singe_stream_t stream, void *out, float *lse, const void *query, const void *key, const void *value,
     size_t kv_row_stride, const int32_t *lens_q, const int32_t *lens_kv, const int32_t *offsets_q,
     const int32_t *offsets_kv, const void *gate, size_t gate_row_stride, size_t batch, size_t total_query_tokens,
-    size_t total_kv_tokens, size_t heads, size_t head_dim, size_t window, float scale) {
+    size_t total_kv_tokens, size_t heads, size_t kv_heads, size_t head_dim, size_t window, float scale) {
     using namespace singe;
-    if (batch == 0 || total_query_tokens == 0 || total_kv_tokens == 0 || heads == 0 || window == 0 ||
-        kv_row_stride < heads * head_dim || (gate != nullptr && gate_row_stride < heads) || !(scale == scale)) {
+    if (batch == 0 || total_query_tokens == 0 || total_kv_tokens == 0 || heads == 0 || kv_heads == 0 || heads % kv_heads != 0 ||
+        window == 0 || kv_row_stride < kv_heads * head_dim || (gate != nullptr && gate_row_stride < heads) || !(scale == scale)) {
         return SINGE_ERR_INVALID_LENGTH;
     }
     if (!fits_i32(batch) || !fits_i32(total_query_tokens) || !fits_i32(total_kv_tokens) || !fits_i32(heads) ||
@@ -1063,10 +1063,10 @@ extern "C" int singe_windowed_prefill_attention_bf16(
         lens_kv == nullptr || offsets_q == nullptr || offsets_kv == nullptr) {
         return SINGE_ERR_NULL_POINTER;
     }
-    if (kv_row_stride % 8 != 0 || !prefill_fast_path(heads, heads, head_dim, total_query_tokens, query, key, value, out)) {
+    if (kv_row_stride % 8 != 0 || !prefill_fast_path(heads, kv_heads, head_dim, total_query_tokens, query, key, value, out)) {
         return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     }
     return prefill_tcgen05_windowed(static_cast<cudaStream_t>(stream), out, lse, query, key, value, kv_row_stride, lens_q,
                                     lens_kv, offsets_q, offsets_kv, gate, gate_row_stride, batch, total_query_tokens,
-                                    total_kv_tokens, heads, head_dim, window, scale);
+                                    total_kv_tokens, heads, kv_heads, head_dim, window, scale);
 }

@@ -6,80 +6,10 @@
 //   layer_norm(x) = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w        (deviations squared, not x^2 - mean^2)
 //   rms_norm(x)   = x / sqrt(mean(x^2) + eps) * w
 // One CTA per row; a row is read once and kept in registers between the passes.
-#include "common.cuh"
+#include "row_pack.cuh"
 
 namespace singe {
 namespace {
-
-bool aligned_to(const void *pointer, size_t bytes) { return (reinterpret_cast<uintptr_t>(pointer) & (bytes - 1)) == 0; }
-
-// Sum over the CTA, the same value in every thread.  `scratch` holds 32 floats; usable back to back.
-__device__ __forceinline__ float cta_sum(float value, float *scratch) {
-    value = warp_sum(value);
-    const int warps = (blockDim.x + 31) >> 5;
-    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = value;
-    __syncthreads();
-    float total = 0.0f;
-    for (int i = 0; i < warps; ++i) total += scratch[i];
-    __syncthreads();
-    return total;
-}
-
-template <int VEC>
-struct Pack {
-    float v[VEC];
-};
-
-template <int VEC>
-__device__ __forceinline__ Pack<VEC> load_pack(const float *p) {
-    Pack<VEC> out;
-    if constexpr (VEC == 4) {
-        const float4 raw = *reinterpret_cast<const float4 *>(p);
-        out.v[0] = raw.x;
-        out.v[1] = raw.y;
-        out.v[2] = raw.z;
-        out.v[3] = raw.w;
-    } else {
-        out.v[0] = *p;
-    }
-    return out;
-}
-
-template <int VEC>
-__device__ __forceinline__ Pack<VEC> load_pack(const __nv_bfloat16 *p) {
-    Pack<VEC> out;
-    if constexpr (VEC == 4) {
-        const uint2 raw = *reinterpret_cast<const uint2 *>(p);
-        out.v[0] = __uint_as_float(raw.x << 16);
-        out.v[1] = __uint_as_float(raw.x & 0xffff0000u);
-        out.v[2] = __uint_as_float(raw.y << 16);
-        out.v[3] = __uint_as_float(raw.y & 0xffff0000u);
-    } else {
-        out.v[0] = __bfloat162float(*p);
-    }
-    return out;
-}
-
-template <int VEC>
-__device__ __forceinline__ void store_pack(float *p, const Pack<VEC> &x) {
-    if constexpr (VEC == 4) {
-        *reinterpret_cast<float4 *>(p) = make_float4(x.v[0], x.v[1], x.v[2], x.v[3]);
-    } else {
-        *p = x.v[0];
-    }
-}
-
-template <int VEC>
-__device__ __forceinline__ void store_pack(__nv_bfloat16 *p, const Pack<VEC> &x) {
-    if constexpr (VEC == 4) {
-        *reinterpret_cast<uint2 *>(p) = make_uint2(pack2<__nv_bfloat16>(x.v[0], x.v[1]), pack2<__nv_bfloat16>(x.v[2], x.v[3]));
-    } else {
-        *p = __float2bfloat16_rn(x.v[0]);
-    }
-}
-
-constexpr int kHeldPacks = 8;      // packs a thread keeps of its row
-constexpr int kNormThreads = 512;  // at most: rows up to 512 * 8 * VEC wide
 
 // The layer norm of the row held in `x` (kHeldPacks packs per thread), in place.
 template <typename T, int VEC>
@@ -237,10 +167,10 @@ __global__ void __launch_bounds__(256)
     }
 }
 
-// out[i, :] = source[rows[i], :] in 16-byte pieces.
+// out[targets[i], :] = source[rows[i], :] in 16-byte pieces (targets == nullptr: out[i, :]).
 __global__ void __launch_bounds__(256)
-    gather_rows_kernel(uint4 *out, const uint4 *source, const int32_t *rows, long long count, int pieces,
-                       long long source_rows, uint32_t *status) {
+    gather_rows_kernel(uint4 *out, const uint4 *source, const int32_t *rows, const int32_t *targets, long long count, int pieces,
+                       long long source_rows, long long out_rows, uint32_t *status) {
     grid_launch_dependents();
     grid_dependency_wait();
     const long long total = count * pieces;
@@ -248,12 +178,18 @@ __global__ void __launch_bounds__(256)
          index += static_cast<long long>(gridDim.x) * blockDim.x) {
         const long long row = index / pieces;
         const long long from = rows[row];
-        if (from < 0 || from >= source_rows) {
+        const long long piece = index - row * pieces;
+        const long long to = targets == nullptr ? row : targets[row];
+        if (to < 0 || to >= out_rows) {
             report_status(status, kStatusIndexOutOfBounds);
-            out[index] = make_uint4(0u, 0u, 0u, 0u);
             continue;
         }
-        out[index] = source[from * pieces + (index - row * pieces)];
+        if (from < 0 || from >= source_rows) {
+            report_status(status, kStatusIndexOutOfBounds);
+            out[to * pieces + piece] = make_uint4(0u, 0u, 0u, 0u);
+            continue;
+        }
+        out[to * pieces + piece] = source[from * pieces + piece];
     }
 }
 
@@ -317,16 +253,6 @@ __global__ void __launch_bounds__(1024)
         best_index[blockIdx.x] = static_cast<long long>(where) + index_offset;
     }
 }
-
-unsigned norm_threads(size_t width, int vec) {
-    // four packs a thread: fewer warps to bring together than with one, and loads enough in flight
-    const size_t packs = (width + vec - 1) / vec;
-    size_t threads = ((packs + 3) / 4 + 31) / 32 * 32;
-    if (threads > kNormThreads) threads = kNormThreads;
-    return static_cast<unsigned>(threads);
-}
-
-bool row_fits(size_t width, int vec) { return width <= static_cast<size_t>(kNormThreads) * kHeldPacks * vec; }
 
 template <typename T>
 int embedding_layer_norm(singe_stream_t stream, float *residual, const void *table, const int64_t *ids,
@@ -432,9 +358,9 @@ SINGE_RESIDUAL_NORM_ENTRIES(bf16, __nv_bfloat16)
 SINGE_RESIDUAL_NORM_ENTRIES(f32, float)
 #undef SINGE_RESIDUAL_NORM_ENTRIES
 
-int singe_gather_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, size_t count,
-                      size_t row_bytes, size_t source_rows, uint32_t *status) {
-    if (count == 0 || row_bytes == 0 || source_rows == 0) return SINGE_ERR_INVALID_LENGTH;
+static int gather_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, const int32_t *targets,
+                       size_t count, size_t row_bytes, size_t source_rows, size_t out_rows, uint32_t *status) {
+    if (count == 0 || row_bytes == 0 || source_rows == 0 || out_rows == 0) return SINGE_ERR_INVALID_LENGTH;
     if (out == nullptr || source == nullptr || rows == nullptr) return SINGE_ERR_NULL_POINTER;
     if (row_bytes % 16 != 0 || !aligned_to(out, 16) || !aligned_to(source, 16)) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     if (!fits_i32(row_bytes) || !fits_i32(count)) return SINGE_ERR_LENGTH_EXCEEDS_I32;
@@ -444,9 +370,21 @@ int singe_gather_rows(singe_stream_t stream, void *out, const void *source, cons
     if (blocks > most) blocks = most;
     SINGE_CUDA_TRY(launch_dependent(gather_rows_kernel, dim3(static_cast<unsigned>(blocks)), dim3(256), 0,
                                     static_cast<cudaStream_t>(stream), kLaunchGlue, 1, static_cast<uint4 *>(out),
-                                    static_cast<const uint4 *>(source), rows, static_cast<long long>(count),
-                                    static_cast<int>(pieces), static_cast<long long>(source_rows), status));
+                                    static_cast<const uint4 *>(source), rows, targets, static_cast<long long>(count),
+                                    static_cast<int>(pieces), static_cast<long long>(source_rows),
+                                    static_cast<long long>(out_rows), status));
     return launch_status();
+}
+
+int singe_gather_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, size_t count,
+                      size_t row_bytes, size_t source_rows, uint32_t *status) {
+    return gather_rows(stream, out, source, rows, nullptr, count, row_bytes, source_rows, count, status);
+}
+
+int singe_move_rows(singe_stream_t stream, void *out, const void *source, const int32_t *rows, const int32_t *targets,
+                    size_t count, size_t row_bytes, size_t source_rows, size_t out_rows, uint32_t *status) {
+    if (targets == nullptr) return SINGE_ERR_NULL_POINTER;
+    return gather_rows(stream, out, source, rows, targets, count, row_bytes, source_rows, out_rows, status);
 }
 
 int singe_argmax_f32(singe_stream_t stream, float *best_value, int64_t *best_index, const float *logits,

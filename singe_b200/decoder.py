@@ -55,13 +55,15 @@ class PageTable:
 
     ``window`` (0: none) is the most tokens any layer looks back over, the token itself included: a page that no later
     token of its sequence can see goes back to the pool at the sequence's next step, and the scratch page takes its
-    place in the sequence's list."""
+    place in the sequence's list.  ``chunks`` are the sizes of the chunks of positions that layers see instead of a window: such
+    a layer sees nothing before the chunk the token stands in."""
 
-    def __init__(self, sequences: int, capacity: int, page_size: int, pool: int, window: int = 0):
+    def __init__(self, sequences: int, capacity: int, page_size: int, pool: int, window: int = 0, chunks=()):
         self.page_size = page_size
         self.capacity = capacity
         self.pool = pool
         self.window = window
+        self.chunks = tuple(chunks)
         self.padding = 0
         self.free: list[int] = []
         self.pages: list[list[int]] = [[] for _ in range(sequences)]
@@ -76,10 +78,10 @@ class PageTable:
 
     @classmethod
     def create_shared(cls, sequences: int, capacity: int, page_size: int, cache_tokens: int,
-                      window: int = 0) -> "PageTable":
-        if sequences == 0 or capacity <= 0 or page_size <= 0 or cache_tokens <= 0 or window < 0:
+                      window: int = 0, chunks=()) -> "PageTable":
+        if sequences == 0 or capacity <= 0 or page_size <= 0 or cache_tokens <= 0 or window < 0 or any(c <= 0 for c in chunks):
             raise PageTableError("page table size")
-        return cls(sequences, capacity, page_size, (cache_tokens - 1) // page_size + 1, window)
+        return cls(sequences, capacity, page_size, (cache_tokens - 1) // page_size + 1, window, chunks)
 
     def with_padding(self, padding: int) -> "PageTable":
         self.padding = padding
@@ -109,14 +111,18 @@ class PageTable:
 
     def _unseen(self, row: int) -> list:
         """Places in a sequence's page list that its next token and all after it cannot see any more."""
-        if self.window == 0:
+        if self.window == 0 and not self.chunks:
             return []
-        dead = max(self.lengths[row] - self.window + 1, 0) // self.page_size
+        length = self.lengths[row]   # the next token's position
+        oldest = [length // size * size for size in self.chunks]
+        if self.window > 0:
+            oldest.append(max(length - self.window + 1, 0))
+        dead = min(oldest) // self.page_size
         return [place for place in range(dead) if self.pages[row][place] != self.pool]
 
     def table_length(self) -> int:
         held = self.pool
-        if self.window > 0:  # lists also name the scratch page, once for every page given back
+        if self.window > 0 or self.chunks:  # lists also name the scratch page, once for every page given back
             held = max(held, len(self.pages) * ((self.capacity - 1) // self.page_size + 1))
         return held + len(self.pages) + (self.padding + self.page_size - 1) // self.page_size
 

@@ -1,7 +1,7 @@
 """Decoder whose configuration lists its layers one by one, each with its own mixer and an optional feed-forward.
 
 ``HybridDecoder`` is a ``PagedDecoder``: the page table, the one-token step and its CUDA graph, the generation loop and
-the checkpoint reader are the ones every decoder here uses.  What is new stands beside them:
+the checkpoint reader are the ones every decoder here uses.  Its parts:
 
   ``LatentAttention``   attention over a low-rank latent of the context.  The cache holds one normalised latent row per
                         token, shared by all heads, behind the page table; a sliding window bounds what a token sees and
@@ -9,9 +9,11 @@ the checkpoint reader are the ones every decoder here uses.  What is new stands 
   ``GatedLinear``       gated linear attention: a recurrent state per sequence, [heads, dim, vdim] in f32, in the
                         sequence's row; a sequence's first token starts it from zero, so a row that is used again needs
                         no clearing.
-  feed-forward          down(relu(up(h))^2)
+  ``ParallelMixer``     chunked attention and the gated delta rule side by side (``parallel_mixer``)
+  feed-forward          down(relu(up(h))^2) or down(silu(gate(h)) * up(h))
+  residual              one stream with layer norms, or several with RMS norms (``residual``)
 
-A layer may borrow another layer's weights; its cache or state is always its own.  The residual stream and all norms
+A layer may borrow another layer's weights; its cache or state is always its own.  The residual streams and all norms
 are f32.  ``dtype`` "bfloat16" keeps weights and activations in bf16 (f32 accumulation, tensor-core kernels); "float32"
 computes everything in true 32-bit with the library's f32 kernels.
 
@@ -28,6 +30,9 @@ import numpy as np
 
 from . import kernel_sys as ks
 from .decoder import PagedDecoder, PageTable
+from .layer_ops import BlockRows, ChunkRows, ExpandedRows, Ops, StepRows, plan_chunks, round_up
+from .parallel_mixer import ParallelConfig, ParallelMixer
+from .residual import LayerNormResidual, StreamResidual, Sublayer
 
 EXPANDED_HEAD_SIZES = (64, 128)  # head sizes of the tensor-core prompt attention; smaller heads are padded with zeros
 ABSORBED_LATENT_LIMIT = 512      # widest latent the tensor-core decode attention takes
@@ -65,6 +70,7 @@ class LayerConfig:
     mixer: object
     ffn: int = 0               # 0: the layer has no feed-forward
     weights_of: int | None = None
+    gated: bool = False        # the feed-forward is silu(gate) * up instead of relu(up)^2
 
 
 @dataclass
@@ -73,7 +79,9 @@ class HybridConfig:
     width: int = 0
     vocab: int = 0
     eps: float = 1e-6
-    page_size: int = 64        # a page of this size is one tile of the decode attention
+    page_size: int = 64        # a page of this size is one tile of the decode attention over latents
+    streams: int = 0           # 0: one residual stream with layer norms; else that many, with RMS norms
+    logit_scale: float = 1.0   # with streams
 
     def owner(self, index: int) -> int:
         """The layer whose weights layer ``index`` uses."""
@@ -86,141 +94,13 @@ class HybridConfig:
         return index
 
     def window(self) -> int:
-        """The most tokens any layer looks back over through the cache."""
+        """The most tokens any layer with a sliding window looks back over through the cache; 0 when chunks alone bound it."""
         return max((layer.mixer.window for layer in self.layers if isinstance(layer.mixer, LatentAttentionConfig)),
-                   default=1)
+                   default=0 if self.chunks() else 1)
 
-
-def round_up(value: int, multiple: int) -> int:
-    return (value + multiple - 1) // multiple * multiple
-
-
-# ------------------------------------------------------------------------------------------------
-# kernels behind one activation type
-# ------------------------------------------------------------------------------------------------
-
-class Ops:
-    """The library's entry points for one activation type, and buffers laid out the way they want them (rows of whole
-    16-byte pieces)."""
-
-    def __init__(self, dtype: str):
-        import torch
-
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"activation type {dtype}")
-        self.torch = torch
-        self.dtype = getattr(torch, dtype)
-        self.is_bf16 = dtype == "bfloat16"
-        self.suffix = "bf16" if self.is_bf16 else "f32"
-
-    def call(self, name: str, *arguments) -> None:
-        code = getattr(ks.lib(), name)(*[a.data_ptr() if hasattr(a, "data_ptr") else a for a in arguments])
-        if code != ks.OK:
-            raise RuntimeError(f"{name}: status {code} ({ks.status_string(code)})")
-
-    def rows(self, rows: int, columns: int):
-        """[rows, columns] of the activation type with padded row stride."""
-        return self.torch.empty((rows, round_up(columns, 8)), dtype=self.dtype, device="cuda")[:, :columns]
-
-    def weight(self, array):
-        """A matrix on the device with padded row stride, or a vector; the padding is zero."""
-        torch = self.torch
-        tensor = torch.as_tensor(array).to("cuda").to(self.dtype)
-        if tensor.dim() < 2:
-            return tensor.contiguous()
-        out = torch.zeros((tensor.shape[0], round_up(tensor.shape[1], 8)), dtype=self.dtype, device="cuda")
-        out[:, : tensor.shape[1]] = tensor
-        return out[:, : tensor.shape[1]]
-
-    def linear(self, stream, out, x, weight, activation: int = 0) -> None:
-        m, k = x.shape
-        n = weight.shape[0]
-        if self.is_bf16:
-            self.call("singe_linear_bf16", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0), out.stride(0),
-                      activation, ks.HINT_STABLE_WEIGHTS)
-        else:
-            self.call("singe_linear_f32", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0), out.stride(0),
-                      activation)
-
-    def linear_f32_out(self, stream, out, x, weight) -> None:
-        """f32 results whatever the activation type (logits)."""
-        m, k = x.shape
-        n = weight.shape[0]
-        if self.is_bf16:
-            self.call("singe_matmul_bf16_f32", stream, out, x, weight, m, n, k, x.stride(0), weight.stride(0),
-                      out.stride(0), 0, 1)
-        else:
-            self.linear(stream, out, x, weight)
-
-    def head_linear(self, stream, out, x, weight, heads: int, gate=None) -> None:
-        """out[t, h] = x[t, h] . weight[h]^T (* sigmoid(gate[t, h])); x and out hold the heads side by side, weight stacks
-        them [heads, columns, reduction]."""
-        columns, reduction = weight.shape[1], weight.shape[2]
-        arguments = [stream, out, x, weight, x.shape[0], heads, columns, reduction, x.stride(0), x.shape[1] // heads,
-                     weight.stride(1), weight.stride(0) // weight.stride(1), out.stride(0), out.shape[1] // heads,
-                     gate, 0 if gate is None else gate.stride(0)]
-        if self.is_bf16:
-            arguments.append(ks.HINT_STABLE_WEIGHTS)
-        self.call(f"singe_head_linear_{self.suffix}", *arguments)
-
-    def add_layer_norm(self, stream, residual, delta, normed, weight, eps: float) -> None:
-        self.call(f"singe_add_layer_norm_{self.suffix}", stream, residual, delta,
-                  0 if delta is None else delta.stride(0), normed, 0 if normed is None else normed.stride(0), weight,
-                  residual.shape[0], residual.shape[1], eps)
-
-
-# ------------------------------------------------------------------------------------------------
-# one step's rows, as the mixers read them
-# ------------------------------------------------------------------------------------------------
-
-@dataclass
-class StepRows:
-    """Device inputs of a step.  int64: tokens, positions, pages, slots per packed row and the paging lists of the
-    Tensor-surface attention; int32: each sequence's first row, new tokens and earlier tokens, the block table, and the
-    rows that take the decode attention with the sequence and the number of visible keys of each."""
-    count: int
-    tokens: object
-    pages: object
-    slots: object
-    query_offsets: object
-    page_offsets: object
-    page_list: object
-    last_page_lengths: object
-    first: object
-    fresh_tokens: object
-    context: object
-    table: object
-    short_rows: object        # int32 [n], or None: row i of the step is query i
-    short_sequences: object
-    short_lens: object
-    short_count: int
-    expanded: dict = field(default_factory=dict)   # window -> ExpandedRows of the longer sequences
-    blocks: dict = field(default_factory=dict)     # heads -> BlockRows of the longer sequences
-
-
-@dataclass
-class ExpandedRows:
-    """What the prompt attention reads for one window: the cache rows whose keys and values it needs, packed sequence by
-    sequence, and each sequence's lengths and offsets."""
-    gather: object
-    keys: int
-    lens_q: object
-    lens_kv: object
-    offsets_q: object
-    offsets_kv: object
-    sequences: int
-
-
-@dataclass
-class BlockRows:
-    """What the recurrence's prompt kernel reads: the blocks of the longer sequences and the segments that run side by side."""
-    rows: object
-    tokens: object
-    blocks: int
-    segments: object
-    last: object
-    count: int
-    cut: bool
+    def chunks(self) -> list:
+        """The chunk sizes of the layers whose tokens see their own chunk."""
+        return sorted({layer.mixer.left.chunk for layer in self.layers if isinstance(layer.mixer, ParallelConfig)})
 
 
 def plan_segments(blocks_of, heads: int, sms: int):
@@ -366,7 +246,7 @@ class LatentAttention:
         ops.call("singe_windowed_prefill_attention_bf16", stream, attended, lse, query, keys_values,
                  keys_values.data_ptr() + c.heads * size * 2, keys_values.stride(0), rows.lens_q, rows.lens_kv,
                  rows.offsets_q, rows.offsets_kv, gate, gate.stride(0), rows.sequences, query.shape[0], rows.keys,
-                 c.heads, size, c.window, c.scale)
+                 c.heads, c.heads, size, c.window, c.scale)
 
 
 class GatedLinear:
@@ -410,7 +290,7 @@ class GatedLinear:
         ops.linear(stream, delta, attended, self.out)
 
 
-MIXERS = {LatentAttentionConfig: LatentAttention, GatedLinearConfig: GatedLinear}
+MIXERS = {LatentAttentionConfig: LatentAttention, GatedLinearConfig: GatedLinear, ParallelConfig: ParallelMixer}
 
 
 # ------------------------------------------------------------------------------------------------
@@ -420,10 +300,11 @@ MIXERS = {LatentAttentionConfig: LatentAttention, GatedLinearConfig: GatedLinear
 @dataclass
 class _Layer:
     mixer: object
-    norm1: object
-    norm2: object = None
-    up: object = None
+    first: Sublayer
+    second: Sublayer = None
+    up: object = None      # with gated: gate and up together
     down: object = None
+    gated: bool = False
 
 
 class HybridDecoder(PagedDecoder):
@@ -439,24 +320,26 @@ class HybridDecoder(PagedDecoder):
         self.dtype = dtype
         self.ops = ops = Ops(dtype)
         whole = sequences * round_up(capacity, config.page_size)
-        table = PageTable.create_shared(sequences, capacity, config.page_size, cache_tokens or whole, config.window())
+        table = PageTable.create_shared(sequences, capacity, config.page_size, cache_tokens or whole, config.window(),
+                                        config.chunks())
         self._init_step_inputs(table, sequences, capacity, config.page_size)
         take = lambda name: torch.as_tensor(weights[name])
+        self.residual = (StreamResidual if config.streams else LayerNormResidual)(config, take, ops)
         built = {}
         for index, layer in enumerate(config.layers):
             if layer.weights_of is not None:
                 continue
             prefix = f"l{index}."
             mixer = MIXERS[type(layer.mixer)](layer.mixer, lambda name, p=prefix: take(p + "mix." + name), ops, config.eps)
-            built[index] = _Layer(mixer, ops.weight(take(prefix + "norm1")))
+            norms = getattr(mixer, "output_norms", None)
+            built[index] = _Layer(mixer, self.residual.sublayer(take, prefix, 1, norms), gated=layer.gated)
             if layer.ffn:
-                built[index].norm2 = ops.weight(take(prefix + "norm2"))
-                built[index].up = ops.weight(take(prefix + "mlp.up"))
+                built[index].second = self.residual.sublayer(take, prefix, 2)
+                built[index].up = (ops.gate_up_weight(take(prefix + "mlp.gate"), take(prefix + "mlp.up")) if layer.gated
+                                   else ops.weight(take(prefix + "mlp.up")))
                 built[index].down = ops.weight(take(prefix + "mlp.down"))
         self.layers = [built[config.owner(index)] for index in range(len(config.layers))]
         self.caches = [layer.mixer.new_cache(table, sequences) for layer in self.layers]
-        self.embed = torch.as_tensor(weights["embed"]).to("cuda").to(ops.dtype).contiguous()
-        self.embed_norm, self.final_norm = ops.weight(take("embed.norm")), ops.weight(take("final.norm"))
         self.head = ops.weight(take("head"))
         # persistent inputs of the one-token step beyond those every decoder has
         i32, i64 = torch.int32, torch.int64
@@ -473,8 +356,8 @@ class HybridDecoder(PagedDecoder):
                           for layer in built.values()}
         self.decode_rows = StepRows(sequences, self.d_tokens, self.d_pages, self.d_slots, self.d_query_offsets,
                                     self.d_page_offsets, self.d_page_list, self.d_last_lengths, self.d_first,
-                                    self.d_fresh, self.d_context, self.d_table, None, self.d_first, self.d_lens,
-                                    sequences)
+                                    self.d_fresh, self.d_context, self.d_table, self.d_positions, self.d_first,
+                                    self.d_lens, 1, None, self.d_first, self.d_lens, sequences)
         self.sms = torch.cuda.get_device_properties(0).multi_processor_count
         self.trail = None   # set to a list to collect the residual stream after every layer (for inspection)
 
@@ -485,33 +368,39 @@ class HybridDecoder(PagedDecoder):
         self.table.place_prompts([tokens_per_sequence] * self.sequences)
         generator = torch.Generator(device="cuda").manual_seed(seed)
         for cache in self.caches:
-            cache.normal_(generator=generator)
+            for part in cache if isinstance(cache, tuple) else (cache,):
+                part.normal_(generator=generator)
         self._refresh_block_table()
 
     # ---- the layers, over a step of any shape ----
 
     def _layers(self, rows: StepRows, scratches):
         """Runs the layers; returns the final norm's output for the step's rows."""
-        torch, ops, c = self.torch, self.ops, self.config
+        ops, c = self.ops, self.config
         stream = self._stream()
         t = rows.count
-        residual = torch.empty((t, c.width), dtype=torch.float32, device="cuda")
-        normed, delta = ops.rows(t, c.width), ops.rows(t, c.width)
-        ops.call(f"singe_embedding_layer_norm_{ops.suffix}", stream, residual, self.embed, rows.tokens, self.embed_norm, t,
-                 c.width, c.vocab, c.eps, self.status)
-        pending = None   # the sublayer output not yet added to the residual
+        normed = ops.rows(t, c.width)
+        residual, done, delta = None, None, None   # done, delta: the sublayer whose output the residual has not taken in yet
         for layer, cache in zip(self.layers, self.caches):
-            ops.add_layer_norm(stream, residual, pending, normed, layer.norm1, c.eps)
+            if done is None:
+                residual = self.residual.start(stream, rows, layer.first, normed, self.status)
+            else:
+                self.residual.advance(stream, residual, delta, done, layer.first, normed)
+            done = layer.first
+            delta = ops.rows(t, c.width if done.output_norms is None else round_up(c.width, 8) + c.width)
             layer.mixer.run(stream, rows, normed, cache, delta, self.status, scratches.get(id(layer)))
-            pending = delta
-            if layer.up is not None:
-                ops.add_layer_norm(stream, residual, pending, normed, layer.norm2, c.eps)
-                inner = ops.rows(t, layer.up.shape[0])
-                ops.linear(stream, inner, normed, layer.up, activation=2)
+            if layer.second is not None:
+                self.residual.advance(stream, residual, delta, done, layer.second, normed)
+                done, delta = layer.second, ops.rows(t, c.width)
+                inner = ops.rows(t, layer.down.shape[1])
+                if layer.gated:
+                    ops.gated_linear_unit(stream, inner, normed, layer.up)
+                else:
+                    ops.linear(stream, inner, normed, layer.up, activation=2)
                 ops.linear(stream, delta, inner, layer.down)
             if self.trail is not None:
-                self.trail.append(residual + delta.float())
-        ops.add_layer_norm(stream, residual, pending, normed, self.final_norm, c.eps)
+                self.trail.append(self.residual.peek(stream, residual, delta, done))
+        self.residual.finish(stream, residual, delta, done, normed)
         return normed
 
     def forward(self) -> None:
@@ -602,9 +491,20 @@ class HybridDecoder(PagedDecoder):
                 narrow[f"segments{heads}"] = np.stack([long[plan[:, 0]], plan[:, 1], plan[:, 2], plan[:, 3]], 1).reshape(-1)
                 narrow[f"segment_last{heads}"] = plan[:, 4]
                 cut[heads] = bool((plan[:, 4] == 0).any())
+        narrow.update({"sequence_of": step.sequence_ids,
+                       "row_lens": np.where(fresh[step.sequence_ids] > 0, step.positions + 1, 0)})
+        plans = {size: plan_chunks(size, context, fresh, first, long) for size in c.chunks() if len(long)}
+        for size, plan in plans.items():
+            at = np.asarray(plan["moved"], dtype=np.int64).reshape(-1, 2)
+            narrow[f"moved{size}"] = block_table[at[:, 0], at[:, 1] // c.page_size] * c.page_size + at[:, 1] % c.page_size
+            narrow.update({f"{name}{size}": plan[name]
+                           for name in ("packed", "moved_to", "lens_q", "lens_kv", "offsets_q", "offsets_kv")})
+        if c.chunks() and len(long):
+            counts = [len(start) for start in starts]
+            narrow["whole"] = np.stack([long, np.cumsum(counts) - counts, counts], 1).reshape(-1)
         wide = {"tokens": step.tokens, "pages": step.write_pages, "slots": step.write_slots,
                 "query_offsets": step.query_offsets, "page_offsets": step.page_offsets, "page_list": step.pages,
-                "last": step.last_page_lengths, "short_rows": short}
+                "last": step.last_page_lengths, "short_rows": short, "positions": step.positions}
         w, n = self._send(wide, np.int64), self._send(narrow, np.int32)
         expanded = {}
         for window in windows if len(long) else []:
@@ -614,11 +514,21 @@ class HybridDecoder(PagedDecoder):
         blocks = {heads: BlockRows(n["block_rows"], n["block_tokens"], n["block_rows"].numel(), n[f"segments{heads}"],
                                    n[f"segment_last{heads}"], n[f"segment_last{heads}"].numel(), cut[heads])
                   for heads in cut}
+        chunks = {}
+        for size, plan in plans.items():
+            part = lambda name: n[f"{name}{size}"]
+            chunks[size] = ChunkRows(part("packed"), torch.from_numpy(plan["cached"]).cuda(), plan["keys"], part("moved"),
+                                     part("moved_to"), part("lens_q"), part("lens_kv"), part("offsets_q"), part("offsets_kv"),
+                                     len(plan["lens_q"]))
+        whole = None
+        if "whole" in n:
+            whole = BlockRows(n["block_rows"], n["block_tokens"], n["block_rows"].numel(), n["whole"], None, len(long), False)
         everything = len(short) == len(step.tokens)
         return StepRows(len(step.tokens), w["tokens"], w["pages"], w["slots"], w["query_offsets"], w["page_offsets"],
                         w["page_list"], w["last"], n["first"], n["fresh"], n["context"],
-                        n["table"].view(block_table.shape), None if everything else w["short_rows"],
-                        n["short_sequences"], n["short_lens"], len(short), expanded, blocks)
+                        n["table"].view(block_table.shape), w["positions"], n["sequence_of"], n["row_lens"],
+                        int(fresh.max()), None if everything else w["short_rows"], n["short_sequences"], n["short_lens"],
+                        len(short), expanded, blocks, chunks, whole)
 
     def _send(self, arrays: dict, kind) -> dict:
         torch = self.torch

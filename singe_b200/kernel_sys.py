@@ -132,8 +132,26 @@ SIGNATURES = {
                                     _z],
     "singe_latent_decode_bf16": [_p, _p, _p, _p, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z, _z, _z, _z, _f, _p],
     "singe_windowed_prefill_attention_bf16": [_p, _p, _p, _p, _p, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _z,
-                                              _z, _f],
-    "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _z, _p, _z, _z, _z, _z, _f, _f, _f, _p, _p,
+                                              _z, _z, _f],
+    "singe_move_rows": [_p, _p, _p, _p, _p, _z, _z, _z, _z, _p],
+    "singe_stream_embedding_norm_bf16": [_p, _p, _p, _p, _p, _p, _z, _p, _z, _z, _z, _z, _f, _p],
+    "singe_stream_embedding_norm_f32": [_p, _p, _p, _p, _p, _p, _z, _p, _z, _z, _z, _z, _f, _p],
+    "singe_stream_step_norm_bf16": [_p, _p, _p, _z, _i, _z, _p, _p, _f, _p, _p, _p, _i, _p, _z, _p, _f, _z, _z,
+                                    _z, _f],
+    "singe_stream_step_norm_f32": [_p, _p, _p, _z, _i, _z, _p, _p, _f, _p, _p, _p, _i, _p, _z, _p, _f, _z, _z,
+                                    _z, _f],
+    "singe_chunked_attention_bf16": [_p] * 10 + [_z] * 10 + [_f, _p],
+    "singe_chunked_attention_f32": [_p] * 8 + [_z] * 9 + [_f, _p],
+    "singe_conv_attention_inputs_bf16": [_p, _p, _z] + [_p] * 5 + [_z] + [_p] * 6 + [_z, _f] + [_p] * 9 + [_z] * 15 + [_f, _p],
+    "singe_conv_attention_inputs_f32": [_p, _p, _z] + [_p] * 5 + [_z] + [_p] * 6 + [_z, _f] + [_p] * 9 + [_z] * 15 + [_f, _p],
+    "singe_conv_recurrence_inputs_bf16": [_p, _p, _z, _p, _p, _z] + [_p] * 6 + [_z] * 7 + [_f],
+    "singe_conv_recurrence_inputs_f32": [_p, _p, _z, _p, _p, _z] + [_p] * 6 + [_z] * 7 + [_f],
+    "singe_conv_state_bf16": [_p, _p, _z, _p, _p, _p, _z, _z, _z, _z],
+    "singe_conv_state_f32": [_p, _p, _z, _p, _p, _p, _z, _z, _z, _z],
+    "singe_gated_delta_step_bf16": [_p, _p, _z, _p, _z, _p, _p, _z, _p, _z] + [_p] * 7 + [_z] * 9 + [_f, _z],
+    "singe_gated_delta_step_f32": [_p, _p, _z, _p, _z, _p, _p, _z, _p, _z] + [_p] * 7 + [_z] * 9 + [_f, _z],
+    "singe_silu_mul_f32": [_p, _p, _z, _p, _p, _z, _z, _z],
+    "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _f, _f, _f, _p, _p,
                                        _z, _p, _p, _z, _i, _p],
     "singe_gated_linear_prompt_scratch": [_z, _z, _z, _z, _z],
     "singe_latent_decode_splits": [_z, _z, _z, _z],

@@ -33,6 +33,7 @@ class Model:
 MODELS = {
     "LlamaForCausalLM": Model(_llama, ("bfloat16",)),
     "Kavalorn": Model(_hybrid, ("bfloat16", "float32")),
+    "Vatolorn": Model(_hybrid, ("bfloat16", "float32")),
 }
 _BY_TYPE = {"llama": "LlamaForCausalLM"}   # model_type of configurations that name no architecture
 

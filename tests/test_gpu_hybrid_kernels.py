@@ -259,7 +259,7 @@ def test_prompt_attention_at_window_edges(heads, size, window):
     lse = torch.zeros((total_q, heads), dtype=torch.float32, device="cuda")
     ops.call("singe_windowed_prefill_attention_bf16", stream(), out, lse, dev(query).to(torch.bfloat16), d_rows,
              d_rows.data_ptr() + heads * size * 2, 2 * heads * size, i32(fresh), i32(lens_kv), i32(offsets_q),
-             i32(offsets_kv), d_gate.data_ptr() + 4, gate.shape[1], len(fresh), total_q, total_kv, heads, size, window, scale)
+             i32(offsets_kv), d_gate.data_ptr() + 4, gate.shape[1], len(fresh), total_q, total_kv, heads, heads, size, window, scale)
     got = host(out)
     for b, n in enumerate(fresh):
         assert np.abs(got[offsets_q[b]: offsets_q[b] + n] - expect[b]).max() < 3e-2, f"sequence {b}"
@@ -282,7 +282,7 @@ def test_prompt_attention_with_scores_that_leave_the_single_pass_range(window):
     lse = torch.zeros((tokens, heads), dtype=torch.float32, device="cuda")
     ops.call("singe_windowed_prefill_attention_bf16", stream(), out, lse, dev(query).to(torch.bfloat16), d_rows,
              d_rows.data_ptr() + heads * size * 2, 2 * heads * size, i32([tokens]), i32([tokens]), i32([0]), i32([0]), None, 0,
-             1, tokens, tokens, heads, size, window, 1.0)
+             1, tokens, tokens, heads, heads, size, window, 1.0)
     assert np.abs(host(out) - expect).max() < 3e-2
 
 
