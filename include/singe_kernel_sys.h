@@ -790,7 +790,7 @@ int singe_conv_attention_inputs_f32(
     size_t packed_count, size_t rows, size_t sequences, size_t tap_count, size_t heads, size_t kv_heads, size_t dim,
     size_t vdim, size_t key_size, size_t value_size, size_t key_at, size_t value_at, size_t span, size_t pages,
     size_t page_size, float eps, uint32_t *status);
-/* Recurrence: mixed = silu(convolution) for all columns (idle rows are left alone); inverse [rows, 2 * unit_heads] holds
+/* Recurrence: mixed = silu(convolution) for all columns (idle rows become zeros); inverse [rows, 2 * unit_heads] holds
  * 1 / sqrt(sum(x^2) + eps) of the first unit_heads pieces of `dim` columns and of as many from second_at on. */
 int singe_conv_recurrence_inputs_bf16(singe_stream_t stream, void *mixed, size_t mixed_stride, float *inverse,
                                       const void *projected, size_t projected_stride, const void *taps, void *state,
@@ -828,6 +828,19 @@ int singe_gated_delta_step_f32(singe_stream_t stream, void *out, size_t out_stri
                                float *state, const int32_t *first, const int32_t *count, const int32_t *context, size_t rows,
                                size_t sequences, size_t heads, size_t kv_heads, size_t dim, size_t vdim, size_t key_at,
                                size_t value_at, size_t gate_at, float eps, size_t longest);
+
+/* The same over prompts, block by block on the tensor core (two-term bf16 operands for what is f32; the state stays f32).  The
+ * blocks of 16 tokens of all sequences served, in order: block_row / block_tokens [blocks], a sequence's last block may be short;
+ * runs [run_count][3] = {sequence, first block, blocks}.  Rows of `mixed` hold finite values.  scratch:
+ * singe_gated_delta_prompt_scratch bytes, which is 0 for sizes this form does not take (dim <= 256 and vdim in eights). */
+int singe_gated_delta_prompt_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *mixed, size_t mixed_stride,
+                                  const float *inverse, const void *strength, size_t strength_stride, const void *decay,
+                                  size_t decay_stride, const float *rate, const float *bias, const void *norm_weight,
+                                  float *state, const int32_t *context, size_t rows, size_t heads, size_t kv_heads, size_t dim,
+                                  size_t vdim, size_t key_at, size_t value_at, size_t gate_at, float eps,
+                                  const int32_t *block_row, const int32_t *block_tokens, size_t blocks, const int32_t *runs,
+                                  size_t run_count, void *scratch);
+size_t singe_gated_delta_prompt_scratch(size_t heads, size_t dim, size_t vdim, size_t rows, size_t blocks);
 
 /* out = silu(gate) * up, elementwise in f32. */
 int singe_silu_mul_f32(singe_stream_t stream, float *out, size_t output_row_stride, const float *gate, const float *up,

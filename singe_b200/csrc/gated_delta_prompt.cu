@@ -1,0 +1,687 @@
+// Gated delta rule over prompts: the recurrence of gated_delta.cu (same operands, same meaning), block by block on the tensor
+// core.
+//
+// In a block of 16 tokens let a_t be the running sum of log g per key channel (A the last one's) and S the state before the
+// block.  The written rows u_t solve a unit lower-triangular system,
+//     (I + M) u = beta (v - (k exp(a))^T S),     M_tj = beta_t sum_c k_tc k_jc exp(a_tc - a_jc)  for j < t,
+// so that with T = (I + M)^-1 diag(beta) and W = T (k exp(a)),
+//     u   = T v - W S,
+//     o_t = (q_t exp(a_t))^T S + sum_(j <= t) P_tj u_j,     P_tj = sum_c q_tc k_jc exp(a_tc - a_jc),
+//     S'  = exp(A) S + sum_j (k_j exp(A - a_j)) u_j^T.
+// Every exponent that reaches a product is <= 0 except in the factored form of M and P, which is only used where the block's
+// whole decay stays above e^-60.
+//
+// 32-bit without 32-bit tensor cores: operands that are f32 by nature enter the bf16 MMA as two terms hi + lo (2^-17 of the
+// value is lost) and their products keep hi hi + hi lo + lo hi; v is bf16 from its convolution and enters as it is.
+// Accumulators, and the state between the blocks, are f32.
+//
+//   prepare   one warp per (block, head): decays, M and its inverse, P and the split operands, to scratch, laid out as the next
+//             kernel's shared memory wants them, so that a block arrives in one bulk copy
+//   advance   one CTA per (sequence, head, slice of the values): the blocks in order, the state in registers as S^T [vdim, dim],
+//             whose accumulator layout is the A-operand layout of the next product.  A warp owns 16 value rows.  The columns of
+//             the state do not meet, so slices run side by side.
+//   finish    RMS norm over a head's values, gate, store
+#include "row_pack.cuh"
+#include "split_bf16.cuh"
+
+namespace singe {
+namespace {
+
+constexpr int kPrepareWarps = 2;
+constexpr int kMaxStages = 6;
+constexpr float kFactoredLimit = -60.0f;
+constexpr int kPitchP = kBlock * 2 + 16;  // bytes of a padded row of P or T
+
+// The operands of one (block, head), bytes: q exp(a) hi, lo; W hi, lo; k exp(A - a) hi, lo; P hi, lo; T hi, lo; exp(A).
+struct DeltaLayout {
+    int pitch;  // bytes of a padded row of q, W or k
+    int w, k, p, t, decay, bytes;
+};
+
+__host__ __device__ constexpr DeltaLayout delta_layout(int dim_pad) {
+    DeltaLayout l = {};
+    l.pitch = dim_pad * 2 + 16;
+    l.w = 2 * kBlock * l.pitch;
+    l.k = 2 * l.w;
+    l.p = 3 * l.w;
+    l.t = l.p + 2 * kBlock * kPitchP;
+    l.decay = l.t + 2 * kBlock * kPitchP;
+    l.bytes = l.decay + dim_pad * 4;
+    return l;
+}
+
+struct DeltaParams {
+    int heads, kv_heads, dim, vdim, key_at, value_at, gate_at;
+    int dim_pad, slice;       // slice: value columns of an advance CTA, 16 per warp
+    __nv_bfloat16 *out;
+    long long out_stride;
+    const __nv_bfloat16 *mixed;
+    long long mixed_stride;
+    const float *inverse;
+    const __nv_bfloat16 *strength;
+    long long strength_stride;
+    const __nv_bfloat16 *decay;
+    long long decay_stride;
+    const float *rate, *bias;
+    const __nv_bfloat16 *norm_weight;
+    float *state;
+    const int32_t *context;
+    const int32_t *block_row, *block_tokens;  // first packed row and tokens of each block
+    const int32_t *runs;                      // [n][3]: sequence, first block, blocks
+    int blocks;
+    uint8_t *operands;                        // [blocks, heads] packs
+    float *attended;                          // [rows, heads * vdim]: o before its norm
+    float eps;
+    uint32_t *error;
+    int stages;
+};
+
+// Shared memory of one warp of the prepare kernel: (q exp(a)), (k exp(-a)) and (k exp(a)), each hi and lo, and a 16 x 17 matrix.
+__host__ __device__ constexpr int prepare_bytes(int dim_pad) { return 6 * kBlock * (dim_pad * 2 + 16) + kBlock * 17 * 4 + 64; }
+
+// acc (two n tiles of 8) += A[16, 16 rows at a] . B[16 rows at b, same columns]^T over `columns`, split operands.
+__device__ __forceinline__ void product_rows(float (&acc)[2][4], uint32_t a_at, uint32_t b_at, int pitch, int columns) {
+    for (int k0 = 0; k0 < columns; k0 += 16) {
+        uint32_t a[2][4], b[2][4];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const uint32_t offset = half * kBlock * pitch + k0 * 2;
+            ldmatrix_x4(a_at + offset, a[half][0], a[half][1], a[half][2], a[half][3]);
+            ldmatrix_x4(b_at + offset, b[half][0], b[half][1], b[half][2], b[half][3]);
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[0][2 * n], b[0][2 * n + 1]);
+            mma_m16n8k16<__nv_bfloat16>(acc[n], a[0][0], a[0][1], a[0][2], a[0][3], b[1][2 * n], b[1][2 * n + 1]);
+            mma_m16n8k16<__nv_bfloat16>(acc[n], a[1][0], a[1][1], a[1][2], a[1][3], b[0][2 * n], b[0][2 * n + 1]);
+        }
+    }
+}
+
+__device__ __forceinline__ float low_half(uint32_t pair) { return __uint_as_float(pair << 16); }
+__device__ __forceinline__ float high_half(uint32_t pair) { return __uint_as_float(pair & 0xffff0000u); }
+
+__global__ void __launch_bounds__(kPrepareWarps * 32) gated_delta_prepare_kernel(const DeltaParams p) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int block = blockIdx.x;
+    const int row0 = p.block_row[block], tokens = p.block_tokens[block];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y * kPrepareWarps + warp;
+    if (head >= p.heads) return;  // warps work alone
+    const DeltaLayout layout = delta_layout(p.dim_pad);
+    extern __shared__ __align__(16) uint8_t prepare_shared[];
+    uint8_t *own = prepare_shared + warp * prepare_bytes(p.dim_pad);
+    const int half_bytes = kBlock * layout.pitch;  // from the hi to the lo part
+    uint8_t *fq = own, *fk = own + 2 * half_bytes, *fa = own + 4 * half_bytes;
+    float *matrix = reinterpret_cast<float *>(own + 6 * half_bytes);  // [16][17]
+    float *betas = matrix + kBlock * 17;                              // [16]
+    const int source = head / (p.heads / p.kv_heads);
+    uint8_t *pack = p.operands + (static_cast<size_t>(block) * p.heads + head) * layout.bytes;
+    float *whole_decay = reinterpret_cast<float *>(pack + layout.decay);
+    const float rate = expf(p.rate[head]);
+    const float query_scale = 1.0f / sqrtf(static_cast<float>(p.dim));
+
+    // a lane's own token: unit lengths and write strength
+    float unit_q = 0.0f, unit_k = 0.0f;
+    if (lane < kBlock) {
+        float beta = 0.0f;
+        if (lane < tokens) {
+            const long long row = row0 + lane;
+            unit_q = p.inverse[row * 2 * p.kv_heads + source] * query_scale;
+            unit_k = p.inverse[row * 2 * p.kv_heads + p.kv_heads + source];
+            beta = 1.0f / (1.0f + expf(-__bfloat162float(p.strength[row * p.strength_stride + head])));
+        }
+        betas[lane] = beta;
+    }
+    // log decay of token t in channel c, and its running sum
+    auto running_decay = [&](int c, float (&sum)[2][kBlock]) {
+        const bool real = c < p.dim;
+        const int channel = head * p.dim + (real ? c : 0);
+        const float2 bias = real ? make_float2(p.bias[channel], p.bias[channel + 1]) : make_float2(0.0f, 0.0f);
+        uint32_t z[kBlock];
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            z[t] = real && t < tokens ? *reinterpret_cast<const uint32_t *>(p.decay + (row0 + t) * p.decay_stride + channel) : 0u;
+        }
+        float total[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            if (real && t < tokens) {
+                const float x = low_half(z[t]) + bias.x, y = high_half(z[t]) + bias.y;
+                total[0] -= rate * (fmaxf(x, 0.0f) + log1pf(__expf(-fabsf(x))));
+                total[1] -= rate * (fmaxf(y, 0.0f) + log1pf(__expf(-fabsf(y))));
+            }
+            sum[0][t] = total[0];
+            sum[1][t] = total[1];
+        }
+    };
+
+    bool strong = false;
+    for (int c = 2 * lane; c < p.dim_pad + 2 * lane; c += 64) {  // a lane takes two adjacent channels
+        const bool inside = c < p.dim_pad;                        // (every lane takes part in the shuffles)
+        const bool real = c < p.dim;                              // dim is a multiple of eight
+        float a[2][kBlock];
+        running_decay(inside ? c : p.dim_pad, a);
+        const float total[2] = {a[0][kBlock - 1], a[1][kBlock - 1]};
+        const bool factors = fminf(total[0], total[1]) >= kFactoredLimit;
+        strong = strong || !factors;
+        const float whole[2] = {__expf(total[0]), __expf(total[1])};
+        if (inside) *reinterpret_cast<float2 *>(whole_decay + c) = make_float2(whole[0], whole[1]);
+        const __nv_bfloat16 *rows = p.mixed + row0 * p.mixed_stride + source * p.dim + (real ? c : 0);
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            const bool live = real && t < tokens;
+            const uint32_t q_raw = live ? *reinterpret_cast<const uint32_t *>(rows + t * p.mixed_stride) : 0u;
+            const uint32_t k_raw = live ? *reinterpret_cast<const uint32_t *>(rows + t * p.mixed_stride + p.key_at) : 0u;
+            const float uq = __shfl_sync(0xffffffffu, unit_q, t), uk = __shfl_sync(0xffffffffu, unit_k, t);
+            float before[2], after[2], back[2];  // exp(a_t), exp(A - a_t), exp(-a_t)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                before[i] = __expf(a[i][t]);
+                if (factors) {
+                    back[i] = __expf(-a[i][t]);
+                    after[i] = whole[i] * back[i];
+                } else {
+                    back[i] = 0.0f;
+                    after[i] = __expf(total[i] - a[i][t]);
+                }
+            }
+            if (!inside) continue;
+            const float q0 = low_half(q_raw) * uq, q1 = high_half(q_raw) * uq;
+            const float k0 = low_half(k_raw) * uk, k1 = high_half(k_raw) * uk;
+            const int at = t * layout.pitch + c * 2;
+            uint32_t hi, lo;
+            split_pair(q0 * before[0], q1 * before[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(pack + at) = hi;
+            *reinterpret_cast<uint32_t *>(pack + half_bytes + at) = lo;
+            *reinterpret_cast<uint32_t *>(fq + at) = hi;
+            *reinterpret_cast<uint32_t *>(fq + half_bytes + at) = lo;
+            split_pair(k0 * after[0], k1 * after[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(pack + layout.k + at) = hi;
+            *reinterpret_cast<uint32_t *>(pack + layout.k + half_bytes + at) = lo;
+            split_pair(k0 * back[0], k1 * back[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(fk + at) = hi;
+            *reinterpret_cast<uint32_t *>(fk + half_bytes + at) = lo;
+            split_pair(k0 * before[0], k1 * before[1], hi, lo);
+            *reinterpret_cast<uint32_t *>(fa + at) = hi;
+            *reinterpret_cast<uint32_t *>(fa + half_bytes + at) = lo;
+        }
+    }
+    __syncwarp();
+    // ---- P, and M (not yet times beta) ----
+    uint8_t *p_hi = pack + layout.p, *p_lo = p_hi + kBlock * kPitchP;
+    uint8_t *t_hi = pack + layout.t, *t_lo = t_hi + kBlock * kPitchP;
+    const int a_offset = (lane & 15) * layout.pitch + (lane >> 4) * 16;
+    const int b_offset = ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch + ((lane >> 3) & 1) * 16;
+    if (!__any_sync(0xffffffffu, strong)) {
+        float scores[2][4] = {}, keys[2][4] = {};
+        product_rows(scores, smem_u32(fq) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
+        product_rows(keys, smem_u32(fa) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int t = (lane >> 2) + half * 8, j = n * 8 + (lane & 3) * 2;
+                uint32_t hi, lo;
+                split_pair(j <= t ? scores[n][2 * half] : 0.0f, j + 1 <= t ? scores[n][2 * half + 1] : 0.0f, hi, lo);
+                *reinterpret_cast<uint32_t *>(p_hi + t * kPitchP + j * 2) = hi;
+                *reinterpret_cast<uint32_t *>(p_lo + t * kPitchP + j * 2) = lo;
+                matrix[t * 17 + j] = j < t ? keys[n][2 * half] : 0.0f;
+                matrix[t * 17 + j + 1] = j + 1 < t ? keys[n][2 * half + 1] : 0.0f;
+            }
+        }
+    } else {
+        // Decays too strong to factor: every pair's decay is taken as one exponential.  The running sums go where k exp(-a)
+        // was; the lanes are the channels.
+        float *sums = reinterpret_cast<float *>(fk);  // [16][dim_pad]
+        for (int c = 2 * lane; c < p.dim_pad; c += 64) {
+            float a[2][kBlock];
+            running_decay(c, a);
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) *reinterpret_cast<float2 *>(sums + t * p.dim_pad + c) = make_float2(a[0][t], a[1][t]);
+        }
+        __syncwarp();
+        const __nv_bfloat16 *queries = p.mixed + row0 * p.mixed_stride + source * p.dim, *keys = queries + p.key_at;
+        for (int t = 0; t < kBlock; ++t) {
+            const float uq = __shfl_sync(0xffffffffu, unit_q, t), kt = __shfl_sync(0xffffffffu, unit_k, t);
+            for (int j = 0; j <= t; ++j) {
+                const float kj = __shfl_sync(0xffffffffu, unit_k, j);
+                float score = 0.0f, dot = 0.0f;
+                if (t < tokens) {
+                    for (int c = lane; c < p.dim; c += 32) {
+                        const float carried = __bfloat162float(keys[j * p.mixed_stride + c]) * kj *
+                                              __expf(sums[t * p.dim_pad + c] - sums[j * p.dim_pad + c]);
+                        score = fmaf(__bfloat162float(queries[t * p.mixed_stride + c]) * uq, carried, score);
+                        dot = fmaf(__bfloat162float(keys[t * p.mixed_stride + c]) * kt, carried, dot);
+                    }
+                }
+                score = warp_sum(score);
+                dot = warp_sum(dot);
+                if (lane == 0) {
+                    __nv_bfloat16 hi, lo;
+                    split_bf16(score, hi, lo);
+                    *reinterpret_cast<__nv_bfloat16 *>(p_hi + t * kPitchP + j * 2) = hi;
+                    *reinterpret_cast<__nv_bfloat16 *>(p_lo + t * kPitchP + j * 2) = lo;
+                    matrix[t * 17 + j] = j < t ? dot : 0.0f;
+                }
+            }
+            for (int j = t + 1 + lane; j < kBlock; j += 32) {
+                *reinterpret_cast<uint16_t *>(p_hi + t * kPitchP + j * 2) = 0;
+                *reinterpret_cast<uint16_t *>(p_lo + t * kPitchP + j * 2) = 0;
+                matrix[t * 17 + j] = 0.0f;
+            }
+        }
+    }
+    __syncwarp();
+    // ---- T = (I + diag(beta) M)^-1 diag(beta): a lane solves for one column ----
+    {
+        float x[kBlock];
+        const int j = lane & 15;
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            float sum = 0.0f;
+#pragma unroll
+            for (int i = 0; i < t; ++i) sum = fmaf(matrix[t * 17 + i], x[i], sum);
+            x[t] = (t == j ? 1.0f : 0.0f) - betas[t] * sum;
+        }
+        __syncwarp();
+        const float beta = betas[j];
+        if (lane < kBlock) {
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) {
+                const float value = x[t] * beta;
+                matrix[t * 17 + j] = value;
+                __nv_bfloat16 hi, lo;
+                split_bf16(value, hi, lo);
+                *reinterpret_cast<__nv_bfloat16 *>(t_hi + t * kPitchP + j * 2) = hi;
+                *reinterpret_cast<__nv_bfloat16 *>(t_lo + t * kPitchP + j * 2) = lo;
+            }
+        }
+    }
+    __syncwarp();
+    // ---- W = T (k exp(a)) ----
+    uint32_t sh[4], sl[4];  // T as A operand
+    {
+        const int t = lane >> 2, j = (lane & 3) * 2;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float *cell = matrix + (t + (i & 1) * 8) * 17 + j + (i >> 1) * 8;
+            split_pair(cell[0], cell[1], sh[i], sl[i]);
+        }
+    }
+    const uint32_t w_at = smem_u32(fa) + (lane & 15) * layout.pitch + (lane >> 4) * 16;
+    for (int c0 = 0; c0 < p.dim_pad; c0 += 16) {
+        uint32_t hi[4], lo[4];
+        ldmatrix_x4_trans(w_at + c0 * 2, hi[0], hi[1], hi[2], hi[3]);
+        ldmatrix_x4_trans(w_at + half_bytes + c0 * 2, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            float acc[4] = {};
+            mma_m16n8k16<__nv_bfloat16>(acc, sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
+            mma_m16n8k16<__nv_bfloat16>(acc, sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+            mma_m16n8k16<__nv_bfloat16>(acc, sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int at = ((lane >> 2) + half * 8) * layout.pitch + (c0 + n * 8 + (lane & 3) * 2) * 2;
+                uint32_t x, y;
+                split_pair(acc[2 * half], acc[2 * half + 1], x, y);
+                *reinterpret_cast<uint32_t *>(pack + layout.w + at) = x;
+                *reinterpret_cast<uint32_t *>(pack + layout.w + half_bytes + at) = y;
+            }
+        }
+    }
+}
+
+// Stage of the advance kernel (bytes): the operands as prepared, then the slice's values in TMA boxes.
+__host__ __device__ inline int delta_values_at(int dim_pad) { return (delta_layout(dim_pad).bytes + 1023) / 1024 * 1024; }
+__host__ __device__ inline int delta_stage_bytes(int dim_pad, int slice) {
+    return delta_values_at(dim_pad) + (slice + 63) / 64 * kValueBox;
+}
+
+// KT = dim_pad / 16.  A warp owns 16 value rows of the slice.
+template <int KT>
+__global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kernel(const __grid_constant__ CUtensorMap value_map,
+                                                                                  const DeltaParams p) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    constexpr int kDim = KT * 16;
+    constexpr DeltaLayout kLayout = delta_layout(kDim);
+    constexpr int kHalf = kBlock * kLayout.pitch;
+    const int run = blockIdx.x, head = blockIdx.y, slice0 = blockIdx.z * p.slice;
+    const int sequence = p.runs[3 * run], first_block = p.runs[3 * run + 1], blocks = p.runs[3 * run + 2];
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int g = lane >> 2, q2 = (lane & 3) * 2;
+    const int stages = p.stages;
+    const int stage_bytes = delta_stage_bytes(kDim, p.slice), values_at = delta_values_at(kDim);
+    extern __shared__ uint8_t advance_raw[];
+    uint8_t *advance_shared = advance_raw + ((1024u - (smem_u32(advance_raw) & 1023u)) & 1023u);
+    const int pitch_o = p.slice + 4;  // floats of a padded row of the outputs on their way to memory
+    float *outputs = reinterpret_cast<float *>(advance_shared + stages * stage_bytes);  // [16][pitch_o]
+    const uint32_t bars = smem_u32(outputs + kBlock * pitch_o);
+    if (tid == 0) {
+        for (int i = 0; i < stages; ++i) mbar_init(bars + 8 * i, 1);
+        mbar_init_fence();
+    }
+    __syncthreads();
+
+    const int value0 = warp * 16;  // within the slice
+    float state[2 * KT][4];        // S^T: rows v, columns k
+    float *home = p.state + (static_cast<size_t>(sequence) * p.heads + head) * p.dim * p.vdim;
+    const bool fresh = p.context[sequence] == 0;
+#pragma unroll
+    for (int n = 0; n < 2 * KT; ++n) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int v = slice0 + value0 + g + (i >> 1) * 8, k = n * 8 + q2 + (i & 1);
+            state[n][i] = !fresh && v < p.vdim && k < p.dim ? home[static_cast<size_t>(k) * p.vdim + v] : 0.0f;
+        }
+    }
+
+    // One warp brings a block in.  What a box holds past a short block or past the head's columns belongs to other rows or
+    // columns (finite values): it meets zeros in T, or is never stored.
+    const int boxes = (p.slice + 63) / 64;
+    auto load_block = [&](int index) {
+        if (warp != 0) return;
+        const int block = first_block + index;
+        const uint32_t bar = bars + 8 * (index % stages);
+        const uint32_t stage = smem_u32(advance_shared) + (index % stages) * stage_bytes;
+        if (lane == 0) {
+            mbar_expect_tx(bar, kLayout.bytes + boxes * kValueBox);
+            bulk_load(stage, p.operands + (static_cast<size_t>(block) * p.heads + head) * kLayout.bytes, kLayout.bytes, bar);
+        }
+        __syncwarp();
+        if (lane < boxes) {
+            tma_load_2d(stage + values_at + lane * kValueBox, &value_map, bar,
+                        p.value_at + head * p.vdim + slice0 + lane * 64, p.block_row[block]);
+        }
+    };
+    for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
+    bool failed = false;
+    const int width = min(p.slice, p.vdim - slice0);  // real columns of the slice, a multiple of eight
+
+    for (int index = 0; index < blocks; ++index) {
+        const int row0 = p.block_row[first_block + index], tokens = p.block_tokens[first_block + index];
+        const bool arrived = mbar_wait(bars + 8 * (index % stages), (index / stages) & 1);
+        fence_proxy_async_shared();
+        // the block has arrived for every thread, everyone is done with the stage loaded next, and with the outputs before
+        if (__syncthreads_or(arrived ? 0 : 1) != 0) {
+            failed = true;
+            break;
+        }
+        if (index + stages - 1 < blocks) load_block(index + stages - 1);
+        uint8_t *here = advance_shared + (index % stages) * stage_bytes;
+        const uint32_t stage = smem_u32(here);
+        const int t = (lane & 7) + ((lane >> 4) << 3);
+
+        uint32_t value[4];  // v^T of this warp: rows v, columns tokens
+        ldmatrix_x4_trans(stage + values_at + value_at(t, value0 + ((lane >> 3) & 1) * 8), value[0], value[1], value[2], value[3]);
+        // ---- S^T W^T and S^T (q exp(a))^T; the small terms are dependency chains of their own ----
+        float o[2][4] = {}, o_low[2][4] = {}, u[2][4] = {}, u_low[2][4] = {};
+#pragma unroll
+        for (int kt = 0; kt < KT; ++kt) {
+            const uint32_t at = stage + t * kLayout.pitch + (kt * 16 + ((lane >> 3) & 1) * 8) * 2;
+            uint32_t sh[4], sl[4], hi[4], lo[4];
+            split_pair(state[2 * kt][0], state[2 * kt][1], sh[0], sl[0]);
+            split_pair(state[2 * kt][2], state[2 * kt][3], sh[1], sl[1]);
+            split_pair(state[2 * kt + 1][0], state[2 * kt + 1][1], sh[2], sl[2]);
+            split_pair(state[2 * kt + 1][2], state[2 * kt + 1][3], sh[3], sl[3]);
+            ldmatrix_x4(at + kLayout.w, hi[0], hi[1], hi[2], hi[3]);
+            ldmatrix_x4(at + kLayout.w + kHalf, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma_m16n8k16<__nv_bfloat16>(u[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(u_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(u_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+            }
+            ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
+            ldmatrix_x4(at + kHalf, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma_m16n8k16<__nv_bfloat16>(o[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+            }
+        }
+        // ---- u^T = v^T T^T - S^T W^T ----
+        uint32_t uh[4], ul[4];
+        {
+            const uint32_t at = stage + kLayout.t + t * kPitchP + ((lane >> 3) & 1) * 16;
+            uint32_t hi[4], lo[4];
+            ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
+            ldmatrix_x4(at + kBlock * kPitchP, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                float direct[4] = {};
+                mma_m16n8k16<__nv_bfloat16>(direct, value[0], value[1], value[2], value[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(direct, value[0], value[1], value[2], value[3], lo[2 * n], lo[2 * n + 1]);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) u[n][i] = direct[i] - (u[n][i] + u_low[n][i]);
+                split_pair(u[n][0], u[n][1], uh[2 * n], ul[2 * n]);
+                split_pair(u[n][2], u[n][3], uh[2 * n + 1], ul[2 * n + 1]);
+            }
+        }
+        // ---- S^T = S^T exp(A) + u^T (k exp(A - a)) ----
+#pragma unroll
+        for (int kt = 0; kt < KT; ++kt) {
+            const uint32_t at = stage + kLayout.k + (lane & 15) * kLayout.pitch + (kt * 16 + (lane >> 4) * 8) * 2;
+            uint32_t hi[4], lo[4];
+            ldmatrix_x4_trans(at, hi[0], hi[1], hi[2], hi[3]);
+            ldmatrix_x4_trans(at + kHalf, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const float2 d = *reinterpret_cast<const float2 *>(here + kLayout.decay + (kt * 16 + n * 8 + q2) * 4);
+                float(&x)[4] = state[2 * kt + n];
+                x[0] *= d.x;
+                x[1] *= d.y;
+                x[2] *= d.x;
+                x[3] *= d.y;
+                mma_m16n8k16<__nv_bfloat16>(x, uh[0], uh[1], uh[2], uh[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(x, uh[0], uh[1], uh[2], uh[3], lo[2 * n], lo[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(x, ul[0], ul[1], ul[2], ul[3], hi[2 * n], hi[2 * n + 1]);
+            }
+        }
+        // ---- o^T += u^T P^T, out through shared memory ----
+        {
+            const uint32_t at = stage + kLayout.p + t * kPitchP + ((lane >> 3) & 1) * 16;
+            uint32_t hi[4], lo[4];
+            ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
+            ldmatrix_x4(at + kBlock * kPitchP, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma_m16n8k16<__nv_bfloat16>(o[n], uh[0], uh[1], uh[2], uh[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o_low[n], uh[0], uh[1], uh[2], uh[3], lo[2 * n], lo[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o_low[n], ul[0], ul[1], ul[2], ul[3], hi[2 * n], hi[2 * n + 1]);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    outputs[(n * 8 + q2 + (i & 1)) * pitch_o + value0 + g + (i >> 1) * 8] = o[n][i] + o_low[n][i];
+                }
+            }
+        }
+        __syncthreads();
+        const int pieces = width / 4;
+        for (int i = tid; i < tokens * pieces; i += blockDim.x) {
+            const int token = i / pieces, piece = i - token * pieces;
+            *reinterpret_cast<float4 *>(p.attended + static_cast<size_t>(row0 + token) * p.heads * p.vdim + head * p.vdim + slice0 +
+                                        piece * 4) = *reinterpret_cast<const float4 *>(outputs + token * pitch_o + piece * 4);
+        }
+    }
+    if (failed) {
+        if (tid == 0) report_status(p.error, kStatusWaitTimeout);
+        linger_after_timeout();
+        return;
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * KT; ++n) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int v = slice0 + value0 + g + (i >> 1) * 8, k = n * 8 + q2 + (i & 1);
+            if (v < p.vdim && k < p.dim) home[static_cast<size_t>(k) * p.vdim + v] = state[n][i];
+        }
+    }
+}
+
+// One warp per (token, head): out = rms_norm(o) * weight * sigmoid(gate).
+__global__ void __launch_bounds__(256) gated_delta_finish_kernel(const DeltaParams p) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int block = blockIdx.x;
+    const int row0 = p.block_row[block], tokens = p.block_tokens[block];
+    const int lane = threadIdx.x & 31, packs = p.vdim / 4;
+    for (int item = blockIdx.y * 8 + (threadIdx.x >> 5); item < tokens * p.heads; item += gridDim.y * 8) {
+        const int token = item / p.heads, head = item - token * p.heads;
+        const size_t row = row0 + token;
+        const float *o = p.attended + row * p.heads * p.vdim + head * p.vdim;
+        float square = 0.0f;
+        for (int i = lane; i < packs; i += 32) {
+            const Pack<4> x = load_pack<4>(o + i * 4);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) square = square_chain(square, x.v[j]);
+        }
+        const float scale = 1.0f / sqrtf(warp_sum(square) / static_cast<float>(p.vdim) + p.eps);
+        const __nv_bfloat16 *gates = p.decay + row * p.decay_stride + p.gate_at + head * p.vdim;
+        __nv_bfloat16 *out = p.out + row * p.out_stride + head * p.vdim;
+        for (int i = lane; i < packs; i += 32) {
+            Pack<4> x = load_pack<4>(o + i * 4);
+            const Pack<4> gate = load_pack<4>(gates + i * 4), weight = load_pack<4>(p.norm_weight + i * 4);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) x.v[j] = x.v[j] * scale * weight.v[j] * __fdividef(1.0f, 1.0f + __expf(-gate.v[j]));
+            store_pack<4>(out + i * 4, x);
+        }
+    }
+}
+
+template <int KT>
+int launch_advance(cudaStream_t stream, const CUtensorMap &value_map, DeltaParams p, size_t runs) {
+    const auto bytes_of = [&](int stages) {
+        return stages * delta_stage_bytes(KT * 16, p.slice) + kBlock * (p.slice + 4) * 4 + kMaxStages * 8 + 1024;
+    };
+    p.stages = kMaxStages;  // as many as leave room for a second CTA, three at least
+    while (p.stages > 3 && bytes_of(p.stages) > 112 * 1024) --p.stages;
+    if (bytes_of(p.stages) > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    static int configured[kMaxDevices] = {0};
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_advance_kernel<KT>, bytes_of(p.stages), configured));
+    const dim3 grid(static_cast<unsigned>(runs), static_cast<unsigned>(p.heads),
+                    static_cast<unsigned>((p.vdim + p.slice - 1) / p.slice));
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_advance_kernel<KT>, grid, dim3(p.slice * 2), bytes_of(p.stages), stream, kLaunchGlue,
+                                    1, value_map, p));
+    return launch_status();
+}
+
+// The padded key size, or 0 for sizes the block form does not take.
+int delta_dim_pad(size_t dim, size_t vdim) {
+    if (dim == 0 || vdim == 0 || dim > 256 || dim % 8 != 0 || vdim % 8 != 0) return 0;
+    int pad = 16;
+    while (static_cast<size_t>(pad) < dim) pad *= 2;
+    return pad;
+}
+
+// Value columns of a CTA: all of a head's up to 128, fewer while (run, head, slice) triples leave SMs idle.
+int delta_slice(size_t runs, size_t heads, size_t vdim) {
+    int slice = 16;
+    while (slice < 128 && static_cast<size_t>(slice) < vdim) slice *= 2;
+    while (slice > 16 && runs * heads * ((vdim + slice - 1) / slice) < static_cast<size_t>(device_sm_count())) slice /= 2;
+    return slice;
+}
+
+}  // namespace
+}  // namespace singe
+
+using namespace singe;
+
+extern "C" {
+
+size_t singe_gated_delta_prompt_scratch(size_t heads, size_t dim, size_t vdim, size_t rows, size_t blocks) {
+    const int dim_pad = delta_dim_pad(dim, vdim);
+    if (dim_pad == 0) return 0;
+    return align256(blocks * heads * delta_layout(dim_pad).bytes) + align256(rows * heads * vdim * sizeof(float));
+}
+
+int singe_gated_delta_prompt_bf16(singe_stream_t stream, void *out, size_t out_stride, const void *mixed, size_t mixed_stride,
+                                  const float *inverse, const void *strength, size_t strength_stride, const void *decay,
+                                  size_t decay_stride, const float *rate, const float *bias, const void *norm_weight, float *state,
+                                  const int32_t *context, size_t rows, size_t heads, size_t kv_heads, size_t dim, size_t vdim,
+                                  size_t key_at, size_t value_at, size_t gate_at, float eps, const int32_t *block_row,
+                                  const int32_t *block_tokens, size_t blocks, const int32_t *runs, size_t run_count, void *scratch) {
+    if (rows == 0 || heads == 0 || kv_heads == 0 || heads % kv_heads != 0 || blocks == 0 || run_count == 0 ||
+        key_at < kv_heads * dim || value_at < key_at + kv_heads * dim || mixed_stride < value_at + heads * vdim ||
+        gate_at < heads * dim || decay_stride < gate_at + heads * vdim || strength_stride < heads || out_stride < heads * vdim) {
+        return SINGE_ERR_INVALID_LENGTH;
+    }
+    if (!fits_i32(rows) || !fits_i32(blocks) || !fits_i32(run_count) || !fits_i32(mixed_stride) || !fits_i32(decay_stride) ||
+        heads > 65535) {
+        return SINGE_ERR_LENGTH_EXCEEDS_I32;
+    }
+    if (out == nullptr || mixed == nullptr || inverse == nullptr || strength == nullptr || decay == nullptr || rate == nullptr ||
+        bias == nullptr || norm_weight == nullptr || state == nullptr || context == nullptr || block_row == nullptr ||
+        block_tokens == nullptr || runs == nullptr || scratch == nullptr) {
+        return SINGE_ERR_NULL_POINTER;
+    }
+    const int dim_pad = delta_dim_pad(dim, vdim);
+    if (dim_pad == 0 || mixed_stride % 8 != 0 || decay_stride % 8 != 0 || out_stride % 8 != 0 || key_at % 8 != 0 ||
+        value_at % 8 != 0 || gate_at % 8 != 0 || !aligned_to(mixed, 16) || !aligned_to(decay, 16) || !aligned_to(out, 16) ||
+        !aligned_to(norm_weight, 8) || !aligned_to(bias, 8) || !aligned_to(scratch, 16)) {
+        return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    }
+    DeltaParams p = {};
+    p.heads = static_cast<int>(heads);
+    p.kv_heads = static_cast<int>(kv_heads);
+    p.dim = static_cast<int>(dim);
+    p.vdim = static_cast<int>(vdim);
+    p.key_at = static_cast<int>(key_at);
+    p.value_at = static_cast<int>(value_at);
+    p.gate_at = static_cast<int>(gate_at);
+    p.dim_pad = dim_pad;
+    p.slice = delta_slice(run_count, heads, vdim);
+    p.out = static_cast<__nv_bfloat16 *>(out);
+    p.out_stride = static_cast<long long>(out_stride);
+    p.mixed = static_cast<const __nv_bfloat16 *>(mixed);
+    p.mixed_stride = static_cast<long long>(mixed_stride);
+    p.inverse = inverse;
+    p.strength = static_cast<const __nv_bfloat16 *>(strength);
+    p.strength_stride = static_cast<long long>(strength_stride);
+    p.decay = static_cast<const __nv_bfloat16 *>(decay);
+    p.decay_stride = static_cast<long long>(decay_stride);
+    p.rate = rate;
+    p.bias = bias;
+    p.norm_weight = static_cast<const __nv_bfloat16 *>(norm_weight);
+    p.state = state;
+    p.context = context;
+    p.block_row = block_row;
+    p.block_tokens = block_tokens;
+    p.runs = runs;
+    p.blocks = static_cast<int>(blocks);
+    p.operands = static_cast<uint8_t *>(scratch);
+    p.attended = reinterpret_cast<float *>(p.operands + align256(blocks * heads * delta_layout(dim_pad).bytes));
+    p.eps = eps;
+    p.error = device_error_word();
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const int shared = kPrepareWarps * prepare_bytes(dim_pad);
+    static int configured[kMaxDevices] = {0};
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_prepare_kernel, shared, configured));
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_prepare_kernel,
+                                    dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((heads + kPrepareWarps - 1) / kPrepareWarps)),
+                                    dim3(kPrepareWarps * 32), shared, s, kLaunchGlue, 1, p));
+    CUtensorMap value_map;
+    {
+        const uint64_t dims[2] = {value_at + heads * vdim, rows};
+        const uint64_t strides[1] = {mixed_stride * 2};
+        const uint32_t box[2] = {64, kBlock};
+        SINGE_TRY(encode_tensor_map(&value_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, mixed, dims, strides, box,
+                                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
+    }
+    int launched = SINGE_ERR_UNSUPPORTED_CONFIGURATION;
+    if (dim_pad == 16) launched = launch_advance<1>(s, value_map, p, run_count);
+    if (dim_pad == 32) launched = launch_advance<2>(s, value_map, p, run_count);
+    if (dim_pad == 64) launched = launch_advance<4>(s, value_map, p, run_count);
+    if (dim_pad == 128) launched = launch_advance<8>(s, value_map, p, run_count);
+    if (dim_pad == 256) launched = launch_advance<16>(s, value_map, p, run_count);
+    SINGE_TRY(launched);
+    const size_t items = kBlock * heads;
+    const unsigned groups = static_cast<unsigned>(items > 256 ? (items + 255) / 256 : 1);  // 32 (token, head) pairs a warp
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_finish_kernel, dim3(static_cast<unsigned>(blocks), groups), dim3(256), 0, s,
+                                    kLaunchGlue, 1, p));
+    return launch_status();
+}
+
+}  // extern "C"

@@ -207,7 +207,14 @@ __global__ void __launch_bounds__(kConvThreads) recurrence_inputs_kernel(const R
     float *inverse = p.inverse + static_cast<size_t>(token) * 2 * p.unit_heads;
     T *state;
     int fresh;
-    if (!locate_taps<T>(p.rows, token, taps, state, fresh)) return;  // nothing reads an idle row
+    if (!locate_taps<T>(p.rows, token, taps, state, fresh)) {
+        // nothing uses an idle row, but a box of neighbouring rows may take it along: it has to be finite
+        for (int c = threadIdx.x * VEC; c < p.rows.span; c += blockDim.x * VEC) {
+            Pack<VEC> zero = {};
+            store_pack<VEC>(mixed + c, zero);
+        }
+        return;
+    }
     __syncthreads();
     for (int c = threadIdx.x * VEC; c < p.rows.span; c += blockDim.x * VEC) {
         Pack<VEC> y = convolve<T, VEC>(p.rows, taps, state, fresh == 1, c);

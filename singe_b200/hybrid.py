@@ -30,13 +30,12 @@ import numpy as np
 
 from . import kernel_sys as ks
 from .decoder import PagedDecoder, PageTable
-from .layer_ops import BlockRows, ChunkRows, ExpandedRows, Ops, StepRows, plan_chunks, round_up
+from .layer_ops import FEW_TOKENS, BlockRows, ChunkRows, ExpandedRows, Ops, StepRows, plan_chunks, round_up
 from .parallel_mixer import ParallelConfig, ParallelMixer
 from .residual import LayerNormResidual, StreamResidual, Sublayer
 
 EXPANDED_HEAD_SIZES = (64, 128)  # head sizes of the tensor-core prompt attention; smaller heads are padded with zeros
 ABSORBED_LATENT_LIMIT = 512      # widest latent the tensor-core decode attention takes
-FEW_TOKENS = 8                   # a sequence with at most this many new tokens takes the decode kernels
 BLOCK_TOKENS = 16                # tokens of a block of the recurrence's prompt kernel
 LEAST_SEGMENT = 8                # blocks a long sequence's segments have at least
 

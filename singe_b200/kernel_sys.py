@@ -150,6 +150,8 @@ SIGNATURES = {
     "singe_conv_state_f32": [_p, _p, _z, _p, _p, _p, _z, _z, _z, _z],
     "singe_gated_delta_step_bf16": [_p, _p, _z, _p, _z, _p, _p, _z, _p, _z] + [_p] * 7 + [_z] * 9 + [_f, _z],
     "singe_gated_delta_step_f32": [_p, _p, _z, _p, _z, _p, _p, _z, _p, _z] + [_p] * 7 + [_z] * 9 + [_f, _z],
+    "singe_gated_delta_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _z, _p, _z] + [_p] * 5 + [_z] * 8 + [_f, _p, _p, _z, _p, _z, _p],
+    "singe_gated_delta_prompt_scratch": [_z, _z, _z, _z, _z],
     "singe_silu_mul_f32": [_p, _p, _z, _p, _p, _z, _z, _z],
     "singe_gated_linear_prompt_bf16": [_p, _p, _z, _p, _z, _p, _p, _p, _p, _p, _z, _z, _z, _z, _z, _f, _f, _f, _p, _p,
                                        _z, _p, _p, _z, _i, _p],
@@ -159,6 +161,7 @@ SIGNATURES = {
 
 _RESTYPES = {
     "singe_gated_linear_prompt_scratch": ctypes.c_size_t,
+    "singe_gated_delta_prompt_scratch": ctypes.c_size_t,
     "singe_latent_decode_splits": ctypes.c_size_t,
     "singe_status_string": ctypes.c_char_p,
     "singe_paged_kv_decode_split_tokens": ctypes.c_size_t,

@@ -6,6 +6,8 @@ from dataclasses import dataclass, field
 
 from . import kernel_sys as ks
 
+FEW_TOKENS = 8                   # a sequence with at most this many new tokens takes the decode kernels
+
 
 def round_up(value: int, multiple: int) -> int:
     return (value + multiple - 1) // multiple * multiple

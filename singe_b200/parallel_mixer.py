@@ -6,7 +6,8 @@
                         for few tokens, the tensor-core prompt kernel for more, which takes every (sequence, chunk) piece as a
                         sequence of its own.
   ``GatedDelta``        the gated delta rule: short convolutions with silu, unit queries and keys, a recurrent state per
-                        sequence, [heads, dim, vdim] in f32, with one decay per key channel.
+                        sequence, [heads, dim, vdim] in f32, with one decay per key channel; token by token for few tokens,
+                        block by block on the tensor core for more.
   ``ParallelMixer``     one projection GEMM for both; their outputs side by side, RMS-normed and averaged by the residual.
 
 Caches and states: keys and values in pages behind the page table; the last projected rows of each sequence for the
@@ -22,7 +23,7 @@ import numpy as np
 
 from . import kernel_sys as ks
 from .decoder import PageTable
-from .layer_ops import Ops, StepRows, round_up
+from .layer_ops import FEW_TOKENS, Ops, StepRows, round_up
 
 TILED_HEAD_SIZES = (64, 128)   # head sizes of the tensor-core kernels; smaller heads are padded with zeros
 TILED_GROUP = 8                # most query heads per key/value head of the split decode kernel
@@ -232,6 +233,8 @@ class GatedDelta:
         self.decay_rate, self.decay_bias = ops.scalars(source("A_log")), ops.scalars(source("dt_bias"))
         self.norm = take("norm").contiguous()
         self.out = ops.weight(take("o"))
+        # the block form, for sizes it takes
+        self.blocked = ops.is_bf16 and ks.lib().singe_gated_delta_prompt_scratch(c.heads, c.dim, c.vdim, 1, 1) > 0
 
     def new_cache(self, table: PageTable, sequences: int):
         torch, c = self.ops.torch, self.config
@@ -257,10 +260,18 @@ class GatedDelta:
         ops.head_linear(stream, decay, projected[:, self.low_at: self.low_at + 2 * self.rank], self.second, 2)
         attended = ops.rows(t, c.heads * c.vdim)
         strength = projected[:, self.strength_at:]
-        ops.call(f"singe_gated_delta_step_{ops.suffix}", stream, attended, attended.stride(0), mixed, mixed.stride(0), inverse,
-                 strength, strength.stride(0), decay, decay.stride(0), self.decay_rate, self.decay_bias, self.norm, state,
-                 step.first, step.fresh_tokens, step.context, t, sequences, c.heads, c.kv_heads, c.dim, c.vdim, self.key_at,
-                 self.value_at, self.columns, self.eps, 0x7fffffff)
+        operands = [attended, attended.stride(0), mixed, mixed.stride(0), inverse, strength, strength.stride(0), decay,
+                    decay.stride(0), self.decay_rate, self.decay_bias, self.norm, state]
+        sizes = [c.heads, c.kv_heads, c.dim, c.vdim, self.key_at, self.value_at, self.columns, self.eps]
+        rows = step.whole if self.blocked else None
+        if rows is not None:
+            scratch = torch.empty(int(ks.lib().singe_gated_delta_prompt_scratch(c.heads, c.dim, c.vdim, t, rows.blocks)),
+                                  dtype=torch.uint8, device="cuda")
+            ops.call("singe_gated_delta_prompt_bf16", stream, *operands, step.context, t, *sizes, rows.rows, rows.tokens, rows.blocks,
+                     rows.segments, rows.count, scratch)
+        if rows is None or step.short_count > 0:
+            ops.call(f"singe_gated_delta_step_{ops.suffix}", stream, *operands, step.first, step.fresh_tokens, step.context, t,
+                     sequences, *sizes, 0x7fffffff if rows is None else FEW_TOKENS)
         ops.linear(stream, out, attended, self.out)
 
 

@@ -11,16 +11,14 @@ import torch
 
 from oracle import hybrid_ref
 from singe_b200 import hybrid, models
-from singe_b200.checkpoint import load_hybrid
 from singe_b200.decoder import CachedDecoder, PageTableError
 from singe_b200.generation import GenerationOptions, PromptChunks, RunningBatch, generate_batch
 from tests import hybrid_util as util
 from tests.conftest import ROOT
+from tests.decoder_checks import Expect, check, greedy, run_portions, small_pages, tokens_of
 
 pytestmark = pytest.mark.gpu
 
-# root mean square of a position's logit error over that of its logits
-LIMIT = {"float32": 3e-5, "bfloat16": 6e-2}
 CONFIGS = {"mixed": util.MIXED, "odd": util.ODD, "ones": util.ONES, "wide": util.WIDE}
 
 
@@ -35,52 +33,9 @@ def snapshots(tmp_path_factory):
     return made
 
 
-class Expect:
-    """Oracle logits of whole sequences, computed once each."""
-
-    def __init__(self, config, weights):
-        self.config, self.weights, self.known = config, weights, {}
-
-    def __call__(self, tokens):
-        key = tuple(tokens)
-        if key not in self.known:
-            self.known[key] = hybrid_ref.forward(self.config, self.weights, tokens)[0]
-        return self.known[key]
-
-
 @pytest.fixture(scope="module")
 def expects(snapshots):
-    return {name: Expect(config, weights) for name, (config, weights, _) in snapshots.items()}
-
-
-def small_pages(directory, sequences, capacity, dtype, cache_tokens):
-    """A decoder whose cache pages hold 16 tokens, so that a small pool still has pages to move around."""
-    config, weights = load_hybrid(directory)
-    config.page_size = 16
-    return hybrid.HybridDecoder(config, sequences, capacity, weights, dtype, cache_tokens)
-
-
-def tokens_of(config, seed, count):
-    return [int(t) for t in np.random.default_rng(seed).integers(0, config["vocab"], size=count)]
-
-
-def check(got, expect, dtype, what):
-    got, expect = got.float().cpu().numpy().astype(np.float64), np.asarray(expect)
-    error = np.sqrt(((got - expect) ** 2).mean(1) / (expect ** 2).mean(1))
-    assert np.isfinite(got).all(), what
-    assert error.max() < LIMIT[dtype], f"{what}: position {error.argmax()} of {len(error)}: {error.max():.2e}"
-
-
-def run_portions(decoder, row, tokens, portions):
-    """Steps one row through ``tokens`` in portions, everything wanted; returns all logits."""
-    outs, at = [], 0
-    for n in portions:
-        part, want = [[] for _ in range(decoder.sequences)], [[] for _ in range(decoder.sequences)]
-        part[row], want[row] = tokens[at: at + n], list(range(len(tokens[at: at + n])))
-        outs.append(decoder.step_tokens(part, want=want).clone())
-        at += n
-    assert at >= len(tokens) and int(decoder.status.item()) == 0
-    return torch.cat(outs)
+    return {name: Expect(hybrid_ref, config, weights) for name, (config, weights, _) in snapshots.items()}
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -197,13 +152,6 @@ def test_a_step_without_room_changes_nothing(snapshots, expects):
         decoder.step_tokens([[1] * 100, []])
     rest = run_portions(decoder, 0, tokens[40:], [20])
     check(torch.cat([first, rest]), expects["mixed"](tokens), "float32", "around a refused step")
-
-
-def greedy(expect, prompt, count):
-    tokens = list(prompt)
-    for _ in range(count):
-        tokens.append(int(expect(tokens)[-1].argmax()))
-    return tokens[len(prompt):]
 
 
 def test_greedy_generation_through_the_scheduler(snapshots, expects):
