@@ -710,16 +710,17 @@ def run_only(args):
 
 
 def run_model(args):
-    """``--model kavalorn``: one JSON line of decode and prompt throughput and kernel rooflines (bench_hybrid.py)."""
+    """``--model``: one JSON line of decode and prompt throughput and kernel rooflines (bench_hybrid.py, bench_vatolorn.py)."""
     import torch
 
     if not torch.cuda.is_available():
         raise SystemExit("bench.py needs a CUDA device: the operators have no CPU path")
     import bench_hybrid
+    import bench_vatolorn
 
     peaks = measured_peaks()
     with ClockSampler(0) as clocks:
-        figures = bench_hybrid.run(peaks)
+        figures = {"kavalorn": bench_hybrid, "vatolorn": bench_vatolorn}[args.model].run(peaks)
     print(json.dumps({"model": args.model, "dtype": "bf16", "data": "synthetic", "peaks": peaks, "clocks": clocks.summary(),
                       "sizes": figures}), flush=True)
 
@@ -734,8 +735,8 @@ def main():
     parser.add_argument("--no-decode-step", action="store_true", help="skip the Llama-shaped decode step figure")
     parser.add_argument("--collective", default="peer", choices=["peer", "oneshot", "twophase", "pushall", "nccl"],
                         help="how the decode step's two collectives per layer run at --gpus > 1")
-    parser.add_argument("--model", default="", choices=["", "kavalorn"],
-                        help="instead of the headline workload: this model beside the Llama-shaped one at equal size "
+    parser.add_argument("--model", default="", choices=["", "kavalorn", "vatolorn"],
+                        help="instead of the headline workload: this model beside the closest other ones at equal size "
                         "(throughput and kernels; one GPU)")
     parser.add_argument("--only", default="", help="profiling aid: launch one kernel a few times and exit "
                         "(decode | paged_attention | gemm:M,N,K | prefill[:len,len,...] | kvwrite | step:LAYERS[:TP])")

@@ -30,6 +30,7 @@ def hybrid_config(size: str, pattern: str = PATTERN) -> hybrid.HybridConfig:
 
 
 def hybrid_decoder(config, sequences: int, capacity: int) -> hybrid.HybridDecoder:
+    """A layer-list decoder with random weights."""
     weights = hybrid.random_weights(config, checkpoint.hybrid_names(config))
     return hybrid.HybridDecoder(config, sequences, capacity, weights)
 

@@ -541,32 +541,50 @@ class HybridDecoder(PagedDecoder):
 
 
 def random_weights(config: HybridConfig, names: dict, seed: int = 4) -> dict:
-    """Random bf16 weights on the GPU for ``names`` (name -> shape): matrices ~ N(0, 1 / columns), norms 1, decay biases 2."""
+    """Random bf16 weights on the GPU for ``names`` (name -> shape): matrices ~ N(0, 1 / columns), norms 1, decays that keep a few
+    hundred tokens, streams that blend into one another a little."""
     import torch
 
     generator = torch.Generator(device="cuda").manual_seed(seed)
+    constants = {"a2.b": 2.0, "A_log": -3.0, "dt_bias": 0.0, "q.b": 0.0, "k.b": 0.0, "v.b": 0.0}
     weights = {}
     for name, shape in names.items():
         if len(shape) == 1:
-            weights[name] = torch.full(shape, 2.0 if name.endswith("a2.b") else 1.0, dtype=torch.bfloat16, device="cuda")
+            value = next((value for ending, value in constants.items() if name.endswith(ending)), 1.0)
+            if name.endswith((".in", ".out")) and ".hc" in name:
+                value = 1.0 / shape[0]
+            weights[name] = torch.full(shape, value, dtype=torch.bfloat16, device="cuda")
         else:
             values = torch.randn(shape, generator=generator, device="cuda", dtype=torch.float32)
-            weights[name] = (values * (1.0 if name == "embed" else shape[1] ** -0.5)).to(torch.bfloat16)
+            values *= 1.0 if name == "embed" else shape[1] ** -0.5
+            if name.endswith(".mix") and ".hc" in name:
+                values = 0.1 * values + torch.eye(shape[0], device="cuda")
+            weights[name] = values.to(torch.bfloat16)
     return weights
 
 
 def decode_step_bytes(config: HybridConfig, sequences: int, context: int) -> dict:
-    """Algorithmic HBM bytes of one bf16 decode step: every weight once (borrowed layers read their owner's again), the
-    visible latents of every sequence, the recurrent states read and written."""
-    weights, cache, state = config.vocab * config.width, 0, 0
+    """Algorithmic HBM bytes of one bf16 decode step: every weight once (borrowed layers read their owner's again), the visible
+    latents or keys and values of every sequence, the recurrent states read and written, the residual streams where there are
+    several."""
+    weights, cache, state, streams = config.vocab * config.width, 0, 0, 0
     for layer in config.layers:
         m, w = layer.mixer, config.width
-        weights += 2 * layer.ffn * w
+        weights += (3 if layer.gated else 2) * layer.ffn * w
+        streams += sequences * config.streams * w * (2 if layer.ffn else 1)
         if isinstance(m, LatentAttentionConfig):
             weights += (m.q_rank + m.kv_rank + m.heads) * w + m.heads * m.dim * (m.q_rank + m.kv_rank)
             weights += m.heads * m.vdim * (m.kv_rank + w)
             cache += sequences * min(context, m.window) * m.kv_rank
+        elif isinstance(m, ParallelConfig):
+            a, r = m.left, m.right
+            weights += (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim)) * w
+            weights += (2 * r.kv_heads * r.dim + 2 * r.heads * r.vdim + r.heads + r.rank + r.gate_rank) * w
+            weights += r.heads * (r.dim * r.rank + r.vdim * r.gate_rank)
+            cache += sequences * (context % a.chunk + 1) * a.kv_heads * (a.dim + a.vdim)
+            state += sequences * r.heads * r.dim * r.vdim
         else:
             weights += (2 * m.heads * (m.dim + m.vdim) + m.rank) * w + m.heads * m.dim * m.rank + m.heads * m.vdim * w
             state += sequences * m.heads * m.dim * m.vdim
-    return {"weights": 2 * weights, "latents": 2 * cache, "states": 8 * state, "total": 2 * weights + 2 * cache + 8 * state}
+    total = 2 * weights + 2 * cache + 8 * state + 8 * streams
+    return {"weights": 2 * weights, "latents": 2 * cache, "states": 8 * state, "streams": 8 * streams, "total": total}

@@ -144,8 +144,8 @@ def test_long_decoding(snapshots, expects, dtype):
 
 
 def test_a_chunk_is_left_behind_at_its_edge(snapshots, expects):
-    """One layer whose attention singles out a key: the logits change with that key exactly as long as its chunk lasts."""
-    config = util.model(64, 50, 2, 1.0, 1e-6, util.layer(util.left(2, 1, 16, 16, 24, 1, util.rot(2, 10.0, (1.0, 16, 1.0, 1.0)), 4.0),
+    """One layer, soft attention, no recurrence: the logits change with a token exactly as long as its chunk lasts."""
+    config = util.model(64, 50, 2, 1.0, 1e-6, util.layer(util.left(2, 1, 16, 16, 24, 1, util.rot(2, 10.0, (1.0, 16, 1.0, 1.0)), 0.2),
                                                          util.right(1, 1, 8, 8, 1)))
     weights = util.make_weights(config, seed=9)
     weights["l0.mix.right.v"][:] = 0.0   # the recurrence carries nothing
@@ -160,9 +160,10 @@ def test_a_chunk_is_left_behind_at_its_edge(snapshots, expects):
                 decoder = models.load_decoder(directory, 1, 64, dtype)
                 outs.append(run_portions(decoder, 0, tokens, [30] + [1] * 10 + [20]))
                 check(outs[-1], vatolorn_ref.forward(config, weights, tokens)[0], dtype, f"target {target}")
-            changed = [bool(v) for v in ((outs[0] - outs[1]).abs().amax(1) > 1e-6).tolist()]
+            changed = ((outs[0] - outs[1]).abs().amax(1) > 1e-5).tolist()
             last = (target // 24 + 1) * 24
-            assert not any(changed[:target]) and all(changed[target: min(last, 60)]) and not any(changed[last:])
+            assert not any(changed[:target]) and not any(changed[last:])
+            assert all(changed[target:last]) if dtype == "float32" else changed[target]
 
 
 def test_a_step_without_room_changes_nothing(snapshots, expects):

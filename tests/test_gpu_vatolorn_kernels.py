@@ -292,9 +292,12 @@ class DeltaCase:
         self.value_at = 2 * self.key_at
         self.columns = round_up(max(heads * dim, heads * vdim), 8)
         self.mixed = draw(rng, rows, self.value_at + round_up(heads * vdim, 8))
-        self.mixed[:, self.key_at: self.value_at] *= 0.7
-        # neighbouring tokens' keys resemble one another, so that the writes of a block interact
-        self.mixed[1:, self.key_at: self.value_at] = bf16(self.mixed[1:, self.key_at: self.value_at] + self.mixed[:-1, self.key_at: self.value_at])
+        # neighbouring tokens' keys resemble one another, so that the writes of a block interact, and every token's key its query,
+        # so that no first read-out all but vanishes
+        keys = self.mixed[:, self.key_at: self.value_at] * 0.7
+        keys[1:] += keys[:-1].copy()
+        keys[:, : kv_heads * dim] += 0.5 * self.mixed[:, : kv_heads * dim]
+        self.mixed[:, self.key_at: self.value_at] = bf16(keys)
         self.strength, self.decay = draw(rng, rows, heads, scale=2.0), draw(rng, rows, 2 * self.columns, scale=spread)
         self.rate = (rate + 0.1 * rng.standard_normal(heads)).astype(np.float32)
         self.bias = (bias + 0.3 * rng.standard_normal(heads * dim)).astype(np.float32)
