@@ -15,11 +15,11 @@
 // value is lost) and their products keep hi hi + hi lo + lo hi; v is bf16 from its convolution and enters as it is.
 // Accumulators, and the state between the blocks, are f32.
 //
-//   prepare   one warp per (block, head): decays, M and its inverse, P and the split operands, to scratch, laid out as the next
+//   prepare   one CTA per (block, head): decays, M and its inverse, P and the split operands, to scratch, laid out as the next
 //             kernel's shared memory wants them, so that a block arrives in one bulk copy
 //   advance   one CTA per (sequence, head, slice of the values): the blocks in order, the state in registers as S^T [vdim, dim],
-//             whose accumulator layout is the A-operand layout of the next product.  A warp owns 16 value rows.  The columns of
-//             the state do not meet, so slices run side by side.
+//             whose accumulator layout is the A-operand layout of the next product.  The columns of the state do not meet, so
+//             slices run side by side.
 //   finish    RMS norm over a head's values, gate, store
 #include "row_pack.cuh"
 #include "split_bf16.cuh"
@@ -27,7 +27,6 @@
 namespace singe {
 namespace {
 
-constexpr int kPrepareWarps = 2;
 constexpr int kMaxStages = 6;
 constexpr float kFactoredLimit = -60.0f;
 constexpr int kPitchP = kBlock * 2 + 16;  // bytes of a padded row of P or T
@@ -76,8 +75,11 @@ struct DeltaParams {
     int stages;
 };
 
-// Shared memory of one warp of the prepare kernel: (q exp(a)), (k exp(-a)) and (k exp(a)), each hi and lo, and a 16 x 17 matrix.
-__host__ __device__ constexpr int prepare_bytes(int dim_pad) { return 6 * kBlock * (dim_pad * 2 + 16) + kBlock * 17 * 4 + 64; }
+// Shared memory of the prepare kernel: (q exp(a)), (k exp(-a)) and (k exp(a)), each hi and lo, a 16 x 17 matrix, three numbers a
+// token, and the decay of either half of the block per channel.
+__host__ __device__ constexpr int prepare_bytes(int dim_pad) {
+    return 6 * kBlock * (dim_pad * 2 + 16) + kBlock * 17 * 4 + 3 * kBlock * 4 + dim_pad * 8;
+}
 
 // acc (two n tiles of 8) += A[16, 16 rows at a] . B[16 rows at b, same columns]^T over `columns`, split operands.
 __device__ __forceinline__ void product_rows(float (&acc)[2][4], uint32_t a_at, uint32_t b_at, int pitch, int columns) {
@@ -101,189 +103,190 @@ __device__ __forceinline__ void product_rows(float (&acc)[2][4], uint32_t a_at, 
 __device__ __forceinline__ float low_half(uint32_t pair) { return __uint_as_float(pair << 16); }
 __device__ __forceinline__ float high_half(uint32_t pair) { return __uint_as_float(pair & 0xffff0000u); }
 
-__global__ void __launch_bounds__(kPrepareWarps * 32) gated_delta_prepare_kernel(const DeltaParams p) {
+// One CTA per (block, head); a thread takes two adjacent channels of one half of the block's tokens.
+__global__ void __launch_bounds__(256) gated_delta_prepare_kernel(const DeltaParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
-    const int block = blockIdx.x;
+    constexpr int kHalf = kBlock / 2;
+    const int block = blockIdx.x, head = blockIdx.y;
     const int row0 = p.block_row[block], tokens = p.block_tokens[block];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y * kPrepareWarps + warp;
-    if (head >= p.heads) return;  // warps work alone
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
     const DeltaLayout layout = delta_layout(p.dim_pad);
     extern __shared__ __align__(16) uint8_t prepare_shared[];
-    uint8_t *own = prepare_shared + warp * prepare_bytes(p.dim_pad);
     const int half_bytes = kBlock * layout.pitch;  // from the hi to the lo part
-    uint8_t *fq = own, *fk = own + 2 * half_bytes, *fa = own + 4 * half_bytes;
-    float *matrix = reinterpret_cast<float *>(own + 6 * half_bytes);  // [16][17]
-    float *betas = matrix + kBlock * 17;                              // [16]
+    uint8_t *fq = prepare_shared, *fk = fq + 2 * half_bytes, *fa = fk + 2 * half_bytes;
+    float *matrix = reinterpret_cast<float *>(fa + 2 * half_bytes);  // [16][17]
+    float *betas = matrix + kBlock * 17, *units_q = betas + kBlock, *units_k = units_q + kBlock;
+    float2 *totals = reinterpret_cast<float2 *>(units_k + kBlock);   // [2 halves][dim_pad / 2]
     const int source = head / (p.heads / p.kv_heads);
     uint8_t *pack = p.operands + (static_cast<size_t>(block) * p.heads + head) * layout.bytes;
-    float *whole_decay = reinterpret_cast<float *>(pack + layout.decay);
     const float rate = expf(p.rate[head]);
-    const float query_scale = 1.0f / sqrtf(static_cast<float>(p.dim));
 
-    // a lane's own token: unit lengths and write strength
-    float unit_q = 0.0f, unit_k = 0.0f;
-    if (lane < kBlock) {
-        float beta = 0.0f;
-        if (lane < tokens) {
-            const long long row = row0 + lane;
-            unit_q = p.inverse[row * 2 * p.kv_heads + source] * query_scale;
+    if (tid < kBlock) {
+        float beta = 0.0f, unit_q = 0.0f, unit_k = 0.0f;
+        if (tid < tokens) {
+            const long long row = row0 + tid;
+            unit_q = p.inverse[row * 2 * p.kv_heads + source] / sqrtf(static_cast<float>(p.dim));
             unit_k = p.inverse[row * 2 * p.kv_heads + p.kv_heads + source];
             beta = 1.0f / (1.0f + expf(-__bfloat162float(p.strength[row * p.strength_stride + head])));
         }
-        betas[lane] = beta;
+        betas[tid] = beta;
+        units_q[tid] = unit_q;
+        units_k[tid] = unit_k;
     }
-    // log decay of token t in channel c, and its running sum
-    auto running_decay = [&](int c, float (&sum)[2][kBlock]) {
-        const bool real = c < p.dim;
-        const int channel = head * p.dim + (real ? c : 0);
-        const float2 bias = real ? make_float2(p.bias[channel], p.bias[channel + 1]) : make_float2(0.0f, 0.0f);
-        uint32_t z[kBlock];
+    const int pairs = p.dim_pad / 2;
+    const int c = 2 * (tid % pairs), half = tid / pairs;
+    const bool inside = half < 2, real = inside && c < p.dim;  // dim is a multiple of eight
+    const int t0 = half * kHalf, channel = head * p.dim + (real ? c : 0);
+    uint32_t q_raw[kHalf], k_raw[kHalf], z_raw[kHalf];
+    {
+        const __nv_bfloat16 *rows = p.mixed + (row0 + t0) * p.mixed_stride + source * p.dim + (real ? c : 0);
+        const __nv_bfloat16 *decays = p.decay + (row0 + t0) * p.decay_stride + channel;
 #pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            z[t] = real && t < tokens ? *reinterpret_cast<const uint32_t *>(p.decay + (row0 + t) * p.decay_stride + channel) : 0u;
+        for (int i = 0; i < kHalf; ++i) {
+            const bool live = real && t0 + i < tokens;
+            z_raw[i] = live ? *reinterpret_cast<const uint32_t *>(decays + i * p.decay_stride) : 0u;
+            q_raw[i] = live ? *reinterpret_cast<const uint32_t *>(rows + i * p.mixed_stride) : 0u;
+            k_raw[i] = live ? *reinterpret_cast<const uint32_t *>(rows + i * p.mixed_stride + p.key_at) : 0u;
         }
-        float total[2] = {0.0f, 0.0f};
+    }
+    // running sums of the log decays, over this half and then over the block
+    float2 sum[kHalf];
+    {
+        const float2 bias = real ? *reinterpret_cast<const float2 *>(p.bias + channel) : make_float2(0.0f, 0.0f);
+        float2 running = make_float2(0.0f, 0.0f);
 #pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            if (real && t < tokens) {
-                const float x = low_half(z[t]) + bias.x, y = high_half(z[t]) + bias.y;
-                total[0] -= rate * (fmaxf(x, 0.0f) + log1pf(__expf(-fabsf(x))));
-                total[1] -= rate * (fmaxf(y, 0.0f) + log1pf(__expf(-fabsf(y))));
+        for (int i = 0; i < kHalf; ++i) {
+            if (real && t0 + i < tokens) {
+                const float x = low_half(z_raw[i]) + bias.x, y = high_half(z_raw[i]) + bias.y;
+                running.x -= rate * (fmaxf(x, 0.0f) + log1pf(__expf(-fabsf(x))));
+                running.y -= rate * (fmaxf(y, 0.0f) + log1pf(__expf(-fabsf(y))));
             }
-            sum[0][t] = total[0];
-            sum[1][t] = total[1];
+            sum[i] = running;
         }
-    };
-
+        if (inside) totals[half * pairs + c / 2] = running;
+    }
+    __syncthreads();
     bool strong = false;
-    for (int c = 2 * lane; c < p.dim_pad + 2 * lane; c += 64) {  // a lane takes two adjacent channels
-        const bool inside = c < p.dim_pad;                        // (every lane takes part in the shuffles)
-        const bool real = c < p.dim;                              // dim is a multiple of eight
-        float a[2][kBlock];
-        running_decay(inside ? c : p.dim_pad, a);
-        const float total[2] = {a[0][kBlock - 1], a[1][kBlock - 1]};
-        const bool factors = fminf(total[0], total[1]) >= kFactoredLimit;
-        strong = strong || !factors;
-        const float whole[2] = {__expf(total[0]), __expf(total[1])};
-        if (inside) *reinterpret_cast<float2 *>(whole_decay + c) = make_float2(whole[0], whole[1]);
-        const __nv_bfloat16 *rows = p.mixed + row0 * p.mixed_stride + source * p.dim + (real ? c : 0);
+    if (inside) {
+        const float2 first = totals[c / 2], second = totals[pairs + c / 2];
+        const float2 total = make_float2(first.x + second.x, first.y + second.y);
+        if (half == 1) {
 #pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            const bool live = real && t < tokens;
-            const uint32_t q_raw = live ? *reinterpret_cast<const uint32_t *>(rows + t * p.mixed_stride) : 0u;
-            const uint32_t k_raw = live ? *reinterpret_cast<const uint32_t *>(rows + t * p.mixed_stride + p.key_at) : 0u;
-            const float uq = __shfl_sync(0xffffffffu, unit_q, t), uk = __shfl_sync(0xffffffffu, unit_k, t);
-            float before[2], after[2], back[2];  // exp(a_t), exp(A - a_t), exp(-a_t)
+            for (int i = 0; i < kHalf; ++i) sum[i] = make_float2(sum[i].x + first.x, sum[i].y + first.y);
+        }
+        const bool factors = fminf(total.x, total.y) >= kFactoredLimit;
+        strong = !factors;
+        const float2 whole = make_float2(__expf(total.x), __expf(total.y));
+        if (half == 0) *reinterpret_cast<float2 *>(pack + layout.decay + c * 4) = whole;
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                before[i] = __expf(a[i][t]);
-                if (factors) {
-                    back[i] = __expf(-a[i][t]);
-                    after[i] = whole[i] * back[i];
-                } else {
-                    back[i] = 0.0f;
-                    after[i] = __expf(total[i] - a[i][t]);
-                }
+        for (int i = 0; i < kHalf; ++i) {
+            const float uq = units_q[t0 + i], uk = units_k[t0 + i];
+            // exp(a_t), exp(A - a_t), exp(-a_t)
+            const float2 before = make_float2(__expf(sum[i].x), __expf(sum[i].y));
+            float2 after, back = make_float2(0.0f, 0.0f);
+            if (factors) {
+                back = make_float2(__expf(-sum[i].x), __expf(-sum[i].y));
+                after = make_float2(whole.x * back.x, whole.y * back.y);
+            } else {
+                after = make_float2(__expf(total.x - sum[i].x), __expf(total.y - sum[i].y));
             }
-            if (!inside) continue;
-            const float q0 = low_half(q_raw) * uq, q1 = high_half(q_raw) * uq;
-            const float k0 = low_half(k_raw) * uk, k1 = high_half(k_raw) * uk;
-            const int at = t * layout.pitch + c * 2;
+            const float q0 = low_half(q_raw[i]) * uq, q1 = high_half(q_raw[i]) * uq;
+            const float k0 = low_half(k_raw[i]) * uk, k1 = high_half(k_raw[i]) * uk;
+            const int at = (t0 + i) * layout.pitch + c * 2;
             uint32_t hi, lo;
-            split_pair(q0 * before[0], q1 * before[1], hi, lo);
+            split_pair(q0 * before.x, q1 * before.y, hi, lo);
             *reinterpret_cast<uint32_t *>(pack + at) = hi;
             *reinterpret_cast<uint32_t *>(pack + half_bytes + at) = lo;
             *reinterpret_cast<uint32_t *>(fq + at) = hi;
             *reinterpret_cast<uint32_t *>(fq + half_bytes + at) = lo;
-            split_pair(k0 * after[0], k1 * after[1], hi, lo);
+            split_pair(k0 * after.x, k1 * after.y, hi, lo);
             *reinterpret_cast<uint32_t *>(pack + layout.k + at) = hi;
             *reinterpret_cast<uint32_t *>(pack + layout.k + half_bytes + at) = lo;
-            split_pair(k0 * back[0], k1 * back[1], hi, lo);
+            split_pair(k0 * back.x, k1 * back.y, hi, lo);
             *reinterpret_cast<uint32_t *>(fk + at) = hi;
             *reinterpret_cast<uint32_t *>(fk + half_bytes + at) = lo;
-            split_pair(k0 * before[0], k1 * before[1], hi, lo);
+            split_pair(k0 * before.x, k1 * before.y, hi, lo);
             *reinterpret_cast<uint32_t *>(fa + at) = hi;
             *reinterpret_cast<uint32_t *>(fa + half_bytes + at) = lo;
         }
     }
-    __syncwarp();
     // ---- P, and M (not yet times beta) ----
     uint8_t *p_hi = pack + layout.p, *p_lo = p_hi + kBlock * kPitchP;
     uint8_t *t_hi = pack + layout.t, *t_lo = t_hi + kBlock * kPitchP;
-    const int a_offset = (lane & 15) * layout.pitch + (lane >> 4) * 16;
-    const int b_offset = ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch + ((lane >> 3) & 1) * 16;
-    if (!__any_sync(0xffffffffu, strong)) {
-        float scores[2][4] = {}, keys[2][4] = {};
-        product_rows(scores, smem_u32(fq) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
-        product_rows(keys, smem_u32(fa) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
+    if (__syncthreads_or(strong ? 1 : 0) == 0) {
+        const int a_offset = (lane & 15) * layout.pitch + (lane >> 4) * 16;
+        const int b_offset = ((lane & 7) + ((lane >> 4) << 3)) * layout.pitch + ((lane >> 3) & 1) * 16;
+        if (warp == 0) {
+            float scores[2][4] = {};
+            product_rows(scores, smem_u32(fq) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
+            for (int n = 0; n < 2; ++n) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int t = (lane >> 2) + half * 8, j = n * 8 + (lane & 3) * 2;
-                uint32_t hi, lo;
-                split_pair(j <= t ? scores[n][2 * half] : 0.0f, j + 1 <= t ? scores[n][2 * half + 1] : 0.0f, hi, lo);
-                *reinterpret_cast<uint32_t *>(p_hi + t * kPitchP + j * 2) = hi;
-                *reinterpret_cast<uint32_t *>(p_lo + t * kPitchP + j * 2) = lo;
-                matrix[t * 17 + j] = j < t ? keys[n][2 * half] : 0.0f;
-                matrix[t * 17 + j + 1] = j + 1 < t ? keys[n][2 * half + 1] : 0.0f;
+                for (int i = 0; i < 2; ++i) {
+                    const int t = (lane >> 2) + i * 8, j = n * 8 + (lane & 3) * 2;
+                    uint32_t hi, lo;
+                    split_pair(j <= t ? scores[n][2 * i] : 0.0f, j + 1 <= t ? scores[n][2 * i + 1] : 0.0f, hi, lo);
+                    *reinterpret_cast<uint32_t *>(p_hi + t * kPitchP + j * 2) = hi;
+                    *reinterpret_cast<uint32_t *>(p_lo + t * kPitchP + j * 2) = lo;
+                }
+            }
+        }
+        if (warp == warps - 1) {
+            float keys[2][4] = {};
+            product_rows(keys, smem_u32(fa) + a_offset, smem_u32(fk) + b_offset, layout.pitch, p.dim_pad);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const int t = (lane >> 2) + (i >> 1) * 8, j = n * 8 + (lane & 3) * 2 + (i & 1);
+                    matrix[t * 17 + j] = j < t ? keys[n][i] : 0.0f;
+                }
             }
         }
     } else {
         // Decays too strong to factor: every pair's decay is taken as one exponential.  The running sums go where k exp(-a)
-        // was; the lanes are the channels.
+        // was; the lanes are the channels, the warps take the pairs in turn.
         float *sums = reinterpret_cast<float *>(fk);  // [16][dim_pad]
-        for (int c = 2 * lane; c < p.dim_pad; c += 64) {
-            float a[2][kBlock];
-            running_decay(c, a);
+        if (inside) {
 #pragma unroll
-            for (int t = 0; t < kBlock; ++t) *reinterpret_cast<float2 *>(sums + t * p.dim_pad + c) = make_float2(a[0][t], a[1][t]);
+            for (int i = 0; i < kHalf; ++i) *reinterpret_cast<float2 *>(sums + (t0 + i) * p.dim_pad + c) = sum[i];
         }
-        __syncwarp();
+        __syncthreads();
         const __nv_bfloat16 *queries = p.mixed + row0 * p.mixed_stride + source * p.dim, *keys = queries + p.key_at;
-        for (int t = 0; t < kBlock; ++t) {
-            const float uq = __shfl_sync(0xffffffffu, unit_q, t), kt = __shfl_sync(0xffffffffu, unit_k, t);
-            for (int j = 0; j <= t; ++j) {
-                const float kj = __shfl_sync(0xffffffffu, unit_k, j);
-                float score = 0.0f, dot = 0.0f;
-                if (t < tokens) {
-                    for (int c = lane; c < p.dim; c += 32) {
-                        const float carried = __bfloat162float(keys[j * p.mixed_stride + c]) * kj *
-                                              __expf(sums[t * p.dim_pad + c] - sums[j * p.dim_pad + c]);
-                        score = fmaf(__bfloat162float(queries[t * p.mixed_stride + c]) * uq, carried, score);
-                        dot = fmaf(__bfloat162float(keys[t * p.mixed_stride + c]) * kt, carried, dot);
-                    }
+        for (int item = warp; item < kBlock * kBlock; item += warps) {
+            const int t = item / kBlock, j = item % kBlock;
+            float score = 0.0f, dot = 0.0f;
+            if (j <= t && t < tokens) {
+                for (int d = lane; d < p.dim; d += 32) {
+                    const float carried = __bfloat162float(keys[j * p.mixed_stride + d]) * units_k[j] *
+                                          __expf(sums[t * p.dim_pad + d] - sums[j * p.dim_pad + d]);
+                    score = fmaf(__bfloat162float(queries[t * p.mixed_stride + d]) * units_q[t], carried, score);
+                    dot = fmaf(__bfloat162float(keys[t * p.mixed_stride + d]) * units_k[t], carried, dot);
                 }
                 score = warp_sum(score);
                 dot = warp_sum(dot);
-                if (lane == 0) {
-                    __nv_bfloat16 hi, lo;
-                    split_bf16(score, hi, lo);
-                    *reinterpret_cast<__nv_bfloat16 *>(p_hi + t * kPitchP + j * 2) = hi;
-                    *reinterpret_cast<__nv_bfloat16 *>(p_lo + t * kPitchP + j * 2) = lo;
-                    matrix[t * 17 + j] = j < t ? dot : 0.0f;
-                }
             }
-            for (int j = t + 1 + lane; j < kBlock; j += 32) {
-                *reinterpret_cast<uint16_t *>(p_hi + t * kPitchP + j * 2) = 0;
-                *reinterpret_cast<uint16_t *>(p_lo + t * kPitchP + j * 2) = 0;
-                matrix[t * 17 + j] = 0.0f;
+            if (lane == 0) {
+                __nv_bfloat16 hi, lo;
+                split_bf16(score, hi, lo);
+                *reinterpret_cast<__nv_bfloat16 *>(p_hi + t * kPitchP + j * 2) = hi;
+                *reinterpret_cast<__nv_bfloat16 *>(p_lo + t * kPitchP + j * 2) = lo;
+                matrix[t * 17 + j] = j < t ? dot : 0.0f;
             }
         }
     }
-    __syncwarp();
+    __syncthreads();
     // ---- T = (I + diag(beta) M)^-1 diag(beta): a lane solves for one column ----
-    {
+    if (warp == 0) {
         float x[kBlock];
         const int j = lane & 15;
 #pragma unroll
         for (int t = 0; t < kBlock; ++t) {
-            float sum = 0.0f;
+            float known = 0.0f;
 #pragma unroll
-            for (int i = 0; i < t; ++i) sum = fmaf(matrix[t * 17 + i], x[i], sum);
-            x[t] = (t == j ? 1.0f : 0.0f) - betas[t] * sum;
+            for (int i = 0; i < t; ++i) known = fmaf(matrix[t * 17 + i], x[i], known);
+            x[t] = (t == j ? 1.0f : 0.0f) - betas[t] * known;
         }
         __syncwarp();
         const float beta = betas[j];
@@ -299,7 +302,7 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) gated_delta_prepare_kernel
             }
         }
     }
-    __syncwarp();
+    __syncthreads();
     // ---- W = T (k exp(a)) ----
     uint32_t sh[4], sl[4];  // T as A operand
     {
@@ -311,7 +314,7 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) gated_delta_prepare_kernel
         }
     }
     const uint32_t w_at = smem_u32(fa) + (lane & 15) * layout.pitch + (lane >> 4) * 16;
-    for (int c0 = 0; c0 < p.dim_pad; c0 += 16) {
+    for (int c0 = warp * 16; c0 < p.dim_pad; c0 += warps * 16) {
         uint32_t hi[4], lo[4];
         ldmatrix_x4_trans(w_at + c0 * 2, hi[0], hi[1], hi[2], hi[3]);
         ldmatrix_x4_trans(w_at + half_bytes + c0 * 2, lo[0], lo[1], lo[2], lo[3]);
@@ -322,10 +325,10 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) gated_delta_prepare_kernel
             mma_m16n8k16<__nv_bfloat16>(acc, sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
             mma_m16n8k16<__nv_bfloat16>(acc, sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int at = ((lane >> 2) + half * 8) * layout.pitch + (c0 + n * 8 + (lane & 3) * 2) * 2;
+            for (int i = 0; i < 2; ++i) {
+                const int at = ((lane >> 2) + i * 8) * layout.pitch + (c0 + n * 8 + (lane & 3) * 2) * 2;
                 uint32_t x, y;
-                split_pair(acc[2 * half], acc[2 * half + 1], x, y);
+                split_pair(acc[2 * i], acc[2 * i + 1], x, y);
                 *reinterpret_cast<uint32_t *>(pack + layout.w + at) = x;
                 *reinterpret_cast<uint32_t *>(pack + layout.w + half_bytes + at) = y;
             }
@@ -339,41 +342,42 @@ __host__ __device__ inline int delta_stage_bytes(int dim_pad, int slice) {
     return delta_values_at(dim_pad) + (slice + 63) / 64 * kValueBox;
 }
 
-// KT = dim_pad / 16.  A warp owns 16 value rows of the slice.
-template <int KT>
-__global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kernel(const __grid_constant__ CUtensorMap value_map,
-                                                                                  const DeltaParams p) {
+// KT = dim_pad / 16.  16 value rows of the slice belong to KS warps, each with KT / KS of the key tiles: with few (sequence, head)
+// pairs one warp's products are what a block waits for, and sharing them pays for bringing the sums together.
+template <int KT, int KS>
+__global__ void __launch_bounds__(256, KT / KS <= 8 ? 2 : 1) gated_delta_advance_kernel(const __grid_constant__ CUtensorMap value_map,
+                                                                                       const DeltaParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
-    constexpr int kDim = KT * 16;
+    constexpr int kDim = KT * 16, kTiles = KT / KS;
     constexpr DeltaLayout kLayout = delta_layout(kDim);
     constexpr int kHalf = kBlock * kLayout.pitch;
     const int run = blockIdx.x, head = blockIdx.y, slice0 = blockIdx.z * p.slice;
     const int sequence = p.runs[3 * run], first_block = p.runs[3 * run + 1], blocks = p.runs[3 * run + 2];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, q2 = (lane & 3) * 2;
+    const int share = warp % KS, tile0 = share * kTiles;  // this warp's key tiles
     const int stages = p.stages;
     const int stage_bytes = delta_stage_bytes(kDim, p.slice), values_at = delta_values_at(kDim);
     extern __shared__ uint8_t advance_raw[];
     uint8_t *advance_shared = advance_raw + ((1024u - (smem_u32(advance_raw) & 1023u)) & 1023u);
-    const int pitch_o = p.slice + 4;  // floats of a padded row of the outputs on their way to memory
-    float *outputs = reinterpret_cast<float *>(advance_shared + stages * stage_bytes);  // [16][pitch_o]
-    const uint32_t bars = smem_u32(outputs + kBlock * pitch_o);
+    float4 *sums = reinterpret_cast<float4 *>(advance_shared + stages * stage_bytes);  // [warps][4][32], KS > 1
+    const uint32_t bars = smem_u32(sums + (KS > 1 ? blockDim.x * 4 : 0));
     if (tid == 0) {
         for (int i = 0; i < stages; ++i) mbar_init(bars + 8 * i, 1);
         mbar_init_fence();
     }
     __syncthreads();
 
-    const int value0 = warp * 16;  // within the slice
-    float state[2 * KT][4];        // S^T: rows v, columns k
+    const int value0 = warp / KS * 16;  // within the slice
+    float state[2 * kTiles][4];         // S^T: rows v, columns k
     float *home = p.state + (static_cast<size_t>(sequence) * p.heads + head) * p.dim * p.vdim;
     const bool fresh = p.context[sequence] == 0;
 #pragma unroll
-    for (int n = 0; n < 2 * KT; ++n) {
+    for (int n = 0; n < 2 * kTiles; ++n) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const int v = slice0 + value0 + g + (i >> 1) * 8, k = n * 8 + q2 + (i & 1);
+            const int v = slice0 + value0 + g + (i >> 1) * 8, k = tile0 * 16 + n * 8 + q2 + (i & 1);
             state[n][i] = !fresh && v < p.vdim && k < p.dim ? home[static_cast<size_t>(k) * p.vdim + v] : 0.0f;
         }
     }
@@ -398,13 +402,12 @@ __global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kern
     };
     for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
     bool failed = false;
-    const int width = min(p.slice, p.vdim - slice0);  // real columns of the slice, a multiple of eight
 
     for (int index = 0; index < blocks; ++index) {
         const int row0 = p.block_row[first_block + index], tokens = p.block_tokens[first_block + index];
         const bool arrived = mbar_wait(bars + 8 * (index % stages), (index / stages) & 1);
         fence_proxy_async_shared();
-        // the block has arrived for every thread, everyone is done with the stage loaded next, and with the outputs before
+        // the block has arrived for every thread, and everyone is done with the stage loaded next and with the sums
         if (__syncthreads_or(arrived ? 0 : 1) != 0) {
             failed = true;
             break;
@@ -417,30 +420,71 @@ __global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kern
         uint32_t value[4];  // v^T of this warp: rows v, columns tokens
         ldmatrix_x4_trans(stage + values_at + value_at(t, value0 + ((lane >> 3) & 1) * 8), value[0], value[1], value[2], value[3]);
         // ---- S^T W^T and S^T (q exp(a))^T; the small terms are dependency chains of their own ----
-        float o[2][4] = {}, o_low[2][4] = {}, u[2][4] = {}, u_low[2][4] = {};
+        float o[2][4] = {}, u[2][4] = {};
+        {
+            float o_low[2][4] = {}, u_low[2][4] = {};
 #pragma unroll
-        for (int kt = 0; kt < KT; ++kt) {
-            const uint32_t at = stage + t * kLayout.pitch + (kt * 16 + ((lane >> 3) & 1) * 8) * 2;
-            uint32_t sh[4], sl[4], hi[4], lo[4];
-            split_pair(state[2 * kt][0], state[2 * kt][1], sh[0], sl[0]);
-            split_pair(state[2 * kt][2], state[2 * kt][3], sh[1], sl[1]);
-            split_pair(state[2 * kt + 1][0], state[2 * kt + 1][1], sh[2], sl[2]);
-            split_pair(state[2 * kt + 1][2], state[2 * kt + 1][3], sh[3], sl[3]);
-            ldmatrix_x4(at + kLayout.w, hi[0], hi[1], hi[2], hi[3]);
-            ldmatrix_x4(at + kLayout.w + kHalf, lo[0], lo[1], lo[2], lo[3]);
+            for (int kt = 0; kt < kTiles; ++kt) {
+                const uint32_t at = stage + t * kLayout.pitch + ((tile0 + kt) * 16 + ((lane >> 3) & 1) * 8) * 2;
+                uint32_t sh[4], sl[4], hi[4], lo[4];
+                split_pair(state[2 * kt][0], state[2 * kt][1], sh[0], sl[0]);
+                split_pair(state[2 * kt][2], state[2 * kt][3], sh[1], sl[1]);
+                split_pair(state[2 * kt + 1][0], state[2 * kt + 1][1], sh[2], sl[2]);
+                split_pair(state[2 * kt + 1][2], state[2 * kt + 1][3], sh[3], sl[3]);
+                ldmatrix_x4(at + kLayout.w, hi[0], hi[1], hi[2], hi[3]);
+                ldmatrix_x4(at + kLayout.w + kHalf, lo[0], lo[1], lo[2], lo[3]);
 #pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                mma_m16n8k16<__nv_bfloat16>(u[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(u_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(u_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+                for (int n = 0; n < 2; ++n) {
+                    mma_m16n8k16<__nv_bfloat16>(u[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
+                    mma_m16n8k16<__nv_bfloat16>(u_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+                    mma_m16n8k16<__nv_bfloat16>(u_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+                }
+                ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
+                ldmatrix_x4(at + kHalf, lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+                for (int n = 0; n < 2; ++n) {
+                    mma_m16n8k16<__nv_bfloat16>(o[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
+                    mma_m16n8k16<__nv_bfloat16>(o_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
+                    mma_m16n8k16<__nv_bfloat16>(o_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+                }
             }
-            ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
-            ldmatrix_x4(at + kHalf, lo[0], lo[1], lo[2], lo[3]);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                mma_m16n8k16<__nv_bfloat16>(o[n], sh[0], sh[1], sh[2], sh[3], hi[2 * n], hi[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(o_low[n], sh[0], sh[1], sh[2], sh[3], lo[2 * n], lo[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(o_low[n], sl[0], sl[1], sl[2], sl[3], hi[2 * n], hi[2 * n + 1]);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    o[n][i] += o_low[n][i];
+                    u[n][i] += u_low[n][i];
+                }
+            }
+        }
+        if (KS > 1) {
+            float4 *mine = sums + warp * 128 + lane;
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mine[n * 32] = make_float4(u[n][0], u[n][1], u[n][2], u[n][3]);
+                mine[(2 + n) * 32] = make_float4(o[n][0], o[n][1], o[n][2], o[n][3]);
+            }
+            __syncthreads();
+            const float4 *all = sums + (warp - share) * 128 + lane;
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) u[n][i] = o[n][i] = 0.0f;
+#pragma unroll
+                for (int other = 0; other < KS; ++other) {
+                    const float4 x = all[other * 128 + n * 32];
+                    u[n][0] += x.x;
+                    u[n][1] += x.y;
+                    u[n][2] += x.z;
+                    u[n][3] += x.w;
+                    if (share == 0) {
+                        const float4 y = all[other * 128 + (2 + n) * 32];
+                        o[n][0] += y.x;
+                        o[n][1] += y.y;
+                        o[n][2] += y.z;
+                        o[n][3] += y.w;
+                    }
+                }
             }
         }
         // ---- u^T = v^T T^T - S^T W^T ----
@@ -456,21 +500,21 @@ __global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kern
                 mma_m16n8k16<__nv_bfloat16>(direct, value[0], value[1], value[2], value[3], hi[2 * n], hi[2 * n + 1]);
                 mma_m16n8k16<__nv_bfloat16>(direct, value[0], value[1], value[2], value[3], lo[2 * n], lo[2 * n + 1]);
 #pragma unroll
-                for (int i = 0; i < 4; ++i) u[n][i] = direct[i] - (u[n][i] + u_low[n][i]);
+                for (int i = 0; i < 4; ++i) u[n][i] = direct[i] - u[n][i];
                 split_pair(u[n][0], u[n][1], uh[2 * n], ul[2 * n]);
                 split_pair(u[n][2], u[n][3], uh[2 * n + 1], ul[2 * n + 1]);
             }
         }
         // ---- S^T = S^T exp(A) + u^T (k exp(A - a)) ----
 #pragma unroll
-        for (int kt = 0; kt < KT; ++kt) {
-            const uint32_t at = stage + kLayout.k + (lane & 15) * kLayout.pitch + (kt * 16 + (lane >> 4) * 8) * 2;
+        for (int kt = 0; kt < kTiles; ++kt) {
+            const uint32_t at = stage + kLayout.k + (lane & 15) * kLayout.pitch + ((tile0 + kt) * 16 + (lane >> 4) * 8) * 2;
             uint32_t hi[4], lo[4];
             ldmatrix_x4_trans(at, hi[0], hi[1], hi[2], hi[3]);
             ldmatrix_x4_trans(at + kHalf, lo[0], lo[1], lo[2], lo[3]);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
-                const float2 d = *reinterpret_cast<const float2 *>(here + kLayout.decay + (kt * 16 + n * 8 + q2) * 4);
+                const float2 d = *reinterpret_cast<const float2 *>(here + kLayout.decay + ((tile0 + kt) * 16 + n * 8 + q2) * 4);
                 float(&x)[4] = state[2 * kt + n];
                 x[0] *= d.x;
                 x[1] *= d.y;
@@ -481,29 +525,24 @@ __global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kern
                 mma_m16n8k16<__nv_bfloat16>(x, ul[0], ul[1], ul[2], ul[3], hi[2 * n], hi[2 * n + 1]);
             }
         }
-        // ---- o^T += u^T P^T, out through shared memory ----
-        {
+        // ---- o^T += u^T P^T; eight lanes hold eight adjacent values of a token ----
+        if (share == 0) {
             const uint32_t at = stage + kLayout.p + t * kPitchP + ((lane >> 3) & 1) * 16;
             uint32_t hi[4], lo[4];
             ldmatrix_x4(at, hi[0], hi[1], hi[2], hi[3]);
             ldmatrix_x4(at + kBlock * kPitchP, lo[0], lo[1], lo[2], lo[3]);
+            float *target = p.attended + static_cast<size_t>(row0) * p.heads * p.vdim + head * p.vdim + slice0 + value0;
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 mma_m16n8k16<__nv_bfloat16>(o[n], uh[0], uh[1], uh[2], uh[3], hi[2 * n], hi[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(o_low[n], uh[0], uh[1], uh[2], uh[3], lo[2 * n], lo[2 * n + 1]);
-                mma_m16n8k16<__nv_bfloat16>(o_low[n], ul[0], ul[1], ul[2], ul[3], hi[2 * n], hi[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o[n], uh[0], uh[1], uh[2], uh[3], lo[2 * n], lo[2 * n + 1]);
+                mma_m16n8k16<__nv_bfloat16>(o[n], ul[0], ul[1], ul[2], ul[3], hi[2 * n], hi[2 * n + 1]);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
-                    outputs[(n * 8 + q2 + (i & 1)) * pitch_o + value0 + g + (i >> 1) * 8] = o[n][i] + o_low[n][i];
+                    const int token = n * 8 + q2 + (i & 1), v = g + (i >> 1) * 8;
+                    if (token < tokens && slice0 + value0 + v < p.vdim) target[static_cast<size_t>(token) * p.heads * p.vdim + v] = o[n][i];
                 }
             }
-        }
-        __syncthreads();
-        const int pieces = width / 4;
-        for (int i = tid; i < tokens * pieces; i += blockDim.x) {
-            const int token = i / pieces, piece = i - token * pieces;
-            *reinterpret_cast<float4 *>(p.attended + static_cast<size_t>(row0 + token) * p.heads * p.vdim + head * p.vdim + slice0 +
-                                        piece * 4) = *reinterpret_cast<const float4 *>(outputs + token * pitch_o + piece * 4);
         }
     }
     if (failed) {
@@ -512,58 +551,91 @@ __global__ void __launch_bounds__(256, KT <= 8 ? 2 : 1) gated_delta_advance_kern
         return;
     }
 #pragma unroll
-    for (int n = 0; n < 2 * KT; ++n) {
+    for (int n = 0; n < 2 * kTiles; ++n) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const int v = slice0 + value0 + g + (i >> 1) * 8, k = n * 8 + q2 + (i & 1);
+            const int v = slice0 + value0 + g + (i >> 1) * 8, k = tile0 * 16 + n * 8 + q2 + (i & 1);
             if (v < p.vdim && k < p.dim) home[static_cast<size_t>(k) * p.vdim + v] = state[n][i];
         }
     }
 }
 
-// One warp per (token, head): out = rms_norm(o) * weight * sigmoid(gate).
+// One warp per (token, head), four in turn: out = rms_norm(o) * weight * sigmoid(gate).  HELD: a head's values are at most one pack a
+// lane, and everything is asked for before the sums.
+template <bool HELD>
 __global__ void __launch_bounds__(256) gated_delta_finish_kernel(const DeltaParams p) {
     grid_launch_dependents();
     grid_dependency_wait();
+    constexpr int kTurns = 4;
     const int block = blockIdx.x;
     const int row0 = p.block_row[block], tokens = p.block_tokens[block];
-    const int lane = threadIdx.x & 31, packs = p.vdim / 4;
-    for (int item = blockIdx.y * 8 + (threadIdx.x >> 5); item < tokens * p.heads; item += gridDim.y * 8) {
-        const int token = item / p.heads, head = item - token * p.heads;
-        const size_t row = row0 + token;
-        const float *o = p.attended + row * p.heads * p.vdim + head * p.vdim;
-        float square = 0.0f;
-        for (int i = lane; i < packs; i += 32) {
-            const Pack<4> x = load_pack<4>(o + i * 4);
+    const int lane = threadIdx.x & 31, packs = p.vdim / 4, items = tokens * p.heads;
+    const float inverse_vdim = 1.0f / static_cast<float>(p.vdim);
+    auto store = [&](Pack<4> x, const Pack<4> &gate, const Pack<4> &weight, float scale, __nv_bfloat16 *out) {
 #pragma unroll
-            for (int j = 0; j < 4; ++j) square = square_chain(square, x.v[j]);
-        }
-        const float scale = 1.0f / sqrtf(warp_sum(square) / static_cast<float>(p.vdim) + p.eps);
-        const __nv_bfloat16 *gates = p.decay + row * p.decay_stride + p.gate_at + head * p.vdim;
-        __nv_bfloat16 *out = p.out + row * p.out_stride + head * p.vdim;
-        for (int i = lane; i < packs; i += 32) {
-            Pack<4> x = load_pack<4>(o + i * 4);
-            const Pack<4> gate = load_pack<4>(gates + i * 4), weight = load_pack<4>(p.norm_weight + i * 4);
+        for (int j = 0; j < 4; ++j) x.v[j] = x.v[j] * scale * weight.v[j] * __fdividef(1.0f, 1.0f + __expf(-gate.v[j]));
+        store_pack<4>(out, x);
+    };
+    Pack<4> held_weight = {};
+    if (HELD && lane < packs) held_weight = load_pack<4>(p.norm_weight + lane * 4);
+    for (int item0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * kTurns; item0 < items; item0 += gridDim.y * 8 * kTurns) {
+        if (HELD) {
+            Pack<4> x[kTurns], gate[kTurns];
+            __nv_bfloat16 *out[kTurns];
 #pragma unroll
-            for (int j = 0; j < 4; ++j) x.v[j] = x.v[j] * scale * weight.v[j] * __fdividef(1.0f, 1.0f + __expf(-gate.v[j]));
-            store_pack<4>(out + i * 4, x);
+            for (int turn = 0; turn < kTurns; ++turn) {
+                const int item = item0 + turn, token = item / p.heads, head = item - token * p.heads;
+                const size_t row = row0 + token;
+                x[turn] = {};
+                out[turn] = p.out + row * p.out_stride + head * p.vdim + lane * 4;
+                if (item < items && lane < packs) {
+                    x[turn] = load_pack<4>(p.attended + row * p.heads * p.vdim + head * p.vdim + lane * 4);
+                    gate[turn] = load_pack<4>(p.decay + row * p.decay_stride + p.gate_at + head * p.vdim + lane * 4);
+                }
+            }
+#pragma unroll
+            for (int turn = 0; turn < kTurns; ++turn) {
+                float square = 0.0f;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) square = square_chain(square, x[turn].v[j]);
+                const float scale = 1.0f / sqrtf(warp_sum(square) * inverse_vdim + p.eps);
+                if (item0 + turn < items && lane < packs) store(x[turn], gate[turn], held_weight, scale, out[turn]);
+            }
+        } else {
+            for (int item = item0; item < min(item0 + kTurns, items); ++item) {
+                const int token = item / p.heads, head = item - token * p.heads;
+                const size_t row = row0 + token;
+                const float *o = p.attended + row * p.heads * p.vdim + head * p.vdim;
+                float square = 0.0f;
+                for (int i = lane; i < packs; i += 32) {
+                    const Pack<4> x = load_pack<4>(o + i * 4);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) square = square_chain(square, x.v[j]);
+                }
+                const float scale = 1.0f / sqrtf(warp_sum(square) * inverse_vdim + p.eps);
+                for (int i = lane; i < packs; i += 32) {
+                    store(load_pack<4>(o + i * 4), load_pack<4>(p.decay + row * p.decay_stride + p.gate_at + head * p.vdim + i * 4),
+                          load_pack<4>(p.norm_weight + i * 4), scale, p.out + row * p.out_stride + head * p.vdim + i * 4);
+                }
+            }
         }
     }
 }
 
-template <int KT>
+template <int KT, int KS>
 int launch_advance(cudaStream_t stream, const CUtensorMap &value_map, DeltaParams p, size_t runs) {
+    const int threads = p.slice * 2 * KS;
     const auto bytes_of = [&](int stages) {
-        return stages * delta_stage_bytes(KT * 16, p.slice) + kBlock * (p.slice + 4) * 4 + kMaxStages * 8 + 1024;
+        return stages * delta_stage_bytes(KT * 16, p.slice) + (KS > 1 ? threads * 64 : 0) + kMaxStages * 8 + 1024;
     };
     p.stages = kMaxStages;  // as many as leave room for a second CTA, three at least
     while (p.stages > 3 && bytes_of(p.stages) > 112 * 1024) --p.stages;
     if (bytes_of(p.stages) > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
     static int configured[kMaxDevices] = {0};
-    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_advance_kernel<KT>, bytes_of(p.stages), configured));
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_advance_kernel<KT, KS>, bytes_of(p.stages), configured));
     const dim3 grid(static_cast<unsigned>(runs), static_cast<unsigned>(p.heads),
                     static_cast<unsigned>((p.vdim + p.slice - 1) / p.slice));
-    SINGE_CUDA_TRY(launch_dependent(gated_delta_advance_kernel<KT>, grid, dim3(p.slice * 2), bytes_of(p.stages), stream, kLaunchGlue,
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_advance_kernel<KT, KS>, grid, dim3(threads), bytes_of(p.stages), stream, kLaunchGlue,
                                     1, value_map, p));
     return launch_status();
 }
@@ -576,11 +648,15 @@ int delta_dim_pad(size_t dim, size_t vdim) {
     return pad;
 }
 
-// Value columns of a CTA: all of a head's up to 128, fewer while (run, head, slice) triples leave SMs idle.
-int delta_slice(size_t runs, size_t heads, size_t vdim) {
+// Value columns of a CTA: all of a head's up to 128, fewer while (run, head, slice) triples leave SMs idle.  `shared_keys`: so few
+// that the key tiles are shared out among four warps as well.
+int delta_slice(size_t runs, size_t heads, size_t vdim, int dim_pad, bool &shared_keys) {
+    const size_t sms = static_cast<size_t>(device_sm_count());
+    shared_keys = dim_pad >= 64 && runs * heads * ((vdim + 15) / 16) < 4 * sms;
+    if (shared_keys) return vdim > 16 ? 32 : 16;
     int slice = 16;
     while (slice < 128 && static_cast<size_t>(slice) < vdim) slice *= 2;
-    while (slice > 16 && runs * heads * ((vdim + slice - 1) / slice) < static_cast<size_t>(device_sm_count())) slice /= 2;
+    while (slice > 16 && runs * heads * ((vdim + slice - 1) / slice) < sms) slice /= 2;
     return slice;
 }
 
@@ -632,7 +708,8 @@ int singe_gated_delta_prompt_bf16(singe_stream_t stream, void *out, size_t out_s
     p.value_at = static_cast<int>(value_at);
     p.gate_at = static_cast<int>(gate_at);
     p.dim_pad = dim_pad;
-    p.slice = delta_slice(run_count, heads, vdim);
+    bool shared_keys = false;
+    p.slice = delta_slice(run_count, heads, vdim, dim_pad, shared_keys);
     p.out = static_cast<__nv_bfloat16 *>(out);
     p.out_stride = static_cast<long long>(out_stride);
     p.mixed = static_cast<const __nv_bfloat16 *>(mixed);
@@ -656,12 +733,10 @@ int singe_gated_delta_prompt_bf16(singe_stream_t stream, void *out, size_t out_s
     p.eps = eps;
     p.error = device_error_word();
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    const int shared = kPrepareWarps * prepare_bytes(dim_pad);
     static int configured[kMaxDevices] = {0};
-    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_prepare_kernel, shared, configured));
-    SINGE_CUDA_TRY(launch_dependent(gated_delta_prepare_kernel,
-                                    dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((heads + kPrepareWarps - 1) / kPrepareWarps)),
-                                    dim3(kPrepareWarps * 32), shared, s, kLaunchGlue, 1, p));
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_prepare_kernel, prepare_bytes(dim_pad), configured));
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_prepare_kernel, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>(heads)),
+                                    dim3(dim_pad < 32 ? 32 : dim_pad), prepare_bytes(dim_pad), s, kLaunchGlue, 1, p));
     CUtensorMap value_map;
     {
         const uint64_t dims[2] = {value_at + heads * vdim, rows};
@@ -671,16 +746,21 @@ int singe_gated_delta_prompt_bf16(singe_stream_t stream, void *out, size_t out_s
                                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B));
     }
     int launched = SINGE_ERR_UNSUPPORTED_CONFIGURATION;
-    if (dim_pad == 16) launched = launch_advance<1>(s, value_map, p, run_count);
-    if (dim_pad == 32) launched = launch_advance<2>(s, value_map, p, run_count);
-    if (dim_pad == 64) launched = launch_advance<4>(s, value_map, p, run_count);
-    if (dim_pad == 128) launched = launch_advance<8>(s, value_map, p, run_count);
-    if (dim_pad == 256) launched = launch_advance<16>(s, value_map, p, run_count);
+    if (dim_pad == 16) launched = launch_advance<1, 1>(s, value_map, p, run_count);
+    if (dim_pad == 32) launched = launch_advance<2, 1>(s, value_map, p, run_count);
+    if (dim_pad == 64) {
+        launched = shared_keys ? launch_advance<4, 4>(s, value_map, p, run_count) : launch_advance<4, 1>(s, value_map, p, run_count);
+    }
+    if (dim_pad == 128) {
+        launched = shared_keys ? launch_advance<8, 4>(s, value_map, p, run_count) : launch_advance<8, 1>(s, value_map, p, run_count);
+    }
+    if (dim_pad == 256) {
+        launched = shared_keys ? launch_advance<16, 4>(s, value_map, p, run_count) : launch_advance<16, 1>(s, value_map, p, run_count);
+    }
     SINGE_TRY(launched);
-    const size_t items = kBlock * heads;
-    const unsigned groups = static_cast<unsigned>(items > 256 ? (items + 255) / 256 : 1);  // 32 (token, head) pairs a warp
-    SINGE_CUDA_TRY(launch_dependent(gated_delta_finish_kernel, dim3(static_cast<unsigned>(blocks), groups), dim3(256), 0, s,
-                                    kLaunchGlue, 1, p));
+    const unsigned groups = static_cast<unsigned>((heads * kBlock + 127) / 128);  // four (token, head) pairs, four times, a warp
+    SINGE_CUDA_TRY(launch_dependent(vdim <= 128 ? gated_delta_finish_kernel<true> : gated_delta_finish_kernel<false>,
+                                    dim3(static_cast<unsigned>(blocks), groups), dim3(256), 0, s, kLaunchGlue, 1, p));
     return launch_status();
 }
 

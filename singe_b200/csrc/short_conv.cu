@@ -10,7 +10,7 @@
 // A step's rows: token t belongs to sequence sequence_of[t], which owns rows [first, first + fresh) and had `context` tokens
 // before.  A sequence with fresh == 0 has one idle row: nothing is kept of it.  Sequences with one new token have their state
 // brought up to date by the same threads that read it; for the others the state kernel follows.
-// One CTA per token; arithmetic is f32.
+// Arithmetic is f32.
 #include "row_pack.cuh"
 
 namespace singe {
@@ -257,6 +257,285 @@ __global__ void __launch_bounds__(kConvThreads) conv_state_kernel(const ConvRows
     }
 }
 
+// ---- bf16 in packs of eight columns: what the sizes of real models take ----
+//
+// A thread owns eight adjacent columns and walks `tile` neighbouring tokens with the taps' rows in registers, so that a row is
+// read once however many taps there are.
+
+constexpr int kWideTaps = 4;
+constexpr int kTileTokens = 8;
+
+struct Eight {
+    float v[8];
+};
+
+__device__ __forceinline__ Eight widen(const uint4 &raw) {
+    Eight x;
+    const uint32_t words[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        x.v[2 * i] = __uint_as_float(words[i] << 16);
+        x.v[2 * i + 1] = __uint_as_float(words[i] & 0xffff0000u);
+    }
+    return x;
+}
+
+__device__ __forceinline__ uint4 narrow(const Eight &x) {
+    return make_uint4(pack2<__nv_bfloat16>(x.v[0], x.v[1]), pack2<__nv_bfloat16>(x.v[2], x.v[3]), pack2<__nv_bfloat16>(x.v[4], x.v[5]),
+                      pack2<__nv_bfloat16>(x.v[6], x.v[7]));
+}
+
+__device__ __forceinline__ uint4 load_eight(const void *base, long long element) {
+    return *reinterpret_cast<const uint4 *>(static_cast<const __nv_bfloat16 *>(base) + element);
+}
+
+// The convolution's moving window over one thread's columns.
+template <int N>
+struct TapWindow {
+    uint4 taps[N], bias;
+    uint4 past[N > 1 ? N - 1 : 1];  // past[j]: the row j + 1 tokens back
+    bool there[N > 1 ? N - 1 : 1];  // false: before the sequence's start
+    bool biased, follows;           // follows: the window stands just before the next token of its sequence
+
+    __device__ __forceinline__ void start(const ConvRows &p, int c) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) taps[j] = load_eight(p.taps, static_cast<long long>(j) * p.span + c);
+        biased = p.bias != nullptr;
+        bias = biased ? load_eight(p.bias, c) : make_uint4(0u, 0u, 0u, 0u);
+        follows = false;
+    }
+
+    // The convolution at `token`, a sequence's new token number `at`; moves the window on, and with `shift` the sequence's state.
+    __device__ __forceinline__ Eight step(const ConvRows &p, int c, int token, int sequence, int at, int context, bool shift) {
+        __nv_bfloat16 *state = static_cast<__nv_bfloat16 *>(p.state) + static_cast<size_t>(sequence) * (N - 1) * p.span + c;
+        if (!follows || at == 0) {
+#pragma unroll
+            for (int j = 0; j < N - 1; ++j) {
+                const int from = at - 1 - j;
+                there[j] = context + from >= 0;
+                past[j] = make_uint4(0u, 0u, 0u, 0u);
+                if (from >= 0) {
+                    past[j] = load_eight(p.projected, (token - 1 - j) * p.stride + c);
+                } else if (there[j]) {
+                    past[j] = *reinterpret_cast<const uint4 *>(state + static_cast<size_t>(N - 1 + from) * p.span);
+                }
+            }
+        }
+        const uint4 now = load_eight(p.projected, token * p.stride + c);
+        const Eight b = widen(bias);
+        Eight y;
+        {
+            const Eight x = widen(now), w = widen(taps[N - 1]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y.v[i] = w.v[i] * (x.v[i] + b.v[i]);
+        }
+#pragma unroll
+        for (int j = 0; j < N - 1; ++j) {
+            if (!there[j]) continue;
+            const Eight x = widen(past[j]), w = widen(taps[N - 2 - j]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y.v[i] = fmaf(w.v[i], x.v[i] + b.v[i], y.v[i]);
+        }
+        if (shift) {
+#pragma unroll
+            for (int j = 0; j < N - 1; ++j) {
+                uint4 *slot = reinterpret_cast<uint4 *>(state + static_cast<size_t>(N - 2 - j) * p.span);
+                if (j == 0) {
+                    *slot = now;
+                } else if (there[j - 1]) {
+                    *slot = past[j - 1];
+                }
+            }
+        }
+#pragma unroll
+        for (int j = N - 2; j > 0; --j) {
+            past[j] = past[j - 1];
+            there[j] = there[j - 1];
+        }
+        if (N > 1) {
+            past[0] = now;
+            there[0] = true;
+        }
+        follows = true;
+        return y;
+    }
+};
+
+// One thread per eight columns of the whole row, so that the norms over all queries and keys meet in the CTA.
+template <int N>
+__global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const AttentionInputs p, int rows, int tile) {
+    using T = __nv_bfloat16;
+    grid_launch_dependents();
+    __shared__ float2 scratch[32];
+    extern __shared__ float2 turns[];  // [tile][pairs]: cosine, sine
+    const int c = threadIdx.x * 8, warps = (blockDim.x + 31) >> 5;
+    const int token0 = blockIdx.x * tile;
+    const bool live = c < p.rows.span;
+    TapWindow<N> window;
+    if (live) window.start(p.rows, c);  // weights: they do not wait for the kernel before
+    grid_dependency_wait();
+    for (int i = threadIdx.x; i < tile * p.pairs; i += blockDim.x) {
+        const int token = token0 + i / p.pairs;
+        if (token >= rows) break;
+        // the angle modulo a turn in double, so that far positions keep the precision of near ones
+        const double angle = static_cast<double>(p.positions[token]) * p.frequencies[i % p.pairs];
+        float sine, cosine;
+        sincosf(static_cast<float>(angle - 6.283185307179586 * rint(angle * 0.15915494309189535)), &sine, &cosine);
+        turns[i] = make_float2(cosine * p.rotation_scale, sine * p.rotation_scale);
+    }
+    const int queries = p.heads * p.dim, keys = p.kv_heads * p.dim;
+    const bool is_query = c < queries, is_key = c >= p.key_at && c < p.key_at + keys;
+    const bool is_value = live && c >= p.value_at;
+    // where the columns go within a head-padded row
+    const int within = is_query ? c : is_key ? c - p.key_at : c - p.value_at;
+    const int head_dim = is_value ? p.vdim : p.dim, size = is_value ? p.value_size : p.key_size;
+    const int head = within / head_dim, d = within - head * head_dim;
+    const int target = head * size + d;
+    Eight gain = {};
+    if (is_query) gain = widen(load_eight(p.query_norm, within));
+    if (is_key) gain = widen(load_eight(p.key_norm, within));
+    const bool normed = is_query || is_key;
+    const size_t key_width = static_cast<size_t>(p.kv_heads) * p.key_size, value_width = static_cast<size_t>(p.kv_heads) * p.value_size;
+    for (int i = 0; i < tile && token0 + i < rows; ++i) {
+        const int token = token0 + i;
+        const int sequence = p.rows.sequence_of[token];
+        T *query = static_cast<T *>(p.query) + token * p.query_stride;
+        const int fresh = sequence >= 0 && sequence < p.rows.sequences ? p.rows.fresh[sequence] : 0;
+        if (fresh <= 0) {
+            for (int at = c; at < p.heads * p.key_size; at += blockDim.x * 8) {
+                *reinterpret_cast<uint4 *>(query + at) = make_uint4(0u, 0u, 0u, 0u);
+            }
+            window.follows = false;
+            continue;
+        }
+        Eight y = {};
+        if (live) y = window.step(p.rows, c, token, sequence, token - p.rows.first[sequence], p.rows.context[sequence], fresh == 1);
+        float square = 0.0f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) square = square_chain(square, y.v[e]);
+        // sums of the queries' and of the keys' squares
+        const float own_q = warp_sum(is_query ? square : 0.0f), own_k = warp_sum(is_key ? square : 0.0f);
+        __syncthreads();  // the sums before have been read (and, the first time, the turns are there)
+        if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = make_float2(own_q, own_k);
+        __syncthreads();
+        float total_q = 0.0f, total_k = 0.0f;
+        for (int w = 0; w < warps; ++w) {
+            total_q += scratch[w].x;
+            total_k += scratch[w].y;
+        }
+        const float scale = is_query ? 1.0f / sqrtf(total_q / static_cast<float>(queries) + p.eps)
+                                     : 1.0f / sqrtf(total_k / static_cast<float>(keys) + p.eps);
+        if (normed) {
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) {
+                float u = y.v[e] * scale * gain.v[e], v = y.v[e + 1] * scale * gain.v[e + 1];
+                const int pair = (d + e) >> 1;
+                if (pair < p.pairs) {
+                    const float2 turn = turns[i * p.pairs + pair];
+                    const float turned = fmaf(u, turn.x, -(v * turn.y));
+                    v = fmaf(v, turn.x, u * turn.y);
+                    u = turned;
+                }
+                y.v[e] = u;
+                y.v[e + 1] = v;
+            }
+        }
+        const uint4 out = narrow(y);
+        long long page = p.write_pages[token], slot = p.write_slots[token];
+        if (page < 0) page += p.pages;
+        if (slot < 0) slot += p.page_size;
+        const bool inside = page >= 0 && page < p.pages && slot >= 0 && slot < p.page_size;
+        if (!inside && threadIdx.x == 0) report_status(p.status, kStatusIndexOutOfBounds);
+        const bool keep = inside && (p.cached == nullptr || p.cached[token] != 0);
+        const long long packed = p.packed_rows == nullptr ? -1 : p.packed_rows[token];
+        const bool pack = packed >= 0 && packed < p.packed_count;
+        const size_t cell = keep ? static_cast<size_t>(page * p.page_size + slot) : 0;
+        T *cached_keys = static_cast<T *>(p.key_cache) + cell * key_width, *cached_values = static_cast<T *>(p.value_cache) + cell * value_width;
+        T *packed_keys = static_cast<T *>(p.packed_keys) + (pack ? packed : 0) * key_width;
+        T *packed_values = static_cast<T *>(p.packed_values) + (pack ? packed : 0) * value_width;
+        if (is_query) *reinterpret_cast<uint4 *>(query + target) = out;
+        if (keep && is_key) *reinterpret_cast<uint4 *>(cached_keys + target) = out;
+        if (keep && is_value) *reinterpret_cast<uint4 *>(cached_values + target) = out;
+        if (pack && is_key) *reinterpret_cast<uint4 *>(packed_keys + target) = out;
+        if (pack && is_value) *reinterpret_cast<uint4 *>(packed_values + target) = out;
+        // heads narrower than their rows: the rest is zero
+        const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+        const int key_rest = (p.key_size - p.dim) / 8, value_rest = (p.value_size - p.vdim) / 8;
+        for (int at = threadIdx.x; at < (p.heads + p.kv_heads) * key_rest; at += blockDim.x) {
+            const int h = at / key_rest, rest = p.dim + (at - h * key_rest) * 8;
+            if (h < p.heads) {
+                *reinterpret_cast<uint4 *>(query + h * p.key_size + rest) = zero;
+            } else {
+                const int place = (h - p.heads) * p.key_size + rest;
+                if (keep) *reinterpret_cast<uint4 *>(cached_keys + place) = zero;
+                if (pack) *reinterpret_cast<uint4 *>(packed_keys + place) = zero;
+            }
+        }
+        for (int at = threadIdx.x; at < p.kv_heads * value_rest; at += blockDim.x) {
+            const int h = at / value_rest, place = h * p.value_size + p.vdim + (at - h * value_rest) * 8;
+            if (keep) *reinterpret_cast<uint4 *>(cached_values + place) = zero;
+            if (pack) *reinterpret_cast<uint4 *>(packed_values + place) = zero;
+        }
+    }
+}
+
+// blockIdx.y takes a slice of the columns; the lanes of a head are neighbours, a power of two of them.
+template <int N>
+__global__ void __launch_bounds__(kConvThreads) recurrence_inputs_wide_kernel(const RecurrenceInputs p, int rows, int tile) {
+    grid_launch_dependents();
+    const int c = (blockIdx.y * kConvThreads + threadIdx.x) * 8;
+    const int token0 = blockIdx.x * tile;
+    const bool live = c < p.rows.span;
+    TapWindow<N> window;
+    if (live) window.start(p.rows, c);
+    grid_dependency_wait();
+    const int units = p.unit_heads * p.dim, lanes = p.dim / 8;
+    const bool first = c < units, second = c >= p.second_at && c < p.second_at + units;
+    const int unit = first ? c / p.dim : p.unit_heads + (c - p.second_at) / p.dim;
+    for (int i = 0; i < tile && token0 + i < rows; ++i) {
+        const int token = token0 + i;
+        const int sequence = p.rows.sequence_of[token];
+        const int fresh = sequence >= 0 && sequence < p.rows.sequences ? p.rows.fresh[sequence] : 0;
+        uint4 out = make_uint4(0u, 0u, 0u, 0u);
+        float square = 0.0f;
+        if (fresh <= 0) {
+            window.follows = false;
+        } else if (live) {
+            Eight y = window.step(p.rows, c, token, sequence, token - p.rows.first[sequence], p.rows.context[sequence], fresh == 1);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y.v[e] = __fdividef(y.v[e], 1.0f + __expf(-y.v[e]));
+            out = narrow(y);
+            const Eight kept = widen(out);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) square = square_chain(square, kept.v[e]);
+        }
+        if (live) *reinterpret_cast<uint4 *>(static_cast<__nv_bfloat16 *>(p.mixed) + token * p.mixed_stride + c) = out;
+        for (int offset = lanes >> 1; offset > 0; offset >>= 1) square += __shfl_xor_sync(0xffffffffu, square, offset);
+        if ((first || second) && fresh > 0 && (threadIdx.x & (lanes - 1)) == 0) {
+            p.inverse[static_cast<size_t>(token) * 2 * p.unit_heads + unit] = 1.0f / sqrtf(square + p.eps);
+        }
+    }
+}
+
+// Tokens of a tile: one where there are few rows (a decode batch), else enough to read each row once.
+int conv_tile(size_t rows, size_t slices) { return rows * slices >= 4 * static_cast<size_t>(device_sm_count()) * kTileTokens ? kTileTokens : 1; }
+
+bool conv_eights(const ConvRows &p) {
+    return p.count <= kWideTaps && p.span % 8 == 0 && p.stride % 8 == 0 && aligned_to(p.projected, 16) && aligned_to(p.bias, 16) &&
+           aligned_to(p.taps, 16) && aligned_to(p.state, 16);
+}
+
+#define SINGE_WIDE_CONV(KERNEL, GRID, THREADS, SHARED)                                                                     \
+    do {                                                                                                                   \
+        auto kernel = KERNEL<1>;                                                                                           \
+        if (p.rows.count == 2) kernel = KERNEL<2>;                                                                         \
+        if (p.rows.count == 3) kernel = KERNEL<3>;                                                                         \
+        if (p.rows.count == 4) kernel = KERNEL<4>;                                                                         \
+        SINGE_CUDA_TRY(launch_dependent(kernel, GRID, dim3(THREADS), SHARED, static_cast<cudaStream_t>(stream), kLaunchGlue, 1, p, \
+                                        static_cast<int>(rows), tile));                                                    \
+        return launch_status();                                                                                            \
+    } while (0)
+
 int validate(const ConvRows &p, size_t rows) {
     if (rows == 0 || p.span <= 0 || p.count <= 0 || p.sequences <= 0 || p.stride < p.span) return SINGE_ERR_INVALID_LENGTH;
     if (p.count > kMaxTaps) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
@@ -309,6 +588,16 @@ int attention_inputs(singe_stream_t stream, const AttentionInputs &p, size_t row
         (p.packed_rows != nullptr && (p.packed_keys == nullptr || p.packed_values == nullptr))) {
         return SINGE_ERR_NULL_POINTER;
     }
+    if (sizeof(T) == 2 && conv_eights(p.rows) && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.key_at % 8 == 0 && p.value_at % 8 == 0 &&
+        p.key_size % 8 == 0 && p.value_size % 8 == 0 && p.query_stride % 8 == 0 && p.rows.span <= 8192 && p.pairs <= 256 &&
+        p.key_at == p.heads * p.dim && p.value_at == p.key_at + p.kv_heads * p.dim && p.rows.span == p.value_at + p.kv_heads * p.vdim &&
+        aligned_to(p.query, 16) && aligned_to(p.key_cache, 16) && aligned_to(p.value_cache, 16) && aligned_to(p.packed_keys, 16) &&
+        aligned_to(p.packed_values, 16) && aligned_to(p.query_norm, 16) && aligned_to(p.key_norm, 16)) {
+        const int tile = conv_tile(rows, 1);
+        const unsigned threads = static_cast<unsigned>((p.rows.span / 8 + 31) / 32 * 32);
+        const dim3 grid(static_cast<unsigned>((rows + tile - 1) / tile));
+        SINGE_WIDE_CONV(attention_inputs_wide_kernel, grid, threads, static_cast<size_t>(tile) * p.pairs * sizeof(float2));
+    }
     const size_t bytes = 4 * sizeof(T);
     const bool out_wide = p.key_size % 4 == 0 && p.value_size % 4 == 0 && p.query_stride % 4 == 0 && aligned_to(p.query, bytes) &&
                           aligned_to(p.key_cache, bytes) && aligned_to(p.value_cache, bytes) &&
@@ -332,6 +621,14 @@ int recurrence_inputs(singe_stream_t stream, const RecurrenceInputs &p, size_t r
         return SINGE_ERR_INVALID_LENGTH;
     }
     if (p.mixed == nullptr || p.inverse == nullptr) return SINGE_ERR_NULL_POINTER;
+    const int lanes = p.dim / 8;
+    if (sizeof(T) == 2 && conv_eights(p.rows) && p.dim % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 &&
+        p.second_at == p.unit_heads * p.dim && p.mixed_stride % 8 == 0 && aligned_to(p.mixed, 16)) {
+        const size_t slices = (static_cast<size_t>(p.rows.span) / 8 + kConvThreads - 1) / kConvThreads;
+        const int tile = conv_tile(rows, slices);
+        const dim3 grid(static_cast<unsigned>((rows + tile - 1) / tile), static_cast<unsigned>(slices));
+        SINGE_WIDE_CONV(recurrence_inputs_wide_kernel, grid, kConvThreads, 0);
+    }
     const bool wide = conv_wide<T>(p.rows) && p.mixed_stride % 4 == 0 && aligned_to(p.mixed, 4 * sizeof(T));
     auto kernel = wide ? recurrence_inputs_kernel<T, 4> : recurrence_inputs_kernel<T, 1>;
     static int configured_wide[kMaxDevices] = {0}, configured[kMaxDevices] = {0};

@@ -113,6 +113,45 @@ def test_convolution_with_silu_and_unit_lengths_over_portions(dtype, taps, heads
             assert np.abs(unit - ref.unit(pieces)).max() < 1e-5
 
 
+@pytest.mark.parametrize("taps", [1, 3, 4])
+def test_convolution_over_a_long_ragged_prompt(taps):
+    """Enough rows for tiles of several tokens: sequences end and begin inside tiles, some idle, some continue."""
+    rng = np.random.default_rng(taps)
+    ops, heads, dim, rest = Ops("bfloat16"), 3, 32, 40
+    span = 2 * heads * dim + rest
+    fresh = [700, 0, 1, 2, 3, 5, 0, 0, 1500, 9, 1, 1, 3000]
+    context = [0, 5, 7, 0, 1, 2, 0, 9, 0, 4, 0, 1, 2]
+    counts = [max(n, 1) for n in fresh]
+    first, rows = np.cumsum([0] + counts)[:-1], sum(counts)
+    past = [draw(rng, min(c, taps - 1), span) for c in context]
+    projected, weight = draw(rng, rows, span), draw(rng, taps, span)
+    state = torch.full((len(fresh), taps - 1, span), float("nan"), dtype=ops.dtype, device="cuda")
+    for s, values in enumerate(past):
+        if len(values):
+            state[s, taps - 1 - len(values):] = dev(values).to(ops.dtype)
+    mixed, inverse = ops.rows(rows, span), torch.empty((rows, 2 * heads), device="cuda")
+    sequence_of = np.repeat(np.arange(len(fresh)), counts)
+    d_projected, d_taps, d_first, d_fresh = ops.weight(projected), dev(weight).to(ops.dtype), i32(first), i32(fresh)
+    ops.call("singe_conv_recurrence_inputs_bf16", stream(), mixed, mixed.stride(0), inverse, d_projected, d_projected.stride(0), d_taps, state,
+             i32(sequence_of), d_first, d_fresh, i32(context), rows, len(fresh), taps, heads, dim, heads * dim, span, 1e-6)
+    ops.call("singe_conv_state_bf16", stream(), d_projected, d_projected.stride(0), state, d_first, d_fresh, rows, len(fresh), taps, span)
+    got, lengths, after = host(mixed), host(inverse), host(state)
+    for s, n in enumerate(fresh):
+        if n == 0:
+            assert (got[first[s]] == 0).all()
+            continue
+        wide = np.concatenate([past[s], projected[first[s]: first[s] + n]])
+        expect = ref.silu(ref.causal_convolution(wide.astype(np.float64), weight.T.astype(np.float64)))[len(past[s]):]
+        part = got[first[s]: first[s] + n]
+        assert relative(part, expect) < LIMIT["bfloat16"], f"sequence {s}"
+        for place in range(2):
+            pieces = part[:, place * heads * dim: (place + 1) * heads * dim].reshape(n, heads, dim)
+            unit = pieces * lengths[first[s]: first[s] + n, place * heads: (place + 1) * heads, None]
+            assert np.abs(unit - ref.unit(pieces)).max() < 1e-5
+        kept = wide[max(len(wide) - taps + 1, 0):] if taps > 1 else wide[:0]
+        assert np.array_equal(after[s, taps - 1 - len(kept):], kept), f"state of sequence {s}"
+
+
 ROTATIONS = [{"dims": 16, "base": 10000.0}, {"dims": 24, "base": 500.0, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 1.0}},
              {"dims": 2, "base": 100.0, "scaling": {"factor": 1.0, "original": 4096, "fast": 32.0, "slow": 32.0}}]
 
@@ -351,10 +390,13 @@ def test_delta_rule_token_by_token(dtype, case):
             assert relative(after[s], end) < 1e-5
 
 
-@pytest.mark.parametrize("case", CASES)
-def test_delta_rule_block_by_block(case):
+@pytest.mark.parametrize("case,many", [(case, False) for case in CASES] + [(case, True) for case in CASES[2:7]])
+def test_delta_rule_block_by_block(case, many):
+    """``many``: enough sequences to fill the machine, so that a block's key tiles stay with one warp."""
     rng = np.random.default_rng(case[2] + case[3] + case[0])
     counts, contexts, eps = [16, 9, 1, 333, 15, 17, 600, 0], [0, 3, 7, 0, 0, 20, 5, 2], 1e-6
+    if many:
+        counts, contexts = [21] * 90 + [40], [0, 2, 0] * 30 + [5]
     delta = DeltaCase(rng, counts, *case)
     heads, kv_heads, dim, vdim = delta.sizes
     before = draw(rng, len(counts), heads, dim, vdim, exact16=False)
