@@ -354,6 +354,8 @@ __global__ void __launch_bounds__(256, KT / KS <= 8 ? 2 : 1) gated_delta_advance
     constexpr int kHalf = kBlock * kLayout.pitch;
     const int run = blockIdx.x, head = blockIdx.y, slice0 = blockIdx.z * p.slice;
     const int sequence = p.runs[3 * run], first_block = p.runs[3 * run + 1], blocks = p.runs[3 * run + 2];
+    // a run's rows are adjacent, and only its last block may be short
+    const int first_row = p.block_row[first_block], last_tokens = p.block_tokens[first_block + blocks - 1];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = lane >> 2, q2 = (lane & 3) * 2;
     const int share = warp % KS, tile0 = share * kTiles;  // this warp's key tiles
@@ -387,24 +389,23 @@ __global__ void __launch_bounds__(256, KT / KS <= 8 ? 2 : 1) gated_delta_advance
     const int boxes = (p.slice + 63) / 64;
     auto load_block = [&](int index) {
         if (warp != 0) return;
-        const int block = first_block + index;
         const uint32_t bar = bars + 8 * (index % stages);
         const uint32_t stage = smem_u32(advance_shared) + (index % stages) * stage_bytes;
         if (lane == 0) {
             mbar_expect_tx(bar, kLayout.bytes + boxes * kValueBox);
-            bulk_load(stage, p.operands + (static_cast<size_t>(block) * p.heads + head) * kLayout.bytes, kLayout.bytes, bar);
+            bulk_load(stage, p.operands + (static_cast<size_t>(first_block + index) * p.heads + head) * kLayout.bytes, kLayout.bytes, bar);
         }
         __syncwarp();
         if (lane < boxes) {
             tma_load_2d(stage + values_at + lane * kValueBox, &value_map, bar,
-                        p.value_at + head * p.vdim + slice0 + lane * 64, p.block_row[block]);
+                        p.value_at + head * p.vdim + slice0 + lane * 64, first_row + index * kBlock);
         }
     };
     for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
     bool failed = false;
 
     for (int index = 0; index < blocks; ++index) {
-        const int row0 = p.block_row[first_block + index], tokens = p.block_tokens[first_block + index];
+        const int row0 = first_row + index * kBlock, tokens = index + 1 < blocks ? kBlock : last_tokens;
         const bool arrived = mbar_wait(bars + 8 * (index % stages), (index / stages) & 1);
         fence_proxy_async_shared();
         // the block has arrived for every thread, and everyone is done with the stage loaded next and with the sums

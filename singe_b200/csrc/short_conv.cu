@@ -295,18 +295,22 @@ struct TapWindow {
     uint4 taps[N], bias;
     uint4 past[N > 1 ? N - 1 : 1];  // past[j]: the row j + 1 tokens back
     bool there[N > 1 ? N - 1 : 1];  // false: before the sequence's start
-    bool biased, follows;           // follows: the window stands just before the next token of its sequence
+    uint4 ahead;                    // the next row, on its way while this one is worked on
+    bool follows;                   // the window stands just before the next token of its sequence
 
     __device__ __forceinline__ void start(const ConvRows &p, int c) {
 #pragma unroll
         for (int j = 0; j < N; ++j) taps[j] = load_eight(p.taps, static_cast<long long>(j) * p.span + c);
-        biased = p.bias != nullptr;
-        bias = biased ? load_eight(p.bias, c) : make_uint4(0u, 0u, 0u, 0u);
+        bias = p.bias != nullptr ? load_eight(p.bias, c) : make_uint4(0u, 0u, 0u, 0u);
         follows = false;
     }
 
-    // The convolution at `token`, a sequence's new token number `at`; moves the window on, and with `shift` the sequence's state.
-    __device__ __forceinline__ Eight step(const ConvRows &p, int c, int token, int sequence, int at, int context, bool shift) {
+    __device__ __forceinline__ void fetch(const ConvRows &p, int c, int token) { ahead = load_eight(p.projected, token * p.stride + c); }
+
+    // The convolution at `token`, a sequence's new token number `at`, whose row is `now`; moves the window on, and with `shift` the
+    // sequence's state.
+    __device__ __forceinline__ Eight step(const ConvRows &p, int c, const uint4 &now, int token, int sequence, int at, int context,
+                                          bool shift) {
         __nv_bfloat16 *state = static_cast<__nv_bfloat16 *>(p.state) + static_cast<size_t>(sequence) * (N - 1) * p.span + c;
         if (!follows || at == 0) {
 #pragma unroll
@@ -321,7 +325,6 @@ struct TapWindow {
                 }
             }
         }
-        const uint4 now = load_eight(p.projected, token * p.stride + c);
         const Eight b = widen(bias);
         Eight y;
         {
@@ -361,19 +364,50 @@ struct TapWindow {
     }
 };
 
+// What a tile's tokens need to know, looked up once for all threads.
+struct TileToken {
+    int sequence, at, context, fresh;
+};
+
+__device__ __forceinline__ void look_up_tile(const ConvRows &p, TileToken *tokens, int token0, int tile, int rows) {
+    for (int i = threadIdx.x; i < tile && token0 + i < rows; i += blockDim.x) {
+        TileToken t = {p.sequence_of[token0 + i], 0, 0, 0};
+        if (t.sequence >= 0 && t.sequence < p.sequences) {
+            t.at = token0 + i - p.first[t.sequence];
+            t.context = p.context[t.sequence];
+            t.fresh = p.fresh[t.sequence];
+        }
+        tokens[i] = t;
+    }
+}
+
 // One thread per eight columns of the whole row, so that the norms over all queries and keys meet in the CTA.
-template <int N>
-__global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const AttentionInputs p, int rows, int tile) {
+template <int N, int THREADS>
+__global__ void __launch_bounds__(THREADS, THREADS <= 384 ? 2 : 1) attention_inputs_wide_kernel(const AttentionInputs p, int rows, int tile) {
     using T = __nv_bfloat16;
     grid_launch_dependents();
-    __shared__ float2 scratch[32];
-    extern __shared__ float2 turns[];  // [tile][pairs]: cosine, sine
+    __shared__ float2 scratch[2][32];
+    __shared__ TileToken tokens[kTileTokens];
+    __shared__ long long cells[kTileTokens], packs[kTileTokens];  // rows of the cache and of the packed arrays, or negative
+    extern __shared__ float2 turns[];                             // [tile][pairs]: cosine, sine
     const int c = threadIdx.x * 8, warps = (blockDim.x + 31) >> 5;
     const int token0 = blockIdx.x * tile;
     const bool live = c < p.rows.span;
     TapWindow<N> window;
     if (live) window.start(p.rows, c);  // weights: they do not wait for the kernel before
     grid_dependency_wait();
+    if (live) window.fetch(p.rows, c, token0);
+    look_up_tile(p.rows, tokens, token0, tile, rows);
+    for (int i = threadIdx.x; i < tile && token0 + i < rows; i += blockDim.x) {
+        long long page = p.write_pages[token0 + i], slot = p.write_slots[token0 + i];
+        if (page < 0) page += p.pages;
+        if (slot < 0) slot += p.page_size;
+        const bool inside = page >= 0 && page < p.pages && slot >= 0 && slot < p.page_size;
+        if (!inside) report_status(p.status, kStatusIndexOutOfBounds);
+        cells[i] = inside && (p.cached == nullptr || p.cached[token0 + i] != 0) ? page * p.page_size + slot : -1;
+        const long long packed = p.packed_rows == nullptr ? -1 : p.packed_rows[token0 + i];
+        packs[i] = packed < p.packed_count ? packed : -1;
+    }
     for (int i = threadIdx.x; i < tile * p.pairs; i += blockDim.x) {
         const int token = token0 + i / p.pairs;
         if (token >= rows) break;
@@ -396,12 +430,15 @@ __global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const Atten
     if (is_key) gain = widen(load_eight(p.key_norm, within));
     const bool normed = is_query || is_key;
     const size_t key_width = static_cast<size_t>(p.kv_heads) * p.key_size, value_width = static_cast<size_t>(p.kv_heads) * p.value_size;
+    __syncthreads();
+    int parity = 0;
     for (int i = 0; i < tile && token0 + i < rows; ++i) {
         const int token = token0 + i;
-        const int sequence = p.rows.sequence_of[token];
+        const TileToken now = tokens[i];
+        const uint4 row = window.ahead;
+        if (live && i + 1 < tile && token + 1 < rows) window.fetch(p.rows, c, token + 1);
         T *query = static_cast<T *>(p.query) + token * p.query_stride;
-        const int fresh = sequence >= 0 && sequence < p.rows.sequences ? p.rows.fresh[sequence] : 0;
-        if (fresh <= 0) {
+        if (now.fresh <= 0) {
             for (int at = c; at < p.heads * p.key_size; at += blockDim.x * 8) {
                 *reinterpret_cast<uint4 *>(query + at) = make_uint4(0u, 0u, 0u, 0u);
             }
@@ -409,20 +446,18 @@ __global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const Atten
             continue;
         }
         Eight y = {};
-        if (live) y = window.step(p.rows, c, token, sequence, token - p.rows.first[sequence], p.rows.context[sequence], fresh == 1);
+        if (live) y = window.step(p.rows, c, row, token, now.sequence, now.at, now.context, now.fresh == 1);
         float square = 0.0f;
 #pragma unroll
         for (int e = 0; e < 8; ++e) square = square_chain(square, y.v[e]);
         // sums of the queries' and of the keys' squares
         const float own_q = warp_sum(is_query ? square : 0.0f), own_k = warp_sum(is_key ? square : 0.0f);
-        __syncthreads();  // the sums before have been read (and, the first time, the turns are there)
-        if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = make_float2(own_q, own_k);
+        float2 *sums = scratch[parity];  // last used two barriers ago
+        parity ^= 1;
+        if ((threadIdx.x & 31) == 0) sums[threadIdx.x >> 5] = make_float2(own_q, own_k);
         __syncthreads();
-        float total_q = 0.0f, total_k = 0.0f;
-        for (int w = 0; w < warps; ++w) {
-            total_q += scratch[w].x;
-            total_k += scratch[w].y;
-        }
+        const float2 part = (threadIdx.x & 31) < warps ? sums[threadIdx.x & 31] : make_float2(0.0f, 0.0f);
+        const float total_q = warp_sum(part.x), total_k = warp_sum(part.y);
         const float scale = is_query ? 1.0f / sqrtf(total_q / static_cast<float>(queries) + p.eps)
                                      : 1.0f / sqrtf(total_k / static_cast<float>(keys) + p.eps);
         if (normed) {
@@ -441,18 +476,11 @@ __global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const Atten
             }
         }
         const uint4 out = narrow(y);
-        long long page = p.write_pages[token], slot = p.write_slots[token];
-        if (page < 0) page += p.pages;
-        if (slot < 0) slot += p.page_size;
-        const bool inside = page >= 0 && page < p.pages && slot >= 0 && slot < p.page_size;
-        if (!inside && threadIdx.x == 0) report_status(p.status, kStatusIndexOutOfBounds);
-        const bool keep = inside && (p.cached == nullptr || p.cached[token] != 0);
-        const long long packed = p.packed_rows == nullptr ? -1 : p.packed_rows[token];
-        const bool pack = packed >= 0 && packed < p.packed_count;
-        const size_t cell = keep ? static_cast<size_t>(page * p.page_size + slot) : 0;
+        const bool keep = cells[i] >= 0, pack = packs[i] >= 0;
+        const size_t cell = keep ? static_cast<size_t>(cells[i]) : 0, packed = pack ? static_cast<size_t>(packs[i]) : 0;
         T *cached_keys = static_cast<T *>(p.key_cache) + cell * key_width, *cached_values = static_cast<T *>(p.value_cache) + cell * value_width;
-        T *packed_keys = static_cast<T *>(p.packed_keys) + (pack ? packed : 0) * key_width;
-        T *packed_values = static_cast<T *>(p.packed_values) + (pack ? packed : 0) * value_width;
+        T *packed_keys = static_cast<T *>(p.packed_keys) + packed * key_width;
+        T *packed_values = static_cast<T *>(p.packed_values) + packed * value_width;
         if (is_query) *reinterpret_cast<uint4 *>(query + target) = out;
         if (keep && is_key) *reinterpret_cast<uint4 *>(cached_keys + target) = out;
         if (keep && is_value) *reinterpret_cast<uint4 *>(cached_values + target) = out;
@@ -481,27 +509,32 @@ __global__ void __launch_bounds__(1024) attention_inputs_wide_kernel(const Atten
 
 // blockIdx.y takes a slice of the columns; the lanes of a head are neighbours, a power of two of them.
 template <int N>
-__global__ void __launch_bounds__(kConvThreads) recurrence_inputs_wide_kernel(const RecurrenceInputs p, int rows, int tile) {
+__global__ void __launch_bounds__(kConvThreads, 4) recurrence_inputs_wide_kernel(const RecurrenceInputs p, int rows, int tile) {
     grid_launch_dependents();
+    __shared__ TileToken tokens[kTileTokens];
     const int c = (blockIdx.y * kConvThreads + threadIdx.x) * 8;
     const int token0 = blockIdx.x * tile;
     const bool live = c < p.rows.span;
     TapWindow<N> window;
     if (live) window.start(p.rows, c);
     grid_dependency_wait();
+    if (live) window.fetch(p.rows, c, token0);
+    look_up_tile(p.rows, tokens, token0, tile, rows);
+    __syncthreads();
     const int units = p.unit_heads * p.dim, lanes = p.dim / 8;
     const bool first = c < units, second = c >= p.second_at && c < p.second_at + units;
     const int unit = first ? c / p.dim : p.unit_heads + (c - p.second_at) / p.dim;
     for (int i = 0; i < tile && token0 + i < rows; ++i) {
         const int token = token0 + i;
-        const int sequence = p.rows.sequence_of[token];
-        const int fresh = sequence >= 0 && sequence < p.rows.sequences ? p.rows.fresh[sequence] : 0;
+        const TileToken now = tokens[i];
+        const uint4 row = window.ahead;
+        if (live && i + 1 < tile && token + 1 < rows) window.fetch(p.rows, c, token + 1);
         uint4 out = make_uint4(0u, 0u, 0u, 0u);
         float square = 0.0f;
-        if (fresh <= 0) {
+        if (now.fresh <= 0) {
             window.follows = false;
         } else if (live) {
-            Eight y = window.step(p.rows, c, token, sequence, token - p.rows.first[sequence], p.rows.context[sequence], fresh == 1);
+            Eight y = window.step(p.rows, c, row, token, now.sequence, now.at, now.context, now.fresh == 1);
 #pragma unroll
             for (int e = 0; e < 8; ++e) y.v[e] = __fdividef(y.v[e], 1.0f + __expf(-y.v[e]));
             out = narrow(y);
@@ -511,7 +544,7 @@ __global__ void __launch_bounds__(kConvThreads) recurrence_inputs_wide_kernel(co
         }
         if (live) *reinterpret_cast<uint4 *>(static_cast<__nv_bfloat16 *>(p.mixed) + token * p.mixed_stride + c) = out;
         for (int offset = lanes >> 1; offset > 0; offset >>= 1) square += __shfl_xor_sync(0xffffffffu, square, offset);
-        if ((first || second) && fresh > 0 && (threadIdx.x & (lanes - 1)) == 0) {
+        if ((first || second) && now.fresh > 0 && (threadIdx.x & (lanes - 1)) == 0) {
             p.inverse[static_cast<size_t>(token) * 2 * p.unit_heads + unit] = 1.0f / sqrtf(square + p.eps);
         }
     }
@@ -525,12 +558,23 @@ bool conv_eights(const ConvRows &p) {
            aligned_to(p.taps, 16) && aligned_to(p.state, 16);
 }
 
-#define SINGE_WIDE_CONV(KERNEL, GRID, THREADS, SHARED)                                                                     \
+template <int N>
+auto attention_inputs_kernel_for(unsigned threads) {
+    return threads <= 384 ? attention_inputs_wide_kernel<N, 384>
+                          : threads <= 768 ? attention_inputs_wide_kernel<N, 768> : attention_inputs_wide_kernel<N, 1024>;
+}
+
+template <int N>
+auto recurrence_inputs_kernel_for(unsigned) {
+    return recurrence_inputs_wide_kernel<N>;
+}
+
+#define SINGE_WIDE_CONV(CHOOSE, GRID, THREADS, SHARED)                                                                     \
     do {                                                                                                                   \
-        auto kernel = KERNEL<1>;                                                                                           \
-        if (p.rows.count == 2) kernel = KERNEL<2>;                                                                         \
-        if (p.rows.count == 3) kernel = KERNEL<3>;                                                                         \
-        if (p.rows.count == 4) kernel = KERNEL<4>;                                                                         \
+        auto kernel = CHOOSE<1>(THREADS);                                                                                  \
+        if (p.rows.count == 2) kernel = CHOOSE<2>(THREADS);                                                                \
+        if (p.rows.count == 3) kernel = CHOOSE<3>(THREADS);                                                                \
+        if (p.rows.count == 4) kernel = CHOOSE<4>(THREADS);                                                                \
         SINGE_CUDA_TRY(launch_dependent(kernel, GRID, dim3(THREADS), SHARED, static_cast<cudaStream_t>(stream), kLaunchGlue, 1, p, \
                                         static_cast<int>(rows), tile));                                                    \
         return launch_status();                                                                                            \
@@ -596,7 +640,7 @@ int attention_inputs(singe_stream_t stream, const AttentionInputs &p, size_t row
         const int tile = conv_tile(rows, 1);
         const unsigned threads = static_cast<unsigned>((p.rows.span / 8 + 31) / 32 * 32);
         const dim3 grid(static_cast<unsigned>((rows + tile - 1) / tile));
-        SINGE_WIDE_CONV(attention_inputs_wide_kernel, grid, threads, static_cast<size_t>(tile) * p.pairs * sizeof(float2));
+        SINGE_WIDE_CONV(attention_inputs_kernel_for, grid, threads, static_cast<size_t>(tile) * p.pairs * sizeof(float2));
     }
     const size_t bytes = 4 * sizeof(T);
     const bool out_wide = p.key_size % 4 == 0 && p.value_size % 4 == 0 && p.query_stride % 4 == 0 && aligned_to(p.query, bytes) &&
@@ -627,7 +671,7 @@ int recurrence_inputs(singe_stream_t stream, const RecurrenceInputs &p, size_t r
         const size_t slices = (static_cast<size_t>(p.rows.span) / 8 + kConvThreads - 1) / kConvThreads;
         const int tile = conv_tile(rows, slices);
         const dim3 grid(static_cast<unsigned>((rows + tile - 1) / tile), static_cast<unsigned>(slices));
-        SINGE_WIDE_CONV(recurrence_inputs_wide_kernel, grid, kConvThreads, 0);
+        SINGE_WIDE_CONV(recurrence_inputs_kernel_for, grid, kConvThreads, 0);
     }
     const bool wide = conv_wide<T>(p.rows) && p.mixed_stride % 4 == 0 && aligned_to(p.mixed, 4 * sizeof(T));
     auto kernel = wide ? recurrence_inputs_kernel<T, 4> : recurrence_inputs_kernel<T, 1>;
