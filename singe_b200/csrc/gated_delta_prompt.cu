@@ -75,10 +75,10 @@ struct DeltaParams {
     int stages;
 };
 
-// Shared memory of the prepare kernel: (q exp(a)), (k exp(-a)) and (k exp(a)), each hi and lo, a 16 x 17 matrix, three numbers a
+// Shared memory of the prepare kernel: the operands as they will go out, (k exp(-a)) hi and lo, a 16 x 17 matrix, three numbers a
 // token, and the decay of either half of the block per channel.
 __host__ __device__ constexpr int prepare_bytes(int dim_pad) {
-    return 6 * kBlock * (dim_pad * 2 + 16) + kBlock * 17 * 4 + 3 * kBlock * 4 + dim_pad * 8;
+    return delta_layout(dim_pad).bytes + 2 * kBlock * (dim_pad * 2 + 16) + kBlock * 17 * 4 + 3 * kBlock * 4 + dim_pad * 8;
 }
 
 // acc (two n tiles of 8) += A[16, 16 rows at a] . B[16 rows at b, same columns]^T over `columns`, split operands.
@@ -112,14 +112,15 @@ __global__ void __launch_bounds__(256) gated_delta_prepare_kernel(const DeltaPar
     const int row0 = p.block_row[block], tokens = p.block_tokens[block];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
     const DeltaLayout layout = delta_layout(p.dim_pad);
-    extern __shared__ __align__(16) uint8_t prepare_shared[];
+    extern __shared__ __align__(128) uint8_t prepare_shared[];
     const int half_bytes = kBlock * layout.pitch;  // from the hi to the lo part
-    uint8_t *fq = prepare_shared, *fk = fq + 2 * half_bytes, *fa = fk + 2 * half_bytes;
-    float *matrix = reinterpret_cast<float *>(fa + 2 * half_bytes);  // [16][17]
+    uint8_t *pack = prepare_shared;
+    uint8_t *fq = pack, *fa = pack + layout.w;  // k exp(a) is where W goes, column tile by column tile
+    uint8_t *fk = pack + layout.bytes;
+    float *matrix = reinterpret_cast<float *>(fk + 2 * half_bytes);  // [16][17]
     float *betas = matrix + kBlock * 17, *units_q = betas + kBlock, *units_k = units_q + kBlock;
     float2 *totals = reinterpret_cast<float2 *>(units_k + kBlock);   // [2 halves][dim_pad / 2]
     const int source = head / (p.heads / p.kv_heads);
-    uint8_t *pack = p.operands + (static_cast<size_t>(block) * p.heads + head) * layout.bytes;
     const float rate = expf(p.rate[head]);
 
     if (tid < kBlock) {
@@ -196,8 +197,6 @@ __global__ void __launch_bounds__(256) gated_delta_prepare_kernel(const DeltaPar
             const int at = (t0 + i) * layout.pitch + c * 2;
             uint32_t hi, lo;
             split_pair(q0 * before.x, q1 * before.y, hi, lo);
-            *reinterpret_cast<uint32_t *>(pack + at) = hi;
-            *reinterpret_cast<uint32_t *>(pack + half_bytes + at) = lo;
             *reinterpret_cast<uint32_t *>(fq + at) = hi;
             *reinterpret_cast<uint32_t *>(fq + half_bytes + at) = lo;
             split_pair(k0 * after.x, k1 * after.y, hi, lo);
@@ -318,6 +317,7 @@ __global__ void __launch_bounds__(256) gated_delta_prepare_kernel(const DeltaPar
         uint32_t hi[4], lo[4];
         ldmatrix_x4_trans(w_at + c0 * 2, hi[0], hi[1], hi[2], hi[3]);
         ldmatrix_x4_trans(w_at + half_bytes + c0 * 2, lo[0], lo[1], lo[2], lo[3]);
+        __syncwarp();  // the tile has been read by all lanes
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
             float acc[4] = {};
@@ -333,6 +333,14 @@ __global__ void __launch_bounds__(256) gated_delta_prepare_kernel(const DeltaPar
                 *reinterpret_cast<uint32_t *>(pack + layout.w + half_bytes + at) = y;
             }
         }
+    }
+    // ---- out in one bulk copy ----
+    fence_proxy_async_shared();
+    __syncthreads();
+    if (tid == 0) {
+        bulk_store(p.operands + (static_cast<size_t>(block) * p.heads + head) * layout.bytes, smem_u32(pack), layout.bytes);
+        tma_store_commit();
+        tma_store_wait<0>();
     }
 }
 
@@ -387,10 +395,10 @@ __global__ void __launch_bounds__(256, KT / KS <= 8 ? 2 : 1) gated_delta_advance
     // One warp brings a block in.  What a box holds past a short block or past the head's columns belongs to other rows or
     // columns (finite values): it meets zeros in T, or is never stored.
     const int boxes = (p.slice + 63) / 64;
-    auto load_block = [&](int index) {
+    auto load_block = [&](int index, int slot) {
         if (warp != 0) return;
-        const uint32_t bar = bars + 8 * (index % stages);
-        const uint32_t stage = smem_u32(advance_shared) + (index % stages) * stage_bytes;
+        const uint32_t bar = bars + 8 * slot;
+        const uint32_t stage = smem_u32(advance_shared) + slot * stage_bytes;
         if (lane == 0) {
             mbar_expect_tx(bar, kLayout.bytes + boxes * kValueBox);
             bulk_load(stage, p.operands + (static_cast<size_t>(first_block + index) * p.heads + head) * kLayout.bytes, kLayout.bytes, bar);
@@ -401,20 +409,24 @@ __global__ void __launch_bounds__(256, KT / KS <= 8 ? 2 : 1) gated_delta_advance
                         p.value_at + head * p.vdim + slice0 + lane * 64, first_row + index * kBlock);
         }
     };
-    for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i);
+    for (int i = 0; i < stages - 1 && i < blocks; ++i) load_block(i, i);
     bool failed = false;
+    int slot = 0, round = 0;
 
-    for (int index = 0; index < blocks; ++index) {
+    for (int index = 0; index < blocks; ++index, round ^= slot == 0) {
+        const int here_slot = slot, next_slot = slot == 0 ? stages - 1 : slot - 1;
+        const int parity = round;
+        slot = slot + 1 == stages ? 0 : slot + 1;
         const int row0 = first_row + index * kBlock, tokens = index + 1 < blocks ? kBlock : last_tokens;
-        const bool arrived = mbar_wait(bars + 8 * (index % stages), (index / stages) & 1);
+        const bool arrived = mbar_wait(bars + 8 * here_slot, parity);
         fence_proxy_async_shared();
         // the block has arrived for every thread, and everyone is done with the stage loaded next and with the sums
         if (__syncthreads_or(arrived ? 0 : 1) != 0) {
             failed = true;
             break;
         }
-        if (index + stages - 1 < blocks) load_block(index + stages - 1);
-        uint8_t *here = advance_shared + (index % stages) * stage_bytes;
+        if (index + stages - 1 < blocks) load_block(index + stages - 1, next_slot);
+        uint8_t *here = advance_shared + here_slot * stage_bytes;
         const uint32_t stage = smem_u32(here);
         const int t = (lane & 7) + ((lane >> 4) << 3);
 
@@ -653,8 +665,8 @@ int delta_dim_pad(size_t dim, size_t vdim) {
 // that the key tiles are shared out among four warps as well.
 int delta_slice(size_t runs, size_t heads, size_t vdim, int dim_pad, bool &shared_keys) {
     const size_t sms = static_cast<size_t>(device_sm_count());
-    shared_keys = dim_pad >= 64 && runs * heads * ((vdim + 15) / 16) < 4 * sms;
-    if (shared_keys) return vdim > 16 ? 32 : 16;
+    shared_keys = dim_pad >= 64 && runs * heads * ((vdim + 15) / 16) < 2 * sms;
+    if (shared_keys) return runs * heads * ((vdim + 15) / 16) <= sms ? 16 : 32;
     int slice = 16;
     while (slice < 128 && static_cast<size_t>(slice) < vdim) slice *= 2;
     while (slice > 16 && runs * heads * ((vdim + slice - 1) / slice) < sms) slice /= 2;

@@ -30,6 +30,11 @@ __device__ __forceinline__ void bulk_load(uint32_t target, const void *source, u
                  : "memory");
 }
 
+// Bulk copy shared -> global as part of the thread's current bulk group (16-byte aligned addresses and size).
+__device__ __forceinline__ void bulk_store(void *target, uint32_t source, uint32_t bytes) {
+    asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(target), "r"(source), "r"(bytes) : "memory");
+}
+
 // ldmatrix_x4_trans's inverse: four 8x8 matrices out of MMA fragments, transposed.
 __device__ __forceinline__ void stmatrix_x4_trans(uint32_t address, uint32_t r0, uint32_t r1, uint32_t r2, uint32_t r3) {
     asm volatile("stmatrix.sync.aligned.m8n8.x4.trans.shared.b16 [%0], {%1, %2, %3, %4};" ::"r"(address), "r"(r0), "r"(r1),
