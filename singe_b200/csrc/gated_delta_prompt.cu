@@ -644,12 +644,16 @@ int launch_advance(cudaStream_t stream, const CUtensorMap &value_map, DeltaParam
     p.stages = kMaxStages;  // as many as leave room for a second CTA, three at least
     while (p.stages > 3 && bytes_of(p.stages) > 112 * 1024) --p.stages;
     if (bytes_of(p.stages) > 227 * 1024) return SINGE_ERR_UNSUPPORTED_CONFIGURATION;
-    static int configured[kMaxDevices] = {0};
-    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_advance_kernel<KT, KS>, bytes_of(p.stages), configured));
     const dim3 grid(static_cast<unsigned>(runs), static_cast<unsigned>(p.heads),
                     static_cast<unsigned>((p.vdim + p.slice - 1) / p.slice));
-    SINGE_CUDA_TRY(launch_dependent(gated_delta_advance_kernel<KT, KS>, grid, dim3(threads), bytes_of(p.stages), stream, kLaunchGlue,
-                                    1, value_map, p));
+    // A grid that leaves SMs idle must not put two CTAs on one: those that launch while the kernel before drains would.  More than
+    // half of an SM's shared memory keeps them apart.
+    int bytes = bytes_of(p.stages);
+    const size_t ctas = static_cast<size_t>(grid.x) * grid.y * grid.z;
+    if (ctas <= static_cast<size_t>(device_sm_count()) && bytes < 120 * 1024) bytes = 120 * 1024;
+    static int configured[kMaxDevices] = {0};
+    SINGE_CUDA_TRY(ensure_dynamic_shared(gated_delta_advance_kernel<KT, KS>, bytes, configured));
+    SINGE_CUDA_TRY(launch_dependent(gated_delta_advance_kernel<KT, KS>, grid, dim3(threads), bytes, stream, kLaunchGlue, 1, value_map, p));
     return launch_status();
 }
 
